@@ -87,7 +87,8 @@ typedef struct {
                                 src/models/cpu.rs:26-56; quantize_weights, rust.rs:1354-1376); the embedding lookup
                                 keeps FP32 rows as in the reference. Decode steps of at most 8 sequences stream the
                                 1-byte copies; prefill and larger batches multiply the dequantised values q * scale */
-  int32_t reserved[1];
+  int32_t max_context;  /* models without a position limit of their own (see pg_model_architecture): the most tokens a
+                           sequence may hold, 0 = 32768; unused by GPT-2, whose n_positions is the limit */
 } pg_backend_config;
 
 /* TextGenerationConfig, src/models/generation.rs:60-85. None is encoded as a negative value. */
@@ -169,6 +170,14 @@ int pg_model_load_dir(const char* dir, const pg_backend_config* backend, pg_mode
 int pg_model_from_host_weights(const pg_gpt2_config* cfg, const float* const* tensors,
                                const uint64_t* lens, uint64_t n_tensors,
                                const pg_backend_config* backend, pg_model** out);
+/* Name of the model's design: "gpt2", or the "architecture" entry of its config.json. pg_model_load_dir picks the
+ * model class by that entry (a GPT-2 configuration has none). For other designs than GPT-2 pg_model_config fills in
+ * vocab_size, n_positions (the backend's max_context), n_embd (the width) and n_layer, sets n_head and n_inner to 1,
+ * and the arithmetic modes are PG_MATH_FP32 and PG_MATH_BF16 (BF16 weights, product inputs and cached keys and values;
+ * FP32 sums, norms, residual stream and recurrent state). No counterpart. */
+const char* pg_model_architecture(const pg_model* model);
+/* Comma-separated names of the designs that pg_model_load_dir knows. No counterpart. */
+const char* pg_registered_architectures(void);
 /* Gpt2Model.config */
 int pg_model_config(const pg_model* model, pg_gpt2_config* out);
 /* AutoregressiveDecoder::max_context_len, src/models/gpt2/rust.rs:1258-1260 */
@@ -215,6 +224,17 @@ int pg_forward_one(const pg_model* model, pg_cache* cache, const int32_t* ids, i
  * sequence, no cache. logits_out holds t * vocab_size floats. */
 int pg_forward(const pg_model* model, const int32_t* ids, int32_t t, float* logits_out);
 
+/* Appends a portion to each of `n` sequences in one pass: lens[i] tokens (ids concatenated) to slot slots[i] (distinct),
+ * after what the slot holds (pg_cache_clear_slot starts a new sequence). `want` lists rows of the concatenated ids, in
+ * any order; logits_out receives n_want * vocab_size floats in that order. argmax_out (n, optional) is the arg-max at
+ * each portion's last token, last_logits_out (n * vocab_size, optional) its logits. A prompt may be cut anywhere. When
+ * every portion is one token and slots are 0..n-1 the pass is a decode step. GPT-2 takes several tokens for slots that
+ * are empty and 0..n-1, else the portions run token by token and must be of equal length. The reference runs whole
+ * prompts only (prefill, src/models/gpt2/rust.rs:906-927). */
+int pg_extend(const pg_model* model, pg_cache* cache, const int32_t* slots, const int32_t* ids, const int32_t* lens,
+              int32_t n, const int32_t* want, int32_t n_want, float* logits_out, int32_t* argmax_out,
+              float* last_logits_out);
+
 /* Greedy decode with every step's token fed back on the device (no host round trip per step):
  * runs `steps` forward_one calls on slots 0..batch-1 starting from first_ids, each next id being
  * the argmax of the step before. tokens_out (steps * batch, step-major) receives the argmax of
@@ -228,6 +248,12 @@ int pg_decode_greedy(const pg_model* model, pg_cache* cache, const int32_t* firs
  * operation buckets. Advances the cache like pg_forward_one. */
 int pg_profile_forward_one(const pg_model* model, pg_cache* cache, const int32_t* ids, int32_t batch,
                            pg_operation_profile* out);
+/* The same for a prefill of `batch` prompts (arguments as pg_prefill): device time of its kernels by operation class.
+ * Layered models only. No reference counterpart. */
+int pg_profile_prefill(const pg_model* model, pg_cache* cache, const int32_t* ids, const int32_t* lens, int32_t batch,
+                       pg_operation_profile* out);
+/* Bytes of recurrent state one sequence carries (0 for GPT-2). No counterpart. */
+uint64_t pg_model_state_bytes_per_sequence(const pg_model* model);
 /* Device-side stopwatch on the cache's own stream (where every kernel of this cache runs):
  * begin drains the stream and records an event; end records a second event, waits for it and
  * returns the elapsed seconds. The reference times with Instant::now() around the same calls

@@ -23,7 +23,7 @@ class PgConfig(C.Structure):
 class PgBackendConfig(C.Structure):
     _fields_ = [("device", C.c_int32), ("math_mode", C.c_int32), ("page_tokens", C.c_int32),
                 ("use_graphs", C.c_int32), ("attn_splits", C.c_int32), ("persistent_step", C.c_int32),
-                ("quantized_weights", C.c_int32), ("reserved", C.c_int32 * 1)]
+                ("quantized_weights", C.c_int32), ("max_context", C.c_int32)]
 
 
 class PgGenerationConfig(C.Structure):
@@ -67,6 +67,11 @@ SIGNATURES = {
     "pg_model_load_dir": (C.c_int, [C.c_char_p, C.POINTER(PgBackendConfig), C.POINTER(_vp)]),
     "pg_model_from_host_weights": (C.c_int, [C.POINTER(PgConfig), C.POINTER(_fp), _u64p, C.c_uint64,
                                              C.POINTER(PgBackendConfig), C.POINTER(_vp)]),
+    "pg_model_architecture": (C.c_char_p, [_vp]),
+    "pg_registered_architectures": (C.c_char_p, []),
+    "pg_model_state_bytes_per_sequence": (C.c_uint64, [_vp]),
+    "pg_profile_prefill": (C.c_int, [_vp, _vp, _ip, _ip, C.c_int32, C.POINTER(PgOperationProfile)]),
+    "pg_extend": (C.c_int, [_vp, _vp, _ip, _ip, _ip, C.c_int32, _ip, C.c_int32, _fp, _ip, _fp]),
     "pg_model_config": (C.c_int, [_vp, C.POINTER(PgConfig)]),
     "pg_model_max_context_len": (C.c_uint64, [_vp]),
     "pg_model_weight_bytes_per_step": (C.c_uint64, [_vp]),

@@ -8,6 +8,7 @@ import os
 import shutil
 import subprocess
 import sys
+from concurrent.futures import ThreadPoolExecutor
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
@@ -42,7 +43,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
     os.makedirs(OBJ_DIR, exist_ok=True)
     nvcc = _nvcc()
     newest_header = max(os.path.getmtime(h) for h in _headers())
-    objs, rebuilt = [], False
+    objs, commands = [], []
     for src in _sources():
         path = os.path.join(CSRC, src)
         obj = os.path.join(OBJ_DIR, src + ".o")
@@ -54,16 +55,22 @@ def build(force: bool = False, verbose: bool = False) -> str:
             cmd = [nvcc, *NVCC_FLAGS, "-c", path, "-o", obj]
         else:
             cmd = [os.environ.get("CXX", "g++"), *CXX_FLAGS, "-c", path, "-o", obj]
+        # the largest sources first: the build ends with its longest compile
+        commands.append((-os.path.getsize(path), cmd))
+
+    def run(cmd):
         if verbose:
             print(" ".join(cmd), file=sys.stderr)
         subprocess.run(cmd, check=True)
-        rebuilt = True
-    if rebuilt or not os.path.exists(LIB):
-        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", LIB, *objs,
+
+    with ThreadPoolExecutor(max_workers=max(1, min(len(commands), os.cpu_count() or 1))) as pool:
+        list(pool.map(run, [cmd for _, cmd in sorted(commands)]))
+    if commands or not os.path.exists(LIB):
+        part = f"{LIB}.{os.getpid()}"  # renamed into place: a process that starts meanwhile never loads half a library
+        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", part, *objs,
                "-cudart", "static", "-lpthread"]
-        if verbose:
-            print(" ".join(cmd), file=sys.stderr)
-        subprocess.run(cmd, check=True)
+        run(cmd)
+        os.replace(part, LIB)
     return LIB
 
 

@@ -1,0 +1,486 @@
+// Attention of the layered models: grouped key / value heads, separate key and value sizes, optional per-head RMS norms
+// of queries, keys and values, and keys that are visible inside one block of `span` positions only (or always, when
+// the span is the whole context). Keys and values live in pages indexed by position % span.
+#include <algorithm>
+#include <cfloat>
+
+#include "device_util.cuh"
+#include "layered_kernels.cuh"
+
+namespace pg {
+namespace {
+
+// First element of the key (which = 0) or value row of cache index c of one kv head.
+template <typename T>
+__device__ __forceinline__ T* page_row(const AttentionLayer& l, T* pool, const int* table_row, int c, int head, int which) {
+  const size_t page_elems = (size_t)l.kv_heads * l.page_tokens * (l.dimp + l.vdimp);
+  T* page = pool + (size_t)table_row[c / l.page_tokens] * page_elems;
+  const int off = c % l.page_tokens;
+  if (which == 0) return page + ((size_t)head * l.page_tokens + off) * l.dimp;
+  return page + (size_t)l.kv_heads * l.page_tokens * l.dimp + ((size_t)head * l.page_tokens + off) * l.vdimp;
+}
+
+// One warp: out[0..np) = norm(x[0..n)) * weight * mul, zero past n. `normed` false: only the copy.
+template <typename T>
+__device__ __forceinline__ void warp_norm_row(const float* x, int n, int np, const float* weight, bool normed, float eps,
+                                              float mul, T* out, int lane) {
+  float s = 0.f;
+  if (normed)
+    for (int c = lane; c < n; c += 32) s += x[c] * x[c];
+  const float r = normed ? 1.f / sqrtf(lane_sum(s) / (float)n + eps) : 1.f;
+  for (int c = lane; c < np; c += 32) {
+    float v = 0.f;
+    if (c < n) {
+      v = x[c] * r;
+      if (weight) v *= weight[c];
+      v *= mul;
+    }
+    out[c] = from_f32<T>(v);
+  }
+}
+
+// ------------------------------------------------------------------ one token per sequence
+// Block = one kv head of one sequence and one part of its visible keys, for RB query heads of the group at a time.
+// Eight lanes share a key (16-byte pieces of the row), the probabilities go through shared memory, and threads then own
+// eight value columns each for a subset of the keys. Partial results of the parts are merged by the last block.
+constexpr int STEP_THREADS = 256, STEP_KEYS = 256, RB = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(STEP_THREADS) attention_step_kernel(AttentionStepArgs a, int y_bf16) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ int last_flag;
+  const AttentionLayer& l = a.l;
+  const int rep = l.heads / l.kv_heads;
+  const int kvh = blockIdx.x, seq = blockIdx.y, split = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* qs = sm;                            // [rep][dimp]
+  float* kn = qs + rep * l.dimp;             // [dimp] new key as stored
+  float* vn = kn + l.dimp;                   // [vdimp] new value as stored
+  float* sc = vn + l.vdimp;                  // [RB][STEP_KEYS]
+  float* acc_s = sc + RB * STEP_KEYS;        // [groups][RB][vdimp] cross-thread sums
+  __shared__ float red_m[RB], red_l[RB], corr_s[RB];
+
+  grid_dep_launch();
+  grid_dep_wait();
+  const float* p = a.p + (size_t)seq * a.ldp;
+  const int pos = a.pos[seq], last = pos % l.span;  // keys 0..last of this block of positions; `last` is the new one
+  const int per = (last + 1 + a.splits - 1) / a.splits;
+  const int k0 = split * per, k1 = min(last + 1, k0 + per);
+  const int* table = a.page_table + (size_t)seq * l.pages_per_seq;
+  T* pool = static_cast<T*>(a.pool);
+  const bool owner = k0 <= last && last < k1;
+
+  for (int i = warp; i < rep + 2; i += STEP_THREADS / 32) {
+    if (i < rep)
+      warp_norm_row<float>(p + l.off_q + (kvh * rep + i) * l.dim, l.dim, l.dimp, l.q_norm, l.q_norm != nullptr, l.eps, 1.f,
+                           qs + i * l.dimp, lane);
+    else if (i == rep)
+      warp_norm_row<float>(p + l.off_k + kvh * l.dim, l.dim, l.dimp, l.k_norm, l.k_norm != nullptr, l.eps, 1.f, kn, lane);
+    else
+      warp_norm_row<float>(p + l.off_v + kvh * l.vdim, l.vdim, l.vdimp, nullptr, l.v_norm != 0, l.eps, 1.f, vn, lane);
+  }
+  __syncthreads();
+  if (owner) {  // append; later reads of this row use the rounded copy in shared memory
+    T* krow = page_row(l, pool, table, last, kvh, 0);
+    T* vrow = page_row(l, pool, table, last, kvh, 1);
+    for (int c = tid; c < l.dimp; c += STEP_THREADS) krow[c] = from_f32<T>(kn[c]);
+    for (int c = tid; c < l.vdimp; c += STEP_THREADS) vrow[c] = from_f32<T>(vn[c]);
+  }
+  __syncthreads();
+  for (int c = tid; c < l.dimp; c += STEP_THREADS) kn[c] = to_f32(from_f32<T>(kn[c]));
+  for (int c = tid; c < l.vdimp; c += STEP_THREADS) vn[c] = to_f32(from_f32<T>(vn[c]));
+  __syncthreads();
+
+  const int nvec = l.vdimp / 8, groups = STEP_THREADS / nvec;  // value phase: thread = (8 columns, key subset)
+  const int vc = tid % nvec, vg = tid / nvec;
+  const int sub = lane >> 3, l8 = lane & 7;
+
+  for (int r0 = 0; r0 < rep; r0 += RB) {
+    const int nr = min(RB, rep - r0);
+    float m_run[RB], l_run[RB], acc[RB][8];
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      m_run[r] = -FLT_MAX;
+      l_run[r] = 0.f;
+#pragma unroll
+      for (int c = 0; c < 8; ++c) acc[r][c] = 0.f;
+    }
+    for (int kb = k0; kb < k1; kb += STEP_KEYS) {
+      const int n = min(STEP_KEYS, k1 - kb);
+      for (int j0 = warp * 4; j0 < n; j0 += STEP_THREADS / 32 * 4) {
+        const int j = j0 + sub;
+        float dot[RB];
+#pragma unroll
+        for (int r = 0; r < RB; ++r) dot[r] = 0.f;
+        if (j < n) {
+          const bool self = kb + j == last;
+          const T* krow = self ? nullptr : page_row(l, pool, table, kb + j, kvh, 0);
+          for (int c = l8 * 8; c < l.dimp; c += 64) {
+            float kv[8];
+            if (self) load8(kn + c, kv);
+            else load8(krow + c, kv);
+#pragma unroll
+            for (int r = 0; r < RB; ++r) {
+              if (r < nr) {
+                float qv[8];
+                load8(qs + (r0 + r) * l.dimp + c, qv);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) dot[r] = fmaf(qv[e], kv[e], dot[r]);
+              }
+            }
+          }
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+          for (int r = 0; r < RB; ++r) dot[r] += __shfl_xor_sync(ALL_LANES, dot[r], o);
+        if (j < n && l8 == 0) {
+#pragma unroll
+          for (int r = 0; r < RB; ++r)
+            if (r < nr) sc[r * STEP_KEYS + j] = dot[r] * l.scale;
+        }
+      }
+      __syncthreads();
+      if (warp < nr) {  // one warp per query head: running maximum, probabilities, sum
+        float mx = -FLT_MAX;
+        for (int j = lane; j < n; j += 32) mx = fmaxf(mx, sc[warp * STEP_KEYS + j]);
+        mx = lane_max(mx);
+        float m_old = -FLT_MAX;
+#pragma unroll
+        for (int r = 0; r < RB; ++r)
+          if (r == warp) m_old = m_run[r];
+        const float m_new = fmaxf(m_old, mx);
+        float sum = 0.f;
+        for (int j = lane; j < n; j += 32) {
+          const float e = expf(sc[warp * STEP_KEYS + j] - m_new);
+          sc[warp * STEP_KEYS + j] = e;
+          sum += e;
+        }
+        sum = lane_sum(sum);
+        if (lane == 0) {
+          red_m[warp] = m_new;
+          red_l[warp] = sum;
+          corr_s[warp] = expf(m_old - m_new);
+        }
+      }
+      __syncthreads();
+#pragma unroll
+      for (int r = 0; r < RB; ++r)
+        if (r < nr) {
+          m_run[r] = red_m[r];
+          l_run[r] = l_run[r] * corr_s[r] + red_l[r];
+#pragma unroll
+          for (int c = 0; c < 8; ++c) acc[r][c] *= corr_s[r];
+        }
+      if (vg < groups) {
+        for (int j = vg; j < n; j += groups) {
+          float vv[8];
+          if (kb + j == last) load8(vn + vc * 8, vv);
+          else load8(page_row(l, pool, table, kb + j, kvh, 1) + vc * 8, vv);
+#pragma unroll
+          for (int r = 0; r < RB; ++r)
+            if (r < nr) {
+              const float pr = sc[r * STEP_KEYS + j];
+#pragma unroll
+              for (int e = 0; e < 8; ++e) acc[r][e] = fmaf(pr, vv[e], acc[r][e]);
+            }
+        }
+      }
+      __syncthreads();
+    }
+    // sum over the key subsets
+    if (vg < groups) {
+#pragma unroll
+      for (int r = 0; r < RB; ++r)
+        if (r < nr)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc_s[((size_t)vg * RB + r) * l.vdimp + vc * 8 + e] = acc[r][e];
+    }
+    __syncthreads();
+    for (int i = tid; i < nr * l.vdim; i += STEP_THREADS) {
+      const int r = i / l.vdim, c = i % l.vdim;
+      float s = 0.f;
+      for (int g = 0; g < groups; ++g) s += acc_s[((size_t)g * RB + r) * l.vdimp + c];
+      float lr = 0.f, mr = 0.f;
+#pragma unroll
+      for (int q = 0; q < RB; ++q)
+        if (q == r) {
+          lr = l_run[q];
+          mr = m_run[q];
+        }
+      const int h = kvh * rep + r0 + r;
+      if (a.splits == 1) {
+        const float y = s / lr * l.out_scale;
+        const size_t at = (size_t)seq * a.ldy + h * l.vdim + c;
+        if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
+        else static_cast<float*>(a.y)[at] = y;
+      } else {
+        float* pt = a.part + (((size_t)seq * l.heads + h) * a.splits + split) * (l.vdim + 2);
+        pt[2 + c] = s;
+        if (c == 0) {
+          pt[0] = mr;
+          pt[1] = lr;
+        }
+      }
+    }
+    __syncthreads();
+  }
+  if (a.splits == 1) return;
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {
+    const unsigned n = atomicAdd(&a.counters[seq * l.kv_heads + kvh], 1u);
+    last_flag = n == (unsigned)a.splits - 1;
+    if (last_flag) a.counters[seq * l.kv_heads + kvh] = 0;
+  }
+  __syncthreads();
+  if (!last_flag) return;
+  __threadfence();
+  for (int i = tid; i < rep * l.vdim; i += STEP_THREADS) {
+    const int h = kvh * rep + i / l.vdim, c = i % l.vdim;
+    const volatile float* pt = a.part + ((size_t)seq * l.heads + h) * a.splits * (l.vdim + 2);
+    float m = -FLT_MAX;
+    for (int s = 0; s < a.splits; ++s) m = fmaxf(m, pt[s * (l.vdim + 2)]);
+    float num = 0.f, den = 0.f;
+    for (int s = 0; s < a.splits; ++s) {
+      const float w = expf(pt[s * (l.vdim + 2)] - m);
+      num += w * pt[s * (l.vdim + 2) + 2 + c];
+      den += w * pt[s * (l.vdim + 2) + 1];
+    }
+    const float y = num / den * l.out_scale;
+    const size_t at = (size_t)seq * a.ldy + h * l.vdim + c;
+    if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
+    else static_cast<float*>(a.y)[at] = y;
+  }
+}
+
+// ------------------------------------------------------------------ portions
+// Norms of every row's queries, keys and values; a warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256) attention_prep_kernel(AttentionPortionArgs a) {
+  const AttentionLayer& l = a.l;
+  const int per = l.heads + 2 * l.kv_heads, lane = threadIdx.x & 31;
+  const long long total = (long long)a.rows * per;
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5; i < total;
+       i += ((long long)gridDim.x * blockDim.x) >> 5) {
+    const int row = (int)(i / per), j = (int)(i % per);
+    const float* p = a.p + (size_t)row * a.ldp;
+    const int seq = a.row_seq[row];
+    const int ctx = a.seq_pos[seq] % l.span;  // cached keys the sequence's first row still sees
+    const size_t krow = (size_t)a.key_start[seq] + ctx + (row - a.seq_start[seq]);
+    if (j < l.heads)
+      warp_norm_row<T>(p + l.off_q + j * l.dim, l.dim, l.dimp, l.q_norm, l.q_norm != nullptr, l.eps, 1.f,
+                       static_cast<T*>(a.q) + ((size_t)row * l.heads + j) * l.dimp, lane);
+    else if (j < l.heads + l.kv_heads)
+      warp_norm_row<T>(p + l.off_k + (j - l.heads) * l.dim, l.dim, l.dimp, l.k_norm, l.k_norm != nullptr, l.eps, 1.f,
+                       static_cast<T*>(a.k) + (krow * l.kv_heads + (j - l.heads)) * l.dimp, lane);
+    else
+      warp_norm_row<T>(p + l.off_v + (j - l.heads - l.kv_heads) * l.vdim, l.vdim, l.vdimp, nullptr, l.v_norm != 0, l.eps, 1.f,
+                       static_cast<T*>(a.v) + (krow * l.kv_heads + (j - l.heads - l.kv_heads)) * l.vdimp, lane);
+  }
+}
+
+// Cached keys and values that the first row of each sequence still sees, copied in front of its own. Block = (key, seq).
+template <typename T>
+__global__ void __launch_bounds__(128) attention_context_kernel(AttentionPortionArgs a) {
+  const AttentionLayer& l = a.l;
+  const int seq = blockIdx.y, ctx = a.seq_pos[seq] % l.span;
+  const int* table = a.page_table + (size_t)a.seq_slot[seq] * l.pages_per_seq;
+  for (int c = blockIdx.x; c < ctx; c += gridDim.x) {
+    const size_t krow = (size_t)a.key_start[seq] + c;
+    for (int i = threadIdx.x; i < l.kv_heads * (l.dimp + l.vdimp) / 8; i += blockDim.x) {
+      const int e = i * 8;
+      const bool is_k = e < l.kv_heads * l.dimp;
+      const int x = is_k ? e : e - l.kv_heads * l.dimp, w = is_k ? l.dimp : l.vdimp;
+      const T* src = page_row(l, static_cast<T*>(a.pool), table, c, x / w, is_k ? 0 : 1) + x % w;
+      T* dst = (is_k ? static_cast<T*>(a.k) + krow * l.kv_heads * l.dimp : static_cast<T*>(a.v) + krow * l.kv_heads * l.vdimp) + x;
+      if (sizeof(T) == 2) {
+        *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
+      } else {
+        reinterpret_cast<float4*>(dst)[0] = reinterpret_cast<const float4*>(src)[0];
+        reinterpret_cast<float4*>(dst)[1] = reinterpret_cast<const float4*>(src)[1];
+      }
+    }
+  }
+}
+
+// Stores the portion's keys and values that later tokens can still see: those of the block of positions in which the
+// next token lies or the last one lay.
+template <typename T>
+__global__ void __launch_bounds__(128) attention_store_kernel(AttentionPortionArgs a) {
+  const AttentionLayer& l = a.l;
+  const int row = blockIdx.x, seq = a.row_seq[row];
+  const int first = a.seq_start[seq], n = a.seq_start[seq + 1] - first, p0 = a.seq_pos[seq];
+  const int pos = p0 + (row - first), end = p0 + n - 1;
+  if (pos / l.span != end / l.span) return;
+  const int* table = a.page_table + (size_t)a.seq_slot[seq] * l.pages_per_seq;
+  const size_t krow = (size_t)a.key_start[seq] + p0 % l.span + (row - first);
+  const int c = pos % l.span;
+  for (int i = threadIdx.x; i < l.kv_heads * (l.dimp + l.vdimp) / 8; i += blockDim.x) {
+    const int e = i * 8;
+    const bool is_k = e < l.kv_heads * l.dimp;
+    const int x = is_k ? e : e - l.kv_heads * l.dimp, w = is_k ? l.dimp : l.vdimp;
+    T* dst = page_row(l, static_cast<T*>(a.pool), table, c, x / w, is_k ? 0 : 1) + x % w;
+    const T* src =
+        (is_k ? static_cast<const T*>(a.k) + krow * l.kv_heads * l.dimp : static_cast<const T*>(a.v) + krow * l.kv_heads * l.vdimp) + x;
+    if (sizeof(T) == 2) {
+      *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
+    } else {
+      reinterpret_cast<float4*>(dst)[0] = reinterpret_cast<const float4*>(src)[0];
+      reinterpret_cast<float4*>(dst)[1] = reinterpret_cast<const float4*>(src)[1];
+    }
+  }
+}
+
+// CUDA-core attention over the workspaces. Block = 32 query rows of one head of one sequence, 128 threads: four lanes
+// per row, key tiles of 32, FP32 scores and sums, online softmax. Key rows of a tile are padded by one float.
+constexpr int QT = 32, KT = 32;
+template <typename T, int VR>
+__global__ void __launch_bounds__(128) attention_rows_kernel(AttentionPortionArgs a) {
+  extern __shared__ __align__(16) float sm[];
+  const AttentionLayer& l = a.l;
+  const int head = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
+  const int first = a.seq_start[seq], n = a.seq_start[seq + 1] - first, q0 = blockIdx.x * QT;
+  if (q0 >= n) return;
+  const int kvh = head / (l.heads / l.kv_heads), p0 = a.seq_pos[seq], ctx = p0 % l.span;
+  const int base_pos = p0 - ctx;  // position of workspace key 0 of this sequence
+  float* qs = sm;                             // [QT][dimp + 1]
+  float* ks = qs + QT * (l.dimp + 1);         // [KT][dimp + 1]
+  float* vs = ks + KT * (l.dimp + 1);         // [KT][vdimp]
+  float* ps = vs + KT * l.vdimp;              // [QT][KT + 1]
+  const int r = tid >> 2, sub = tid & 3;
+  const int qrow = q0 + r;
+  const bool live = qrow < n;
+  for (int i = tid; i < QT * l.dimp; i += 128) {
+    const int rr = i / l.dimp, c = i % l.dimp;
+    qs[rr * (l.dimp + 1) + c] =
+        q0 + rr < n ? to_f32(static_cast<const T*>(a.q)[((size_t)(first + q0 + rr) * l.heads + head) * l.dimp + c]) : 0.f;
+  }
+  // keys [lo_row, hi_row] of the workspace are visible to this thread's row
+  const int pos = p0 + min(qrow, n - 1);
+  const int lo_row = max(pos / l.span * l.span - base_pos, 0), hi_row = pos - base_pos;
+  // range of the block's rows
+  const int pos_a = p0 + q0, pos_b = p0 + min(q0 + QT, n) - 1;
+  const int lo = max(pos_a / l.span * l.span - base_pos, 0), hi = pos_b - base_pos;
+  float m = -FLT_MAX, lsum = 0.f, acc[VR];
+#pragma unroll
+  for (int c = 0; c < VR; ++c) acc[c] = 0.f;
+  for (int kt = lo; kt <= hi; kt += KT) {
+    __syncthreads();
+    for (int i = tid; i < KT * l.dimp; i += 128) {
+      const int rr = i / l.dimp, c = i % l.dimp;
+      ks[rr * (l.dimp + 1) + c] =
+          kt + rr <= hi ? to_f32(static_cast<const T*>(a.k)[((size_t)(a.key_start[seq] + kt + rr) * l.kv_heads + kvh) * l.dimp + c]) : 0.f;
+    }
+    for (int i = tid; i < KT * l.vdimp; i += 128) {
+      const int rr = i / l.vdimp, c = i % l.vdimp;
+      vs[i] = kt + rr <= hi ? to_f32(static_cast<const T*>(a.v)[((size_t)(a.key_start[seq] + kt + rr) * l.kv_heads + kvh) * l.vdimp + c]) : 0.f;
+    }
+    __syncthreads();
+    float s[KT / 4];
+#pragma unroll
+    for (int j = 0; j < KT / 4; ++j) s[j] = 0.f;
+    for (int c = 0; c < l.dim; ++c) {
+      const float q = qs[r * (l.dimp + 1) + c];
+#pragma unroll
+      for (int j = 0; j < KT / 4; ++j) s[j] = fmaf(q, ks[(j * 4 + sub) * (l.dimp + 1) + c], s[j]);
+    }
+    float mx = -FLT_MAX;
+#pragma unroll
+    for (int j = 0; j < KT / 4; ++j) {
+      const int key = kt + j * 4 + sub;
+      s[j] = (live && key >= lo_row && key <= hi_row) ? s[j] * l.scale : -FLT_MAX;
+      mx = fmaxf(mx, s[j]);
+    }
+    mx = fmaxf(mx, __shfl_xor_sync(ALL_LANES, mx, 1));
+    mx = fmaxf(mx, __shfl_xor_sync(ALL_LANES, mx, 2));
+    const float m_new = fmaxf(m, mx), corr = expf(m - m_new);
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < KT / 4; ++j) {
+      const float e = s[j] > -FLT_MAX ? expf(s[j] - m_new) : 0.f;
+      ps[r * (KT + 1) + j * 4 + sub] = e;
+      sum += e;
+    }
+    sum += __shfl_xor_sync(ALL_LANES, sum, 1);
+    sum += __shfl_xor_sync(ALL_LANES, sum, 2);
+    lsum = lsum * corr + sum;
+    m = m_new;
+    __syncwarp();  // the four lanes of a row exchange probabilities
+#pragma unroll
+    for (int c = 0; c < VR; ++c) acc[c] *= corr;
+    for (int j = 0; j < KT; ++j) {
+      const float pr = ps[r * (KT + 1) + j];
+#pragma unroll
+      for (int c = 0; c < VR; ++c) {
+        const int col = c * 4 + sub;
+        if (col < l.vdimp) acc[c] = fmaf(pr, vs[j * l.vdimp + col], acc[c]);
+      }
+    }
+  }
+  if (!live) return;
+  const float inv = l.out_scale / lsum;
+#pragma unroll
+  for (int c = 0; c < VR; ++c) {
+    const int col = c * 4 + sub;
+    if (col < l.vdim) static_cast<T*>(a.y)[(size_t)(first + qrow) * a.ldy + head * l.vdim + col] = from_f32<T>(acc[c] * inv);
+  }
+}
+
+template <typename T>
+cudaError_t portion_t(const AttentionPortionArgs& a, cudaStream_t s) {
+  const AttentionLayer& l = a.l;
+  cudaError_t e;
+  const long long warps = (long long)a.rows * (l.heads + 2 * l.kv_heads);
+  const int pgrid = (int)std::min<long long>((warps + 7) / 8, 148 * 16);
+  if ((e = launch_kernel(attention_prep_kernel<T>, dim3(pgrid), dim3(256), 0, s, false, a)) != cudaSuccess) return e;
+  if (a.krows > a.rows) {
+    const int cgrid = std::min(a.krows - a.rows, 1024);
+    if ((e = launch_kernel(attention_context_kernel<T>, dim3(cgrid, a.nseq), dim3(128), 0, s, false, a)) != cudaSuccess) return e;
+  }
+  const dim3 grid((a.max_len + QT - 1) / QT, l.heads, a.nseq);
+  const size_t smem = ((size_t)(QT + KT) * (l.dimp + 1) + (size_t)KT * l.vdimp + (size_t)QT * (KT + 1)) * sizeof(float);
+#define PG_ROWS(VR_)                                                                                                        \
+  do {                                                                                                                      \
+    e = cudaFuncSetAttribute(attention_rows_kernel<T, VR_>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);       \
+    if (e == cudaSuccess) e = launch_kernel(attention_rows_kernel<T, VR_>, grid, dim3(128), smem, s, false, a);             \
+  } while (0)
+  if (l.vdimp <= 64) PG_ROWS(16);
+  else if (l.vdimp <= 128) PG_ROWS(32);
+  else PG_ROWS(64);
+#undef PG_ROWS
+  if (e != cudaSuccess) return e;
+  return launch_kernel(attention_store_kernel<T>, dim3(a.rows), dim3(128), 0, s, false, a);
+}
+
+size_t step_smem(const AttentionLayer& l) {
+  const int groups = STEP_THREADS / (l.vdimp / 8);
+  return ((size_t)(l.heads / l.kv_heads) * l.dimp + l.dimp + l.vdimp + RB * STEP_KEYS + (size_t)groups * RB * l.vdimp) * sizeof(float);
+}
+
+}  // namespace
+
+size_t attention_page_elems(const AttentionLayer& l) { return (size_t)l.kv_heads * l.page_tokens * (l.dimp + l.vdimp); }
+
+bool attention_supported(const AttentionLayer& l) { return step_smem(l) <= 200 * 1024; }
+
+cudaError_t launch_attention_step(const AttentionStepArgs& a, bool bf16, bool y_bf16, bool pdl, cudaStream_t s) {
+  const AttentionLayer& l = a.l;
+  const size_t smem = step_smem(l);
+  if (smem > 200 * 1024) return cudaErrorInvalidValue;
+  const dim3 grid(l.kv_heads, a.batch, a.splits);
+  const int yb = y_bf16 ? 1 : 0;
+  cudaError_t e;
+  if (bf16) {
+    e = cudaFuncSetAttribute(attention_step_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    return e != cudaSuccess ? e : launch_kernel(attention_step_kernel<__nv_bfloat16>, grid, dim3(STEP_THREADS), smem, s, pdl, a, yb);
+  }
+  e = cudaFuncSetAttribute(attention_step_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  return e != cudaSuccess ? e : launch_kernel(attention_step_kernel<float>, grid, dim3(STEP_THREADS), smem, s, pdl, a, yb);
+}
+
+cudaError_t launch_attention_portion(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
+  if (a.rows <= 0) return cudaSuccess;
+  return bf16 ? portion_t<__nv_bfloat16>(a, s) : portion_t<float>(a, s);
+}
+
+}  // namespace pg

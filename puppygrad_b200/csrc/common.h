@@ -29,6 +29,9 @@ struct Json {
 // Returns false and fills `err` on malformed input.
 bool parse_json(const char* data, size_t len, Json* out, std::string* err);
 
+// Whole file into `out`; false and `err` on failure.
+bool read_file(const std::string& path, std::vector<uint8_t>* out, std::string* err);
+
 // ---- safetensors container (the format of the `safetensors` crate, version 0.7.0) ----
 struct TensorEntry {
   std::string dtype;

@@ -203,7 +203,7 @@ bool parse_json(const char* data, size_t len, Json* out, std::string* err) {
 }
 
 // ------------------------------------------------------------------ safetensors
-static bool read_file(const std::string& path, std::vector<uint8_t>* out, std::string* err) {
+bool read_file(const std::string& path, std::vector<uint8_t>* out, std::string* err) {
   FILE* f = fopen(path.c_str(), "rb");
   if (!f) {
     *err = std::string(strerror(errno));

@@ -16,85 +16,93 @@
 #include <numeric>
 
 #include "common.h"
+#include "design.h"
 #include "kernels.cuh"
+#include "layered.h"
+#include "runtime.h"
 #include "sampler.h"
 
-namespace pg {
-
-#define PG_CUDA_TRY(expr)                                                                      \
-  do {                                                                                         \
-    cudaError_t _e = (expr);                                                                   \
-    if (_e != cudaSuccess)                                                                     \
-      return set_error(PG_CUDA, std::string("CUDA error: ") + cudaGetErrorString(_e) + " at " + \
-                                    __FILE__ + ":" + std::to_string(__LINE__) + " (" #expr ")"); \
-  } while (0)
-
-struct LayerWeights {
-  float *ln1_g, *ln1_b, *w_qkv, *b_qkv, *w_proj, *b_proj, *ln2_g, *ln2_b, *w_fc, *b_fc, *w_proj2, *b_proj2;
-  // copies in the tiled layout of the tensor-core decode kernel (nullptr in fp32 mode)
-  float *t_qkv = nullptr, *t_proj = nullptr, *t_fc = nullptr, *t_proj2 = nullptr;
-  // lo parts (w - hi(w), hi = the upper 19 bits a TF32 tensor core reads) of the four matrices, [out, in] row-major:
-  // second operand of the FP32-grade prefill GEMM (nullptr in fp32 mode)
-  float *l_qkv = nullptr, *l_proj = nullptr, *l_fc = nullptr, *l_proj2 = nullptr;
-  // packed copies for the single-kernel decode step (BF16 or row-quantised int8 weights), [out, in] rows, and,
-  // for int8, one scale per output row
-  void *p_qkv = nullptr, *p_proj = nullptr, *p_fc = nullptr, *p_proj2 = nullptr;
-  float *s_qkv = nullptr, *s_proj = nullptr, *s_fc = nullptr, *s_proj2 = nullptr;
-};
-
-static bool env_flag(const char* name) {
-  const char* v = getenv(name);
-  return v && *v && strcmp(v, "0") != 0;
+pg_model::~pg_model() {
+  if (arena) {
+    cudaSetDevice(device);
+    cudaFree(arena);
+    if (tiled_arena) cudaFree(tiled_arena);
+    if (lo_arena) cudaFree(lo_arena);
+    if (packed_arena) cudaFree(packed_arena);
+    if (scale_arena) cudaFree(scale_arena);
+    if (head_deq) cudaFree(head_deq);
+  }
 }
 
-}  // namespace pg
-
-using namespace pg;
-
-// ------------------------------------------------------------------ model
-struct pg_model {
-  pg_gpt2_config cfg{};
-  pg_backend_config backend{};
-  int device = 0;
-  int num_sms = 148;
-  float* arena = nullptr;  // every weight tensor lives in this one allocation
-  float* tiled_arena = nullptr;  // second copy of the dense matrices, tiled for TMA (tensor-core modes)
-  size_t tiled_floats = 0;
-  float* t_wte = nullptr;
-  float* lo_arena = nullptr;
-  size_t arena_floats = 0;
-  int stream_weight_type = STREAM_W_F32;  // what the single-kernel decode step streams
-  unsigned char* packed_arena = nullptr;  // BF16 / int8 copies of the dense matrices and of wte
-  float* scale_arena = nullptr;           // int8: row scales
-  void* p_wte = nullptr;
-  float* s_wte = nullptr;
-  float* head_w = nullptr;      // FP32 rows of the lm_head: wte itself, or (int8) its dequantised copy
-  float* head_deq = nullptr;    // owned storage of that copy
-  float *wte = nullptr, *wpe = nullptr, *lnf_g = nullptr, *lnf_b = nullptr;
-  std::vector<LayerWeights> layers;
-  bool fused_ok = false;  // LayerNorm/argmax fusion needs n_embd % 4 == 0 and n_embd <= 2048
-  bool use_pdl = true;
-
-  int c() const { return (int)cfg.n_embd; }
-  int f() const { return (int)cfg.n_inner; }
-  int v() const { return (int)cfg.vocab_size; }
-  int heads() const { return (int)cfg.n_head; }
-  int head_dim() const { return (int)(cfg.n_embd / cfg.n_head); }
-  int layers_n() const { return (int)cfg.n_layer; }
-  int positions() const { return (int)cfg.n_positions; }
-
-  ~pg_model() {
-    if (arena) {
-      cudaSetDevice(device);
-      cudaFree(arena);
-      if (tiled_arena) cudaFree(tiled_arena);
-      if (lo_arena) cudaFree(lo_arena);
-      if (packed_arena) cudaFree(packed_arena);
-      if (scale_arena) cudaFree(scale_arena);
-      if (head_deq) cudaFree(head_deq);
+pg_cache::~pg_cache() {
+  if (!model) return;
+  cudaSetDevice(model->device);
+  if (stream) cudaStreamSynchronize(stream);
+#ifdef PG_DEV_TRACE
+  if (d_stream_trace) {
+    const int L = model->layers_n();
+    std::vector<unsigned long long> t((size_t)2 * (L + 1) * 16 + 128);
+    if (cudaMemcpy(t.data(), d_stream_trace, t.size() * 8, cudaMemcpyDeviceToHost) == cudaSuccess) {
+      for (int cta = 0; cta < 2; ++cta)
+        for (int l = 0; l <= L; ++l) {
+          const unsigned long long* r = t.data() + ((size_t)cta * (L + 1) + l) * 16;
+          fprintf(stderr, "stream trace cta %d layer %2d:", cta ? 100 : 0, l);
+          for (int p = 1; p < 10; ++p) fprintf(stderr, " %6lld", r[p] ? (long long)(r[p] - r[p - 1]) : -1LL);
+          fprintf(stderr, "  | start %lld cycles\n", (long long)(r[0] - t[((size_t)cta * (L + 1)) * 16]));
+        }
+    }
+    cudaFree(d_stream_trace);
+  }
+#endif
+#ifdef PG_DEV_TRACE
+  if (d_chain_trace) {
+    std::vector<unsigned long long> t((size_t)chain_ctas * 32 + 512);
+    if (cudaMemcpy(t.data(), d_chain_trace, t.size() * 8, cudaMemcpyDeviceToHost) == cudaSuccess) {
+      unsigned long long t0 = ~0ULL;
+      for (int i = 0; i < chain_ctas; ++i) t0 = std::min(t0, t[(size_t)i * 32 + 31]);
+      for (int sl = 0; sl < 10; ++sl) {
+        unsigned long long lo = ~0ULL, hi = 0, wlo = ~0ULL, whi = 0;
+        for (int i = 0; i < chain_ctas; ++i) {
+          const unsigned long long v = t[(size_t)i * 32 + sl] - t0, w = t[(size_t)i * 32 + 10 + sl] - t0;
+          lo = std::min(lo, v); hi = std::max(hi, v); wlo = std::min(wlo, w); whi = std::max(whi, w);
+        }
+        fprintf(stderr, "chain trace phase %d: work done %6llu..%6llu ns, barrier passed %6llu..%6llu ns\n", sl, wlo, whi, lo, hi);
+      }
+      // the lm_head of the last step: per CTA its SM and the time its share took; then CTA 0's units (see unit_trace)
+      for (int i = 0; i < chain_ctas; ++i) {
+        const unsigned long long* r = t.data() + (size_t)i * 32;
+        fprintf(stderr, "chain trace lm_head cta %3d sm %3llu work %7lld ns\n", i, r[22], (long long)(r[21] - r[20]));
+      }
+      const unsigned long long* u = t.data() + (size_t)chain_ctas * 32;
+      for (int i = 0; i < 48; ++i) {
+        fprintf(stderr, "chain trace unit %2d:", i);
+        for (int e = 0; e < 8; ++e) fprintf(stderr, " %7lld", u[i * 8 + e] ? (long long)(u[i * 8 + e] - u[0]) : -1LL);
+        fprintf(stderr, "\n");
+      }
     }
   }
-};
+#endif
+  for (auto& cp : chain_programs) {
+    if (cp.second.dev) cudaFree(cp.second.dev);
+    if (cp.second.dev_argmax_only) cudaFree(cp.second.dev_argmax_only);
+    if (cp.second.d_times) cudaFree(cp.second.d_times);
+  }
+  for (auto& g : graphs) cudaGraphExecDestroy(g.second);
+  for (auto& t : tables)
+    if (t.d_table) cudaFree(t.d_table);
+  for (void* p : {(void*)kv_pool, (void*)d_ids, (void*)d_pos, (void*)d_argmax, (void*)d_token_log,
+                  (void*)x, (void*)norm, (void*)qkv, (void*)attn, (void*)hbuf, (void*)logits, (void*)part_val,
+                  (void*)part_idx, (void*)attn_part, (void*)attn_counters, (void*)topk_vals, (void*)topk_idx,
+                  (void*)px, (void*)pnorm, (void*)pqkv, (void*)pattn, (void*)ph, (void*)plo, (void*)prow, (void*)norm_lo,
+                  (void*)attn_lo, (void*)h_lo, (void*)d_error, (void*)d_stream_ll, (void*)d_stream_epoch,
+                  (void*)chain_partials, (void*)d_chain_barrier, (void*)d_chain_trace, (void*)d_chain_best})
+    if (p) cudaFree(p);
+  if (t0) cudaEventDestroy(t0);
+  if (t1) cudaEventDestroy(t1);
+  if (h_ids) cudaFreeHost(h_ids);
+  if (h_out) cudaFreeHost(h_out);
+  if (stream) cudaStreamDestroy(stream);
+}
 
 namespace pg {
 
@@ -305,148 +313,27 @@ static int build_model(const pg_gpt2_config& cfg, const float* const* tensors, c
 
 }  // namespace pg
 
-// ------------------------------------------------------------------ cache
-struct pg_cache {
-  const pg_model* model = nullptr;
-  int max_batch = 0;
-  cudaStream_t stream = nullptr;
-  KvLayout kv{};
-  size_t page_floats = 0;  // floats of one page of one layer
-  int num_pages = 0;
-  float* kv_pool = nullptr;  // [layer][page][2][head][page_tokens][head_dim]
-  std::vector<int> free_pages;
-  std::vector<int> h_table;    // [max_batch][pages_per_seq], -1 = unassigned
-  std::vector<int> seq_len;    // host mirror of d_pos
-  int* d_table = nullptr;
-  bool table_dirty = true;
-  int *d_ids = nullptr, *d_pos = nullptr, *d_argmax = nullptr, *d_token_log = nullptr;
-  float *x = nullptr, *norm = nullptr, *qkv = nullptr, *attn = nullptr, *hbuf = nullptr, *logits = nullptr;
-  float* part_val = nullptr;
-  int* part_idx = nullptr;
-  int part_stride = 0;
-  float* attn_part = nullptr;
-  unsigned* attn_counters = nullptr;
-  float* topk_vals = nullptr;
-  int* topk_idx = nullptr;
-  // tensor-core decode path (9..64 sequences): TF32 hi/lo pairs of the GEMM inputs, split-K scratch
-  float *norm_lo = nullptr, *attn_lo = nullptr, *h_lo = nullptr;
-  int* d_error = nullptr;
-  // persistent chain kernel of the tensor-core decode path: partial tiles, grid-barrier word
-  float* chain_partials = nullptr;
-  unsigned* d_chain_barrier = nullptr;
-  unsigned long long* d_chain_best = nullptr;  // row arg-max accumulators of the lm_head phase
-  unsigned long long* d_chain_trace = nullptr;  // developer aid: only allocated in builds with -DPG_DEV_TRACE
-  int chain_ctas = 0;
-  int chain_min_batch = 9;  // smallest batch whose decode step runs as the chain kernel in the tensor-core modes (measured on
-                            // B200, GPT-2 medium, 8 sequences: 1.34 ms as the chain kernel, 1.09 ms as one kernel per operation)
-  struct ChainProgram {  // whole-step phase list of the persistent chain kernel for one batch size
-    ChainPhase* dev = nullptr;            // in device memory (nullptr: this batch size is not supported)
-    ChainPhase* dev_argmax_only = nullptr;  // the same list whose lm_head reduce phase keeps the row arg-max but stores no logits
-    int n = 0;
-    std::vector<int> bucket;              // profile bucket of every phase
-    unsigned long long* d_times = nullptr;  // n + 1 time stamps, written in profiling runs
-  };
-  std::map<int, ChainProgram> chain_programs;
-  bool step_wants_logits = true;  // false: the caller of this step only reads the arg-max (greedy decoding)
-  // single-kernel decode step (at most 8 sequences): layer table, tagged exchange buffers, tag counter
-  unsigned long long* d_stream_ll = nullptr;  // ll_x | ll_qkv | ll_attn | ll_h | ll_part | ll_best
-  unsigned* d_stream_epoch = nullptr;
-  int stream_grid = 0;
-  unsigned dbg_spin_limit = 0, dbg_poison = 0;  // pg_cache_debug_expire_next_wait: consumed by the next decode step
-#ifdef PG_DEV_TRACE
-  unsigned long long* d_stream_trace = nullptr;
-#endif
-  int *h_ids = nullptr, *h_out = nullptr;  // pinned staging
-  // prefill workspace (grow-only)
-  size_t pre_rows = 0;
-  float *px = nullptr, *pnorm = nullptr, *pqkv = nullptr, *pattn = nullptr, *ph = nullptr, *plo = nullptr;
-  int* prow = nullptr;  // [4][pre_rows]: ids, pos, slot, (batch+1 seq_start / last rows)
-  std::map<std::pair<int, int>, cudaGraphExec_t> graphs;  // (batch, splits) -> decode-step graph
-  std::map<std::pair<int, int>, uint64_t> graphs_launches;  // kernel nodes in each graph
-  uint64_t decode_launches = 0;  // kernels launched by decode steps (for gpu_launches accounting)
-  cudaEvent_t t0 = nullptr, t1 = nullptr;  // pg_cache_time_begin / pg_cache_time_end
-
-  float* layer_pool(int l) const { return kv_pool + (size_t)l * num_pages * page_floats; }
-
-  ~pg_cache() {
-    if (!model) return;
-    cudaSetDevice(model->device);
-    if (stream) cudaStreamSynchronize(stream);
-#ifdef PG_DEV_TRACE
-    if (d_stream_trace) {
-      const int L = model->layers_n();
-      std::vector<unsigned long long> t((size_t)2 * (L + 1) * 16 + 128);
-      if (cudaMemcpy(t.data(), d_stream_trace, t.size() * 8, cudaMemcpyDeviceToHost) == cudaSuccess) {
-        for (int cta = 0; cta < 2; ++cta)
-          for (int l = 0; l <= L; ++l) {
-            const unsigned long long* r = t.data() + ((size_t)cta * (L + 1) + l) * 16;
-            fprintf(stderr, "stream trace cta %d layer %2d:", cta ? 100 : 0, l);
-            for (int p = 1; p < 10; ++p) fprintf(stderr, " %6lld", r[p] ? (long long)(r[p] - r[p - 1]) : -1LL);
-            fprintf(stderr, "  | start %lld cycles\n", (long long)(r[0] - t[((size_t)cta * (L + 1)) * 16]));
-          }
-      }
-      cudaFree(d_stream_trace);
-    }
-#endif
-#ifdef PG_DEV_TRACE
-    if (d_chain_trace) {
-      std::vector<unsigned long long> t((size_t)chain_ctas * 32 + 512);
-      if (cudaMemcpy(t.data(), d_chain_trace, t.size() * 8, cudaMemcpyDeviceToHost) == cudaSuccess) {
-        unsigned long long t0 = ~0ULL;
-        for (int i = 0; i < chain_ctas; ++i) t0 = std::min(t0, t[(size_t)i * 32 + 31]);
-        for (int sl = 0; sl < 10; ++sl) {
-          unsigned long long lo = ~0ULL, hi = 0, wlo = ~0ULL, whi = 0;
-          for (int i = 0; i < chain_ctas; ++i) {
-            const unsigned long long v = t[(size_t)i * 32 + sl] - t0, w = t[(size_t)i * 32 + 10 + sl] - t0;
-            lo = std::min(lo, v); hi = std::max(hi, v); wlo = std::min(wlo, w); whi = std::max(whi, w);
-          }
-          fprintf(stderr, "chain trace phase %d: work done %6llu..%6llu ns, barrier passed %6llu..%6llu ns\n", sl, wlo, whi, lo, hi);
-        }
-        // the lm_head of the last step: per CTA its SM and the time its share took; then CTA 0's units (see unit_trace)
-        for (int i = 0; i < chain_ctas; ++i) {
-          const unsigned long long* r = t.data() + (size_t)i * 32;
-          fprintf(stderr, "chain trace lm_head cta %3d sm %3llu work %7lld ns\n", i, r[22], (long long)(r[21] - r[20]));
-        }
-        const unsigned long long* u = t.data() + (size_t)chain_ctas * 32;
-        for (int i = 0; i < 48; ++i) {
-          fprintf(stderr, "chain trace unit %2d:", i);
-          for (int e = 0; e < 8; ++e) fprintf(stderr, " %7lld", u[i * 8 + e] ? (long long)(u[i * 8 + e] - u[0]) : -1LL);
-          fprintf(stderr, "\n");
-        }
-      }
-    }
-#endif
-    for (auto& cp : chain_programs) {
-      if (cp.second.dev) cudaFree(cp.second.dev);
-      if (cp.second.dev_argmax_only) cudaFree(cp.second.dev_argmax_only);
-      if (cp.second.d_times) cudaFree(cp.second.d_times);
-    }
-    for (auto& g : graphs) cudaGraphExecDestroy(g.second);
-    for (void* p : {(void*)kv_pool, (void*)d_table, (void*)d_ids, (void*)d_pos, (void*)d_argmax, (void*)d_token_log,
-                    (void*)x, (void*)norm, (void*)qkv, (void*)attn, (void*)hbuf, (void*)logits, (void*)part_val,
-                    (void*)part_idx, (void*)attn_part, (void*)attn_counters, (void*)topk_vals, (void*)topk_idx,
-                    (void*)px, (void*)pnorm, (void*)pqkv, (void*)pattn, (void*)ph, (void*)plo, (void*)prow, (void*)norm_lo,
-                    (void*)attn_lo, (void*)h_lo, (void*)d_error, (void*)d_stream_ll, (void*)d_stream_epoch,
-                    (void*)chain_partials, (void*)d_chain_barrier, (void*)d_chain_trace, (void*)d_chain_best})
-      if (p) cudaFree(p);
-    if (t0) cudaEventDestroy(t0);
-    if (t1) cudaEventDestroy(t1);
-    if (h_ids) cudaFreeHost(h_ids);
-    if (h_out) cudaFreeHost(h_out);
-    if (stream) cudaStreamDestroy(stream);
-  }
-};
-
 namespace pg {
-
-constexpr int MAX_SPLITS = 16;
-constexpr int MAX_TOPK = 64;
 
 // Words of the tagged exchange buffers of the single-kernel decode step, in the order
 // ll_x [8][C], ll_qkv [8][3C], ll_attn [8][C], ll_h [8][F], ll_part [8 * H][8][66], ll_best [8][grid][2].
 static size_t stream_ll_words(const pg_model* m, int grid) {
   const size_t C = m->c(), F = m->f(), H = m->heads();
   return 8 * (C + 3 * C + C + F) + 8 * H * 8 * 66 + 8 * (size_t)grid * 2;
+}
+
+int page_table_init(PageTable* t, int max_batch, int span, int page_tokens, cudaStream_t s) {
+  t->span = span;
+  t->page_tokens = page_tokens;
+  t->pages_per_seq = (span + page_tokens - 1) / page_tokens;
+  t->num_pages = max_batch * t->pages_per_seq;
+  t->free_pages.resize(t->num_pages);
+  for (int i = 0; i < t->num_pages; ++i) t->free_pages[i] = t->num_pages - 1 - i;  // pop_back hands out page 0 first
+  t->h_table.assign((size_t)t->num_pages, -1);
+  PG_CUDA_TRY(cudaMalloc(&t->d_table, (size_t)t->num_pages * sizeof(int)));
+  PG_CUDA_TRY(cudaMemsetAsync(t->d_table, 0, (size_t)t->num_pages * sizeof(int), s));
+  t->dirty = true;
+  return PG_OK;
 }
 
 static int cache_new(const pg_model* m, int max_batch, pg_cache** out) {
@@ -457,20 +344,10 @@ static int cache_new(const pg_model* m, int max_batch, pg_cache** out) {
   c->model = m;
   c->max_batch = max_batch;
   const int C = m->c(), F = m->f(), V = m->v(), P = m->positions(), H = m->heads(), D = m->head_dim();
-  c->kv = KvLayout{H, D, m->backend.page_tokens, (P + m->backend.page_tokens - 1) / m->backend.page_tokens};
-  c->page_floats = (size_t)2 * H * c->kv.page_tokens * D;
-  c->num_pages = max_batch * c->kv.pages_per_seq;
   PG_CUDA_TRY(cudaStreamCreateWithFlags(&c->stream, cudaStreamNonBlocking));
   const size_t B = (size_t)max_batch;
-  PG_CUDA_TRY(cudaMalloc(&c->kv_pool, (size_t)m->layers_n() * c->num_pages * c->page_floats * sizeof(float)));
-  // KV pages start zeroed like the reference's vec![0.0; len] (rust.rs:258-266)
-  PG_CUDA_TRY(cudaMemsetAsync(c->kv_pool, 0, (size_t)m->layers_n() * c->num_pages * c->page_floats * sizeof(float), c->stream));
-  c->free_pages.resize(c->num_pages);
-  for (int i = 0; i < c->num_pages; ++i) c->free_pages[i] = c->num_pages - 1 - i;  // pop_back hands out page 0 first
-  c->h_table.assign(B * c->kv.pages_per_seq, -1);
+  // step state every family has: token ids and positions of the slots, results, pinned staging
   c->seq_len.assign(B, 0);
-  PG_CUDA_TRY(cudaMalloc(&c->d_table, B * c->kv.pages_per_seq * sizeof(int)));
-  PG_CUDA_TRY(cudaMemsetAsync(c->d_table, 0, B * c->kv.pages_per_seq * sizeof(int), c->stream));
   PG_CUDA_TRY(cudaMalloc(&c->d_ids, B * sizeof(int)));
   PG_CUDA_TRY(cudaMalloc(&c->d_pos, B * sizeof(int)));
   PG_CUDA_TRY(cudaMalloc(&c->d_argmax, B * sizeof(int)));
@@ -478,22 +355,38 @@ static int cache_new(const pg_model* m, int max_batch, pg_cache** out) {
   PG_CUDA_TRY(cudaMemsetAsync(c->d_ids, 0, B * sizeof(int), c->stream));
   PG_CUDA_TRY(cudaMemsetAsync(c->d_pos, 0, B * sizeof(int), c->stream));
   PG_CUDA_TRY(cudaMemsetAsync(c->d_token_log, 0, B * P * sizeof(int), c->stream));
+  PG_CUDA_TRY(cudaMalloc(&c->logits, B * V * sizeof(float)));
+  c->part_stride = linear_decode_grid(V, m->num_sms);
+  PG_CUDA_TRY(cudaMalloc(&c->part_val, B * c->part_stride * sizeof(float)));
+  PG_CUDA_TRY(cudaMalloc(&c->part_idx, B * c->part_stride * sizeof(int)));
+  PG_CUDA_TRY(cudaMalloc(&c->topk_vals, B * MAX_TOPK * sizeof(float)));
+  PG_CUDA_TRY(cudaMalloc(&c->topk_idx, B * MAX_TOPK * sizeof(int)));
+  PG_CUDA_TRY(cudaMalloc(&c->d_error, sizeof(int)));
+  PG_CUDA_TRY(cudaMemsetAsync(c->d_error, 0, sizeof(int), c->stream));
+  PG_CUDA_TRY(cudaMallocHost(&c->h_ids, B * sizeof(int)));
+  PG_CUDA_TRY(cudaMallocHost(&c->h_out, (B * (1 + 2 * MAX_TOPK) + 1) * sizeof(int)));
+  if (m->layered) {
+    if (int r = layered_cache_init(c.get())) return r;
+    PG_CUDA_TRY(cudaStreamSynchronize(c->stream));
+    *out = c.release();
+    return PG_OK;
+  }
+  c->tables.resize(1);
+  if (int r = page_table_init(&c->tables[0], max_batch, P, m->backend.page_tokens, c->stream)) return r;
+  c->kv = KvLayout{H, D, m->backend.page_tokens, c->tables[0].pages_per_seq};
+  c->page_floats = (size_t)2 * H * c->kv.page_tokens * D;
+  const size_t kv_floats = (size_t)m->layers_n() * c->tables[0].num_pages * c->page_floats;
+  PG_CUDA_TRY(cudaMalloc(&c->kv_pool, kv_floats * sizeof(float)));
+  // KV pages start zeroed like the reference's vec![0.0; len] (rust.rs:258-266)
+  PG_CUDA_TRY(cudaMemsetAsync(c->kv_pool, 0, kv_floats * sizeof(float), c->stream));
   PG_CUDA_TRY(cudaMalloc(&c->x, B * C * sizeof(float)));
   PG_CUDA_TRY(cudaMalloc(&c->norm, B * std::max(C, 4) * sizeof(float)));
   PG_CUDA_TRY(cudaMalloc(&c->qkv, B * 3 * C * sizeof(float)));
   PG_CUDA_TRY(cudaMalloc(&c->attn, B * C * sizeof(float)));
   PG_CUDA_TRY(cudaMalloc(&c->hbuf, B * F * sizeof(float)));
-  PG_CUDA_TRY(cudaMalloc(&c->logits, B * V * sizeof(float)));
-  c->part_stride = linear_decode_grid(V, m->num_sms);
-  PG_CUDA_TRY(cudaMalloc(&c->part_val, B * c->part_stride * sizeof(float)));
-  PG_CUDA_TRY(cudaMalloc(&c->part_idx, B * c->part_stride * sizeof(int)));
   PG_CUDA_TRY(cudaMalloc(&c->attn_part, B * H * MAX_SPLITS * (D + 2) * sizeof(float)));
   PG_CUDA_TRY(cudaMalloc(&c->attn_counters, B * H * sizeof(unsigned)));
   PG_CUDA_TRY(cudaMemsetAsync(c->attn_counters, 0, B * H * sizeof(unsigned), c->stream));
-  PG_CUDA_TRY(cudaMalloc(&c->topk_vals, B * MAX_TOPK * sizeof(float)));
-  PG_CUDA_TRY(cudaMalloc(&c->topk_idx, B * MAX_TOPK * sizeof(int)));
-  PG_CUDA_TRY(cudaMalloc(&c->d_error, sizeof(int)));
-  PG_CUDA_TRY(cudaMemsetAsync(c->d_error, 0, sizeof(int), c->stream));
   if (const char* e = getenv("PG_CHAIN_MIN_BATCH")) c->chain_min_batch = std::max(1, std::min(65, atoi(e)));
   if (max_batch >= c->chain_min_batch && C % 32 == 0 && F % 32 == 0) {
     const int bmax = std::min(max_batch, 64);
@@ -533,50 +426,55 @@ static int cache_new(const pg_model* m, int max_batch, pg_cache** out) {
 #endif
     }
   }
-  PG_CUDA_TRY(cudaMallocHost(&c->h_ids, B * sizeof(int)));
-  PG_CUDA_TRY(cudaMallocHost(&c->h_out, (B * (1 + 2 * MAX_TOPK) + 1) * sizeof(int)));
   PG_CUDA_TRY(cudaStreamSynchronize(c->stream));
   *out = c.release();
   return PG_OK;
 }
 
 static void release_slot_pages(pg_cache* c, int slot) {
-  int* row = c->h_table.data() + (size_t)slot * c->kv.pages_per_seq;
-  for (int p = c->kv.pages_per_seq - 1; p >= 0; --p)
-    if (row[p] >= 0) {
-      c->free_pages.push_back(row[p]);
-      row[p] = -1;
-      c->table_dirty = true;
-    }
+  for (PageTable& t : c->tables) {
+    int* row = t.h_table.data() + (size_t)slot * t.pages_per_seq;
+    for (int p = t.pages_per_seq - 1; p >= 0; --p)
+      if (row[p] >= 0) {
+        t.free_pages.push_back(row[p]);
+        row[p] = -1;
+        t.dirty = true;
+      }
+  }
 }
 
-// Makes sure slot `slot` owns pages for positions [0, upto).
+// Makes sure slot `slot` owns pages for positions [0, upto) (for a table with a shorter span: for the indices they map to).
 static int ensure_pages(pg_cache* c, int slot, int upto) {
-  int need = (upto + c->kv.page_tokens - 1) / c->kv.page_tokens;
-  int* row = c->h_table.data() + (size_t)slot * c->kv.pages_per_seq;
-  for (int p = 0; p < need; ++p)
-    if (row[p] < 0) {
-      if (c->free_pages.empty()) return set_error(PG_INVALID_INPUT, "KV page pool exhausted");
-      row[p] = c->free_pages.back();
-      c->free_pages.pop_back();
-      c->table_dirty = true;
-    }
+  for (PageTable& t : c->tables) {
+    int need = (std::min(upto, t.span) + t.page_tokens - 1) / t.page_tokens;
+    int* row = t.h_table.data() + (size_t)slot * t.pages_per_seq;
+    for (int p = 0; p < need; ++p)
+      if (row[p] < 0) {
+        if (t.free_pages.empty()) return set_error(PG_INVALID_INPUT, "KV page pool exhausted");
+        row[p] = t.free_pages.back();
+        t.free_pages.pop_back();
+        t.dirty = true;
+      }
+  }
   return PG_OK;
 }
 
 static int sync_table(pg_cache* c) {
-  if (!c->table_dirty) return PG_OK;
-  // unassigned entries are uploaded as page 0; kernels never index past a slot's seq_len
-  std::vector<int> up(c->h_table.size());
-  for (size_t i = 0; i < up.size(); ++i) up[i] = std::max(c->h_table[i], 0);
-  PG_CUDA_TRY(cudaMemcpyAsync(c->d_table, up.data(), up.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
-  PG_CUDA_TRY(cudaStreamSynchronize(c->stream));  // `up` is a pageable temporary
-  c->table_dirty = false;
+  for (PageTable& t : c->tables) {
+    if (!t.dirty) continue;
+    // unassigned entries are uploaded as page 0; kernels never index past a slot's seq_len
+    std::vector<int> up(t.h_table.size());
+    for (size_t i = 0; i < up.size(); ++i) up[i] = std::max(t.h_table[i], 0);
+    PG_CUDA_TRY(cudaMemcpyAsync(t.d_table, up.data(), up.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
+    PG_CUDA_TRY(cudaStreamSynchronize(c->stream));  // `up` is a pageable temporary
+    t.dirty = false;
+  }
   return PG_OK;
 }
 
 static int choose_splits(const pg_cache* c, int batch, int max_len) {
   const pg_model* m = c->model;
+  if (m->layered) return layered_choose_splits(c, batch, max_len);
   if (m->head_dim() != 64) return 1;
   if (m->backend.attn_splits > 0) return std::min(m->backend.attn_splits, MAX_SPLITS);
   // enough CTAs to cover the SMs twice, but at least 128 keys per split
@@ -585,26 +483,6 @@ static int choose_splits(const pg_cache* c, int batch, int max_len) {
   int s = std::max(1, std::min(std::min(by_fill, by_len), 8));
   return s;
 }
-
-// Per-operation device timing of one decode step: the buckets of Gpt2OperationProfile
-// (rust.rs:336-347). Events around every launch serialise the step, so this is a profiling mode.
-enum Bucket { B_LAYER_NORM = 0, B_QKV, B_ATTN, B_ATTN_PROJ, B_MLP_FC, B_MLP_PROJ, B_LOGITS, B_OTHER, B_COUNT };
-struct StepProfiler {
-  std::vector<cudaEvent_t> ev;
-  std::vector<int> bucket;
-  int chain_event = -1;  // index of the event pair around the persistent chain kernel, if it ran
-  cudaError_t mark(cudaStream_t s, int b) {
-    cudaEvent_t e;
-    cudaError_t r = cudaEventCreate(&e);
-    if (r != cudaSuccess) return r;
-    ev.push_back(e);
-    bucket.push_back(b);
-    return cudaEventRecord(e, s);
-  }
-  ~StepProfiler() {
-    for (auto e : ev) cudaEventDestroy(e);
-  }
-};
 
 // Arguments of the chain kernel for `batch` sequences starting at slot 64 * chunk (steps of more than 64
 // sequences run as one launch per 64: the activation buffers are reused, what belongs to a slot is offset).
@@ -618,7 +496,7 @@ static ChainArgs chain_base_args(const pg_cache* c, int batch, int chunk = 0) {
   base.act_hi[CH_ACT_H] = c->hbuf; base.act_lo[CH_ACT_H] = c->h_lo; base.act_k[CH_ACT_H] = m->f();
   base.partials = c->chain_partials; base.barrier = c->d_chain_barrier; base.error_flag = c->d_error;
   base.trace = c->d_chain_trace;
-  base.kv = c->kv; base.page_table = c->d_table + s0 * c->kv.pages_per_seq; base.pos = c->d_pos + s0;
+  base.kv = c->kv; base.page_table = c->tables[0].d_table + s0 * c->kv.pages_per_seq; base.pos = c->d_pos + s0;
   base.wte = m->wte; base.wpe = m->wpe; base.ids = c->d_ids + s0; base.pos_rw = c->d_pos + s0;
   base.argmax_out = c->d_argmax + s0;
   base.token_log = c->d_token_log + s0 * m->positions(); base.n_positions = m->positions(); base.best = c->d_chain_best;
@@ -741,6 +619,7 @@ static int ensure_chain_programs(pg_cache* c, int batch) {
 // forward_one_profiled_with_scratch + block_forward_one_profiled (rust.rs:943-1006, 1136-1250).
 static cudaError_t enqueue_decode_step(pg_cache* c, int batch, int splits, cudaStream_t s, uint64_t* launches,
                                        StepProfiler* prof = nullptr) {
+  if (c->model->layered) return layered_enqueue_decode(c, batch, splits, s, launches, prof);
   // FP32 weights: the single-kernel step wins up to 4 sequences (measured on B200: 279 against 306 us for one GPT-2
   // small sequence, 1014 against 1168 us for four GPT-2 medium ones; at eight it loses, 1806 against 1548 us);
   // packed weights (BF16, int8) are only read by that kernel
@@ -770,13 +649,13 @@ static cudaError_t enqueue_decode_step(pg_cache* c, int batch, int splits, cudaS
     a.bias[0] = w0.b_qkv; a.bias[1] = w0.b_proj; a.bias[2] = w0.b_fc; a.bias[3] = w0.b_proj2;
     a.ln_g[0] = w0.ln1_g; a.ln_g[1] = w0.ln2_g; a.ln_b[0] = w0.ln1_b; a.ln_b[1] = w0.ln2_b;
     a.p_stride = w1.b_qkv - w0.b_qkv;
-    a.kv_pool = c->layer_pool(0); a.kv_stride = (long long)c->num_pages * (long long)c->page_floats;
+    a.kv_pool = c->layer_pool(0); a.kv_stride = (long long)c->tables[0].num_pages * (long long)c->page_floats;
     a.wte = m->wte; a.wpe = m->wpe; a.lnf_g = m->lnf_g; a.lnf_b = m->lnf_b;
     a.n_layer = m->layers_n(); a.c = m->c(); a.f = m->f(); a.v = m->v(); a.n_positions = m->positions();
     a.eps = m->cfg.layer_norm_epsilon;
     a.ids = c->d_ids; a.pos = c->d_pos; a.argmax = c->d_argmax; a.token_log = c->d_token_log;
     a.logits = c->step_wants_logits ? c->logits : nullptr;
-    a.page_table = c->d_table; a.kv = c->kv;
+    a.page_table = c->tables[0].d_table; a.kv = c->kv;
     a.ll_x = c->d_stream_ll; a.ll_qkv = a.ll_x + 8 * C; a.ll_attn = a.ll_qkv + 8 * 3 * C; a.ll_h = a.ll_attn + 8 * C;
     a.ll_part = a.ll_h + 8 * F; a.ll_best = a.ll_part + 8 * H * 8 * 66;
     a.epoch = c->d_stream_epoch; a.error_flag = c->d_error;
@@ -862,7 +741,7 @@ static cudaError_t enqueue_decode_step(pg_cache* c, int batch, int splits, cudaS
       cur_bucket = B_ATTN;
       DecodeAttnArgs at{};
       at.qkv = c->qkv; at.out = c->attn; at.out_lo = c->attn_lo; at.kv_pool = c->layer_pool(l);
-      at.page_table = c->d_table; at.pos = c->d_pos; at.part = c->attn_part; at.counters = c->attn_counters;
+      at.page_table = c->tables[0].d_table; at.pos = c->d_pos; at.part = c->attn_part; at.counters = c->attn_counters;
       at.kv = c->kv; at.batch = batch; at.splits = splits;
       PG_E(launch_decode_attention(at, pdl, s));
       cur_bucket = B_ATTN_PROJ;
@@ -909,7 +788,7 @@ static cudaError_t enqueue_decode_step(pg_cache* c, int batch, int splits, cudaS
     PG_E(linear(w.w_qkv, w.b_qkv, c->x, c->qkv, 3 * C, C, EPI_NONE, nullptr, w.ln1_g, w.ln1_b));
     cur_bucket = B_ATTN;
     DecodeAttnArgs at{};
-    at.qkv = c->qkv; at.out = c->attn; at.kv_pool = c->layer_pool(l); at.page_table = c->d_table;
+    at.qkv = c->qkv; at.out = c->attn; at.kv_pool = c->layer_pool(l); at.page_table = c->tables[0].d_table;
     at.pos = c->d_pos; at.part = c->attn_part; at.counters = c->attn_counters; at.kv = c->kv;
     at.batch = batch; at.splits = splits;
     PG_E(launch_decode_attention(at, pdl, s));
@@ -1062,7 +941,7 @@ static int run_blocks(const pg_model* m, const BlockWorkspace& ws, const Prefill
     PG_CUDA_TRY(launch_layernorm_rows(ws.x, w.ln1_g, w.ln1_b, eps, ws.norm, rows, C, false, s, lo_c));
     PG_CUDA_TRY(gemm(w.w_qkv, w.l_qkv, w.b_qkv, ws.norm, lo_c, ws.qkv, nullptr, 3 * C, C, EPI_NONE, nullptr));
     if (cache)
-      PG_CUDA_TRY(launch_kv_scatter(ws.qkv, ws.d_slot, ws.d_pos, cache->layer_pool(l), cache->d_table, cache->kv,
+      PG_CUDA_TRY(launch_kv_scatter(ws.qkv, ws.d_slot, ws.d_pos, cache->layer_pool(l), cache->tables[0].d_table, cache->kv,
                                     rows, s));
     PrefillAttnArgs pa{};
     pa.qkv = ws.qkv; pa.out = ws.attn; pa.seq_start = ws.d_seq_start;
@@ -1129,7 +1008,7 @@ static int recover_after_timeout(pg_cache* c, int code) {
     const std::vector<unsigned long long> init(64, chain_argmax_init());
     cudaMemcpyAsync(c->d_chain_best, init.data(), init.size() * sizeof(unsigned long long), cudaMemcpyHostToDevice, c->stream);
   }
-  cudaMemsetAsync(c->attn_counters, 0, (size_t)c->max_batch * c->model->heads() * sizeof(unsigned), c->stream);
+  if (c->attn_counters) cudaMemsetAsync(c->attn_counters, 0, (size_t)c->max_batch * c->model->heads() * sizeof(unsigned), c->stream);
   if (c->d_stream_epoch) {
     // tags of the failed step may sit in the exchange buffers: move the counter far past them
     unsigned e = 0;
@@ -1178,9 +1057,94 @@ static int fetch_outputs(pg_cache* c, int batch, float* logits_out, int32_t* arg
   return PG_OK;
 }
 
+static int prepare_step(const pg_model* m, pg_cache* c, const int32_t* ids, int batch);
+static int do_forward_one(const pg_model* m, pg_cache* c, const int32_t* ids, int batch, float* logits_out,
+                          int32_t* argmax_out, float* topk_vals, int32_t* topk_idx, int k);
+
+// What a portion pass brings back to the host: logits of the wanted rows (plan.out_rows up to n_want), and of the last
+// row of every sequence (left in c->logits, with the arg-max, as after a decode step).
+static int run_layered_portions(const pg_model* m, pg_cache* c, PortionPlan& plan, const int32_t* want, int n_want, float* want_logits,
+                                bool need_last, StepProfiler* prof) {
+  const int V = m->v(), n = plan.n();
+  PG_CUDA_TRY(cudaSetDevice(m->device));
+  for (int i = 0; i < n; ++i)
+    if (int r = ensure_pages(c, plan.slot[i], plan.start_pos[i] + plan.seq_start[i + 1] - plan.seq_start[i])) return r;
+  if (int r = sync_table(c)) return r;
+  plan.out_rows.assign(want, want + n_want);
+  if (need_last)
+    for (int i = 0; i < n; ++i) plan.out_rows.push_back(plan.seq_start[i + 1] - 1);
+  float* logits = nullptr;
+  if (!plan.out_rows.empty())
+    if (int r = layered_logits_buffer(c, plan.out_rows.size(), &logits)) return r;
+  if (int r = layered_run_portions(c, plan, logits, prof)) return r;
+  cudaStream_t s = c->stream;
+  if (need_last) {
+    PG_CUDA_TRY(cudaMemcpyAsync(c->logits, logits + (size_t)n_want * V, (size_t)n * V * sizeof(float), cudaMemcpyDeviceToDevice, s));
+    PG_CUDA_TRY(launch_argmax_rows(c->logits, n, V, c->d_argmax, s));
+  }
+  if (n_want && want_logits)
+    PG_CUDA_TRY(cudaMemcpyAsync(want_logits, logits, (size_t)n_want * V * sizeof(float), cudaMemcpyDeviceToHost, s));
+  std::vector<int> pos(n);
+  for (int i = 0; i < n; ++i) {
+    pos[i] = plan.start_pos[i] + plan.seq_start[i + 1] - plan.seq_start[i];
+    PG_CUDA_TRY(cudaMemcpyAsync(c->d_pos + plan.slot[i], &pos[i], sizeof(int), cudaMemcpyHostToDevice, s));
+    if (need_last)  // the next id of the slot, should a greedy step follow without ids
+      PG_CUDA_TRY(cudaMemcpyAsync(c->d_ids + plan.slot[i], c->d_argmax + i, sizeof(int), cudaMemcpyDeviceToDevice, s));
+  }
+  if (int r = check_device_error(c)) return r;  // waits for the stream
+  for (int i = 0; i < n; ++i) c->seq_len[plan.slot[i]] = pos[i];
+  return PG_OK;
+}
+
+// Portions for slots[i] (nullptr: slots 0..n-1), appended to what the slots hold.
+static int make_plan(const pg_model* m, const pg_cache* c, const int32_t* slots, const int32_t* ids, const int32_t* lens, int n, PortionPlan* plan) {
+  if (n <= 0 || n > c->max_batch)
+    return set_error(PG_INVALID_INPUT, "batch " + std::to_string(n) + " exceeds the cache's max_batch " + std::to_string(c->max_batch));
+  if (!ids || !lens) return set_error(PG_INVALID_INPUT, "null ids or lens");
+  std::vector<char> used(c->max_batch, 0);
+  int off = 0;
+  plan->seq_start.push_back(0);
+  for (int i = 0; i < n; ++i) {
+    const int slot = slots ? slots[i] : i;
+    if (slot < 0 || slot >= c->max_batch) return set_error(PG_INVALID_INPUT, "slot out of range");
+    if (used[slot]) return set_error(PG_INVALID_INPUT, "slot " + std::to_string(slot) + " appears twice");
+    used[slot] = 1;
+    if (int r = validate_sequence(m, ids + off, lens[i])) return r;
+    const int start = c->seq_len[slot];
+    if (start + (long long)lens[i] > m->positions())
+      return set_error(PG_INVALID_INPUT, "sequence length " + std::to_string(start + (long long)lens[i]) + " exceeds n_positions " + std::to_string(m->positions()));
+    for (int t = 0; t < lens[i]; ++t) {
+      plan->ids.push_back(ids[off + t]);
+      plan->pos.push_back(start + t);
+      plan->row_seq.push_back(i);
+    }
+    off += lens[i];
+    plan->seq_start.push_back(off);
+    plan->slot.push_back(slot);
+    plan->start_pos.push_back(start);
+    plan->max_len = std::max(plan->max_len, lens[i]);
+  }
+  return PG_OK;
+}
+
 static int do_prefill(const pg_model* m, pg_cache* c, const int32_t* ids, const int32_t* lens, int batch,
-                      float* logits_out, int32_t* argmax_out) {
+                      float* logits_out, int32_t* argmax_out, StepProfiler* prof = nullptr) {
   if (int r = check_cache(m, c)) return r;
+  if (m->layered) {
+    if (batch <= 0 || batch > c->max_batch)
+      return set_error(PG_INVALID_INPUT, "batch " + std::to_string(batch) + " exceeds the cache's max_batch " + std::to_string(c->max_batch));
+    if (!ids || !lens) return set_error(PG_INVALID_INPUT, "null ids or lens");
+    for (int b = 0, off = 0; b < batch; off += lens[b++])  // nothing is cleared for input that is refused
+      if (int r = validate_sequence(m, ids + off, lens[b])) return r;
+    for (int b = 0; b < batch; ++b) {
+      release_slot_pages(c, b);
+      c->seq_len[b] = 0;
+    }
+    PortionPlan plan;
+    if (int r = make_plan(m, c, nullptr, ids, lens, batch, &plan)) return r;
+    if (int r = run_layered_portions(m, c, plan, nullptr, 0, nullptr, true, prof)) return r;
+    return fetch_outputs(c, batch, logits_out, argmax_out, nullptr, nullptr, 0);
+  }
   if (batch <= 0 || batch > c->max_batch)
     return set_error(PG_INVALID_INPUT, "batch " + std::to_string(batch) + " exceeds the cache's max_batch " + std::to_string(c->max_batch));
   if (!ids || !lens) return set_error(PG_INVALID_INPUT, "null ids or lens");
@@ -1278,6 +1242,52 @@ static int do_forward_one(const pg_model* m, pg_cache* c, const int32_t* ids, in
   return fetch_outputs(c, batch, logits_out, argmax_out, topk_vals, topk_idx, k);
 }
 
+static int do_extend(const pg_model* m, pg_cache* c, const int32_t* slots, const int32_t* ids, const int32_t* lens, int n,
+                     const int32_t* want, int n_want, float* logits_out, int32_t* argmax_out, float* last_logits_out) {
+  if (int r = check_cache(m, c)) return r;
+  if (!slots) return set_error(PG_INVALID_INPUT, "null slots");
+  if (n_want < 0 || (n_want > 0 && (!want || !logits_out))) return set_error(PG_INVALID_INPUT, "null want or logits_out");
+  PortionPlan plan;
+  if (int r = make_plan(m, c, slots, ids, lens, n, &plan)) return r;
+  for (int i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= plan.rows()) return set_error(PG_INVALID_INPUT, "wanted row " + std::to_string(want[i]) + " is outside the portion");
+  const size_t V = m->v();
+  bool in_order = true, fresh = true, equal = true;
+  for (int i = 0; i < n; ++i) {
+    in_order = in_order && plan.slot[i] == i;
+    fresh = fresh && plan.start_pos[i] == 0;
+    equal = equal && lens[i] == lens[0];
+  }
+  auto token_steps = [&](int len) -> int {  // as decode steps of slots 0..n-1, all portions `len` tokens long
+    std::vector<int32_t> step(n);
+    std::vector<float> logits;
+    for (int t = 0; t < len; ++t) {
+      bool wanted = false;
+      for (int i = 0; i < n; ++i) step[i] = ids[plan.seq_start[i] + t];
+      for (int w = 0; w < n_want; ++w)
+        for (int i = 0; i < n; ++i) wanted = wanted || want[w] == plan.seq_start[i] + t;
+      const bool last = t + 1 == len, fetch = wanted || (last && last_logits_out);
+      if (fetch) logits.resize((size_t)n * V);
+      if (int r = do_forward_one(m, c, step.data(), n, fetch ? logits.data() : nullptr, last ? argmax_out : nullptr, nullptr, nullptr, 0)) return r;
+      for (int w = 0; w < n_want; ++w)
+        for (int i = 0; i < n; ++i)
+          if (want[w] == plan.seq_start[i] + t) memcpy(logits_out + (size_t)w * V, logits.data() + (size_t)i * V, V * sizeof(float));
+      if (last && last_logits_out) memcpy(last_logits_out, logits.data(), (size_t)n * V * sizeof(float));
+    }
+    return PG_OK;
+  };
+  if (in_order && plan.max_len == 1) return token_steps(1);
+  if (!m->layered) {
+    if (in_order && fresh && n_want == 0) return do_prefill(m, c, ids, lens, n, last_logits_out, argmax_out);
+    if (!in_order || !equal)
+      return set_error(PG_INVALID_INPUT, "gpt2 portions after the first run token by token: slots must be 0..n-1 and lengths equal");
+    return token_steps(plan.max_len);
+  }
+  const bool need_last = argmax_out || last_logits_out;
+  if (int r = run_layered_portions(m, c, plan, want, n_want, logits_out, need_last, nullptr)) return r;
+  return need_last ? fetch_outputs(c, n, last_logits_out, argmax_out, nullptr, nullptr, 0) : PG_OK;
+}
+
 // Device buffers and stream of the cache-less full-sequence forward, sized for `rows` positions and re-used
 // from call to call (generate_greedy runs one forward per token).
 struct ForwardWorkspace {
@@ -1285,6 +1295,7 @@ struct ForwardWorkspace {
   float *x = nullptr, *norm = nullptr, *qkv = nullptr, *attn = nullptr, *h = nullptr, *logits = nullptr;
   int* meta = nullptr;
   cudaStream_t s = nullptr;
+  std::unique_ptr<pg_cache> cache;  // layered models
   ~ForwardWorkspace() {
     if (s) cudaStreamSynchronize(s);
     for (void* p : {(void*)x, (void*)norm, (void*)qkv, (void*)attn, (void*)h, (void*)logits, (void*)meta})
@@ -1327,6 +1338,21 @@ static int do_forward(const pg_model* m, const int32_t* ids, int t, float* logit
   if (!m) return set_error(PG_INVALID_INPUT, "null model");
   if (int r = validate_sequence(m, ids, t)) return r;
   if (int r = ensure_device(m->device)) return r;
+  if (m->layered) {  // one portion through a cache of its own
+    if (!ws.cache) {
+      pg_cache* c = nullptr;
+      if (int r = cache_new(m, 1, &c)) return r;
+      ws.cache.reset(c);
+    }
+    release_slot_pages(ws.cache.get(), 0);
+    ws.cache->seq_len[0] = 0;
+    PortionPlan plan;
+    const int32_t len = t;
+    if (int r = make_plan(m, ws.cache.get(), nullptr, ids, &len, 1, &plan)) return r;
+    std::vector<int32_t> rows;
+    for (int i = last_only ? t - 1 : 0; i < t; ++i) rows.push_back(i);
+    return run_layered_portions(m, ws.cache.get(), plan, rows.data(), (int)rows.size(), logits_out, false, nullptr);
+  }
   const size_t C = m->c(), V = m->v(), R = t;
   const size_t out_rows = last_only ? 1 : R;
   if (int r = ws.reserve(m, std::max(R, reserve_rows), out_rows)) return r;
@@ -1353,6 +1379,15 @@ static int do_forward(const pg_model* m, const int32_t* ids, int t, float* logit
   PG_CUDA_TRY(cudaMemcpyAsync(logits_out, ws.logits, out_rows * V * sizeof(float), cudaMemcpyDeviceToHost, s));
   PG_CUDA_TRY(cudaStreamSynchronize(s));  // also keeps `hm` alive long enough
   return PG_OK;
+}
+
+static void fill_profile(const double* sec, const uint64_t* cnt, pg_operation_profile* out) {
+  memset(out, 0, sizeof(*out));
+  out->layer_norm = sec[B_LAYER_NORM]; out->qkv_projection = sec[B_QKV]; out->attention = sec[B_ATTN];
+  out->attention_projection = sec[B_ATTN_PROJ]; out->mlp_fc_projection = sec[B_MLP_FC];
+  out->mlp_projection = sec[B_MLP_PROJ]; out->final_logits = sec[B_LOGITS]; out->other = sec[B_OTHER];
+  const Bucket order[8] = {B_LAYER_NORM, B_QKV, B_ATTN, B_ATTN_PROJ, B_MLP_FC, B_MLP_PROJ, B_LOGITS, B_OTHER};
+  for (int i = 0; i < 8; ++i) out->launches[i] = cnt[order[i]];
 }
 
 static double now_s() {
@@ -1401,6 +1436,15 @@ int pg_model_from_host_weights(const pg_gpt2_config* cfg, const float* const* te
 int pg_model_load_dir(const char* dir, const pg_backend_config* backend, pg_model** out) {
   if (!dir || !out) return set_error(PG_ASSET, "null directory or output");
   std::string d(dir);
+  bool layered = false;
+  LayeredConfig lc;
+  if (int r = load_design_config(d + "/config.json", &layered, &lc)) return r;
+  if (layered) {
+    SafeTensorsFile file;
+    if (int r = read_safetensors(d + "/model.safetensors", &file)) return r;
+    if (int r = check_layered_tensors(file, d + "/model.safetensors", &lc)) return r;
+    return build_layered_model(lc, file, backend, out);
+  }
   pg_gpt2_config cfg{};
   if (int r = load_config_json(d + "/config.json", &cfg)) return r;
   HostWeights hw;
@@ -1414,10 +1458,24 @@ int pg_model_config(const pg_model* model, pg_gpt2_config* out) {
   return PG_OK;
 }
 
+const char* pg_model_architecture(const pg_model* model) {
+  return !model ? "" : model->layered ? layered_config(model).architecture.c_str() : "gpt2";
+}
+
+const char* pg_registered_architectures(void) {
+  static const std::string names = registered_designs();
+  return names.c_str();
+}
+
+uint64_t pg_model_state_bytes_per_sequence(const pg_model* model) {
+  return model && model->layered ? layered_state_bytes_per_sequence(model) : 0;
+}
+
 uint64_t pg_model_max_context_len(const pg_model* model) { return model ? model->cfg.n_positions : 0; }
 
 uint64_t pg_model_weight_bytes_per_step(const pg_model* model) {
   if (!model) return 0;
+  if (model->layered) return layered_weight_bytes_per_step(model);
   const pg_gpt2_config& c = model->cfg;
   // every block matrix, bias and LayerNorm vector once; the tied embedding once as lm_head;
   // ln_f; one wte row and one wpe row are negligible and not counted. With BF16 / int8 weights the
@@ -1476,6 +1534,7 @@ int pg_cache_read_layer(const pg_cache* cache, int32_t slot, uint64_t layer, flo
   if (!cache || !keys || !values) return set_error(PG_INVALID_INPUT, "null argument");
   if (slot < 0 || slot >= cache->max_batch) return set_error(PG_INVALID_INPUT, "slot out of range");
   if (layer >= cache->model->cfg.n_layer) return set_error(PG_INVALID_INPUT, "layer out of range");
+  if (cache->model->layered) return set_error(PG_INVALID_INPUT, "the layers of this model do not have GPT-2's key / value layout");
   const pg_model* m = cache->model;
   PG_CUDA_TRY(cudaSetDevice(m->device));
   size_t n = (size_t)m->positions() * m->c();
@@ -1486,7 +1545,7 @@ int pg_cache_read_layer(const pg_cache* cache, int32_t slot, uint64_t layer, flo
   int rc = sync_table(c);
   cudaError_t e = cudaSuccess;
   if (rc == PG_OK) {
-    e = launch_kv_gather(cache->layer_pool((int)layer), cache->d_table, cache->kv, slot, cache->seq_len[slot],
+    e = launch_kv_gather(cache->layer_pool((int)layer), cache->tables[0].d_table, cache->kv, slot, cache->seq_len[slot],
                          m->positions(), dk, dv, cache->stream);
     if (e == cudaSuccess) e = cudaMemcpyAsync(keys, dk, n * sizeof(float), cudaMemcpyDeviceToHost, cache->stream);
     if (e == cudaSuccess) e = cudaMemcpyAsync(values, dv, n * sizeof(float), cudaMemcpyDeviceToHost, cache->stream);
@@ -1508,6 +1567,11 @@ int pg_prefill(const pg_model* model, pg_cache* cache, const int32_t* ids, const
 int pg_forward_one(const pg_model* model, pg_cache* cache, const int32_t* ids, int32_t batch, float* logits_out,
                    int32_t* argmax_out, float* topk_vals, int32_t* topk_idx, int32_t k) {
   return do_forward_one(model, cache, ids, batch, logits_out, argmax_out, topk_vals, topk_idx, k);
+}
+
+int pg_extend(const pg_model* model, pg_cache* cache, const int32_t* slots, const int32_t* ids, const int32_t* lens, int32_t n,
+              const int32_t* want, int32_t n_want, float* logits_out, int32_t* argmax_out, float* last_logits_out) {
+  return do_extend(model, cache, slots, ids, lens, n, want, n_want, logits_out, argmax_out, last_logits_out);
 }
 
 int pg_forward(const pg_model* model, const int32_t* ids, int32_t t, float* logits_out) {
@@ -1611,14 +1675,27 @@ int pg_profile_forward_one(const pg_model* model, pg_cache* cache, const int32_t
       fused_phases = (uint64_t)it->second.n;
     }
   }
-  memset(out, 0, sizeof(*out));
-  out->layer_norm = sec[B_LAYER_NORM]; out->qkv_projection = sec[B_QKV]; out->attention = sec[B_ATTN];
-  out->attention_projection = sec[B_ATTN_PROJ]; out->mlp_fc_projection = sec[B_MLP_FC];
-  out->mlp_projection = sec[B_MLP_PROJ]; out->final_logits = sec[B_LOGITS]; out->other = sec[B_OTHER];
-  const Bucket order[8] = {B_LAYER_NORM, B_QKV, B_ATTN, B_ATTN_PROJ, B_MLP_FC, B_MLP_PROJ, B_LOGITS, B_OTHER};
-  for (int i = 0; i < 8; ++i) out->launches[i] = cnt[order[i]];
+  fill_profile(sec, cnt, out);
   out->fused_step_kernel = fused_sec;
   out->fused_phases = fused_phases;
+  return PG_OK;
+}
+
+int pg_profile_prefill(const pg_model* model, pg_cache* cache, const int32_t* ids, const int32_t* lens, int32_t batch,
+                       pg_operation_profile* out) {
+  if (!model || !cache || !out) return set_error(PG_INVALID_INPUT, "null argument");
+  if (!model->layered) return set_error(PG_INVALID_INPUT, "pg_profile_prefill is available for layered models");
+  StepProfiler prof;
+  if (int r = do_prefill(model, cache, ids, lens, batch, nullptr, nullptr, &prof)) return r;
+  double sec[B_COUNT] = {0};
+  uint64_t cnt[B_COUNT] = {0};
+  for (size_t i = 0; i + 1 < prof.ev.size(); i += 2) {
+    float ms = 0.f;
+    PG_CUDA_TRY(cudaEventElapsedTime(&ms, prof.ev[i], prof.ev[i + 1]));
+    sec[prof.bucket[i]] += ms * 1e-3;
+    cnt[prof.bucket[i]] += 1;
+  }
+  fill_profile(sec, cnt, out);
   return PG_OK;
 }
 

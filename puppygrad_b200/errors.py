@@ -15,11 +15,24 @@ class Gpt2Error(Exception):
                "Cuda": "GPT-2 CUDA error: ", "Timeout": "GPT-2 device timeout: "}
 
     def __init__(self, kind: str, message: str):
-        super().__init__(self._PREFIX.get(kind, "") + message)
+        super().__init__(self.prefix(kind) + message)
         self.kind = kind
         self.message = message
 
 
-def check(status: int) -> None:
+    @classmethod
+    def prefix(cls, kind: str) -> str:
+        return cls._PREFIX.get(kind, "")
+
+
+class DesignError(Gpt2Error):
+    """The same for models of other designs than GPT-2."""
+
+    @classmethod
+    def prefix(cls, kind: str) -> str:
+        return Gpt2Error._PREFIX.get(kind, "").replace("GPT-2", "model").replace("model asset", "asset")
+
+
+def check(status: int, error=Gpt2Error) -> None:
     if status != N.PG_OK:
-        raise Gpt2Error(Gpt2Error.KINDS.get(status, "Cuda"), N.lib.pg_last_error_message().decode())
+        raise error(Gpt2Error.KINDS.get(status, "Cuda"), N.lib.pg_last_error_message().decode())
