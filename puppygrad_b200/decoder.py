@@ -145,6 +145,10 @@ class DecoderModel:
     cache_class = DecoderCache
 
     @classmethod
+    def default_cuda_config(cls) -> CudaConfig:
+        return CudaConfig()
+
+    @classmethod
     def _check(cls, status: int) -> None:
         check(status, cls.error_class)
 

@@ -23,7 +23,9 @@ from typing import Callable, List, Optional, Sequence, TextIO, Tuple
 
 from .errors import Gpt2Error
 from .generation import GenerationStats, ProfiledGenerationStats, TextGenerationConfig, gpt2_generation_config
-from .gpt2 import Gpt2CudaConfig, Gpt2Model
+from .decoder import DecoderModel
+from .gpt2 import Gpt2CudaConfig
+from .registry import architecture_of, load_model, model_class
 from .streaming import IncrementalTextStreamer, escape_raw_token
 
 
@@ -125,7 +127,7 @@ class Gpt2GenerationStats:
 class Gpt2Runtime:
     """rust.rs:324-327, 377-635."""
 
-    def __init__(self, model: Gpt2Model, tokenizer: Gpt2Tokenizer):
+    def __init__(self, model: DecoderModel, tokenizer: Optional[Gpt2Tokenizer]):
         self.model = model
         self.tokenizer = tokenizer
 
@@ -136,9 +138,16 @@ class Gpt2Runtime:
     @classmethod
     def from_dir_with_backend(cls, model_dir: str, backend: Optional[Gpt2CudaConfig], use_tuning: bool = True,
                               tuning_file: Optional[str] = None) -> "Gpt2Runtime":
+        """Any registered model (the class by config.json) with the directory's tokenizer.json."""
         paths = Gpt2AssetPaths.new(model_dir)
-        model = Gpt2Model.from_dir(paths.model_dir, backend, use_tuning=use_tuning, tuning_file=tuning_file)
+        model = load_model(paths.model_dir, backend, use_tuning=use_tuning, tuning_file=tuning_file)
         return cls(model, Gpt2Tokenizer.from_file(paths.tokenizer))
+
+    @classmethod
+    def ids_only(cls, model_dir: str, backend: Optional[Gpt2CudaConfig], use_tuning: bool = True,
+                 tuning_file: Optional[str] = None) -> "Gpt2Runtime":
+        """Without a tokenizer: token ids in, token ids out (`stream_ids_with_stats`)."""
+        return cls(load_model(model_dir, backend, use_tuning=use_tuning, tuning_file=tuning_file), None)
 
     def generate_greedy_text(self, prompt: str, max_new_tokens: int) -> str:
         input_ids = self.tokenizer.encode(prompt)
@@ -224,11 +233,15 @@ class Gpt2Runtime:
     def stream_token_ids_with_stats(self, prompt: str, generation: TextGenerationConfig,
                                     on_token: Callable[[int], None]) -> Tuple[List[int], Gpt2GenerationStats]:
         """rust.rs:548-635: returns prompt ids + generated ids."""
-        self._check_generation(generation)
-        profile = Gpt2OperationProfile()
         t0 = time.perf_counter()
         input_ids = self.tokenizer.encode(prompt)
-        tokenize_time = time.perf_counter() - t0
+        return self.stream_ids_with_stats(input_ids, generation, on_token, tokenize_time=time.perf_counter() - t0)
+
+    def stream_ids_with_stats(self, input_ids: Sequence[int], generation: TextGenerationConfig, on_token: Callable[[int], None],
+                              tokenize_time: float = 0.0) -> Tuple[List[int], Gpt2GenerationStats]:
+        """The same from token ids."""
+        self._check_generation(generation)
+        profile = Gpt2OperationProfile()
         profile.tokenization += tokenize_time
         failure: List[BaseException] = []
 
@@ -294,10 +307,13 @@ def format_gpt2_stats(load_time: float, stats: Gpt2GenerationStats) -> str:
 
 
 def run_gpt2(argv: Optional[Sequence[str]] = None, stdout: TextIO = sys.stdout, stderr: TextIO = sys.stderr) -> int:
-    """The generation part of `run-gpt2` (main.rs:1305-1388): no download, the model directory must exist."""
+    """The generation part of `run-gpt2` (main.rs:1305-1388): no download, the model directory must exist. Serves every
+    registered model; with `--prompt-ids` no tokenizer is needed and the generated ids are printed."""
     ap = argparse.ArgumentParser(prog="python -m puppygrad_b200.run_gpt2")
     ap.add_argument("--model-dir", required=True)
-    ap.add_argument("--prompt", required=True)
+    prompt = ap.add_mutually_exclusive_group(required=True)
+    prompt.add_argument("--prompt")
+    prompt.add_argument("--prompt-ids", help="token ids with commas between them, instead of text")
     ap.add_argument("--max-new-tokens", type=int, default=32)
     ap.add_argument("--temperature", type=float, default=0.0)
     ap.add_argument("--top-p", type=float, default=None)
@@ -313,6 +329,7 @@ def run_gpt2(argv: Optional[Sequence[str]] = None, stdout: TextIO = sys.stdout, 
     ap.add_argument("--tuning-file", default=None)
     ap.add_argument("--math-mode", default=None, help="fp32, tf32x3, tf32 or bf16 (default: the tuning file's, else fp32)")
     ap.add_argument("--quantized-weights", action="store_true")
+    ap.add_argument("--max-context", type=int, default=0, help="models without a position limit: the most tokens of a sequence")
     a = ap.parse_args(argv)
     generation = gpt2_generation_config(a.max_new_tokens)
     generation.temperature, generation.top_p, generation.top_k = a.temperature, a.top_p, a.top_k
@@ -322,16 +339,27 @@ def run_gpt2(argv: Optional[Sequence[str]] = None, stdout: TextIO = sys.stdout, 
     elif a.eos_token_id is not None:
         generation.eos_token_id = a.eos_token_id
     generation.validate()
+    name = architecture_of(a.model_dir) if os.path.exists(os.path.join(a.model_dir, "config.json")) else "gpt2"
+    if name != "gpt2" and a.eos_token_id is None:
+        generation.eos_token_id = None  # the default is GPT-2's end-of-text token
     backend = None
-    if a.math_mode is not None or a.quantized_weights:
-        backend = Gpt2CudaConfig(math_mode=a.math_mode or "fp32", quantized_weights=a.quantized_weights)
-    stderr.write(f"loading GPT-2 from {a.model_dir}\n")
+    if a.math_mode is not None or a.quantized_weights or a.max_context:
+        default = model_class(name).default_cuda_config().math_mode
+        backend = Gpt2CudaConfig(math_mode=a.math_mode or default, quantized_weights=a.quantized_weights, max_context=a.max_context)
+    stderr.write(f"loading {'GPT-2' if name == 'gpt2' else name} from {a.model_dir}\n")
     t0 = time.perf_counter()
-    runtime = Gpt2Runtime.from_dir_with_backend(a.model_dir, backend, use_tuning=not a.no_tuning, tuning_file=a.tuning_file)
+    load = Gpt2Runtime.ids_only if a.prompt_ids is not None else Gpt2Runtime.from_dir_with_backend
+    runtime = load(a.model_dir, backend, use_tuning=not a.no_tuning, tuning_file=a.tuning_file)
     load_time = time.perf_counter() - t0
     used = getattr(runtime.model, "cuda_config", None)  # the tuning file's when no backend was given
     stderr.write(f"backend: {used.describe() if used is not None else 'cuda'}\n")
-    if a.stream_raw_tokens:
+    if a.prompt_ids is not None:
+        def on_id(token_id: int) -> None:
+            stdout.write(f"{token_id}\n")
+            stdout.flush()
+
+        _, stats = runtime.stream_ids_with_stats([int(t) for t in a.prompt_ids.split(",") if t.strip()], generation, on_id)
+    elif a.stream_raw_tokens:
         for token_id in runtime.tokenizer.encode(a.prompt):
             write_raw_token_event(stdout, None, "prompt", token_id, runtime.tokenizer)
         stdout.flush()

@@ -133,23 +133,25 @@ def uniform_prompt(seed: int, length: int, vocab_size: int) -> np.ndarray:
     return rng.integers(0, vocab_size, size=length, dtype=np.int64)
 
 
-def write_safetensors(path: str, tensors: dict[str, np.ndarray], prefix: str = "") -> None:
-    """Minimal safetensors writer: u64 LE header length, JSON header, raw little-endian data."""
+def write_safetensors(path: str, tensors: dict[str, np.ndarray], prefix: str = "", bf16: bool = False) -> None:
+    """Minimal safetensors writer: u64 LE header length, JSON header, raw little-endian data (F32, or rounded to BF16)."""
     header, offset = {}, 0
     order = list(tensors)
     for name in order:
         a = tensors[name]
         assert a.dtype == np.float32
-        header[prefix + name] = {"dtype": "F32", "shape": list(a.shape),
-                                 "data_offsets": [offset, offset + a.nbytes]}
-        offset += a.nbytes
+        nbytes = a.nbytes // 2 if bf16 else a.nbytes
+        header[prefix + name] = {"dtype": "BF16" if bf16 else "F32", "shape": list(a.shape),
+                                 "data_offsets": [offset, offset + nbytes]}
+        offset += nbytes
     blob = json.dumps(header, separators=(",", ":")).encode()
     blob += b" " * ((8 - len(blob) % 8) % 8)
     with open(path, "wb") as f:
         f.write(len(blob).to_bytes(8, "little"))
         f.write(blob)
         for name in order:
-            f.write(np.ascontiguousarray(tensors[name]).astype("<f4", copy=False).tobytes())
+            a = np.ascontiguousarray(tensors[name]).astype("<f4", copy=False)
+            f.write((round_bf16(a).view(np.uint32) >> np.uint32(16)).astype("<u2").tobytes() if bf16 else a.tobytes())
 
 
 def read_safetensors(path: str) -> dict[str, np.ndarray]:
@@ -178,4 +180,13 @@ def write_model_dir(path: str, cfg: dict, weights: dict[str, np.ndarray], prefix
         json.dump({k: cfg[k] for k in ("vocab_size", "n_positions", "n_embd", "n_layer", "n_head",
                                        "n_inner", "layer_norm_epsilon") if k in cfg}, f)
     write_safetensors(os.path.join(path, "model.safetensors"), weights, prefix)
+    return path
+
+
+def write_design_dir(path: str, cfg: dict, weights: dict[str, np.ndarray], bf16: bool = True) -> str:
+    """A model directory of a design other than GPT-2: `cfg` as config.json, the tensors by name (BF16 unless told)."""
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    write_safetensors(os.path.join(path, "model.safetensors"), weights, bf16=bf16)
     return path
