@@ -279,6 +279,52 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(AttentionPortionArg
   }
 }
 
+// The same when every size and offset is a multiple of four: eight lanes per (row, head), the row in registers.
+template <typename T>
+__global__ void __launch_bounds__(256) attention_prep_vec_kernel(AttentionPortionArgs a) {
+  const AttentionLayer& l = a.l;
+  const int per = l.heads + 2 * l.kv_heads, l8 = threadIdx.x & 7;
+  const long long total = ((long long)a.rows * per + 3) / 4 * 4;  // whole warps stay together
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 3; i < total;
+       i += ((long long)gridDim.x * blockDim.x) >> 3) {
+    const bool on = i < (long long)a.rows * per;
+    const int row = on ? (int)(i / per) : 0, j = on ? (int)(i % per) : 0;
+    const int seq = a.row_seq[row], ctx = a.seq_pos[seq] % l.span;
+    const size_t krow = (size_t)a.key_start[seq] + ctx + (row - a.seq_start[seq]);
+    const bool is_q = j < l.heads, is_k = !is_q && j < l.heads + l.kv_heads;
+    const int h = is_q ? j : is_k ? j - l.heads : j - l.heads - l.kv_heads;
+    const int n = is_q || is_k ? l.dim : l.vdim, np = is_q || is_k ? l.dimp : l.vdimp;
+    const float* x = a.p + (size_t)row * a.ldp + (is_q ? l.off_q : is_k ? l.off_k : l.off_v) + h * n;
+    const float* weight = is_q ? l.q_norm : is_k ? l.k_norm : nullptr;
+    const bool normed = is_q ? l.q_norm != nullptr : is_k ? l.k_norm != nullptr : l.v_norm != 0;
+    T* out = is_q   ? static_cast<T*>(a.q) + ((size_t)row * l.heads + h) * np
+             : is_k ? static_cast<T*>(a.k) + (krow * l.kv_heads + h) * np
+                    : static_cast<T*>(a.v) + (krow * l.kv_heads + h) * np;
+    float4 v[8];
+    float s = 0.f;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const int c = q * 32 + l8 * 4;
+      v[q] = on && c < n ? load4(x + c) : make_float4(0, 0, 0, 0);
+      s += (v[q].x * v[q].x + v[q].y * v[q].y) + (v[q].z * v[q].z + v[q].w * v[q].w);
+    }
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) s += __shfl_xor_sync(ALL_LANES, s, o);
+    const float r = normed ? 1.f / sqrtf(s / (float)n + l.eps) : 1.f;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const int c = q * 32 + l8 * 4;
+      if (on && c < np) {
+        float4 y = make_float4(v[q].x * r, v[q].y * r, v[q].z * r, v[q].w * r);
+        if (weight && c < n) {
+          y.x *= weight[c]; y.y *= weight[c + 1]; y.z *= weight[c + 2]; y.w *= weight[c + 3];
+        }
+        store4(out + c, y);
+      }
+    }
+  }
+}
+
 // Cached keys and values that the first row of each sequence still sees, copied in front of its own. Block = (key, seq).
 template <typename T>
 __global__ void __launch_bounds__(128) attention_context_kernel(AttentionPortionArgs a) {
@@ -432,10 +478,18 @@ cudaError_t portion_t(const AttentionPortionArgs& a, cudaStream_t s) {
   cudaError_t e;
   const long long warps = (long long)a.rows * (l.heads + 2 * l.kv_heads);
   const int pgrid = (int)std::min<long long>((warps + 7) / 8, 148 * 16);
-  if ((e = launch_kernel(attention_prep_kernel<T>, dim3(pgrid), dim3(256), 0, s, false, a)) != cudaSuccess) return e;
+  const bool vec = l.dim % 4 == 0 && l.vdim % 4 == 0 && l.off_q % 4 == 0 && l.off_k % 4 == 0 && l.off_v % 4 == 0 && a.ldp % 4 == 0;
+  const int vgrid = (int)std::min<long long>((warps + 31) / 32, 148 * 16);
+  e = vec ? launch_kernel(attention_prep_vec_kernel<T>, dim3(vgrid), dim3(256), 0, s, false, a)
+          : launch_kernel(attention_prep_kernel<T>, dim3(pgrid), dim3(256), 0, s, false, a);
+  if (e != cudaSuccess) return e;
   if (a.krows > a.rows) {
     const int cgrid = std::min(a.krows - a.rows, 1024);
     if ((e = launch_kernel(attention_context_kernel<T>, dim3(cgrid, a.nseq), dim3(128), 0, s, false, a)) != cudaSuccess) return e;
+  }
+  if (sizeof(T) == 2) {
+    if ((e = launch_attention_tc(a, s)) != cudaSuccess) return e;
+    return launch_kernel(attention_store_kernel<T>, dim3(a.rows), dim3(128), 0, s, false, a);
   }
   const dim3 grid((a.max_len + QT - 1) / QT, l.heads, a.nseq);
   const size_t smem = ((size_t)(QT + KT) * (l.dimp + 1) + (size_t)KT * l.vdimp + (size_t)QT * (KT + 1)) * sizeof(float);

@@ -54,7 +54,7 @@ struct LayeredModel {
   Norm final_norm;
   double* freq = nullptr;
   std::vector<DevLayer> layers;
-  int max_in = 0, max_y = 0, max_ff = 0, max_rec = 0;  // widest projection, mixer output, hidden row, heads * dim of a recurrence
+  int max_in = 0, max_y = 0, max_ff = 0, max_rec = 0, max_rec_out = 0;  // widest projection, mixer output, hidden row, heads * dim and heads * vdim of a recurrence
   int n_pools = 0, n_states = 0;
   std::vector<int> spans;  // one page table each
   std::vector<void*> allocations;
@@ -84,7 +84,7 @@ struct LayeredCache {
   float* attn_part = nullptr;
   unsigned* attn_counters = nullptr;
   // portion workspaces (grow-only)
-  float *decay = nullptr, *unit = nullptr, *rate = nullptr, *segments = nullptr;
+  float *decay = nullptr, *unit = nullptr, *rate = nullptr, *out_raw = nullptr, *segments = nullptr;
   void *q = nullptr, *k = nullptr, *v = nullptr;
   int* meta = nullptr;
   float* logits = nullptr;
@@ -95,7 +95,7 @@ struct LayeredCache {
     for (LayeredRows* r : {&step, &portion})
       for (void* p : {(void*)r->x[0], (void*)r->x[1], (void*)r->p, (void*)r->yo, r->h, r->y, r->ff, (void*)r->h32, (void*)r->y32, (void*)r->ff32})
         if (p) cudaFree(p);
-    for (void* p : {(void*)attn_part, (void*)attn_counters, (void*)decay, (void*)unit, (void*)rate, (void*)segments, q, k, v,
+    for (void* p : {(void*)attn_part, (void*)attn_counters, (void*)decay, (void*)unit, (void*)rate, (void*)out_raw, (void*)segments, q, k, v,
                     (void*)meta, (void*)logits})
       if (p) cudaFree(p);
   }
@@ -237,6 +237,7 @@ int build_layer(Builder& b, const LayerSpec& spec, const std::string& p, int pag
       a.out_scale = bs.scale;
       br.state = m->n_states++;
       m->max_rec = std::max(m->max_rec, K);
+      m->max_rec_out = std::max(m->max_rec_out, V);
     }
     d->branches.push_back(br);
   }
@@ -623,7 +624,7 @@ cudaError_t enqueue_portions(pg_cache* c, const PortionPlan& plan, const Portion
         RecurrenceScanArgs a{};
         a.l = b.rec; a.p = r.p; a.ldp = l.in.np; a.rows = rows; a.nseq = plan.n();
         a.seq_start = d.seq_start; a.seq_slot = d.slot; a.seq_pos = d.start_pos; a.state = lc->states[b.state];
-        a.decay = lc->decay; a.unit = lc->unit; a.rate = lc->rate;
+        a.decay = lc->decay; a.unit = lc->unit; a.rate = lc->rate; a.out_raw = lc->out_raw;
         a.segments = lc->segments; a.seg_tokens = SEGMENT_TOKENS;
         a.max_segs = recurrence_use_segments(b.rec, plan.n(), plan.max_len, max_segs) ? max_segs : 0;
         a.y = y; a.ldy = l.out.kp;
@@ -699,7 +700,8 @@ int layered_run_portions(pg_cache* c, const PortionPlan& plan, float* logits, St
     }
   }
   if (m->max_rec && (size_t)rows > lc->gate_rows) {
-    size_t g = lc->gate_rows, h = g;
+    size_t g = lc->gate_rows, h = g, o = g;
+    if (int r = grow(&lc->out_raw, &o, rows, m->max_rec_out * sizeof(float))) return r;
     if (int r = grow(&lc->decay, &g, rows, m->max_rec * sizeof(float))) return r;
     if (int r = grow(&lc->unit, &h, rows, m->max_rec * sizeof(float))) return r;
     if (int r = grow(&lc->rate, &lc->gate_rows, rows, m->max_rec * sizeof(float))) return r;

@@ -102,6 +102,7 @@ struct RecurrenceScanArgs {  // whole portions of `nseq` sequences
   const int* seq_pos;    // [nseq] position of the first row; 0 starts from a zero state
   float* state;
   float *decay, *unit, *rate;  // [rows, heads * dim] scratch: decay; delta: unit key, a * u
+  float* out_raw;              // [rows, heads * vdim] scratch: outputs before the head norm
   float* segments;             // scratch of the segmented scan (may be nullptr)
   int seg_tokens, max_segs;    // tokens per segment, segments of the longest sequence (0: one pass)
   void* y;
@@ -155,6 +156,7 @@ struct AttentionPortionArgs {
 };
 // Norms the rows' queries, keys and values into the workspaces, copies the cached keys and values that the first rows
 // still see in front of them, attends, and stores what later tokens can still see into the pages.
+cudaError_t launch_attention_tc(const AttentionPortionArgs& a, cudaStream_t s);  // the products of BF16 portions on the tensor cores
 cudaError_t launch_attention_portion(const AttentionPortionArgs& a, bool bf16, cudaStream_t s);
 
 }  // namespace pg

@@ -143,28 +143,35 @@ __global__ void __launch_bounds__(STEP_THREADS) recurrence_step_kernel(Recurrenc
 }
 
 // ------------------------------------------------------------------ gates of whole portions
-constexpr int GATE_ROWS = 4;
+constexpr int GATE_ROWS = 16;
 // decay, and for the delta rule the unit keys u and the removal rates a * u, of GATE_ROWS rows per block
 __global__ void __launch_bounds__(256) recurrence_gates_kernel(RecurrenceScanArgs a) {
-  extern __shared__ __align__(16) float sm[];  // [GATE_ROWS][rank]
+  extern __shared__ __align__(16) float sm[];  // [rank][GATE_ROWS]
   const RecurrenceLayer& l = a.l;
   const int K = l.heads * l.dim, r0 = blockIdx.x * GATE_ROWS, tid = threadIdx.x;
   const int nr = min(GATE_ROWS, a.rows - r0);
   const bool delta = l.kind == KIND_DELTA;
-  for (int i = tid; i < nr * l.rank; i += blockDim.x) {
-    const float t = a.p[(size_t)(r0 + i / l.rank) * a.ldp + l.off_t + i % l.rank];
-    sm[i] = delta ? tanhf(t) : t;
+  for (int i = tid; i < GATE_ROWS * l.rank; i += blockDim.x) {
+    const int j = i / l.rank, r = i % l.rank;
+    const float t = j < nr ? a.p[(size_t)(r0 + j) * a.ldp + l.off_t + r] : 0.f;
+    sm[r * GATE_ROWS + j] = delta ? tanhf(t) : t;
   }
   __syncthreads();
   for (int c = tid; c < K; c += blockDim.x) {
     float z[GATE_ROWS];
 #pragma unroll
     for (int j = 0; j < GATE_ROWS; ++j) z[j] = l.b2[c];
+#pragma unroll 4
     for (int r = 0; r < l.rank; ++r) {
       const float w = l.w2[(size_t)r * K + c];
 #pragma unroll
-      for (int j = 0; j < GATE_ROWS; ++j)
-        if (j < nr) z[j] = fmaf(w, sm[j * l.rank + r], z[j]);
+      for (int j = 0; j < GATE_ROWS; j += 4) {
+        const float4 t = load4(sm + r * GATE_ROWS + j);
+        z[j] = fmaf(w, t.x, z[j]);
+        z[j + 1] = fmaf(w, t.y, z[j + 1]);
+        z[j + 2] = fmaf(w, t.z, z[j + 2]);
+        z[j + 3] = fmaf(w, t.w, z[j + 3]);
+      }
     }
 #pragma unroll
     for (int j = 0; j < GATE_ROWS; ++j)
@@ -203,6 +210,7 @@ struct ScanArgs {
   int mode, tb;
   float *seg_state, *seg_trans;  // [nseq][max_segs][heads][dim][dvp], [nseq][max_segs][heads][dim][dkp] (GLA: [..][dim] decays)
   int dkp;
+  int col_blocks, block_cols;  // column blocks of a head, columns of each (the last may have fewer)
   int vec;      // 16-byte copies are possible
   int y_bf16;
 };
@@ -219,16 +227,65 @@ __device__ __forceinline__ void copy_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
+// Sum of CPL values over the eight lanes of a group. Afterwards every lane holds one column's total: the one
+// owned_column() names.
+template <int CPL>
+__device__ __forceinline__ float group_reduce(const float (&v)[CPL], int lr) {
+  float x;
+  if (CPL == 4) {
+    const bool up = lr & 4;
+    const float a0 = up ? v[2 % CPL] : v[0], a1 = up ? v[3 % CPL] : v[1 % CPL];
+    const float b0 = up ? v[0] : v[2 % CPL], b1 = up ? v[1 % CPL] : v[3 % CPL];
+    const float c0 = a0 + __shfl_xor_sync(ALL_LANES, b0, 4), c1 = a1 + __shfl_xor_sync(ALL_LANES, b1, 4);
+    const bool up2 = lr & 2;
+    x = (up2 ? c1 : c0) + __shfl_xor_sync(ALL_LANES, up2 ? c0 : c1, 2);
+  } else if (CPL == 2) {
+    const bool up = lr & 4;
+    x = (up ? v[1 % CPL] : v[0]) + __shfl_xor_sync(ALL_LANES, up ? v[0] : v[1 % CPL], 4);
+    x += __shfl_xor_sync(ALL_LANES, x, 2);
+  } else {
+    x = v[0] + __shfl_xor_sync(ALL_LANES, v[0], 4);
+    x += __shfl_xor_sync(ALL_LANES, x, 2);
+  }
+  return x + __shfl_xor_sync(ALL_LANES, x, 1);
+}
+template <int CPL>
+__device__ __forceinline__ int owned_column(int lr) {
+  return CPL == 4 ? ((lr & 4) >> 1) | ((lr & 2) >> 1) : CPL == 2 ? (lr & 4) >> 2 : 0;
+}
+// The totals of all columns in every lane.
+template <int CPL>
+__device__ __forceinline__ void group_all_reduce(float (&v)[CPL], int lr) {
+  const float x = group_reduce<CPL>(v, lr);
+  if (CPL == 4) {
+    const float y = __shfl_xor_sync(ALL_LANES, x, 2);
+    const float lo = lr & 2 ? y : x, hi = lr & 2 ? x : y;
+    const float lo2 = __shfl_xor_sync(ALL_LANES, lo, 4), hi2 = __shfl_xor_sync(ALL_LANES, hi, 4);
+    v[0] = lr & 4 ? lo2 : lo;
+    v[1 % CPL] = lr & 4 ? hi2 : hi;
+    v[2 % CPL] = lr & 4 ? lo : lo2;
+    v[3 % CPL] = lr & 4 ? hi : hi2;
+  } else if (CPL == 2) {
+    const float y = __shfl_xor_sync(ALL_LANES, x, 4);
+    v[0] = lr & 4 ? y : x;
+    v[1 % CPL] = lr & 4 ? x : y;
+  } else {
+    v[0] = x;
+  }
+}
+
 template <int KIND, int RPL, int CPL>
-__global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
+__global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(ScanArgs sa) {
   extern __shared__ __align__(16) float sm[];
   constexpr int DKP = 8 * RPL, NA = KIND == KIND_DELTA ? 5 : 3;  // staged key-channel arrays
   const RecurrenceScanArgs& a = sa.a;
   const RecurrenceLayer& l = a.l;
   const int dk = l.dim, K = l.heads * dk, tid = threadIdx.x, nthreads = blockDim.x;
   const bool trans = sa.mode == SCAN_TRANS;
-  const int dv = trans ? dk : l.vdim;  // columns of this launch
-  const int head = blockIdx.x, seq = blockIdx.y, seg = blockIdx.z;
+  // blockIdx.x = head * (column blocks) + column block; with several column blocks per head the outputs leave unnormed
+  const int head = blockIdx.x / sa.col_blocks, cb = blockIdx.x % sa.col_blocks, seq = blockIdx.y, seg = blockIdx.z;
+  const int all_cols = trans ? dk : l.vdim, cbase = cb * sa.block_cols;
+  const int dv = min(sa.block_cols, all_cols - cbase);  // columns of this block
   const int W = nthreads >> 5, COLS = W * 4 * CPL, TB = sa.tb;
   const int stride = NA * DKP + 2 * COLS;  // floats of one staged token: k, decay, q, (u, rate), v, gate
   float* stage = sm;                       // [2][TB][stride]
@@ -260,7 +317,7 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
       }
     };
     const int vec = sa.vec, e = vec ? 4 : 1;
-    const int nk = dk / e, nv = trans ? 0 : dv / e, ng = outputs ? nv : 0;
+    const int nk = dk / e, nv = trans ? 0 : dv / e, ng = outputs && sa.col_blocks == 1 ? nv : 0;
     const int per = NA * nk + nv + ng;
     for (int i = tid; i < n * per; i += nthreads) {
       const int t = i / per, j = i - t * per, row = tb0 + t;
@@ -274,11 +331,11 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
       } else if (j < NA * nk + nv) {
         const int x = (j - NA * nk) * e;
         d += NA * DKP + x;
-        s = a.p + (size_t)row * a.ldp + l.off_v + head * dv + x;
+        s = a.p + (size_t)row * a.ldp + l.off_v + head * l.vdim + cbase + x;
       } else {
         const int x = (j - NA * nk - nv) * e;
         d += NA * DKP + COLS + x;
-        s = a.p + (size_t)row * a.ldp + l.off_g + head * dv + x;
+        s = a.p + (size_t)row * a.ldp + l.off_g + head * l.vdim + cbase + x;
       }
       if (vec) copy_async16(d, s);
       else copy_async4(d, s);
@@ -299,16 +356,12 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
       const int col = col0 + c;
       float v = 0.f;
       if (row < dk && col < dv) {
-        if (init) v = init[(size_t)row * l.dvp + col];
-        else if (trans) v = row == col ? 1.f : 0.f;
+        if (init) v = init[(size_t)row * l.dvp + cbase + col];
+        else if (trans) v = row == cbase + col ? 1.f : 0.f;
       }
       s[r][c] = v;
     }
   }
-  float total[KIND == KIND_GLA ? RPL : 1];  // GLA: product of the segment's decays
-#pragma unroll
-  for (int r = 0; r < (KIND == KIND_GLA ? RPL : 1); ++r) total[r] = 1.f;
-
   load_block(0, t0);
   copy_commit();
   int buf = 0;
@@ -318,6 +371,7 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
     if (tb0 + TB < t1) load_block(buf ^ 1, tb0 + TB);
     copy_commit();
     const int n = min(TB, t1 - tb0);
+#pragma unroll 2
     for (int t = 0; t < n; ++t) {
       const float* x = stage + ((size_t)buf * TB + t) * stride;
       const float* xk = x + lr * 4;
@@ -328,21 +382,23 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
         o[c] = d[c] = 0.f;
       }
       if (KIND == KIND_DELTA) {
+        float d2[CPL];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) d2[c] = 0.f;
 #pragma unroll
         for (int j = 0; j < RPL / 4; ++j) {
           const float4 u = load4(xk + 3 * DKP + j * 32);
 #pragma unroll
           for (int c = 0; c < CPL; ++c) {
             d[c] = fmaf(u.x, s[4 * j][c], d[c]);
-            d[c] = fmaf(u.y, s[4 * j + 1][c], d[c]);
+            d2[c] = fmaf(u.y, s[4 * j + 1][c], d2[c]);
             d[c] = fmaf(u.z, s[4 * j + 2][c], d[c]);
-            d[c] = fmaf(u.w, s[4 * j + 3][c], d[c]);
+            d2[c] = fmaf(u.w, s[4 * j + 3][c], d2[c]);
           }
         }
 #pragma unroll
-        for (int off = 4; off > 0; off >>= 1)
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) d[c] += __shfl_xor_sync(ALL_LANES, d[c], off);
+        for (int c = 0; c < CPL; ++c) d[c] += d2[c];
+        group_all_reduce<CPL>(d, lr);
       }
 #pragma unroll
       for (int j = 0; j < RPL / 4; ++j) {
@@ -361,22 +417,21 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
             s[r][c] = fmaf(ww[i], s[r][c], add);
             o[c] = fmaf(qq[i], s[r][c], o[c]);
           }
-          if (KIND == KIND_GLA) total[KIND == KIND_GLA ? r : 0] *= ww[i];
         }
       }
       if (outputs) {
-#pragma unroll
-        for (int off = 4; off > 0; off >>= 1)
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) o[c] += __shfl_xor_sync(ALL_LANES, o[c], off);
-        if (lr == 0) {
-#pragma unroll
-          for (int c = 0; c < CPL; ++c) os[(size_t)t * COLS + col0 + c] = o[c] * l.q_scale;
-        }
+        const float total = group_reduce<CPL>(o, lr);
+        if (CPL == 4 ? (lr & 1) == 0 : CPL == 2 ? (lr & 3) == 0 : lr == 0)
+          os[(size_t)t * COLS + col0 + owned_column<CPL>(lr)] = total * l.q_scale;
       }
     }
     if (outputs) {
       __syncthreads();
+      if (sa.col_blocks > 1) {  // recurrence_output_kernel finishes the rows
+        for (int i = tid; i < n * dv; i += nthreads)
+          a.out_raw[(size_t)(tb0 + i / dv) * (l.heads * l.vdim) + head * l.vdim + cbase + i % dv] = os[(size_t)(i / dv) * COLS + i % dv];
+        continue;
+      }
       // head norm, gate and branch scale of the block's tokens, a warp per token
       for (int t = warp; t < n; t += W) {
         const float* o = os + (size_t)t * COLS;
@@ -407,11 +462,44 @@ __global__ void __launch_bounds__(512) recurrence_scan_kernel(ScanArgs sa) {
     if (row < dk) {
 #pragma unroll
       for (int c = 0; c < CPL; ++c)
-        if (col0 + c < dv) fin[(size_t)row * pitch + col0 + c] = s[r][c];
-      if (KIND == KIND_GLA && sa.mode == SCAN_LOCAL && warp == 0 && lane < 8)
-        sa.seg_trans[seg_index * dk + row] = total[KIND == KIND_GLA ? r : 0];
+        if (col0 + c < dv) fin[(size_t)row * pitch + cbase + col0 + c] = s[r][c];
     }
   }
+}
+
+// Head norm, gate and branch scale of scan outputs that left in several column blocks; a warp per (row, head).
+__global__ void __launch_bounds__(256) recurrence_output_kernel(RecurrenceScanArgs a, int y_bf16) {
+  const RecurrenceLayer& l = a.l;
+  const int lane = threadIdx.x & 31, dv = l.vdim;
+  const long long total = (long long)a.rows * l.heads;
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5; i < total; i += ((long long)gridDim.x * blockDim.x) >> 5) {
+    const int row = (int)(i / l.heads), head = (int)(i % l.heads);
+    const float* o = a.out_raw + (size_t)row * (l.heads * dv) + head * dv;
+    const float* g = a.p + (size_t)row * a.ldp + l.off_g + head * dv;
+    float sq = 0.f;
+    for (int c = lane; c < dv; c += 32) sq += o[c] * o[c];
+    const float rinv = 1.f / sqrtf(lane_sum(sq) / (float)dv + l.eps);
+    for (int c = lane; c < dv; c += 32) {
+      const float gate = l.kind == KIND_DELTA ? sigmoid_f(g[c]) : silu_f(g[c]);
+      const float y = o[c] * rinv * l.norm[l.kind == KIND_DELTA ? head * dv + c : c] * gate * l.out_scale;
+      const size_t at = (size_t)row * a.ldy + head * dv + c;
+      if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
+      else static_cast<float*>(a.y)[at] = y;
+    }
+  }
+}
+
+// Product of the decays of every segment, per key channel (GLA).
+__global__ void __launch_bounds__(256) segment_decay_kernel(ScanArgs sa) {
+  const RecurrenceScanArgs& a = sa.a;
+  const int K = a.l.heads * a.l.dim, seg = blockIdx.y, seq = blockIdx.z;
+  const int t0 = a.seq_start[seq] + seg * a.seg_tokens, t1 = min(a.seq_start[seq + 1], t0 + a.seg_tokens);
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (t0 >= t1 || c >= K) return;
+  float p = 1.f;
+#pragma unroll 8
+  for (int t = t0; t < t1; ++t) p *= a.decay[(size_t)t * K + c];
+  sa.seg_trans[((size_t)seq * a.max_segs + seg) * K + c] = p;
 }
 
 // Turns the segments' own contributions into their start states, in order: start[0] = cached state (or zero),
@@ -466,6 +554,16 @@ __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(Sca
 // ------------------------------------------------------------------ host side
 constexpr size_t MAX_SMEM = 227 * 1024;
 
+int sm_count() {
+  static const int n = [] {
+    int dev = 0, v = 148;
+    cudaGetDevice(&dev);
+    if (cudaDeviceGetAttribute(&v, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) v = 148;
+    return v;
+  }();
+  return n;
+}
+
 size_t scan_smem(int kind, int rpl, int cpl, int warps, int tb) {
   const size_t na = kind == KIND_DELTA ? 5 : 3, cols = (size_t)warps * 4 * cpl;
   return ((size_t)2 * tb * (na * 8 * rpl + 2 * cols) + (size_t)tb * cols) * sizeof(float);
@@ -484,22 +582,46 @@ cudaError_t launch_scan(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
 }
 
 template <int KIND, int RPL>
-cudaError_t launch_scan_cols(const ScanArgs& sa, dim3 grid, int cols, bool wide, cudaStream_t s) {
-  if (cols > 128 || (wide && RPL <= 16)) return launch_scan<KIND, RPL, 4>(sa, grid, cols, s);
-  if (cols > 64) return launch_scan<KIND, RPL, 2>(sa, grid, cols, s);
+cudaError_t launch_scan_cols(const ScanArgs& sa, dim3 grid, int cols, int cpl, cudaStream_t s) {
+  if (cpl == 4) return launch_scan<KIND, RPL, 4>(sa, grid, cols, s);
+  if (cpl == 2) return launch_scan<KIND, RPL, 2>(sa, grid, cols, s);
   return launch_scan<KIND, RPL, 1>(sa, grid, cols, s);
 }
 
-// `wide`: many blocks are in flight, so lanes take four columns each (fewer shared-memory reads per product)
-cudaError_t launch_scan_any(const ScanArgs& sa, dim3 grid, int cols, bool wide, cudaStream_t s) {
+int tune_int(const char* name, int otherwise) {
+  const char* e = getenv(name);
+  return e && *e ? atoi(e) : otherwise;
+}
+
+// `blocks` heads x sequences x segments are in flight. Few of them: the columns of a head are cut over several blocks
+// (64 at least). Lanes take as many columns as leave every block at least four warps, so that a staged key, decay and
+// query is read from shared memory for many products.
+cudaError_t launch_scan_any(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
   const int dk = sa.a.l.dim;
-#define PG_SCAN(KIND_)                                                                   \
-  (dk <= 32    ? launch_scan_cols<KIND_, 4>(sa, grid, cols, wide, s)                     \
-   : dk <= 64  ? launch_scan_cols<KIND_, 8>(sa, grid, cols, wide, s)                     \
-   : dk <= 128 ? launch_scan_cols<KIND_, 16>(sa, grid, cols, wide, s)                    \
-   : dk <= 256 ? launch_scan_cols<KIND_, 32>(sa, grid, cols, wide, s) : cudaErrorInvalidValue)
-  return sa.a.l.kind == KIND_DELTA ? PG_SCAN(KIND_DELTA) : PG_SCAN(KIND_GLA);
+  const long long blocks = (long long)grid.x * grid.y * grid.z;
+  int nb = (cols + 255) / 256;
+  while (nb * 2 * blocks <= sm_count() && (cols + nb * 2 - 1) / (nb * 2) >= 48) nb *= 2;
+  nb = std::max(nb, tune_int("PG_SCAN_BLOCKS", 0));
+  sa.block_cols = ((cols + nb - 1) / nb + 3) / 4 * 4;
+  sa.col_blocks = (cols + sa.block_cols - 1) / sa.block_cols;
+  grid.x *= sa.col_blocks;
+  const int bc = sa.block_cols;
+  int cpl = bc > 32 ? 4 : bc > 16 ? 2 : 1;
+  if (const int c = tune_int("PG_SCAN_CPL", 0)) cpl = std::max(c, (bc + 63) / 64);
+  if (cpl == 3) cpl = 4;
+#define PG_SCAN(KIND_)                                                                  \
+  (dk <= 32    ? launch_scan_cols<KIND_, 4>(sa, grid, bc, cpl, s)                       \
+   : dk <= 64  ? launch_scan_cols<KIND_, 8>(sa, grid, bc, cpl, s)                       \
+   : dk <= 128 ? launch_scan_cols<KIND_, 16>(sa, grid, bc, cpl, s)                      \
+   : dk <= 256 ? launch_scan_cols<KIND_, 32>(sa, grid, bc, cpl, s) : cudaErrorInvalidValue)
+  cudaError_t e = sa.a.l.kind == KIND_DELTA ? PG_SCAN(KIND_DELTA) : PG_SCAN(KIND_GLA);
 #undef PG_SCAN
+  if (e == cudaSuccess && sa.col_blocks > 1 && (sa.mode == SCAN_FULL || sa.mode == SCAN_OUTPUT)) {
+    const long long warps = (long long)sa.a.rows * sa.a.l.heads;
+    e = launch_kernel(recurrence_output_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 16)), dim3(256), 0, s, false, sa.a,
+                      sa.y_bf16);
+  }
+  return e;
 }
 
 }  // namespace
@@ -541,7 +663,7 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   sa.vec = m4(l.dim) && m4(l.vdim) && m4(l.off_k) && m4(l.off_q) && m4(l.off_v) && m4(l.off_g) && m4(a.ldp) && m4(K);
   if (a.max_segs <= 1 || !a.segments) {
     sa.mode = SCAN_FULL;
-    return launch_scan_any(sa, dim3(l.heads, a.nseq, 1), l.vdim, false, s);
+    return launch_scan_any(sa, dim3(l.heads, a.nseq, 1), l.vdim, s);
   }
   const size_t units = (size_t)a.nseq * a.max_segs * l.heads;
   sa.dkp = (l.dim + 3) / 4 * 4;
@@ -549,10 +671,13 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   sa.seg_trans = a.segments + units * l.dim * l.dvp;
   const dim3 grid(l.heads, a.nseq, a.max_segs);
   sa.mode = SCAN_LOCAL;
-  if ((e = launch_scan_any(sa, grid, l.vdim, true, s)) != cudaSuccess) return e;
+  if ((e = launch_scan_any(sa, grid, l.vdim, s)) != cudaSuccess) return e;
   if (l.kind == KIND_DELTA) {
     sa.mode = SCAN_TRANS;
-    if ((e = launch_scan_any(sa, grid, l.dim, true, s)) != cudaSuccess) return e;
+    if ((e = launch_scan_any(sa, grid, l.dim, s)) != cudaSuccess) return e;
+  } else {
+    e = launch_kernel(segment_decay_kernel, dim3((K + 255) / 256, a.max_segs, a.nseq), dim3(256), 0, s, false, sa);
+    if (e != cudaSuccess) return e;
   }
   const dim3 cgrid(l.heads, a.nseq, (l.vdim + COMBINE_COLS - 1) / COMBINE_COLS);
   const size_t csmem = (size_t)2 * l.dim * COMBINE_COLS * sizeof(float);
@@ -560,7 +685,7 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
                            : launch_kernel(recurrence_combine_kernel<KIND_GLA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa);
   if (e != cudaSuccess) return e;
   sa.mode = SCAN_OUTPUT;
-  return launch_scan_any(sa, grid, l.vdim, true, s);
+  return launch_scan_any(sa, grid, l.vdim, s);
 }
 
 }  // namespace pg
