@@ -19,21 +19,6 @@ namespace {
 
 constexpr int KB = 64;  // BF16 elements per k block: one 128-byte swizzle row
 
-// Two FP32 multiply-adds in one instruction.
-__device__ __forceinline__ unsigned long long pack2(float a, float b) {
-  unsigned long long r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ void unpack2(unsigned long long v, float& a, float& b) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
-}
-__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
-  unsigned long long r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-
 // z * Phi(z) of two values for results that are rounded to BF16 next. Phi(z) - 1/2 = z P(2 z^2 / 4.5^2 - 1) on
 // [-4.5, 4.5] with a degree-9 weighted least-squares fit of (Phi(z) - 1/2) / z on Chebyshev nodes; beyond that range Phi
 // is taken at its end. Absolute error below 1e-5 inside and 5e-5 outside.

@@ -54,7 +54,8 @@ struct LayeredModel {
   Norm final_norm;
   double* freq = nullptr;
   std::vector<DevLayer> layers;
-  int max_in = 0, max_y = 0, max_ff = 0, max_rec = 0, max_rec_out = 0;  // widest projection, mixer output, hidden row, heads * dim and heads * vdim of a recurrence
+  int max_in = 0, max_y = 0, max_ff = 0, max_rec = 0;  // widest projection, mixer output, hidden row, heads * dim ...
+  int max_rec_out = 0, max_rec_heads = 0;                  // ... heads * vdim and heads of a recurrence
   int n_pools = 0, n_states = 0;
   std::vector<int> spans;  // one page table each
   std::vector<void*> allocations;
@@ -84,7 +85,7 @@ struct LayeredCache {
   float* attn_part = nullptr;
   unsigned* attn_counters = nullptr;
   // portion workspaces (grow-only)
-  float *decay = nullptr, *unit = nullptr, *rate = nullptr, *out_raw = nullptr, *segments = nullptr;
+  float *decay = nullptr, *unit = nullptr, *rate = nullptr, *unit_next = nullptr, *pair = nullptr, *out_raw = nullptr, *segments = nullptr;
   void *q = nullptr, *k = nullptr, *v = nullptr;
   int* meta = nullptr;
   float* logits = nullptr;
@@ -95,7 +96,7 @@ struct LayeredCache {
     for (LayeredRows* r : {&step, &portion})
       for (void* p : {(void*)r->x[0], (void*)r->x[1], (void*)r->p, (void*)r->yo, r->h, r->y, r->ff, (void*)r->h32, (void*)r->y32, (void*)r->ff32})
         if (p) cudaFree(p);
-    for (void* p : {(void*)attn_part, (void*)attn_counters, (void*)decay, (void*)unit, (void*)rate, (void*)out_raw, (void*)segments, q, k, v,
+    for (void* p : {(void*)attn_part, (void*)attn_counters, (void*)decay, (void*)unit, (void*)rate, (void*)unit_next, (void*)pair, (void*)out_raw, (void*)segments, q, k, v,
                     (void*)meta, (void*)logits})
       if (p) cudaFree(p);
   }
@@ -238,6 +239,7 @@ int build_layer(Builder& b, const LayerSpec& spec, const std::string& p, int pag
       br.state = m->n_states++;
       m->max_rec = std::max(m->max_rec, K);
       m->max_rec_out = std::max(m->max_rec_out, V);
+      m->max_rec_heads = std::max(m->max_rec_heads, s.heads);
     }
     d->branches.push_back(br);
   }
@@ -624,7 +626,8 @@ cudaError_t enqueue_portions(pg_cache* c, const PortionPlan& plan, const Portion
         RecurrenceScanArgs a{};
         a.l = b.rec; a.p = r.p; a.ldp = l.in.np; a.rows = rows; a.nseq = plan.n();
         a.seq_start = d.seq_start; a.seq_slot = d.slot; a.seq_pos = d.start_pos; a.state = lc->states[b.state];
-        a.decay = lc->decay; a.unit = lc->unit; a.rate = lc->rate; a.out_raw = lc->out_raw;
+        a.decay = lc->decay; a.unit = lc->unit; a.rate = lc->rate; a.unit_next = lc->unit_next; a.pair = lc->pair;
+        a.out_raw = lc->out_raw; a.error_flag = c->d_error;
         a.segments = lc->segments; a.seg_tokens = SEGMENT_TOKENS;
         a.max_segs = recurrence_use_segments(b.rec, plan.n(), plan.max_len, max_segs) ? max_segs : 0;
         a.y = y; a.ldy = l.out.kp;
@@ -700,7 +703,9 @@ int layered_run_portions(pg_cache* c, const PortionPlan& plan, float* logits, St
     }
   }
   if (m->max_rec && (size_t)rows > lc->gate_rows) {
-    size_t g = lc->gate_rows, h = g, o = g;
+    size_t g = lc->gate_rows, h = g, o = g, x = g, y = g;
+    if (int r = grow(&lc->unit_next, &x, rows, m->max_rec * sizeof(float))) return r;
+    if (int r = grow(&lc->pair, &y, rows, m->max_rec_heads * 4 * sizeof(float))) return r;
     if (int r = grow(&lc->out_raw, &o, rows, m->max_rec_out * sizeof(float))) return r;
     if (int r = grow(&lc->decay, &g, rows, m->max_rec * sizeof(float))) return r;
     if (int r = grow(&lc->unit, &h, rows, m->max_rec * sizeof(float))) return r;

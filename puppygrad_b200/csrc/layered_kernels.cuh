@@ -101,7 +101,10 @@ struct RecurrenceScanArgs {  // whole portions of `nseq` sequences
   const int* seq_slot;   // [nseq]
   const int* seq_pos;    // [nseq] position of the first row; 0 starts from a zero state
   float* state;
-  float *decay, *unit, *rate;  // [rows, heads * dim] scratch: decay; delta: unit key, a * u
+  float *decay, *unit, *rate;  // [rows, heads * dim] scratch: decay; delta: unit key u, a * u ...
+  float *unit_next;            // ... and the next token's u times this token's decay
+  float *pair;                 // [rows, heads, 4] delta: next u . (a * u), next u . k
+  int* error_flag;
   float* out_raw;              // [rows, heads * vdim] scratch: outputs before the head norm
   float* segments;             // scratch of the segmented scan (may be nullptr)
   int seg_tokens, max_segs;    // tokens per segment, segments of the longest sequence (0: one pass)

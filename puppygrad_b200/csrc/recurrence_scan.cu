@@ -1,0 +1,726 @@
+// Recurrent mixers over whole portions of prompts: the gates of every row, the scan, and for long portions its
+// segmented form. Everything that enters the recurrence is FP32.
+//
+// Both rules act on every column of a head's [dim, vdim] state on its own (S[:, c] needs only v[c] of the new token), so
+// a column's `dim` entries are spread over eight lanes and the columns over groups of lanes, warps and blocks.
+#include <algorithm>
+#include <cstdlib>
+
+#include "recurrence.cuh"
+#include "tc_common.cuh"
+
+namespace pg {
+namespace {
+
+// ------------------------------------------------------------------ gates
+constexpr int GATE_ROWS = 16;
+// decay of GATE_ROWS rows x 256 key channels per block
+__global__ void __launch_bounds__(256) recurrence_decay_kernel(RecurrenceScanArgs a) {
+  extern __shared__ __align__(16) float sm[];  // [rank][GATE_ROWS]
+  const RecurrenceLayer& l = a.l;
+  const int K = l.heads * l.dim, r0 = blockIdx.x * GATE_ROWS, tid = threadIdx.x, c = blockIdx.y * 256 + tid;
+  const int nr = min(GATE_ROWS, a.rows - r0);
+  for (int i = tid; i < GATE_ROWS * l.rank; i += 256) {
+    const int j = i / l.rank, r = i - j * l.rank;
+    const float t = j < nr ? a.p[(size_t)(r0 + j) * a.ldp + l.off_t + r] : 0.f;
+    sm[r * GATE_ROWS + j] = l.kind == KIND_DELTA ? tanhf(t) : t;
+  }
+  __syncthreads();
+  if (c >= K) return;
+  float z[GATE_ROWS];
+#pragma unroll
+  for (int j = 0; j < GATE_ROWS; ++j) z[j] = l.b2[c];
+  const float* __restrict__ w2 = l.w2 + c;
+#pragma unroll 8
+  for (int r = 0; r < l.rank; ++r) {
+    const float w = w2[(size_t)r * K];
+#pragma unroll
+    for (int j = 0; j < GATE_ROWS; j += 4) {
+      const float4 t = load4(sm + r * GATE_ROWS + j);
+      z[j] = fmaf(w, t.x, z[j]);
+      z[j + 1] = fmaf(w, t.y, z[j + 1]);
+      z[j + 2] = fmaf(w, t.z, z[j + 2]);
+      z[j + 3] = fmaf(w, t.w, z[j + 3]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < GATE_ROWS; ++j)
+    if (j < nr) a.decay[(size_t)(r0 + j) * K + c] = decay_of(l.kind, z[j], l.inv_tau);
+}
+
+// Delta rule, after the decays; a warp per (row, head): the unit key u, the removal rate a * u, and what the scan needs
+// to take two tokens at a time: the next token's u times this one's decay, next u . (a * u), next u . k.
+__global__ void __launch_bounds__(256) delta_gates_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int K = l.heads * l.dim, lane = threadIdx.x & 31;
+  const long long total = (long long)a.rows * l.heads;
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5; i < total; i += ((long long)gridDim.x * blockDim.x) >> 5) {
+    const int row = (int)(i / l.heads), head = (int)(i % l.heads);
+    const float* pr = a.p + (size_t)row * a.ldp;
+    const float* k = pr + l.off_k + head * l.dim;
+    const float* kn = row + 1 < a.rows ? k + a.ldp : k;  // unused where the next row is another sequence's
+    float s = 0.f, sn = 0.f;
+    for (int c = lane; c < l.dim; c += 32) {
+      s += k[c] * k[c];
+      sn += kn[c] * kn[c];
+    }
+    const float inv = 1.f / sqrtf(lane_sum(s) + UNIT_EPS), invn = 1.f / sqrtf(lane_sum(sn) + UNIT_EPS);
+    float ub = 0.f, uk = 0.f;
+    for (int c = lane; c < l.dim; c += 32) {
+      const int ch = head * l.dim + c;
+      const size_t at = (size_t)row * K + ch;
+      const float u = k[c] * inv, un = kn[c] * invn, b = sigmoid_f(pr[l.off_a + ch] + l.a_bias[ch]) * u;
+      a.unit[at] = u;
+      a.rate[at] = b;
+      a.unit_next[at] = un * a.decay[at];
+      ub += un * b;
+      uk += un * k[c];
+    }
+    ub = lane_sum(ub);
+    uk = lane_sum(uk);
+    if (lane == 0) store4(a.pair + (size_t)i * 4, make_float4(ub, uk, 0.f, 0.f));
+  }
+}
+
+// ------------------------------------------------------------------ scan
+// Block = one head of one sequence (or of one segment of it), or a part of its columns. The last warp stages the rows of
+// TB tokens at a time in a ring of shared-memory stages (bulk copies where rows are 16-byte aligned); in the others
+// eight lanes share a column (lane l holds rows 32 j + 4 l + i), a group of eight has CPL columns, a warp four groups.
+// A lane's share of an output goes to shared memory; after TB tokens the shares are added and the head norm and output
+// gate applied.
+enum ScanMode {
+  SCAN_FULL = 0,     // whole sequence: start from the cached state (or zero), outputs, final state to the cache
+  SCAN_LOCAL = 1,    // one segment from a zero state, no outputs: its contribution to the state
+  SCAN_TRANS = 2,    // one segment with identity columns and no values: its transition matrix (delta)
+  SCAN_OUTPUT = 3    // one segment from its known start state: outputs
+};
+constexpr int SCAN_WARPS = 8;   // at most: 32 CPL columns
+constexpr int SCAN_STAGES = 3;
+struct ScanArgs {
+  RecurrenceScanArgs a;
+  int mode, tb;
+  float *seg_state, *seg_trans;  // [nseq][max_segs][heads][dim][dvp], [nseq][max_segs][heads][dim][dkp] (GLA: [..][dim] decays)
+  int dkp;
+  int col_blocks, block_cols;  // column blocks of a head, columns of each (the last may have fewer)
+  int vec;      // rows can be copied in 16-byte pieces
+  int y_bf16;
+};
+
+__device__ __forceinline__ void bulk_row(float* dst, const float* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)), "l"(src),
+               "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
+__device__ __forceinline__ void named_barrier(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+
+// Sums of N values over the eight lanes of a group, in every lane: halves are exchanged on the way down, totals on the
+// way back.
+template <int N, int OFF>
+struct GroupSum {
+  static __device__ __forceinline__ void run(float* v, int lr) {
+    const bool up = lr & OFF;
+    if (N > 1) {
+      constexpr int H = N > 1 ? N / 2 : 1;
+#pragma unroll
+      for (int i = 0; i < H; ++i) {
+        const float send = up ? v[i] : v[i + H], keep = up ? v[i + H] : v[i];
+        v[i] = keep + __shfl_xor_sync(ALL_LANES, send, OFF);
+      }
+      GroupSum<H, OFF / 2>::run(v, lr);
+#pragma unroll
+      for (int i = 0; i < H; ++i) {
+        const float other = __shfl_xor_sync(ALL_LANES, v[i], OFF), own = v[i];
+        v[i] = up ? other : own;
+        v[i + H] = up ? own : other;
+      }
+    } else {
+      v[0] += __shfl_xor_sync(ALL_LANES, v[0], OFF);
+      GroupSum<1, OFF / 2>::run(v, lr);
+    }
+  }
+};
+template <int N>
+struct GroupSum<N, 0> {
+  static __device__ __forceinline__ void run(float*, int) {}
+};
+
+// The delta rule works on two tokens at a time: with e = (u' * w)^T S, where the dash marks the second token,
+// u'^T S_t = e - (u' . b) d + (u' . k) v, so that both reads come from one reduction over the state before the pair.
+template <int KIND, int RPL, int CPL>
+__global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kernel(ScanArgs sa) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ uint64_t full[SCAN_STAGES], empty[SCAN_STAGES];
+  __shared__ int failed_flag;
+  constexpr int DKP = 8 * RPL, NA = KIND == KIND_DELTA ? 6 : 3, J = RPL / 4;  // staged key-channel arrays
+  const RecurrenceScanArgs& a = sa.a;
+  const RecurrenceLayer& l = a.l;
+  const int dk = l.dim, K = l.heads * dk, tid = threadIdx.x;
+  const bool trans = sa.mode == SCAN_TRANS;
+  // blockIdx.x = head * (column blocks) + column block; with several column blocks per head the outputs leave unnormed
+  const int head = blockIdx.x / sa.col_blocks, cb = blockIdx.x % sa.col_blocks, seq = blockIdx.y, seg = blockIdx.z;
+  const int all_cols = trans ? dk : l.vdim, cbase = cb * sa.block_cols;
+  const int dv = min(sa.block_cols, all_cols - cbase);  // columns of this block
+  const int W = (blockDim.x >> 5) - 1, COLS = W * 4 * CPL, TB = sa.tb;
+  // floats of one staged token: k, decay, q, (u, rate, next u * decay), v, gate, (next u . rate, next u . k)
+  const int stride = NA * DKP + 2 * COLS + 4, OP = COLS + 4;
+  float* stage = sm;                                   // [SCAN_STAGES][TB][stride]
+  float* os0 = sm + (size_t)SCAN_STAGES * TB * stride;  // [2][TB][8 lanes of a group][OP]
+  const int lane = tid & 31, warp = tid >> 5;
+  const bool outputs = sa.mode == SCAN_FULL || sa.mode == SCAN_OUTPUT;
+  const bool want_v = !trans, want_g = outputs && sa.col_blocks == 1;
+  volatile int* failed = &failed_flag;
+
+  int t0 = a.seq_start[seq], t1 = a.seq_start[seq + 1];
+  if (sa.mode != SCAN_FULL) {
+    t0 += seg * a.seg_tokens;
+    t1 = min(t1, t0 + a.seg_tokens);
+    if (t0 >= t1) return;
+  }
+  for (int i = tid; i < SCAN_STAGES * TB * stride; i += blockDim.x) stage[i] = 0.f;  // the padding stays zero
+  if (tid == 0) {
+    for (int i = 0; i < SCAN_STAGES; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], (uint32_t)W);
+    }
+    failed_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the zeros come before the bulk copies
+  __syncthreads();
+  const int blocks = (t1 - t0 + TB - 1) / TB;
+
+  if (warp == W) {  // ---- stages rows; lane = (token, array)
+    const int arr = lane & 7;  // key-channel arrays, then values, then gates (GLA: lanes 5..7 idle; delta: all busy)
+    const bool key = arr < NA, value = arr == NA && want_v, gate = arr == NA + 1 && want_g;
+    const bool on = (key && !(arr == 2 && !outputs)) || value || gate;
+    const float* src = nullptr;
+    int pitch = a.ldp, off = 0;
+    if (key) {
+      off = arr * DKP;
+      const float* gates[4] = {a.decay, a.unit, a.rate, a.unit_next};
+      if (arr == 0) src = a.p + l.off_k + head * dk;
+      else if (arr == 2) src = a.p + l.off_q + head * dk;
+      else {
+        src = gates[arr == 1 ? 0 : arr - 2] + head * dk;
+        pitch = K;
+      }
+    } else if (value || gate) {
+      off = NA * DKP + (gate ? COLS : 0);
+      src = a.p + (gate ? l.off_g : l.off_v) + head * l.vdim + cbase;
+    }
+    const int count = key ? dk : dv;
+    const uint32_t token_bytes = 4u * (uint32_t)((NA - (outputs ? 0 : 1)) * dk + (want_v ? dv : 0) + (want_g ? dv : 0)) +
+                                 (KIND == KIND_DELTA ? 16u : 0u);
+    for (int b = 0; b < blocks; ++b) {
+      const int s = b % SCAN_STAGES, tb0 = t0 + b * TB, n = min(TB, t1 - tb0);
+      if (b >= SCAN_STAGES && !mbar_wait(&empty[s], ((b / SCAN_STAGES) - 1) & 1, failed, a.error_flag, 41)) break;
+      __syncwarp();
+      float* dst = stage + (size_t)s * TB * stride;
+      if (sa.vec) {
+        if (lane == 0) mbar_expect_tx(&full[s], (uint32_t)n * token_bytes);
+        __syncwarp();
+        if (on)
+          for (int t = lane >> 3; t < n; t += 4)
+            bulk_row(dst + (size_t)t * stride + off, src + (size_t)(tb0 + t) * pitch, (uint32_t)(4 * count), &full[s]);
+        if (KIND == KIND_DELTA)
+          for (int t = lane; t < n; t += 32)
+            bulk_row(dst + (size_t)t * stride + NA * DKP + 2 * COLS, a.pair + ((size_t)(tb0 + t) * l.heads + head) * 4, 16, &full[s]);
+      } else {
+        if (on)
+          for (int t = lane >> 3; t < n; t += 4)
+            for (int i = 0; i < count; ++i) dst[(size_t)t * stride + off + i] = src[(size_t)(tb0 + t) * pitch + i];
+        if (KIND == KIND_DELTA)
+          for (int t = lane; t < n; t += 32)
+            store4(dst + (size_t)t * stride + NA * DKP + 2 * COLS, load4(a.pair + ((size_t)(tb0 + t) * l.heads + head) * 4));
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&full[s]);
+      }
+    }
+    return;
+  }
+
+  // ---- start state, two neighbouring rows per register pair
+  const int lr = lane & 7, col0 = (warp * 4 + (lane >> 3)) * CPL;
+  unsigned long long s[RPL / 2][CPL];
+  const size_t seg_index = ((size_t)seq * a.max_segs + seg) * l.heads + head;
+  const float* init = nullptr;
+  if (sa.mode == SCAN_FULL && a.seq_pos[seq] > 0) init = a.state + ((size_t)a.seq_slot[seq] * l.heads + head) * dk * l.dvp;
+  if (sa.mode == SCAN_OUTPUT) init = sa.seg_state + seg_index * dk * l.dvp;
+  auto row_of = [&](int r) { return (r >> 2) * 32 + lr * 4 + (r & 3); };
+#pragma unroll
+  for (int r = 0; r < RPL; r += 2) {
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      const int col = col0 + c;
+      float v[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int row = row_of(r + e);
+        v[e] = 0.f;
+        if (row < dk && col < dv) {
+          if (init) v[e] = init[(size_t)row * l.dvp + cbase + col];
+          else if (trans) v[e] = row == cbase + col ? 1.f : 0.f;
+        }
+      }
+      s[r / 2][c] = pack2(v[0], v[1]);
+    }
+  }
+
+  using Row = ulonglong2;  // four entries of a key-channel row
+  for (int b = 0; b < blocks; ++b) {
+    const int sidx = b % SCAN_STAGES, tb0 = t0 + b * TB, n = min(TB, t1 - tb0);
+    mbar_wait(&full[sidx], (b / SCAN_STAGES) & 1, failed, a.error_flag, 42);  // on expiry the numbers are void, the barriers below are kept
+    __syncwarp();
+    const float* x0 = stage + (size_t)sidx * TB * stride;
+    float* os = os0 + (size_t)(b & 1) * TB * 8 * OP;
+
+    auto values = [&](const float* x, float (&v)[CPL]) {
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) v[c] = x[NA * DKP + col0 + c];
+    };
+    auto fetch = [&](const float* x, int arr, Row (&r)[J]) {
+#pragma unroll
+      for (int j = 0; j < J; ++j) r[j] = *reinterpret_cast<const Row*>(x + arr * DKP + j * 32 + lr * 4);
+    };
+    auto dot = [&](const Row (&u)[J], float* d) {
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        unsigned long long e = 0, f = 0;
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+          e = fma2(u[j].x, s[2 * j][c], e);
+          f = fma2(u[j].y, s[2 * j + 1][c], f);
+        }
+        float x, y, z, w;
+        unpack2(e, x, y);
+        unpack2(f, z, w);
+        d[c] = (x + y) + (z + w);
+      }
+    };
+    // one token: S = w S - b d + k v, and this lane's share of S^T q
+    auto token = [&](int t, const Row (&k)[J], const Row (&w)[J], const Row (&q)[J], const Row (&bb)[J], const float (&v)[CPL], const float* d) {
+      unsigned long long o[CPL], vv[CPL], dd[CPL];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        o[c] = 0;
+        vv[c] = pack2(v[c], v[c]);
+        dd[c] = KIND == KIND_DELTA ? pack2(-d[c], -d[c]) : 0;
+      }
+#pragma unroll
+      for (int j = 0; j < J; ++j) {
+        const unsigned long long kk[2] = {k[j].x, k[j].y}, ww[2] = {w[j].x, w[j].y}, qq[2] = {q[j].x, q[j].y}, rr[2] = {bb[j].x, bb[j].y};
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int r = 2 * j + i;
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) {
+            unsigned long long add = mul2(kk[i], vv[c]);
+            if (KIND == KIND_DELTA) add = fma2(rr[i], dd[c], add);
+            s[r][c] = fma2(ww[i], s[r][c], add);
+            o[c] = fma2(qq[i], s[r][c], o[c]);
+          }
+        }
+      }
+      if (outputs) {
+        float* po = os + (size_t)(t * 8 + lr) * OP + col0;
+        float r[CPL];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          float x, y;
+          unpack2(o[c], x, y);
+          r[c] = x + y;
+        }
+        if (CPL == 4) store4(po, make_float4(r[0], r[1 % CPL], r[2 % CPL], r[3 % CPL]));
+        else if (CPL == 2) *reinterpret_cast<float2*>(po) = make_float2(r[0], r[1 % CPL]);
+        else po[0] = r[0];
+      }
+    };
+    if (KIND == KIND_GLA) {
+#pragma unroll 2
+      for (int t = 0; t < n; ++t) {
+        const float* x = x0 + (size_t)t * stride;
+        Row k[J], w[J], q[J];
+        float v[CPL];
+        fetch(x, 0, k);
+        fetch(x, 1, w);
+        fetch(x, 2, q);
+        values(x, v);
+        token(t, k, w, q, k, v, nullptr);
+      }
+    } else {
+      int t = 0;
+      for (; t + 1 < n; t += 2) {
+        const float *xa = x0 + (size_t)t * stride, *xb = xa + stride;
+        float d[2 * CPL], va[CPL], vb[CPL];
+        Row k[J], w[J], q[J], r[J];
+        fetch(xa, 3, k);
+        fetch(xa, 5, w);
+        dot(k, d);
+        dot(w, d + CPL);
+        fetch(xa, 0, k);
+        fetch(xa, 1, w);
+        fetch(xa, 2, q);
+        fetch(xa, 4, r);
+        values(xa, va);
+        const float2 ab = *reinterpret_cast<const float2*>(xa + NA * DKP + 2 * COLS);
+        GroupSum<2 * CPL, 4>::run(d, lr);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) d[CPL + c] = fmaf(ab.y, va[c], fmaf(-ab.x, d[c], d[CPL + c]));
+        token(t, k, w, q, r, va, d);
+        fetch(xb, 0, k);
+        fetch(xb, 1, w);
+        fetch(xb, 2, q);
+        fetch(xb, 4, r);
+        values(xb, vb);
+        token(t + 1, k, w, q, r, vb, d + CPL);
+      }
+      if (t < n) {
+        const float* xa = x0 + (size_t)t * stride;
+        float d[CPL], va[CPL];
+        Row k[J], w[J], q[J], r[J];
+        fetch(xa, 3, k);
+        dot(k, d);
+        fetch(xa, 0, k);
+        fetch(xa, 1, w);
+        fetch(xa, 2, q);
+        fetch(xa, 4, r);
+        values(xa, va);
+        GroupSum<CPL, 4>::run(d, lr);
+        token(t, k, w, q, r, va, d);
+      }
+    }
+    if (outputs) {
+      // every warp's shares are in; this buffer is written again two blocks on, after the next barrier
+      named_barrier(1, W * 32);
+      for (int t = warp; t < n; t += W) {
+        const float* po = os + (size_t)t * 8 * OP;
+        const float* g = x0 + (size_t)t * stride + NA * DKP + COLS;
+        float o[4], sq = 0.f;  // at most 128 columns
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int c = lane + i * 32;
+          float x = 0.f;
+          if (c < dv) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x += po[e * OP + c];
+          }
+          o[i] = x * l.q_scale;
+          sq += o[i] * o[i];
+        }
+        if (sa.col_blocks > 1) {  // recurrence_output_kernel finishes the rows
+          float* out = a.out_raw + (size_t)(tb0 + t) * (l.heads * l.vdim) + head * l.vdim + cbase;
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (lane + i * 32 < dv) out[lane + i * 32] = o[i];
+        } else {
+          const float rinv = 1.f / sqrtf(lane_sum(sq) / (float)dv + l.eps);
+          const size_t base = (size_t)(tb0 + t) * a.ldy + head * dv;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int c = lane + i * 32;
+            if (c < dv) {
+              const float gate = KIND == KIND_DELTA ? sigmoid_f(g[c]) : silu_f(g[c]);
+              const float y = o[i] * rinv * l.norm[KIND == KIND_DELTA ? head * dv + c : c] * gate * l.out_scale;
+              if (sa.y_bf16) static_cast<__nv_bfloat16*>(a.y)[base + c] = __float2bfloat16_rn(y);
+              else static_cast<float*>(a.y)[base + c] = y;
+            }
+          }
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[sidx]);
+  }
+
+  if (sa.mode == SCAN_OUTPUT) return;
+  float* fin = sa.mode == SCAN_FULL ? a.state + ((size_t)a.seq_slot[seq] * l.heads + head) * dk * l.dvp
+               : trans              ? sa.seg_trans + seg_index * dk * sa.dkp
+                                    : sa.seg_state + seg_index * dk * l.dvp;
+  const int pitch = trans ? sa.dkp : l.dvp;
+#pragma unroll
+  for (int r = 0; r < RPL; r += 2)
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      float v[2];
+      unpack2(s[r / 2][c], v[0], v[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (row_of(r + e) < dk && col0 + c < dv) fin[(size_t)row_of(r + e) * pitch + cbase + col0 + c] = v[e];
+    }
+}
+
+// Head norm, gate and branch scale of scan outputs that left in several column blocks; a warp per (row, head), at most
+// 256 columns.
+__global__ void __launch_bounds__(256) recurrence_output_kernel(RecurrenceScanArgs a, int y_bf16) {
+  const RecurrenceLayer& l = a.l;
+  const int lane = threadIdx.x & 31, dv = l.vdim;
+  const long long total = (long long)a.rows * l.heads;
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5; i < total; i += ((long long)gridDim.x * blockDim.x) >> 5) {
+    const int row = (int)(i / l.heads), head = (int)(i % l.heads);
+    const float* o = a.out_raw + (size_t)row * (l.heads * dv) + head * dv;
+    const float* g = a.p + (size_t)row * a.ldp + l.off_g + head * dv;
+    float ov[8], gv[8], sq = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = lane + j * 32;
+      ov[j] = c < dv ? o[c] : 0.f;
+      gv[j] = c < dv ? g[c] : 0.f;
+      sq += ov[j] * ov[j];
+    }
+    const float rinv = 1.f / sqrtf(lane_sum(sq) / (float)dv + l.eps);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = lane + j * 32;
+      if (c >= dv) break;
+      const float gate = l.kind == KIND_DELTA ? sigmoid_f(gv[j]) : silu_f(gv[j]);
+      const float y = ov[j] * rinv * l.norm[l.kind == KIND_DELTA ? head * dv + c : c] * gate * l.out_scale;
+      const size_t at = (size_t)row * a.ldy + head * dv + c;
+      if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
+      else static_cast<float*>(a.y)[at] = y;
+    }
+  }
+}
+
+// Product of the decays of every segment, per key channel (GLA).
+__global__ void __launch_bounds__(256) segment_decay_kernel(ScanArgs sa) {
+  const RecurrenceScanArgs& a = sa.a;
+  const int K = a.l.heads * a.l.dim, seg = blockIdx.y, seq = blockIdx.z;
+  const int t0 = a.seq_start[seq] + seg * a.seg_tokens, t1 = min(a.seq_start[seq + 1], t0 + a.seg_tokens);
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (t0 >= t1 || c >= K) return;
+  float p = 1.f;
+#pragma unroll 8
+  for (int t = t0; t < t1; ++t) p *= a.decay[(size_t)t * K + c];
+  sa.seg_trans[((size_t)seq * a.max_segs + seg) * K + c] = p;
+}
+
+// Turns the segments' own contributions into their start states, in order: start[0] = cached state (or zero),
+// start[i + 1] = transition[i] start[i] + local[i]; the last one goes to the cache. Block = 16 columns of one head of
+// one sequence; the running state stays in shared memory, the next segment's numbers load one segment ahead.
+constexpr int COMBINE_COLS = 16, COMBINE_THREADS = 256;
+template <int KIND>
+__global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(ScanArgs sa) {
+  extern __shared__ __align__(16) float sm[];
+  const RecurrenceScanArgs& a = sa.a;
+  const RecurrenceLayer& l = a.l;
+  const int dk = l.dim, head = blockIdx.x, seq = blockIdx.y, c0 = blockIdx.z * COMBINE_COLS, tid = threadIdx.x;
+  const int nc = min(COMBINE_COLS, l.vdim - c0);
+  const int len = a.seq_start[seq + 1] - a.seq_start[seq], segs = (len + a.seg_tokens - 1) / a.seg_tokens;
+  const int tp = sa.dkp + 4;               // pitch of a transition row in shared memory
+  float* cur = sm;                         // [dk][COMBINE_COLS]
+  float* nxt = sm + dk * COMBINE_COLS;
+  float* tr = sm + 2 * dk * COMBINE_COLS;  // delta: [2][dk][tp], the next one loading
+  float* cached = a.state + ((size_t)a.seq_slot[seq] * l.heads + head) * dk * l.dvp;
+  const bool fresh = a.seq_pos[seq] == 0;
+  constexpr int MAX_PER = 256 * COMBINE_COLS / COMBINE_THREADS;  // dk <= 256
+  const int per = (dk * COMBINE_COLS + COMBINE_THREADS - 1) / COMBINE_THREADS;
+  auto seg_at = [&](int g) { return ((size_t)seq * a.max_segs + g) * l.heads + head; };
+  auto load_trans = [&](int g, float* dst) {
+    const float* src = sa.seg_trans + seg_at(g) * dk * sa.dkp;
+    const int row4 = sa.dkp / 4;
+    for (int i = tid; i < dk * row4; i += COMBINE_THREADS) {
+      const int r = i / row4, x = i - r * row4;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + r * tp + x * 4)), "l"(src + (size_t)i * 4) : "memory");
+    }
+  };
+  float loc[MAX_PER], dec[MAX_PER];
+  auto load_next = [&](int g) {
+    const float* p = sa.seg_state + seg_at(g) * dk * l.dvp;
+#pragma unroll
+    for (int q = 0; q < MAX_PER; ++q) {
+      const int i = tid + q * COMBINE_THREADS, r = i / COMBINE_COLS, c = i % COMBINE_COLS;
+      if (q < per && r < dk) {
+        loc[q] = c < nc ? p[(size_t)r * l.dvp + c0 + c] : 0.f;
+        if (KIND == KIND_GLA) dec[q] = sa.seg_trans[seg_at(g) * dk + r];
+      }
+    }
+  };
+  for (int i = tid; i < dk * COMBINE_COLS; i += COMBINE_THREADS) {
+    const int r = i / COMBINE_COLS, c = i % COMBINE_COLS;
+    cur[i] = (!fresh && c < nc) ? cached[(size_t)r * l.dvp + c0 + c] : 0.f;
+  }
+  load_next(0);
+  if (KIND == KIND_DELTA) load_trans(0, tr);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  for (int g = 0; g < segs; ++g) {
+    float v[MAX_PER], w[MAX_PER];
+#pragma unroll
+    for (int q = 0; q < MAX_PER; ++q) {
+      v[q] = loc[q];
+      w[q] = KIND == KIND_GLA ? dec[q] : 0.f;
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (g + 1 < segs) {
+      load_next(g + 1);
+      if (KIND == KIND_DELTA) load_trans(g + 1, tr + (size_t)((g + 1) & 1) * dk * tp);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    float* start = sa.seg_state + seg_at(g) * dk * l.dvp;
+    const float* m = tr + (size_t)(g & 1) * dk * tp;
+#pragma unroll
+    for (int q = 0; q < MAX_PER; ++q) {
+      const int i = tid + q * COMBINE_THREADS, r = i / COMBINE_COLS, c = i % COMBINE_COLS;
+      if (q < per && r < dk) {
+        const float old = cur[i];
+        float x = v[q];
+        if (KIND == KIND_GLA) {
+          x = fmaf(w[q], old, x);
+        } else {
+          float e = 0.f, f = 0.f;
+          int j = 0;
+          for (; j + 3 < dk; j += 4) {
+            const float4 t = load4(m + (size_t)r * tp + j);
+            e = fmaf(t.x, cur[j * COMBINE_COLS + c], e);
+            f = fmaf(t.y, cur[(j + 1) * COMBINE_COLS + c], f);
+            e = fmaf(t.z, cur[(j + 2) * COMBINE_COLS + c], e);
+            f = fmaf(t.w, cur[(j + 3) * COMBINE_COLS + c], f);
+          }
+          for (; j < dk; ++j) e = fmaf(m[(size_t)r * tp + j], cur[j * COMBINE_COLS + c], e);
+          x += e + f;
+        }
+        if (c < nc) start[(size_t)r * l.dvp + c0 + c] = old;
+        nxt[i] = x;
+      }
+    }
+    __syncthreads();
+    float* t = cur;
+    cur = nxt;
+    nxt = t;
+  }
+  for (int i = tid; i < dk * COMBINE_COLS; i += COMBINE_THREADS) {
+    const int r = i / COMBINE_COLS, c = i % COMBINE_COLS;
+    if (c < nc) cached[(size_t)r * l.dvp + c0 + c] = cur[i];
+  }
+}
+
+// ------------------------------------------------------------------ host side
+constexpr size_t MAX_SMEM = 225 * 1024;  // beside a little static shared memory
+
+int sm_count() {
+  static const int n = [] {
+    int dev = 0, v = 148;
+    cudaGetDevice(&dev);
+    if (cudaDeviceGetAttribute(&v, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) v = 148;
+    return v;
+  }();
+  return n;
+}
+
+int tune_int(const char* name, int otherwise) {
+  const char* e = getenv(name);
+  return e && *e ? atoi(e) : otherwise;
+}
+
+size_t scan_smem(int kind, int rpl, int cpl, int warps, int tb) {
+  const size_t na = kind == KIND_DELTA ? 6 : 3, cols = (size_t)warps * 4 * cpl;
+  return ((size_t)SCAN_STAGES * tb * (na * 8 * rpl + 2 * cols + 4) + (size_t)2 * tb * 8 * (cols + 4)) * sizeof(float);
+}
+
+template <int KIND, int RPL, int CPL>
+cudaError_t launch_scan(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
+  const int warps = (cols + 4 * CPL - 1) / (4 * CPL);
+  if (warps > SCAN_WARPS) return cudaErrorInvalidValue;
+  sa.tb = 16;
+  while (sa.tb > 2 && scan_smem(KIND, RPL, CPL, warps, sa.tb) > MAX_SMEM) sa.tb /= 2;
+  const size_t smem = scan_smem(KIND, RPL, CPL, warps, sa.tb);
+  if (smem > MAX_SMEM) return cudaErrorInvalidValue;
+  cudaError_t e = cudaFuncSetAttribute(recurrence_scan_kernel<KIND, RPL, CPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
+  if (e != cudaSuccess) return e;
+  return launch_kernel(recurrence_scan_kernel<KIND, RPL, CPL>, grid, dim3((warps + 1) * 32), smem, s, false, sa);
+}
+
+template <int KIND, int RPL>
+cudaError_t launch_scan_cols(const ScanArgs& sa, dim3 grid, int cols, int cpl, cudaStream_t s) {
+  if (cpl == 4) return launch_scan<KIND, RPL, 4>(sa, grid, cols, s);
+  if (cpl == 2) return launch_scan<KIND, RPL, 2>(sa, grid, cols, s);
+  return launch_scan<KIND, RPL, 1>(sa, grid, cols, s);
+}
+
+cudaError_t launch_scan_any(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
+  const int dk = sa.a.l.dim;
+  const long long blocks = (long long)grid.x * grid.y * grid.z;
+  // few blocks in flight: the columns of a head are cut over several of them
+  int nb = (cols + 127) / 128;
+  while (nb * 2 * blocks <= sm_count() && (cols + nb * 2 - 1) / (nb * 2) >= 48) nb *= 2;
+  nb = std::max(nb, tune_int("PG_SCAN_BLOCKS", 0));
+  sa.block_cols = ((cols + nb - 1) / nb + 3) / 4 * 4;
+  sa.col_blocks = (cols + sa.block_cols - 1) / sa.block_cols;
+  grid.x *= sa.col_blocks;
+  const int bc = sa.block_cols;
+  int cpl = std::max((bc + 31) / 32, tune_int("PG_SCAN_CPL", 0));
+  if (cpl == 3) cpl = 4;
+#define PG_SCAN(KIND_)                                                                  \
+  (dk <= 32    ? launch_scan_cols<KIND_, 4>(sa, grid, bc, cpl, s)                       \
+   : dk <= 64  ? launch_scan_cols<KIND_, 8>(sa, grid, bc, cpl, s)                       \
+   : dk <= 128 ? launch_scan_cols<KIND_, 16>(sa, grid, bc, cpl, s)                      \
+   : dk <= 256 ? launch_scan_cols<KIND_, 32>(sa, grid, bc, cpl, s) : cudaErrorInvalidValue)
+  cudaError_t e = sa.a.l.kind == KIND_DELTA ? PG_SCAN(KIND_DELTA) : PG_SCAN(KIND_GLA);
+#undef PG_SCAN
+  if (e == cudaSuccess && sa.col_blocks > 1 && (sa.mode == SCAN_FULL || sa.mode == SCAN_OUTPUT)) {
+    const long long warps = (long long)sa.a.rows * sa.a.l.heads;
+    e = launch_kernel(recurrence_output_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 32)), dim3(256), 0, s, false, sa.a,
+                      sa.y_bf16);
+  }
+  return e;
+}
+
+}  // namespace
+
+bool recurrence_use_segments(const RecurrenceLayer& l, int nseq, int max_len, int max_segs) {
+  // the transition matrices of the delta rule must fit shared memory twice
+  return max_segs >= 4 && max_len >= 512 && (long long)nseq * l.heads < 48 && (l.kind != KIND_DELTA || l.dim <= 144);
+}
+
+size_t recurrence_segment_floats(const RecurrenceLayer& l, int nseq, int max_segs) {
+  return (size_t)nseq * max_segs * l.heads * l.dim * (l.dvp + (l.kind == KIND_DELTA ? (l.dim + 3) / 4 * 4 : 1));
+}
+
+cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cudaStream_t s) {
+  if (a.rows <= 0) return cudaSuccess;
+  const RecurrenceLayer& l = a.l;
+  const int K = l.heads * l.dim;
+  cudaError_t e = launch_kernel(recurrence_decay_kernel, dim3((a.rows + GATE_ROWS - 1) / GATE_ROWS, (K + 255) / 256), dim3(256),
+                                (size_t)GATE_ROWS * l.rank * sizeof(float), s, false, a);
+  if (e != cudaSuccess) return e;
+  if (l.kind == KIND_DELTA) {
+    const long long warps = (long long)a.rows * l.heads;
+    e = launch_kernel(delta_gates_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 32)), dim3(256), 0, s, false, a);
+    if (e != cudaSuccess) return e;
+  }
+  ScanArgs sa{};
+  sa.a = a;
+  sa.y_bf16 = y_bf16 ? 1 : 0;
+  auto m4 = [](int v) { return v % 4 == 0; };
+  sa.vec = m4(l.dim) && m4(l.vdim) && m4(l.off_k) && m4(l.off_q) && m4(l.off_v) && m4(l.off_g) && m4(a.ldp);
+  if (a.max_segs <= 1 || !a.segments) {
+    sa.mode = SCAN_FULL;
+    return launch_scan_any(sa, dim3(l.heads, a.nseq, 1), l.vdim, s);
+  }
+  const size_t units = (size_t)a.nseq * a.max_segs * l.heads;
+  sa.dkp = (l.dim + 3) / 4 * 4;
+  sa.seg_state = a.segments;
+  sa.seg_trans = a.segments + units * l.dim * l.dvp;
+  const dim3 grid(l.heads, a.nseq, a.max_segs);
+  sa.mode = SCAN_LOCAL;
+  if ((e = launch_scan_any(sa, grid, l.vdim, s)) != cudaSuccess) return e;
+  if (l.kind == KIND_DELTA) {
+    sa.mode = SCAN_TRANS;
+    e = launch_scan_any(sa, grid, l.dim, s);
+  } else {
+    e = launch_kernel(segment_decay_kernel, dim3((K + 255) / 256, a.max_segs, a.nseq), dim3(256), 0, s, false, sa);
+  }
+  if (e != cudaSuccess) return e;
+  const dim3 cgrid(l.heads, a.nseq, (l.vdim + COMBINE_COLS - 1) / COMBINE_COLS);
+  const size_t csmem = ((size_t)2 * l.dim * COMBINE_COLS + (l.kind == KIND_DELTA ? (size_t)2 * l.dim * (sa.dkp + 4) : 0)) * sizeof(float);
+  if (csmem > MAX_SMEM) return cudaErrorInvalidValue;
+  e = cudaFuncSetAttribute(recurrence_combine_kernel<KIND_DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
+  if (e != cudaSuccess) return e;
+  e = l.kind == KIND_DELTA ? launch_kernel(recurrence_combine_kernel<KIND_DELTA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa)
+                           : launch_kernel(recurrence_combine_kernel<KIND_GLA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa);
+  if (e != cudaSuccess) return e;
+  sa.mode = SCAN_OUTPUT;
+  return launch_scan_any(sa, grid, l.vdim, s);
+}
+
+}  // namespace pg
