@@ -19,7 +19,8 @@ int align_to(int n, int a) { return (n + a - 1) / a * a; }
 constexpr int K_ALIGN = 64;  // input columns of every product: one TMA box of BF16
 constexpr int N_ALIGN = 8;
 constexpr int MAX_ROWS_LINEAR = 8;
-constexpr int SEGMENT_TOKENS = 128;
+// tokens per segment of a recurrence over a long portion: many enough to fill the chip, few enough to combine quickly
+int segment_tokens(int max_len) { return max_len >= 4096 ? 256 : 128; }
 
 struct Matrix {  // [np, kp] row-major in the storage type, zero outside [n, k]
   void* w = nullptr;
@@ -609,7 +610,7 @@ cudaError_t enqueue_portions(pg_cache* c, const PortionPlan& plan, const Portion
     post = nullptr;
     return launch_norm_step(a, rows, m->bf16, false, s);
   };
-  const int max_segs = (plan.max_len + SEGMENT_TOKENS - 1) / SEGMENT_TOKENS;
+  const int max_segs = (plan.max_len + segment_tokens(plan.max_len) - 1) / segment_tokens(plan.max_len);
   for (const DevLayer& l : m->layers) {
     PG_L(B_LAYER_NORM, norm(&l.norm1));
     PG_L(B_QKV, product(m, l.in, r.h, r.p, nullptr, l.in.np, l.in.np, rows, false, c->d_error, false, s));
@@ -628,7 +629,7 @@ cudaError_t enqueue_portions(pg_cache* c, const PortionPlan& plan, const Portion
         a.seq_start = d.seq_start; a.seq_slot = d.slot; a.seq_pos = d.start_pos; a.state = lc->states[b.state];
         a.decay = lc->decay; a.unit = lc->unit; a.rate = lc->rate; a.unit_next = lc->unit_next; a.pair = lc->pair;
         a.out_raw = lc->out_raw; a.error_flag = c->d_error;
-        a.segments = lc->segments; a.seg_tokens = SEGMENT_TOKENS;
+        a.segments = lc->segments; a.seg_tokens = segment_tokens(plan.max_len);
         a.max_segs = recurrence_use_segments(b.rec, plan.n(), plan.max_len, max_segs) ? max_segs : 0;
         a.y = y; a.ldy = l.out.kp;
         PG_L(B_ATTN, launch_recurrence_scan(a, m->bf16, s));
@@ -683,7 +684,7 @@ int layered_run_portions(pg_cache* c, const PortionPlan& plan, float* logits, St
   }
   if (int r = grow(&lc->meta, &lc->meta_ints, meta.size(), sizeof(int))) return r;
   size_t qe = 0, ke = 0, ve = 0, seg = 0;
-  const int max_segs = (plan.max_len + SEGMENT_TOKENS - 1) / SEGMENT_TOKENS;
+  const int max_segs = (plan.max_len + segment_tokens(plan.max_len) - 1) / segment_tokens(plan.max_len);
   for (const DevLayer& l : m->layers)
     for (const DevBranch& b : l.branches) {
       if (b.kind == BranchSpec::ATTENTION) {

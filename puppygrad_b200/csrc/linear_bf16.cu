@@ -69,7 +69,14 @@ __global__ void __launch_bounds__(RL_THREADS, 1) rows_linear_kernel(RowsLinearAr
     }
   };
   // weights do not depend on the previous kernel: the first loads go out before the dependency wait
-  request(blockIdx.x * upc + wu, s0);
+  // (unit u of round q of this block: units are dealt out over the blocks so that every SM streams its share)
+  request(wu * gridDim.x + blockIdx.x, s0);
+  if (a.fuse_norm) {  // the norms' vectors too, as far as L2
+    const int c = (tid & 127) * 32;
+    const float* v = (tid >> 7) == 0 ? a.norm.post_g : (tid >> 7) == 1 ? a.norm.post_b : (tid >> 7) == 2 ? a.norm.pre_g : a.norm.pre_b;
+    if (v)
+      for (int i = c; i < a.norm.ldx; i += 128 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(v + i));
+  }
   grid_dep_wait();
 
   if (!a.fuse_norm) {
@@ -122,13 +129,13 @@ __global__ void __launch_bounds__(RL_THREADS, 1) rows_linear_kernel(RowsLinearAr
 
   float bv = -INFINITY;
   int bi = INT_MAX;
-  for (int u0 = blockIdx.x * upc; u0 < units; u0 += gridDim.x * upc) {
-    const int unit = u0 + wu;
+  for (int round = 0; round * upc * (int)gridDim.x + (int)blockIdx.x < units; ++round) {
+    const int unit = (round * upc + wu) * gridDim.x + blockIdx.x;
     float acc[RL_ROWS * MT];
 #pragma unroll
     for (int i = 0; i < RL_ROWS * MT; ++i) acc[i] = 0.f;
     for (int st = s0; st < s1; st += RL_PRE) {
-      if (st != s0 || u0 != (int)blockIdx.x * upc) request(unit, st);
+      if (st != s0 || round > 0) request(unit, st);
 #pragma unroll
       for (int j = 0; j < RL_PRE; ++j) {
         if (st + j < s1) {
@@ -159,7 +166,7 @@ __global__ void __launch_bounds__(RL_THREADS, 1) rows_linear_kernel(RowsLinearAr
       const int uu = i / (RL_ROWS * MT), e = i % (RL_ROWS * MT), r = e / MT, m = e % MT;
       float v = 0.f;
       for (int q = 0; q < kparts; ++q) v += part[uu * kparts + q][e];
-      const int row = (u0 + uu) * RL_ROWS + r;
+      const int row = ((round * upc + uu) * (int)gridDim.x + (int)blockIdx.x) * RL_ROWS + r;
       if (row < a.n && m < a.m) {
         if (a.epilogue == ROWS_GELU_ERF) v = gelu_erf(v);
         if (a.out) a.out[(size_t)m * a.ldo + row] = v;
@@ -222,8 +229,8 @@ bool rows_linear_supported(int m, int k, bool fuse_norm, int width) {
 
 int rows_linear_grid(int m, int n, int k) {
   (void)m;
-  const int upc = RL_WARPS >> k_part_shift(n, k), units = (n + RL_ROWS - 1) / RL_ROWS;
-  return std::max(1, std::min(sm_count(), (units + upc - 1) / upc));
+  (void)k;
+  return std::max(1, std::min(sm_count(), (n + RL_ROWS - 1) / RL_ROWS));
 }
 
 cudaError_t launch_rows_linear(const RowsLinearArgs& a, bool pdl, cudaStream_t s, int* grid_out) {

@@ -1,6 +1,8 @@
 // One new token per sequence through a recurrent mixer (gated linear attention, generalized delta rule): the cached
 // [dim, vdim] FP32 state of every head is read, advanced and written back, with the gates before it and the head norm and
 // output gate after it in the same kernel. Everything that enters the recurrence is FP32.
+#include <algorithm>
+
 #include "recurrence.cuh"
 
 namespace pg {
@@ -27,7 +29,8 @@ __global__ void __launch_bounds__(STEP_THREADS) recurrence_step_kernel(Recurrenc
   float* vs = ts + rka;      // [dvp]
   float* ds = vs + dvp;      // [dvp] u^T S
   float* os = ds + dvp;      // [dvp]
-  float* part = os + dvp;    // [KG][dvp]
+  float* zs = os + dvp;      // [max(256, dk)] partial sums of the decay projection
+  float* part = zs + (dk > STEP_THREADS ? dka : STEP_THREADS);  // [KG][dvp]
   const int dv4 = dvp / 4, KG = STEP_THREADS / dv4;
   const int c4 = tid % dv4, kg = tid / dv4;
   const bool active = kg < KG;
@@ -56,10 +59,21 @@ __global__ void __launch_bounds__(STEP_THREADS) recurrence_step_kernel(Recurrenc
   for (int c = tid; c < dvp; c += STEP_THREADS) vs[c] = c < dv ? p[l.off_v + head * dv + c] : 0.f;
   kk = block_sum(kk, red);  // also orders the shared-memory writes above
   const float inv_norm = 1.f / sqrtf(kk + UNIT_EPS);
+  // second half of the decay projection: RG threads share a channel, so that its weights arrive in one round trip or two
+  const int RG = dk >= STEP_THREADS ? 1 : STEP_THREADS / dk;
+  for (int i = tid; i < RG * dk; i += STEP_THREADS) {
+    const int c = i % dk, g = i / dk;
+    const float* __restrict__ w2 = l.w2 + head * dk + c;
+    float z = 0.f;
+#pragma unroll 16
+    for (int r = g; r < l.rank; r += RG) z = fmaf(w2[(size_t)r * K], ts[r], z);
+    zs[i] = z;
+  }
+  __syncthreads();
   for (int c = tid; c < dk; c += STEP_THREADS) {
     const int ch = head * dk + c;
     float z = l.b2[ch];
-    for (int r = 0; r < l.rank; ++r) z = fmaf(l.w2[(size_t)r * K + ch], ts[r], z);
+    for (int g = 0; g < RG; ++g) z += zs[g * dk + c];
     ws[c] = decay_of(l.kind, z, l.inv_tau);
     if (delta) {
       const float u = ks[c] * inv_norm;
@@ -135,7 +149,7 @@ cudaError_t launch_recurrence_step(const RecurrenceStepArgs& a, bool y_bf16, boo
   const RecurrenceLayer& l = a.l;
   const int dv4 = l.dvp / 4, kg = STEP_THREADS / dv4, nr = (l.dim + kg - 1) / kg;
   if (dv4 > STEP_THREADS) return cudaErrorInvalidValue;
-  const size_t smem = ((size_t)5 * ((l.dim + 3) & ~3) + ((l.rank + 3) & ~3) + 3 * (size_t)l.dvp + (size_t)kg * l.dvp) * sizeof(float);
+  const size_t smem = ((size_t)5 * ((l.dim + 3) & ~3) + ((l.rank + 3) & ~3) + 3 * (size_t)l.dvp + std::max(STEP_THREADS, (l.dim + 3) & ~3) + (size_t)kg * l.dvp) * sizeof(float);
   const dim3 grid(l.heads, a.batch), block(STEP_THREADS);
   const int yb = y_bf16 ? 1 : 0;
   if (nr <= 4) return launch_kernel(recurrence_step_kernel<4>, grid, block, smem, s, pdl, a, yb);

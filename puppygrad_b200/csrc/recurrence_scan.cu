@@ -82,6 +82,60 @@ __global__ void __launch_bounds__(256) delta_gates_kernel(RecurrenceScanArgs a) 
   }
 }
 
+// The same when every size and offset is a multiple of four: eight lanes per (row, head), four channels at a time.
+__global__ void __launch_bounds__(256) delta_gates_vec_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int K = l.heads * l.dim, l8 = threadIdx.x & 7;
+  const long long total = (long long)a.rows * l.heads, rounded = (total + 3) / 4 * 4;  // whole warps stay together
+  auto eight = [](float v) {
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) v += __shfl_xor_sync(ALL_LANES, v, o);
+    return v;
+  };
+  for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 3; i < rounded; i += ((long long)gridDim.x * blockDim.x) >> 3) {
+    const bool on = i < total;
+    const int row = on ? (int)(i / l.heads) : 0, head = on ? (int)(i % l.heads) : 0;
+    const float* pr = a.p + (size_t)row * a.ldp;
+    const float* k = pr + l.off_k + head * l.dim;
+    const float* kn = row + 1 < a.rows ? k + a.ldp : k;
+    float4 kv[8], nv[8];
+    float s = 0.f, sn = 0.f;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const int c = q * 32 + l8 * 4;
+      const bool in = on && c < l.dim;
+      kv[q] = in ? load4(k + c) : make_float4(0, 0, 0, 0);
+      nv[q] = in ? load4(kn + c) : make_float4(0, 0, 0, 0);
+      s += (kv[q].x * kv[q].x + kv[q].y * kv[q].y) + (kv[q].z * kv[q].z + kv[q].w * kv[q].w);
+      sn += (nv[q].x * nv[q].x + nv[q].y * nv[q].y) + (nv[q].z * nv[q].z + nv[q].w * nv[q].w);
+    }
+    const float inv = 1.f / sqrtf(eight(s) + UNIT_EPS), invn = 1.f / sqrtf(eight(sn) + UNIT_EPS);
+    float ub = 0.f, uk = 0.f;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) {
+      const int c = q * 32 + l8 * 4, ch = head * l.dim + c;
+      if (on && c < l.dim) {
+        const size_t at = (size_t)row * K + ch;
+        const float4 al = load4(pr + l.off_a + ch), dec = load4(a.decay + at);
+        const float* ab = l.a_bias + ch;
+        float4 u, b, un;
+        u.x = kv[q].x * inv; u.y = kv[q].y * inv; u.z = kv[q].z * inv; u.w = kv[q].w * inv;
+        b.x = sigmoid_f(al.x + ab[0]) * u.x; b.y = sigmoid_f(al.y + ab[1]) * u.y;
+        b.z = sigmoid_f(al.z + ab[2]) * u.z; b.w = sigmoid_f(al.w + ab[3]) * u.w;
+        un.x = nv[q].x * invn; un.y = nv[q].y * invn; un.z = nv[q].z * invn; un.w = nv[q].w * invn;
+        ub += (un.x * b.x + un.y * b.y) + (un.z * b.z + un.w * b.w);
+        uk += (un.x * kv[q].x + un.y * kv[q].y) + (un.z * kv[q].z + un.w * kv[q].w);
+        store4(a.unit + at, u);
+        store4(a.rate + at, b);
+        store4(a.unit_next + at, make_float4(un.x * dec.x, un.y * dec.y, un.z * dec.z, un.w * dec.w));
+      }
+    }
+    ub = eight(ub);
+    uk = eight(uk);
+    if (on && l8 == 0) store4(a.pair + (size_t)i * 4, make_float4(ub, uk, 0.f, 0.f));
+  }
+}
+
 // ------------------------------------------------------------------ scan
 // Block = one head of one sequence (or of one segment of it), or a part of its columns. The last warp stages the rows of
 // TB tokens at a time in a ring of shared-memory stages (bulk copies where rows are 16-byte aligned); in the others
@@ -685,7 +739,9 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   if (e != cudaSuccess) return e;
   if (l.kind == KIND_DELTA) {
     const long long warps = (long long)a.rows * l.heads;
-    e = launch_kernel(delta_gates_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 32)), dim3(256), 0, s, false, a);
+    const bool vec = l.dim % 4 == 0 && l.off_k % 4 == 0 && l.off_a % 4 == 0 && a.ldp % 4 == 0;
+    e = vec ? launch_kernel(delta_gates_vec_kernel, dim3((unsigned)std::min<long long>((warps + 31) / 32, 148 * 32)), dim3(256), 0, s, false, a)
+            : launch_kernel(delta_gates_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 32)), dim3(256), 0, s, false, a);
     if (e != cudaSuccess) return e;
   }
   ScanArgs sa{};
