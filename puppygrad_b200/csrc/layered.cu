@@ -24,6 +24,7 @@ int segment_tokens(int max_len) { return max_len >= 4096 ? 256 : 128; }
 
 struct Matrix {  // [np, kp] row-major in the storage type, zero outside [n, k]
   void* w = nullptr;
+  void* tiled = nullptr;  // BF16: the second copy that batches of decode rows stream
   int n = 0, k = 0, np = 0, kp = 0;
 };
 struct Norm {
@@ -143,6 +144,8 @@ struct Builder {
       if (e == cudaSuccess) e = cudaDeviceSynchronize();
       cudaFree(tmp);
       PG_CUDA_TRY(e);
+      if (int r = alloc(tiled_bf16_elems(out->np, out->kp) * 2, &out->tiled)) return r;
+      PG_CUDA_TRY(launch_tile_bf16(out->w, out->tiled, out->np, out->kp, 0));
     } else {
       PG_CUDA_TRY(cudaMemcpy2D(out->w, (size_t)out->kp * 4, v.data(), (size_t)k * 4, (size_t)k * 4, n, cudaMemcpyHostToDevice));
     }
@@ -454,7 +457,7 @@ cudaError_t product(const LayeredModel* m, const Matrix& w, const void* x, float
                     int* error_flag, bool pdl, cudaStream_t s) {
   if (m->bf16) {
     Bf16GemmArgs a{};
-    a.x = x; a.w = w.w; a.out = out; a.out_h = out_h; a.ldo = ldo; a.error_flag = error_flag;
+    a.x = x; a.w = w.w; a.w_tiled = w.tiled; a.out = out; a.out_h = out_h; a.ldo = ldo; a.error_flag = error_flag;
     a.m = rows; a.n = n_out; a.k = w.kp; a.gelu_erf = gelu ? 1 : 0;
     return launch_tc_gemm_bf16(a, pdl, s);
   }
@@ -503,11 +506,22 @@ cudaError_t layered_enqueue_decode(pg_cache* c, int batch, int splits, cudaStrea
     embed = false;
     post = nullptr;
   };
+  // With a few rows every block of a product makes the normed rows itself; with more of them one row kernel is cheaper.
+  const bool fuse_norm = batch <= 4;
   auto rows_linear = [&](const Matrix& w, const float* x, const NormStepArgs* norm, float* out, int ldo, int n_out, int epi, float* pv, int* pi,
                          int* grid) -> cudaError_t {
     RowsLinearArgs a{};
     a.w = w.w; a.x = x; a.ldx = w.kp; a.out = out; a.ldo = ldo; a.m = batch; a.n = n_out; a.k = w.kp; a.epilogue = epi;
-    if (norm) { a.fuse_norm = 1; a.norm = *norm; }
+    if (norm && fuse_norm) {
+      a.fuse_norm = 1;
+      a.norm = *norm;
+    } else if (norm) {
+      NormStepArgs na = *norm;
+      na.h32 = r.h32;
+      if ((e = launch_norm_step(na, batch, true, pdl, s)) != cudaSuccess) return e;
+      ++n;
+      a.x = r.h32;
+    }
     a.part_val = pv; a.part_idx = pi;
     return launch_rows_linear(a, pdl, s, grid);
   };

@@ -23,7 +23,8 @@ struct NormStepArgs {
   const float* y;        // [rows, ldx] sublayer output, or nullptr
   const float *post_g, *post_b;
   const float *pre_g, *pre_b;  // nullptr: no h
-  void* h;               // [rows, ldh] in T
+  void* h;               // [rows, ldh] in T ...
+  float* h32;            // ... or in FP32 (when not nullptr)
   int ldx, ldh, width;
   float eps;
 };
@@ -32,6 +33,10 @@ cudaError_t launch_norm_step(const NormStepArgs& a, int rows, bool bf16, bool pd
 cudaError_t launch_gelu_erf(float* x, size_t n, bool pdl, cudaStream_t s);
 // FP32 [rows, cols] -> BF16 [rows_padded, ld], zero outside rows x cols
 cudaError_t launch_pack_bf16(const float* src, void* dst, int rows, int cols, int rows_padded, int ld, cudaStream_t s);
+// BF16 [rows, ld] (ld % 64 == 0) -> tiles [ceil(rows / 128)][ld / 64][128][64], rows past the end zero: one 128 x 64 tile is
+// one contiguous 16 KB run, which a decode step streams at full DRAM bandwidth (128 rows of 128 bytes each would not be)
+size_t tiled_bf16_elems(int rows, int ld);
+cudaError_t launch_tile_bf16(const void* src, void* dst, int rows, int ld, cudaStream_t s);
 
 // ------------------------------------------------------------------ linear_bf16.cu
 // out[m, n] = f(x)[m, k] . w[n, k]^T for at most 8 rows, BF16 weights, FP32 activations and sums. `norm` (optional)
@@ -59,6 +64,7 @@ cudaError_t launch_rows_linear(const RowsLinearArgs& a, bool pdl, cudaStream_t s
 struct Bf16GemmArgs {
   const void* x;   // [m, k] BF16
   const void* w;   // [n, k] BF16
+  const void* w_tiled;  // the same in 128 x 64 tiles (launch_tile_bf16): used for at most 64 rows
   float* out;      // [m, ldo] FP32, or nullptr
   void* out_h;     // [m, ldo] BF16, or nullptr
   int ldo;

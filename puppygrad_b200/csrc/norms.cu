@@ -60,11 +60,14 @@ __global__ void __launch_bounds__(NORM_THREADS) norm_step_kernel(NormStepArgs a)
   if (a.pre_g) {
     float mean, rstd;
     moments(x, &mean, &rstd);
-    T* h = static_cast<T*>(a.h) + (size_t)row * a.ldh;
 #pragma unroll
     for (int j = 0; j < V4; ++j) {
       const int c = (tid + j * NORM_THREADS) * 4;
-      if (c < a.ldh) store4(h + c, norm_step_apply(x[j], mean, rstd, a.pre_g, a.pre_b, c, a.width));
+      if (c < a.ldh) {
+        const float4 n = norm_step_apply(x[j], mean, rstd, a.pre_g, a.pre_b, c, a.width);
+        if (a.h32) store4(a.h32 + (size_t)row * a.ldh + c, n);
+        else store4(static_cast<T*>(a.h) + (size_t)row * a.ldh + c, n);
+      }
     }
   }
 }
@@ -97,6 +100,18 @@ __global__ void __launch_bounds__(256) pack_bf16_kernel(const float* __restrict_
   }
 }
 
+__global__ void __launch_bounds__(256) tile_bf16_kernel(const uint4* __restrict__ src, uint4* __restrict__ dst, int rows, int ld) {
+  const int nkb = ld / 64;
+  const size_t n = (size_t)((rows + 127) / 128) * nkb * 128 * 8;  // 16-byte pieces
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const int piece = (int)(i & 7), r = (int)((i >> 3) & 127);
+    const size_t tile = i >> 10;
+    const int kb = (int)(tile % nkb);
+    const size_t row = tile / nkb * 128 + r;
+    dst[i] = row < (size_t)rows ? src[row * (ld / 8) + kb * 8 + piece] : make_uint4(0, 0, 0, 0);
+  }
+}
+
 int grid_for(size_t n) { return (int)((n + 255) / 256 < 1184 ? (n + 255) / 256 : 1184); }
 
 }  // namespace
@@ -108,6 +123,13 @@ cudaError_t launch_norm_step(const NormStepArgs& a, int rows, bool bf16, bool pd
 
 cudaError_t launch_gelu_erf(float* x, size_t n, bool pdl, cudaStream_t s) {
   return launch_kernel(gelu_erf_kernel, dim3(grid_for(n)), dim3(256), 0, s, pdl, x, n);
+}
+
+size_t tiled_bf16_elems(int rows, int ld) { return (size_t)((rows + 127) / 128) * 128 * ld; }
+
+cudaError_t launch_tile_bf16(const void* src, void* dst, int rows, int ld, cudaStream_t s) {
+  if (ld % 64 != 0) return cudaErrorInvalidValue;
+  return launch_kernel(tile_bf16_kernel, dim3(1184), dim3(256), 0, s, false, static_cast<const uint4*>(src), static_cast<uint4*>(dst), rows, ld);
 }
 
 cudaError_t launch_pack_bf16(const float* src, void* dst, int rows, int cols, int rows_padded, int ld, cudaStream_t s) {

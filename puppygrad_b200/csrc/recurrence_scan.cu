@@ -4,7 +4,6 @@
 // Both rules act on every column of a head's [dim, vdim] state on its own (S[:, c] needs only v[c] of the new token), so
 // a column's `dim` entries are spread over eight lanes and the columns over groups of lanes, warps and blocks.
 #include <algorithm>
-#include <cstdlib>
 
 #include "recurrence.cuh"
 #include "tc_common.cuh"
@@ -661,11 +660,6 @@ int sm_count() {
   return n;
 }
 
-int tune_int(const char* name, int otherwise) {
-  const char* e = getenv(name);
-  return e && *e ? atoi(e) : otherwise;
-}
-
 size_t scan_smem(int kind, int rpl, int cpl, int warps, int tb) {
   const size_t na = kind == KIND_DELTA ? 6 : 3, cols = (size_t)warps * 4 * cpl;
   return ((size_t)SCAN_STAGES * tb * (na * 8 * rpl + 2 * cols + 4) + (size_t)2 * tb * 8 * (cols + 4)) * sizeof(float);
@@ -697,12 +691,11 @@ cudaError_t launch_scan_any(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
   // few blocks in flight: the columns of a head are cut over several of them
   int nb = (cols + 127) / 128;
   while (nb * 2 * blocks <= sm_count() && (cols + nb * 2 - 1) / (nb * 2) >= 48) nb *= 2;
-  nb = std::max(nb, tune_int("PG_SCAN_BLOCKS", 0));
   sa.block_cols = ((cols + nb - 1) / nb + 3) / 4 * 4;
   sa.col_blocks = (cols + sa.block_cols - 1) / sa.block_cols;
   grid.x *= sa.col_blocks;
   const int bc = sa.block_cols;
-  int cpl = std::max((bc + 31) / 32, tune_int("PG_SCAN_CPL", 0));
+  int cpl = (bc + 31) / 32;
   if (cpl == 3) cpl = 4;
 #define PG_SCAN(KIND_)                                                                  \
   (dk <= 32    ? launch_scan_cols<KIND_, 4>(sa, grid, bc, cpl, s)                       \
