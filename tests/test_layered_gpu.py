@@ -447,3 +447,24 @@ def test_profiles_and_sizes(mixed):
                l["mixer"]["right"]["heads"] * l["mixer"]["right"]["dim"] ** 2 * 4 for l in MIXED["layers"])
     assert model.state_bytes_per_sequence() == want
     assert model.weight_bytes_per_step() > 0
+
+
+# ------------------------------------------------------------------ sizes past one tile of every product
+@pytest.fixture(scope="module")
+def wide():
+    return Case(lo.config(500, 1100, [lo.gla(3, 40, 72, ff=7000), lo.pair(10, 2, 72, 80, 90, 5, 40, ff=300)]), 21, rank=33)
+
+
+@pytest.mark.parametrize("mode", MODES)
+def test_wide_layers(wide, mode):
+    """Several tiles and k blocks of the products, a hidden row too long for the eight-row kernel's shared memory."""
+    model = wide.model(mode)
+    ids = wide.ids(300)
+    assert_rows(model.forward(ids).logits, wide.want(ids), mode)
+    for batch in (1, 3, 8, 40):
+        cache = model.new_kv_cache(batch)
+        prompts = [ids[:100 + 3 * (i % 4)] for i in range(batch)]
+        model.prefill_batch(prompts, cache)
+        for t in range(2):
+            got, _, _, _ = model.forward_one_batch([ids[len(p) + t] for p in prompts], cache, want_logits=True)
+            assert_rows(got, np.stack([wide.want(ids)[len(p) + t] for p in prompts]), mode)
