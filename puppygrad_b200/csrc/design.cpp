@@ -10,7 +10,7 @@ namespace pg {
 namespace {
 
 // Largest sizes the kernels take (per head: shared-memory rows and registers; per model: 32-bit indexing).
-constexpr int MAX_WIDTH = 16384, MAX_HEAD_DIM = 256, MAX_HEADS = 1024, MAX_RANK = 1024;
+constexpr int MAX_WIDTH = 16384, MAX_HEAD_DIM = 256, MAX_HEADS = 1024, MAX_RANK = 512;
 
 struct Reader {
   std::string path;
