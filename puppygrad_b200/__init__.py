@@ -14,6 +14,7 @@ from .gpt2 import Gpt2Config, Gpt2CudaConfig, Gpt2KvCache, Gpt2Model, Gpt2Output
 from .registry import MODELS, load_model, model_class
 from .runtime import (Gpt2AssetPaths, Gpt2GenerationStats, Gpt2OperationProfile, Gpt2Runtime, Gpt2Tokenizer,
                       write_raw_token_event)
+from .sanesun import SanesunConfig, SanesunModel
 from .streaming import IncrementalTextStreamer, escape_raw_token, is_incremental_decode_safe
 
 __all__ = ["generate", "Gpt2Error", "GPT2_EOS_TOKEN_ID", "GenerationStats", "LogitsSampler",
@@ -21,4 +22,4 @@ __all__ = ["generate", "Gpt2Error", "GPT2_EOS_TOKEN_ID", "GenerationStats", "Log
            "Gpt2CudaConfig", "Gpt2KvCache", "Gpt2Model", "Gpt2Output", "IncrementalTextStreamer", "escape_raw_token",
            "is_incremental_decode_safe", "Gpt2AssetPaths", "Gpt2GenerationStats", "Gpt2OperationProfile", "Gpt2Runtime",
            "Gpt2Tokenizer", "write_raw_token_event", "ProfiledGenerationStats", "CudaConfig", "DecoderCache", "DecoderModel", "ModelOutput",
-           "DiruraxConfig", "DiruraxModel", "DesignError", "MODELS", "load_model", "model_class"]
+           "DiruraxConfig", "DiruraxModel", "SanesunConfig", "SanesunModel", "DesignError", "MODELS", "load_model", "model_class"]

@@ -1,24 +1,13 @@
 // Attention of the layered models: grouped key / value heads, separate key and value sizes, optional per-head RMS norms
-// of queries, keys and values, and keys that are visible inside one block of `span` positions only (or always, when
-// the span is the whole context). Keys and values live in pages indexed by position % span.
+// of queries, keys and values. Which keys are visible, and where in the pages they lie, is KeyLife's matter; the single-token
+// kernel here knows blocks of positions only, the portion kernels all of it.
 #include <algorithm>
 #include <cfloat>
 
-#include "device_util.cuh"
-#include "layered_kernels.cuh"
+#include "attn_pages.cuh"
 
 namespace pg {
 namespace {
-
-// First element of the key (which = 0) or value row of cache index c of one kv head.
-template <typename T>
-__device__ __forceinline__ T* page_row(const AttentionLayer& l, T* pool, const int* table_row, int c, int head, int which) {
-  const size_t page_elems = (size_t)l.kv_heads * l.page_tokens * (l.dimp + l.vdimp);
-  T* page = pool + (size_t)table_row[c / l.page_tokens] * page_elems;
-  const int off = c % l.page_tokens;
-  if (which == 0) return page + ((size_t)head * l.page_tokens + off) * l.dimp;
-  return page + (size_t)l.kv_heads * l.page_tokens * l.dimp + ((size_t)head * l.page_tokens + off) * l.vdimp;
-}
 
 // One warp: out[0..np) = norm(x[0..n)) * weight * mul, zero past n. `normed` false: only the copy.
 template <typename T>
@@ -62,7 +51,7 @@ __global__ void __launch_bounds__(STEP_THREADS) attention_step_kernel(AttentionS
   grid_dep_launch();
   grid_dep_wait();
   const float* p = a.p + (size_t)seq * a.ldp;
-  const int pos = a.pos[seq], last = pos % l.span;  // keys 0..last of this block of positions; `last` is the new one
+  const int pos = a.pos[seq], last = pos % l.life.span;  // keys 0..last of this block of positions; `last` is the new one
   const int per = (last + 1 + a.splits - 1) / a.splits;
   const int k0 = split * per, k1 = min(last + 1, k0 + per);
   const int* table = a.page_table + (size_t)seq * l.pages_per_seq;
@@ -265,17 +254,16 @@ __global__ void __launch_bounds__(256) attention_prep_kernel(AttentionPortionArg
     const int row = (int)(i / per), j = (int)(i % per);
     const float* p = a.p + (size_t)row * a.ldp;
     const int seq = a.row_seq[row];
-    const int ctx = a.seq_pos[seq] % l.span;  // cached keys the sequence's first row still sees
-    const size_t krow = (size_t)a.key_start[seq] + ctx + (row - a.seq_start[seq]);
+    const size_t krow = (size_t)a.key_start[seq] + l.life.context(a.seq_pos[seq]) + (row - a.seq_start[seq]);
     if (j < l.heads)
       warp_norm_row<T>(p + l.off_q + j * l.dim, l.dim, l.dimp, l.q_norm, l.q_norm != nullptr, l.eps, 1.f,
                        static_cast<T*>(a.q) + ((size_t)row * l.heads + j) * l.dimp, lane);
     else if (j < l.heads + l.kv_heads)
       warp_norm_row<T>(p + l.off_k + (j - l.heads) * l.dim, l.dim, l.dimp, l.k_norm, l.k_norm != nullptr, l.eps, 1.f,
-                       static_cast<T*>(a.k) + (krow * l.kv_heads + (j - l.heads)) * l.dimp, lane);
+                       static_cast<T*>(a.k) + krow * a.ldk + (j - l.heads) * l.dimp, lane);
     else
       warp_norm_row<T>(p + l.off_v + (j - l.heads - l.kv_heads) * l.vdim, l.vdim, l.vdimp, nullptr, l.v_norm != 0, l.eps, 1.f,
-                       static_cast<T*>(a.v) + (krow * l.kv_heads + (j - l.heads - l.kv_heads)) * l.vdimp, lane);
+                       static_cast<T*>(a.v) + krow * a.ldv + (j - l.heads - l.kv_heads) * l.vdimp, lane);
   }
 }
 
@@ -289,8 +277,8 @@ __global__ void __launch_bounds__(256) attention_prep_vec_kernel(AttentionPortio
        i += ((long long)gridDim.x * blockDim.x) >> 3) {
     const bool on = i < (long long)a.rows * per;
     const int row = on ? (int)(i / per) : 0, j = on ? (int)(i % per) : 0;
-    const int seq = a.row_seq[row], ctx = a.seq_pos[seq] % l.span;
-    const size_t krow = (size_t)a.key_start[seq] + ctx + (row - a.seq_start[seq]);
+    const int seq = a.row_seq[row];
+    const size_t krow = (size_t)a.key_start[seq] + l.life.context(a.seq_pos[seq]) + (row - a.seq_start[seq]);
     const bool is_q = j < l.heads, is_k = !is_q && j < l.heads + l.kv_heads;
     const int h = is_q ? j : is_k ? j - l.heads : j - l.heads - l.kv_heads;
     const int n = is_q || is_k ? l.dim : l.vdim, np = is_q || is_k ? l.dimp : l.vdimp;
@@ -298,8 +286,8 @@ __global__ void __launch_bounds__(256) attention_prep_vec_kernel(AttentionPortio
     const float* weight = is_q ? l.q_norm : is_k ? l.k_norm : nullptr;
     const bool normed = is_q ? l.q_norm != nullptr : is_k ? l.k_norm != nullptr : l.v_norm != 0;
     T* out = is_q   ? static_cast<T*>(a.q) + ((size_t)row * l.heads + h) * np
-             : is_k ? static_cast<T*>(a.k) + (krow * l.kv_heads + h) * np
-                    : static_cast<T*>(a.v) + (krow * l.kv_heads + h) * np;
+             : is_k ? static_cast<T*>(a.k) + krow * a.ldk + h * np
+                    : static_cast<T*>(a.v) + krow * a.ldv + h * np;
     float4 v[8];
     float s = 0.f;
 #pragma unroll
@@ -325,61 +313,56 @@ __global__ void __launch_bounds__(256) attention_prep_vec_kernel(AttentionPortio
   }
 }
 
+// Eight elements between a workspace row (keys of all key heads, then their values) and a cached row.
+template <typename T>
+struct RowPiece {
+  T *cached, *work;
+  __device__ __forceinline__ RowPiece(const AttentionPortionArgs& a, const int* table, int place, size_t krow, int piece) {
+    const AttentionLayer& l = a.l;
+    const int e = piece * 8;
+    const bool is_k = e < l.kv_heads * l.dimp;
+    const int x = is_k ? e : e - l.kv_heads * l.dimp, w = is_k ? l.dimp : l.vrow;
+    cached = page_row(l, static_cast<T*>(a.pool), table, place, x / w, is_k ? 0 : 1) + x % w;
+    work = (is_k ? static_cast<T*>(a.k) + krow * a.ldk : static_cast<T*>(a.v) + krow * a.ldv) + x;
+  }
+  static __device__ __forceinline__ int count(const AttentionLayer& l) { return l.kv_heads * (l.dimp + l.vrow) / 8; }
+  static __device__ __forceinline__ void copy(T* dst, const T* src) {
+    reinterpret_cast<uint4*>(dst)[0] = reinterpret_cast<const uint4*>(src)[0];
+    if (sizeof(T) == 4) reinterpret_cast<uint4*>(dst)[1] = reinterpret_cast<const uint4*>(src)[1];
+  }
+};
+
 // Cached keys and values that the first row of each sequence still sees, copied in front of its own. Block = (key, seq).
 template <typename T>
 __global__ void __launch_bounds__(128) attention_context_kernel(AttentionPortionArgs a) {
   const AttentionLayer& l = a.l;
-  const int seq = blockIdx.y, ctx = a.seq_pos[seq] % l.span;
+  const int seq = blockIdx.y, p0 = a.seq_pos[seq], ctx = l.life.context(p0);
   const int* table = a.page_table + (size_t)a.seq_slot[seq] * l.pages_per_seq;
-  for (int c = blockIdx.x; c < ctx; c += gridDim.x) {
-    const size_t krow = (size_t)a.key_start[seq] + c;
-    for (int i = threadIdx.x; i < l.kv_heads * (l.dimp + l.vdimp) / 8; i += blockDim.x) {
-      const int e = i * 8;
-      const bool is_k = e < l.kv_heads * l.dimp;
-      const int x = is_k ? e : e - l.kv_heads * l.dimp, w = is_k ? l.dimp : l.vdimp;
-      const T* src = page_row(l, static_cast<T*>(a.pool), table, c, x / w, is_k ? 0 : 1) + x % w;
-      T* dst = (is_k ? static_cast<T*>(a.k) + krow * l.kv_heads * l.dimp : static_cast<T*>(a.v) + krow * l.kv_heads * l.vdimp) + x;
-      if (sizeof(T) == 2) {
-        *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
-      } else {
-        reinterpret_cast<float4*>(dst)[0] = reinterpret_cast<const float4*>(src)[0];
-        reinterpret_cast<float4*>(dst)[1] = reinterpret_cast<const float4*>(src)[1];
-      }
+  for (int c = blockIdx.x; c < ctx; c += gridDim.x)
+    for (int i = threadIdx.x; i < RowPiece<T>::count(l); i += blockDim.x) {
+      const RowPiece<T> r(a, table, l.life.place(l.life.context_position(p0, c)), (size_t)a.key_start[seq] + c, i);
+      RowPiece<T>::copy(r.work, r.cached);
     }
-  }
 }
 
-// Stores the portion's keys and values that later tokens can still see: those of the block of positions in which the
-// next token lies or the last one lay.
+// Stores the portion's keys and values that later tokens can still see.
 template <typename T>
 __global__ void __launch_bounds__(128) attention_store_kernel(AttentionPortionArgs a) {
   const AttentionLayer& l = a.l;
   const int row = blockIdx.x, seq = a.row_seq[row];
-  const int first = a.seq_start[seq], n = a.seq_start[seq + 1] - first, p0 = a.seq_pos[seq];
-  const int pos = p0 + (row - first), end = p0 + n - 1;
-  if (pos / l.span != end / l.span) return;
+  const int first = a.seq_start[seq], n = a.seq_start[seq + 1] - first, p0 = a.seq_pos[seq], pos = p0 + (row - first);
+  if (!l.life.lives(pos, p0 + n - 1)) return;
   const int* table = a.page_table + (size_t)a.seq_slot[seq] * l.pages_per_seq;
-  const size_t krow = (size_t)a.key_start[seq] + p0 % l.span + (row - first);
-  const int c = pos % l.span;
-  for (int i = threadIdx.x; i < l.kv_heads * (l.dimp + l.vdimp) / 8; i += blockDim.x) {
-    const int e = i * 8;
-    const bool is_k = e < l.kv_heads * l.dimp;
-    const int x = is_k ? e : e - l.kv_heads * l.dimp, w = is_k ? l.dimp : l.vdimp;
-    T* dst = page_row(l, static_cast<T*>(a.pool), table, c, x / w, is_k ? 0 : 1) + x % w;
-    const T* src =
-        (is_k ? static_cast<const T*>(a.k) + krow * l.kv_heads * l.dimp : static_cast<const T*>(a.v) + krow * l.kv_heads * l.vdimp) + x;
-    if (sizeof(T) == 2) {
-      *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
-    } else {
-      reinterpret_cast<float4*>(dst)[0] = reinterpret_cast<const float4*>(src)[0];
-      reinterpret_cast<float4*>(dst)[1] = reinterpret_cast<const float4*>(src)[1];
-    }
+  for (int i = threadIdx.x; i < RowPiece<T>::count(l); i += blockDim.x) {
+    const RowPiece<T> r(a, table, l.life.place(pos), (size_t)a.key_start[seq] + l.life.row(p0, pos), i);
+    RowPiece<T>::copy(r.cached, r.work);
   }
 }
 
 // CUDA-core attention over the workspaces. Block = 32 query rows of one head of one sequence, 128 threads: four lanes
-// per row, key tiles of 32, FP32 scores and sums, online softmax. Key rows of a tile are padded by one float.
-constexpr int QT = 32, KT = 32;
+// per row, key tiles of 32, FP32 scores and sums, online softmax. Query and key rows are staged in pieces of DC columns, padded
+// by one float.
+constexpr int QT = 32, KT = 32, DC = 128;
 template <typename T, int VR>
 __global__ void __launch_bounds__(128) attention_rows_kernel(AttentionPortionArgs a) {
   extern __shared__ __align__(16) float sm[];
@@ -387,54 +370,60 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttentionPortionArg
   const int head = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
   const int first = a.seq_start[seq], n = a.seq_start[seq + 1] - first, q0 = blockIdx.x * QT;
   if (q0 >= n) return;
-  const int kvh = head / (l.heads / l.kv_heads), p0 = a.seq_pos[seq], ctx = p0 % l.span;
-  const int base_pos = p0 - ctx;  // position of workspace key 0 of this sequence
-  float* qs = sm;                             // [QT][dimp + 1]
-  float* ks = qs + QT * (l.dimp + 1);         // [KT][dimp + 1]
-  float* vs = ks + KT * (l.dimp + 1);         // [KT][vdimp]
-  float* ps = vs + KT * l.vdimp;              // [QT][KT + 1]
+  const int rep = l.heads / l.kv_heads, kvh = head / rep, p0 = a.seq_pos[seq];
+  const int width = l.mix ? l.kv_heads * l.dimp : l.dimp, koff = l.mix ? 0 : kvh * l.dimp, dc = min(width, DC);
+  float* qs = sm;                       // [QT][dc + 1]
+  float* ks = qs + QT * (dc + 1);       // [KT][dc + 1]
+  float* vs = ks + KT * (dc + 1);       // [KT][vdimp]
+  float* ps = vs + KT * l.vdimp;        // [QT][KT + 1]
   const int r = tid >> 2, sub = tid & 3;
   const int qrow = q0 + r;
   const bool live = qrow < n;
-  for (int i = tid; i < QT * l.dimp; i += 128) {
-    const int rr = i / l.dimp, c = i % l.dimp;
-    qs[rr * (l.dimp + 1) + c] =
-        q0 + rr < n ? to_f32(static_cast<const T*>(a.q)[((size_t)(first + q0 + rr) * l.heads + head) * l.dimp + c]) : 0.f;
-  }
-  // keys [lo_row, hi_row] of the workspace are visible to this thread's row
+  auto stage = [&](float* dst, const T* src, size_t pitch, int rows, int c0) {  // rows past `rows` and columns past `width` as zero
+    for (int i = tid; i < QT * dc; i += 128) {
+      const int rr = i / dc, c = i % dc;
+      dst[rr * (dc + 1) + c] = rr < rows && c0 + c < width ? to_f32(src[(size_t)rr * pitch + c0 + c]) : 0.f;
+    }
+  };
+  const size_t qpitch = (size_t)l.heads * width;
+  const T* qsrc = static_cast<const T*>(a.q) + (size_t)(first + q0) * qpitch + (size_t)head * width;
+  if (width <= DC) stage(qs, qsrc, qpitch, n - q0, 0);
+  // workspace keys [lo_row, hi_row] and those below `keep` are visible to this thread's row
   const int pos = p0 + min(qrow, n - 1);
-  const int lo_row = max(pos / l.span * l.span - base_pos, 0), hi_row = pos - base_pos;
-  // range of the block's rows
-  const int pos_a = p0 + q0, pos_b = p0 + min(q0 + QT, n) - 1;
-  const int lo = max(pos_a / l.span * l.span - base_pos, 0), hi = pos_b - base_pos;
-  float m = -FLT_MAX, lsum = 0.f, acc[VR];
+  const int lo_row = l.life.low(p0, pos), hi_row = l.life.row(p0, pos), keep = l.life.keep;
+  const int lo = l.life.low(p0, p0 + q0), hi = l.life.row(p0, p0 + min(q0 + QT, n) - 1);  // moving range of the block's rows
+  const int kept = min(keep, lo);  // ... and the kept keys below it
+  float m = l.sink ? l.sink[head] : -FLT_MAX, lsum = l.sink ? 1.f : 0.f, acc[VR];
 #pragma unroll
   for (int c = 0; c < VR; ++c) acc[c] = 0.f;
-  for (int kt = lo; kt <= hi; kt += KT) {
+  const int kept_tiles = (kept + KT - 1) / KT, tiles = kept_tiles + (hi - lo) / KT + 1;
+  for (int tile = 0; tile < tiles; ++tile) {
+    const int kt = tile < kept_tiles ? tile * KT : lo + (tile - kept_tiles) * KT;
+    const int end = tile < kept_tiles ? min(kept, kt + KT) : min(hi + 1, kt + KT);
     __syncthreads();
-    for (int i = tid; i < KT * l.dimp; i += 128) {
-      const int rr = i / l.dimp, c = i % l.dimp;
-      ks[rr * (l.dimp + 1) + c] =
-          kt + rr <= hi ? to_f32(static_cast<const T*>(a.k)[((size_t)(a.key_start[seq] + kt + rr) * l.kv_heads + kvh) * l.dimp + c]) : 0.f;
-    }
     for (int i = tid; i < KT * l.vdimp; i += 128) {
       const int rr = i / l.vdimp, c = i % l.vdimp;
-      vs[i] = kt + rr <= hi ? to_f32(static_cast<const T*>(a.v)[((size_t)(a.key_start[seq] + kt + rr) * l.kv_heads + kvh) * l.vdimp + c]) : 0.f;
+      vs[i] = kt + rr < end ? to_f32(static_cast<const T*>(a.v)[(size_t)(a.key_start[seq] + kt + rr) * a.ldv + kvh * l.vdimp + c]) : 0.f;
     }
-    __syncthreads();
     float s[KT / 4];
 #pragma unroll
     for (int j = 0; j < KT / 4; ++j) s[j] = 0.f;
-    for (int c = 0; c < l.dim; ++c) {
-      const float q = qs[r * (l.dimp + 1) + c];
+    for (int c0 = 0; c0 < width; c0 += dc) {
+      if (c0 > 0) __syncthreads();
+      stage(ks, static_cast<const T*>(a.k) + (size_t)(a.key_start[seq] + kt) * a.ldk + koff, a.ldk, end - kt, c0);
+      if (width > DC) stage(qs, qsrc, qpitch, n - q0, c0);
+      __syncthreads();
+      for (int c = 0; c < dc; ++c) {
+        const float q = qs[r * (dc + 1) + c];
 #pragma unroll
-      for (int j = 0; j < KT / 4; ++j) s[j] = fmaf(q, ks[(j * 4 + sub) * (l.dimp + 1) + c], s[j]);
+        for (int j = 0; j < KT / 4; ++j) s[j] = fmaf(q, ks[(j * 4 + sub) * (dc + 1) + c], s[j]);
+      }
     }
     float mx = -FLT_MAX;
 #pragma unroll
     for (int j = 0; j < KT / 4; ++j) {
       const int key = kt + j * 4 + sub;
-      s[j] = (live && key >= lo_row && key <= hi_row) ? s[j] * l.scale : -FLT_MAX;
+      s[j] = (live && key < end && key <= hi_row && (key >= lo_row || key < keep)) ? s[j] * l.scale : -FLT_MAX;
       mx = fmaxf(mx, s[j]);
     }
     mx = fmaxf(mx, __shfl_xor_sync(ALL_LANES, mx, 1));
@@ -464,7 +453,8 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttentionPortionArg
     }
   }
   if (!live) return;
-  const float inv = l.out_scale / lsum;
+  float inv = l.out_scale / lsum;
+  if (l.off_gate >= 0) inv *= sigmoid_f(a.p[(size_t)(first + qrow) * a.ldp + l.off_gate + head]);
 #pragma unroll
   for (int c = 0; c < VR; ++c) {
     const int col = c * 4 + sub;
@@ -473,37 +463,33 @@ __global__ void __launch_bounds__(128) attention_rows_kernel(AttentionPortionArg
 }
 
 template <typename T>
-cudaError_t portion_t(const AttentionPortionArgs& a, cudaStream_t s) {
+cudaError_t ready_t(const AttentionPortionArgs& a, cudaStream_t s) {
   const AttentionLayer& l = a.l;
-  cudaError_t e;
+  if (l.rot_dims || l.v_rot || l.mix || l.q_bias) return launch_attention_rotate(a, sizeof(T) == 2, s);
   const long long warps = (long long)a.rows * (l.heads + 2 * l.kv_heads);
   const int pgrid = (int)std::min<long long>((warps + 7) / 8, 148 * 16);
   const bool vec = l.dim % 4 == 0 && l.vdim % 4 == 0 && l.off_q % 4 == 0 && l.off_k % 4 == 0 && l.off_v % 4 == 0 && a.ldp % 4 == 0;
   const int vgrid = (int)std::min<long long>((warps + 31) / 32, 148 * 16);
-  e = vec ? launch_kernel(attention_prep_vec_kernel<T>, dim3(vgrid), dim3(256), 0, s, false, a)
-          : launch_kernel(attention_prep_kernel<T>, dim3(pgrid), dim3(256), 0, s, false, a);
-  if (e != cudaSuccess) return e;
-  if (a.krows > a.rows) {
-    const int cgrid = std::min(a.krows - a.rows, 1024);
-    if ((e = launch_kernel(attention_context_kernel<T>, dim3(cgrid, a.nseq), dim3(128), 0, s, false, a)) != cudaSuccess) return e;
-  }
-  if (sizeof(T) == 2) {
-    if ((e = launch_attention_tc(a, s)) != cudaSuccess) return e;
-    return launch_kernel(attention_store_kernel<T>, dim3(a.rows), dim3(128), 0, s, false, a);
-  }
+  return vec ? launch_kernel(attention_prep_vec_kernel<T>, dim3(vgrid), dim3(256), 0, s, false, a)
+             : launch_kernel(attention_prep_kernel<T>, dim3(pgrid), dim3(256), 0, s, false, a);
+}
+
+cudaError_t rows_core(const AttentionPortionArgs& a, cudaStream_t s) {
+  const AttentionLayer& l = a.l;
+  const int dc = std::min(attention_q_width(l), DC);
   const dim3 grid((a.max_len + QT - 1) / QT, l.heads, a.nseq);
-  const size_t smem = ((size_t)(QT + KT) * (l.dimp + 1) + (size_t)KT * l.vdimp + (size_t)QT * (KT + 1)) * sizeof(float);
-#define PG_ROWS(VR_)                                                                                                        \
-  do {                                                                                                                      \
-    e = cudaFuncSetAttribute(attention_rows_kernel<T, VR_>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);       \
-    if (e == cudaSuccess) e = launch_kernel(attention_rows_kernel<T, VR_>, grid, dim3(128), smem, s, false, a);             \
+  const size_t smem = ((size_t)(QT + KT) * (dc + 1) + (size_t)KT * l.vdimp + (size_t)QT * (KT + 1)) * sizeof(float);
+  cudaError_t e;
+#define PG_ROWS(VR_)                                                                                                          \
+  do {                                                                                                                        \
+    e = cudaFuncSetAttribute(attention_rows_kernel<float, VR_>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);     \
+    if (e == cudaSuccess) e = launch_kernel(attention_rows_kernel<float, VR_>, grid, dim3(128), smem, s, false, a);           \
   } while (0)
   if (l.vdimp <= 64) PG_ROWS(16);
   else if (l.vdimp <= 128) PG_ROWS(32);
   else PG_ROWS(64);
 #undef PG_ROWS
-  if (e != cudaSuccess) return e;
-  return launch_kernel(attention_store_kernel<T>, dim3(a.rows), dim3(128), 0, s, false, a);
+  return e == cudaSuccess && l.v_rot ? launch_attention_turn_back(a, s) : e;
 }
 
 size_t step_smem(const AttentionLayer& l) {
@@ -513,7 +499,7 @@ size_t step_smem(const AttentionLayer& l) {
 
 }  // namespace
 
-size_t attention_page_elems(const AttentionLayer& l) { return (size_t)l.kv_heads * l.page_tokens * (l.dimp + l.vdimp); }
+size_t attention_page_elems(const AttentionLayer& l) { return (size_t)l.kv_heads * l.page_tokens * (l.dimp + l.vrow); }
 
 bool attention_supported(const AttentionLayer& l) { return step_smem(l) <= 200 * 1024; }
 
@@ -532,9 +518,28 @@ cudaError_t launch_attention_step(const AttentionStepArgs& a, bool bf16, bool y_
   return e != cudaSuccess ? e : launch_kernel(attention_step_kernel<float>, grid, dim3(STEP_THREADS), smem, s, pdl, a, yb);
 }
 
+cudaError_t launch_attention_context(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
+  if (a.krows <= a.rows) return cudaSuccess;
+  const dim3 grid(std::min(a.krows - a.rows, 1024), a.nseq);
+  return bf16 ? launch_kernel(attention_context_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, false, a)
+              : launch_kernel(attention_context_kernel<float>, grid, dim3(128), 0, s, false, a);
+}
+
+cudaError_t launch_attention_core(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
+  return bf16 ? launch_attention_tc(a, s) : rows_core(a, s);
+}
+
+cudaError_t launch_attention_store(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
+  return bf16 ? launch_kernel(attention_store_kernel<__nv_bfloat16>, dim3(a.rows), dim3(128), 0, s, false, a)
+              : launch_kernel(attention_store_kernel<float>, dim3(a.rows), dim3(128), 0, s, false, a);
+}
+
 cudaError_t launch_attention_portion(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
   if (a.rows <= 0) return cudaSuccess;
-  return bf16 ? portion_t<__nv_bfloat16>(a, s) : portion_t<float>(a, s);
+  cudaError_t e = bf16 ? ready_t<__nv_bfloat16>(a, s) : ready_t<float>(a, s);
+  if (e == cudaSuccess) e = launch_attention_context(a, bf16, s);
+  if (e == cudaSuccess) e = launch_attention_core(a, bf16, s);
+  return e == cudaSuccess ? launch_attention_store(a, bf16, s) : e;
 }
 
 }  // namespace pg

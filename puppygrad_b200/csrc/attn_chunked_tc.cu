@@ -5,7 +5,9 @@
 // first scores of an item overlap the end of the one before. Warp 0 loads, warp 1 issues the MMAs, warps 2..5 do the
 // softmax (thread = row). S(j + 1) = Q K^T is issued before O += P(j) V, so that the tensor cores work on the next scores
 // while the softmax warps are busy; keys and values have rings of their own. An item walks only the key tiles that some
-// row of it can see. Every wait is bounded: on expiry the error flag is set, work stops, tensor memory is freed.
+// row of it can see: those of the moving range, and before them those of the sequence's kept first keys. Keys come in pieces of
+// 64 columns through a ring; where the queries of an item do not fit beside it, their pieces come with the keys', again for
+// every tile. Every wait is bounded: on expiry the error flag is set, work stops, tensor memory is freed.
 #include <algorithm>
 
 #include "device_util.cuh"
@@ -26,13 +28,26 @@ __device__ __forceinline__ float exp2_fast(float x) {
   return r;
 }
 
-// kstages / vstages: ring depths; dpieces / vpieces: 64-column pieces of a key / value row; vn: columns of O (multiple of 16)
+constexpr int MAX_KSTAGES = 8;
+
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float* v) {
+  uint32_t u[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    u[i] = *reinterpret_cast<const uint32_t*>(&b);
+  }
+  *reinterpret_cast<uint4*>(p) = make_uint4(u[0], u[1], u[2], u[3]);
+}
+
+// kstages / vstages: ring depths (pieces of keys, whole value tiles); dpieces / vpieces: 64-column pieces of a query or key / value
+// row; vn: columns of O (multiple of 16); q_resident: an item's queries stay in shared memory
 struct TcShape {
-  int dpieces, vpieces, ksteps, vn, kstages, vstages, tmem_cols;
+  int dpieces, vpieces, ksteps, vn, kstages, vstages, tmem_cols, q_resident;
 };
 
 struct TcItem {
-  int head, seq, first, n, q0, kvh, p0, base_pos, pos_a, pos_b, lo, tiles;
+  int head, seq, first, n, q0, kvh, p0, pos_a, pos_b, lo, kept, kept_tiles, tiles;
   // false: no rows here
   __device__ __forceinline__ bool set(const AttentionPortionArgs& a, int index, int qtiles) {
     const AttentionLayer& l = a.l;
@@ -45,36 +60,44 @@ struct TcItem {
     if (q0 >= n) return false;
     kvh = head / (l.heads / l.kv_heads);
     p0 = a.seq_pos[seq];
-    base_pos = p0 - p0 % l.span;  // position of the sequence's first workspace key
     pos_a = p0 + q0;
     pos_b = p0 + min(q0 + QROWS, n) - 1;
-    lo = max(pos_a / l.span * l.span - base_pos, 0);
-    tiles = (pos_b - base_pos - lo) / KROWS + 1;
+    lo = l.life.low(p0, pos_a);  // the moving range of the item's rows starts here
+    kept = min(l.life.keep, lo);
+    if (lo < KROWS) lo = kept = 0;
+    kept_tiles = (kept + KROWS - 1) / KROWS;
+    tiles = kept_tiles + (l.life.row(p0, pos_b) - lo) / KROWS + 1;
     return true;
   }
+  // first workspace row of tile j, and the end of the rows that it stands for
+  __device__ __forceinline__ int start(int j) const { return j < kept_tiles ? j * KROWS : lo + (j - kept_tiles) * KROWS; }
+  __device__ __forceinline__ int end(int j) const { return j < kept_tiles ? kept : 1 << 30; }
 };
 
 __global__ void __launch_bounds__(192, 2)
     attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, AttentionPortionArgs a, TcShape t, int items, int qtiles) {
   extern __shared__ uint8_t smem_raw[];
-  __shared__ uint64_t q_full, q_empty, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full, p_ready, pv_done, o_free;
+  __shared__ uint64_t q_full, q_empty, k_full[MAX_KSTAGES], k_empty[MAX_KSTAGES], v_full[2], v_empty[2], s_full, p_ready, pv_done, o_free;
   __shared__ uint32_t tmem_slot;
   __shared__ int failed_flag;
   const AttentionLayer& l = a.l;
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* qs = base;
-  uint8_t* ks = qs + (size_t)t.dpieces * PIECE;
-  uint8_t* vs = ks + (size_t)t.kstages * t.dpieces * PIECE;
+  uint8_t* ks = qs + (t.q_resident ? (size_t)t.dpieces * PIECE : 0);  // a stage: a piece of keys, and one of queries unless resident
+  const uint32_t kstage_bytes = t.q_resident ? PIECE : 2 * PIECE;
+  uint8_t* vs = ks + (size_t)t.kstages * kstage_bytes;
   volatile int* failed = &failed_flag;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
   if (threadIdx.x == 0) {
     mbar_init(&q_full, 1);
     mbar_init(&q_empty, 1);
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < MAX_KSTAGES; ++i) {
       mbar_init(&k_full[i], 1);
       mbar_init(&k_empty[i], 1);
+    }
+    for (int i = 0; i < 2; ++i) {
       mbar_init(&v_full[i], 1);
       mbar_init(&v_empty[i], 1);
     }
@@ -96,19 +119,28 @@ __global__ void __launch_bounds__(192, 2)
 
   if (warp == 0) {
     if (lane == 0) {
+      const int key_head = l.mix ? 0 : 1;  // mixed heads: all key heads are one wide row
+      uint32_t kp = 0;                     // pieces of keys before the current one
       for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
         if (!w.set(a, it, qtiles)) continue;
-        if (done > 0) ok = mbar_wait(&q_empty, (done - 1) & 1, failed, a.error_flag, 20);
-        if (!ok) break;
-        mbar_expect_tx(&q_full, t.dpieces * PIECE);
-        for (int d = 0; d < t.dpieces; ++d) tma_load_3d(qs + (size_t)d * PIECE, &map_q, d * 64, w.head, w.first + w.q0, &q_full);
-        for (int j = 0; j < w.tiles && ok; ++j) {
-          const int krow = a.key_start[w.seq] + w.lo + j * KROWS;
-          const uint32_t gt = g + j, s = gt % t.kstages, v = gt % t.vstages;
-          if (gt >= (uint32_t)t.kstages) ok = mbar_wait(&k_empty[s], ((gt / t.kstages) - 1) & 1, failed, a.error_flag, 21);
+        if (t.q_resident) {
+          if (done > 0) ok = mbar_wait(&q_empty, (done - 1) & 1, failed, a.error_flag, 20);
           if (!ok) break;
-          mbar_expect_tx(&k_full[s], t.dpieces * PIECE);
-          for (int d = 0; d < t.dpieces; ++d) tma_load_3d(ks + (size_t)(s * t.dpieces + d) * PIECE, &map_k, d * 64, w.kvh, krow, &k_full[s]);
+          mbar_expect_tx(&q_full, t.dpieces * PIECE);
+          for (int d = 0; d < t.dpieces; ++d) tma_load_3d(qs + (size_t)d * PIECE, &map_q, d * 64, w.head, w.first + w.q0, &q_full);
+        }
+        for (int j = 0; j < w.tiles && ok; ++j) {
+          const int krow = a.key_start[w.seq] + w.start(j);
+          const uint32_t gt = g + j, v = gt % t.vstages;
+          for (int d = 0; d < t.dpieces; ++d, ++kp) {
+            const uint32_t s = kp % t.kstages;
+            if (kp >= (uint32_t)t.kstages) ok = mbar_wait(&k_empty[s], ((kp / t.kstages) - 1) & 1, failed, a.error_flag, 21);
+            if (!ok) break;
+            mbar_expect_tx(&k_full[s], kstage_bytes);
+            tma_load_3d(ks + (size_t)s * kstage_bytes, &map_k, d * 64, key_head * w.kvh, krow, &k_full[s]);
+            if (!t.q_resident) tma_load_3d(ks + (size_t)s * kstage_bytes + PIECE, &map_q, d * 64, w.head, w.first + w.q0, &k_full[s]);
+          }
+          if (!ok) break;
           if (gt >= (uint32_t)t.vstages) ok = mbar_wait(&v_empty[v], ((gt / t.vstages) - 1) & 1, failed, a.error_flag, 22);
           if (!ok) break;
           mbar_expect_tx(&v_full[v], t.vpieces * PIECE);
@@ -121,17 +153,20 @@ __global__ void __launch_bounds__(192, 2)
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc_bf16(QROWS, KROWS), idesc_o = umma_idesc_bf16(QROWS, t.vn, true);
-      auto scores = [&](uint32_t gt, bool last) -> bool {
-        const uint32_t s = gt % t.kstages;
-        if (!mbar_wait(&k_full[s], (gt / t.kstages) & 1, failed, a.error_flag, 23)) return false;
-        tc_fence_after();
-        for (int k = 0; k < t.ksteps; ++k) {
-          const uint64_t dq = umma_desc_sw128(qs + (size_t)(k >> 2) * PIECE) + (uint64_t)((k & 3) * 2);
-          const uint64_t dk = umma_desc_sw128(ks + (size_t)(s * t.dpieces + (k >> 2)) * PIECE) + (uint64_t)((k & 3) * 2);
-          umma_bf16_ss(tmem + COL_S, dq, dk, idesc_s, k != 0);
+      uint32_t kp = 0;
+      auto scores = [&](bool last) -> bool {
+        for (int d = 0; d < t.dpieces; ++d, ++kp) {
+          const uint32_t s = kp % t.kstages;
+          if (!mbar_wait(&k_full[s], (kp / t.kstages) & 1, failed, a.error_flag, 23)) return false;
+          tc_fence_after();
+          const uint8_t* kt = ks + (size_t)s * kstage_bytes;
+          const uint8_t* qt = t.q_resident ? qs + (size_t)d * PIECE : kt + PIECE;
+          const int steps = min(4, t.ksteps - d * 4);
+          for (int k = 0; k < steps; ++k)
+            umma_bf16_ss(tmem + COL_S, umma_desc_sw128(qt) + (uint64_t)(k * 2), umma_desc_sw128(kt) + (uint64_t)(k * 2), idesc_s, (d | k) != 0);
+          umma_commit(&k_empty[s]);
         }
-        umma_commit(&k_empty[s]);
-        if (last) umma_commit(&q_empty);
+        if (last && t.q_resident) umma_commit(&q_empty);
         umma_commit(&s_full);
         return true;
       };
@@ -139,13 +174,13 @@ __global__ void __launch_bounds__(192, 2)
       // but the very first one follows such a wait.
       for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
         if (!w.set(a, it, qtiles)) continue;
-        ok = mbar_wait(&q_full, done & 1, failed, a.error_flag, 24) && scores(g, w.tiles == 1);
+        ok = (!t.q_resident || mbar_wait(&q_full, done & 1, failed, a.error_flag, 24)) && scores(w.tiles == 1);
         for (int j = 0; j < w.tiles && ok; ++j) {
           const uint32_t gt = g + j;
           ok = mbar_wait(&p_ready, gt & 1, failed, a.error_flag, 25);  // P is written, S has been read
           if (!ok) break;
           tc_fence_after();
-          if (j + 1 < w.tiles) ok = scores(gt + 1, j + 2 == w.tiles);
+          if (j + 1 < w.tiles) ok = scores(j + 2 == w.tiles);
           const uint32_t v = gt % t.vstages;
           ok = ok && mbar_wait(&v_full[v], (gt / t.vstages) & 1, failed, a.error_flag, 26);
           if (ok && j == 0 && done > 0) ok = mbar_wait(&o_free, (done - 1) & 1, failed, a.error_flag, 30);  // O of the item before has been read
@@ -168,9 +203,9 @@ __global__ void __launch_bounds__(192, 2)
     for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
       if (!w.set(a, it, qtiles)) continue;
       const int qrow = w.q0 + r, pos = w.p0 + min(qrow, w.n - 1);
-      const int lo_row = max(pos / l.span * l.span - w.base_pos, 0), hi_row = pos - w.base_pos;
-      const int lo_all = max(w.pos_b / l.span * l.span - w.base_pos, 0), hi_all = w.pos_a - w.base_pos;  // keys every row sees
-      float m_ref = -1e30f, sum = 0.f;
+      const int lo_row = l.life.low(w.p0, pos), hi_row = l.life.row(w.p0, pos), keep = l.life.keep;
+      const int lo_all = l.life.low(w.p0, w.pos_b), hi_all = l.life.row(w.p0, w.pos_a);  // keys every row sees
+      float m_ref = l.sink ? l.sink[w.head] * LOG2E : -1e30f, sum = l.sink ? 1.f : 0.f;
       for (int j = 0; j < w.tiles && ok; ++j) {
         const uint32_t gt = g + j;
         ok = __all_sync(ALL_LANES, mbar_wait(&s_full, gt & 1, failed, a.error_flag, 27));
@@ -184,12 +219,12 @@ __global__ void __launch_bounds__(192, 2)
 #pragma unroll
           for (int i = 0; i < 32; ++i) s[c * 32 + i] = v[i];
         }
-        const int k0 = w.lo + j * KROWS;
-        if (k0 < lo_all || k0 + KROWS - 1 > hi_all) {
-          const int lo_i = lo_row - k0, hi_i = hi_row - k0;
+        const int k0 = w.start(j), k1 = w.end(j);
+        if (j < w.kept_tiles ? k0 + KROWS > k1 : k0 < lo_all || k0 + KROWS - 1 > hi_all) {
+          const int lo_i = lo_row - k0, hi_i = min(hi_row, k1 - 1) - k0, keep_i = keep - k0;
 #pragma unroll
           for (int i = 0; i < 128; ++i)
-            if (i < lo_i || i > hi_i) s[i] = scale2 < 0.f ? INFINITY : -INFINITY;
+            if ((i < lo_i && i >= keep_i) || i > hi_i) s[i] = scale2 < 0.f ? INFINITY : -INFINITY;
         }
         float mx[4];
 #pragma unroll
@@ -246,9 +281,54 @@ __global__ void __launch_bounds__(192, 2)
       if (ok) ok = __all_sync(ALL_LANES, mbar_wait(&pv_done, (g + w.tiles - 1) & 1, failed, a.error_flag, 29));
       if (!ok) break;
       tc_fence_after();
-      const float inv = l.out_scale / sum;
+      float inv = l.out_scale / sum;
+      if (l.off_gate >= 0 && qrow < w.n) inv *= sigmoid_f(a.p[(size_t)(w.first + qrow) * a.ldp + l.off_gate + w.head]);
       __nv_bfloat16* y = static_cast<__nv_bfloat16*>(a.y) + (size_t)(w.first + qrow) * a.ldy + w.head * l.vdim;
       const bool vec = l.vdim % 8 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+      if (l.v_rot) {  // pairs (c, c + half) are turned back by the row's angle
+        const int half = l.vdim >> 1;
+        const float2* cs = a.v_rot + (size_t)(w.first + min(qrow, w.n - 1)) * half;
+        const bool vec2 = vec && half % 8 == 0;
+        for (int c = 0; c < half; c += 16) {
+          float u[16], v[16];
+          tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)c, u);
+          tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)(half + c), v);
+          if (c + 16 >= half) {
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&o_free);
+          }
+          if (qrow < w.n) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i)
+              if (c + i < half) {
+                const float2 r = cs[c + i];
+                const float x = u[i] * inv, z = v[i] * inv;
+                u[i] = x * r.x + z * r.y;
+                v[i] = z * r.x - x * r.y;
+              }
+            if (vec2) {
+#pragma unroll
+              for (int h = 0; h < 2; ++h)
+                if (c + h * 8 < half) {
+                  store8(y + c + h * 8, u + h * 8);
+                  store8(y + half + c + h * 8, v + h * 8);
+                }
+            } else {
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                if (c + i < half) {
+                  y[c + i] = __float2bfloat16_rn(u[i]);
+                  y[half + c + i] = __float2bfloat16_rn(v[i]);
+                }
+            }
+          }
+          __syncwarp();
+        }
+        g += w.tiles;
+        ++done;
+        continue;
+      }
       for (int c = 0; c < t.vn; c += 16) {
         float o[16];
         tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)c, o);
@@ -262,13 +342,9 @@ __global__ void __launch_bounds__(192, 2)
 #pragma unroll
           for (int h = 0; h < 2; ++h)
             if (c + h * 8 < l.vdim) {
-              uint32_t u[4];
 #pragma unroll
-              for (int i = 0; i < 4; ++i) {
-                const __nv_bfloat162 b = __floats2bfloat162_rn(o[h * 8 + 2 * i] * inv, o[h * 8 + 2 * i + 1] * inv);
-                u[i] = *reinterpret_cast<const uint32_t*>(&b);
-              }
-              *reinterpret_cast<uint4*>(y + c + h * 8) = make_uint4(u[0], u[1], u[2], u[3]);
+              for (int i = 0; i < 8; ++i) o[h * 8 + i] *= inv;
+              store8(y + c + h * 8, o + h * 8);
             }
         } else {
 #pragma unroll
@@ -286,13 +362,13 @@ __global__ void __launch_bounds__(192, 2)
   if (warp == 1) tmem_dealloc(tmem, (uint32_t)t.tmem_cols);
 }
 
-// BF16 [rows][heads][dim] (dim % 8 == 0), box = 64 elements of one head of 128 rows, 128-byte swizzle; columns past dim and
+// BF16 [rows][heads][dim] (dim % 8 == 0), rows `pitch` elements apart, box = 64 elements of one head of 128 rows, 128-byte swizzle; columns past dim and
 // rows past the end read as zero.
-bool make_head_map(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t heads, uint64_t dim) {
+bool make_head_map(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t heads, uint64_t dim, uint64_t pitch) {
   EncodeTiledFn fn = encode_fn();
   if (!fn) return false;
   cuuint64_t dims[3] = {dim, heads, rows};
-  cuuint64_t strides[2] = {dim * 2, heads * dim * 2};
+  cuuint64_t strides[2] = {dim * 2, pitch * 2};
   cuuint32_t box[3] = {64, 1, 128};
   cuuint32_t estr[3] = {1, 1, 1};
   return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -306,18 +382,35 @@ constexpr size_t TC_MAX_SMEM = 225 * 1024;
 cudaError_t launch_attention_tc(const AttentionPortionArgs& a, cudaStream_t s) {
   const AttentionLayer& l = a.l;
   TcShape t;
-  t.dpieces = (l.dimp + 63) / 64;
+  const int width = attention_q_width(l);
+  t.dpieces = (width + 63) / 64;
   t.vpieces = (l.vdimp + 63) / 64;
-  t.ksteps = (l.dimp + 15) / 16;
+  t.ksteps = (width + 15) / 16;
   t.vn = (l.vdimp + 15) / 16 * 16;
   t.tmem_cols = (int)COL_O + t.vn <= 256 ? 256 : 512;
-  auto bytes = [&](int stages) { return (size_t)(t.dpieces + stages * (t.dpieces + t.vpieces)) * PIECE + 1024; };
-  const int stages = bytes(2) <= TC_MAX_SMEM ? 2 : 1;
-  t.kstages = t.vstages = stages;
-  if (bytes(stages) > TC_MAX_SMEM) return cudaErrorInvalidValue;
+  // queries stay resident while two value tiles and a few key pieces fit beside them
+  auto bytes = [&] { return ((size_t)(t.q_resident ? t.dpieces + t.kstages : 2 * t.kstages) + (size_t)t.vstages * t.vpieces) * PIECE + 1024; };
+  t.vstages = 2;
+  t.q_resident = 1;
+  t.kstages = std::min(t.dpieces == 1 ? 2 : 4, 2 * t.dpieces);
+  if (bytes() > TC_MAX_SMEM) t.vstages = 1;
+  if (bytes() > TC_MAX_SMEM) {
+    t.q_resident = 0;
+    t.vstages = 2;
+    if (bytes() > TC_MAX_SMEM) t.vstages = 1;
+  }
+  if (bytes() > TC_MAX_SMEM) return cudaErrorInvalidValue;
+  for (const int most = std::min(MAX_KSTAGES, 2 * t.dpieces); t.kstages < most && t.dpieces > 1;) {  // deeper rings where there is room
+    ++t.kstages;
+    if (bytes() > TC_MAX_SMEM) {
+      --t.kstages;
+      break;
+    }
+  }
   CUtensorMap mq, mk, mv;
-  if (!make_head_map(&mq, a.q, a.rows, l.heads, l.dimp) || !make_head_map(&mk, a.k, a.krows, l.kv_heads, l.dimp) ||
-      !make_head_map(&mv, a.v, a.krows, l.kv_heads, l.vdimp))
+  const int key_heads = l.mix ? 1 : l.kv_heads;
+  if (!make_head_map(&mq, a.q, a.rows, l.heads, width, (uint64_t)l.heads * width) || !make_head_map(&mk, a.k, a.krows, key_heads, width, a.ldk) ||
+      !make_head_map(&mv, a.v, a.krows, l.kv_heads, l.vdimp, a.ldv))
     return cudaErrorInvalidValue;
   cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_MAX_SMEM);
   if (e != cudaSuccess) return e;
@@ -325,8 +418,8 @@ cudaError_t launch_attention_tc(const AttentionPortionArgs& a, cudaStream_t s) {
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-  const int per_sm = t.tmem_cols <= 256 && bytes(stages) <= 110 * 1024 ? 2 : 1;
-  return launch_kernel(attention_tc_kernel, dim3(std::min(items, sms * per_sm)), dim3(192), bytes(stages), s, false, mq, mk, mv, a, t, items,
+  const int per_sm = t.tmem_cols <= 256 && bytes() <= 110 * 1024 ? 2 : 1;
+  return launch_kernel(attention_tc_kernel, dim3(std::min(items, sms * per_sm)), dim3(192), bytes(), s, false, mq, mk, mv, a, t, items,
                        qtiles);
 }
 

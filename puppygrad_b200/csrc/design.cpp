@@ -10,7 +10,7 @@ namespace pg {
 namespace {
 
 // Largest sizes the kernels take (per head: shared-memory rows and registers; per model: 32-bit indexing).
-constexpr int MAX_WIDTH = 16384, MAX_HEAD_DIM = 256, MAX_HEADS = 1024, MAX_RANK = 512;
+constexpr int MAX_WIDTH = 16384, MAX_HEAD_DIM = 256, MAX_HEADS = 1024, MAX_RANK = 512, MAX_LATENT = 1024, MAX_TAPS = 64;
 
 struct Reader {
   std::string path;
@@ -36,19 +36,34 @@ struct Reader {
     *out = (float)f->num;
     return PG_OK;
   }
+  int number(const Json& j, const std::string& where, const char* key, double* out) const {
+    float f = 0.f;
+    if (int e = number(j, where, key, &f)) return e;
+    *out = j.get(key)->num;
+    return PG_OK;
+  }
 };
+
+int heads_divide(const Reader& r, const std::string& where, int heads, int kv_heads) {
+  if (heads % kv_heads == 0) return PG_OK;
+  return r.fail(where + ": heads " + std::to_string(heads) + " must be divisible by kv_heads " + std::to_string(kv_heads));
+}
+
+// heads, kv_heads, dim, vdim, scale of grouped-head attention.
+int read_head_sizes(const Reader& r, const Json& m, const std::string& where, AttentionSpec* a) {
+  if (int e = r.integer(m, where, "heads", 1, MAX_HEADS, &a->heads)) return e;
+  if (int e = r.integer(m, where, "kv_heads", 1, MAX_HEADS, &a->kv_heads)) return e;
+  if (int e = r.integer(m, where, "dim", 1, MAX_HEAD_DIM, &a->dim)) return e;
+  if (int e = r.integer(m, where, "vdim", 1, MAX_HEAD_DIM, &a->vdim)) return e;
+  if (int e = r.number(m, where, "scale", &a->scale)) return e;
+  return heads_divide(r, where, a->heads, a->kv_heads);
+}
 
 // Grouped-head attention: heads, kv_heads, dim, vdim, scale and an optional mask {size}.
 int read_attention(const Reader& r, const Json& m, const std::string& where, BranchSpec* b) {
   b->kind = BranchSpec::ATTENTION;
   AttentionSpec& a = b->attn;
-  if (int e = r.integer(m, where, "heads", 1, MAX_HEADS, &a.heads)) return e;
-  if (int e = r.integer(m, where, "kv_heads", 1, MAX_HEADS, &a.kv_heads)) return e;
-  if (int e = r.integer(m, where, "dim", 1, MAX_HEAD_DIM, &a.dim)) return e;
-  if (int e = r.integer(m, where, "vdim", 1, MAX_HEAD_DIM, &a.vdim)) return e;
-  if (int e = r.number(m, where, "scale", &a.scale)) return e;
-  if (a.heads % a.kv_heads != 0)
-    return r.fail(where + ": heads " + std::to_string(a.heads) + " must be divisible by kv_heads " + std::to_string(a.kv_heads));
+  if (int e = read_head_sizes(r, m, where, &a)) return e;
   const Json* mask = m.get("mask");
   if (mask && mask->kind == Json::Object) {
     if (int e = r.integer(*mask, where + ".mask", "size", 1, 1 << 30, &a.chunk)) return e;
@@ -80,10 +95,10 @@ int read_delta(const Reader& r, const Json& m, const std::string& where, BranchS
   return PG_OK;
 }
 
-// Dirurax: layers of type "gla" (gated linear attention) and "parallel" (chunked attention with normed queries, keys
-// and values beside a generalized delta rule), each with an optional dense feed-forward.
-int parse_dirurax(const Json& root, const std::string& path, LayeredConfig* out) {
-  Reader r{path};
+// Sizes, eps and the list of layers, each with an optional dense feed-forward; `mixer(type, entry, where, layer, known)` fills in
+// the branches of a layer.
+int read_layers(const Reader& r, const Json& root, LayeredConfig* out,
+                const std::function<int(const std::string&, const Json&, const std::string&, LayerSpec*, bool*)>& mixer) {
   if (int e = r.integer(root, "model", "vocab", 1, 1 << 24, &out->vocab)) return e;
   if (int e = r.integer(root, "model", "width", 1, MAX_WIDTH, &out->width)) return e;
   const Json* norm = r.object(root, "norm");
@@ -95,33 +110,14 @@ int parse_dirurax(const Json& root, const std::string& path, LayeredConfig* out)
   for (size_t i = 0; i < layers->arr.size(); ++i) {
     const Json& j = layers->arr[i];
     const std::string where = "layers[" + std::to_string(i) + "]";
-    const Json* type = j.get("type");
-    const Json* mixer = r.object(j, "mixer");
+    const Json *type = j.get("type"), *mix = r.object(j, "mixer");
     if (!type || type->kind != Json::String) return r.fail(where + ": missing `type`");
-    if (!mixer) return r.fail(where + ": missing `mixer`");
+    if (!mix) return r.fail(where + ": missing `mixer`");
     LayerSpec l;
     l.type = type->str;
-    if (l.type == "gla") {
-      BranchSpec b;
-      b.prefix = "mix";
-      if (int e = read_gla(r, *mixer, where + ".mixer", &b)) return e;
-      l.branches.push_back(b);
-    } else if (l.type == "parallel") {
-      const Json *left = r.object(*mixer, "left"), *right = r.object(*mixer, "right");
-      if (!left || !right) return r.fail(where + ".mixer: missing `left` or `right`");
-      BranchSpec a, d;
-      a.prefix = "mix.left";
-      d.prefix = "mix.right";
-      if (int e = read_attention(r, *left, where + ".mixer.left", &a)) return e;
-      a.attn.qk_norm = a.attn.v_norm = true;
-      if (int e = read_delta(r, *right, where + ".mixer.right", &d)) return e;
-      if (int e = r.number(*mixer, where + ".mixer", "left_scale", &a.scale)) return e;
-      if (int e = r.number(*mixer, where + ".mixer", "right_scale", &d.scale)) return e;
-      l.branches.push_back(a);
-      l.branches.push_back(d);
-    } else {
-      return r.fail(where + ": unknown type \"" + l.type + "\"");
-    }
+    bool known = true;
+    if (int e = mixer(l.type, *mix, where + ".mixer", &l, &known)) return e;
+    if (!known) return r.fail(where + ": unknown type \"" + l.type + "\"");
     const Json* mlp = j.get("mlp");
     if (mlp && mlp->kind == Json::Object) {
       const Json* kind = mlp->get("kind");
@@ -135,7 +131,105 @@ int parse_dirurax(const Json& root, const std::string& path, LayeredConfig* out)
   return PG_OK;
 }
 
-const Design kDesigns[] = {{"Dirurax", parse_dirurax}};
+// Dirurax: layers of type "gla" (gated linear attention) and "parallel" (chunked attention with normed queries, keys
+// and values beside a generalized delta rule), each with an optional dense feed-forward.
+int parse_dirurax(const Json& root, const std::string& path, LayeredConfig* out) {
+  Reader r{path};
+  return read_layers(r, root, out, [&](const std::string& type, const Json& mixer, const std::string& where, LayerSpec* l, bool* known) -> int {
+    if (type == "gla") {
+      BranchSpec b;
+      b.prefix = "mix";
+      if (int e = read_gla(r, mixer, where, &b)) return e;
+      l->branches.push_back(b);
+    } else if (type == "parallel") {
+      const Json *left = r.object(mixer, "left"), *right = r.object(mixer, "right");
+      if (!left || !right) return r.fail(where + ": missing `left` or `right`");
+      BranchSpec a, d;
+      a.prefix = "mix.left";
+      d.prefix = "mix.right";
+      if (int e = read_attention(r, *left, where + ".left", &a)) return e;
+      a.attn.qk_norm = a.attn.v_norm = true;
+      if (int e = read_delta(r, *right, where + ".right", &d)) return e;
+      if (int e = r.number(mixer, where, "left_scale", &a.scale)) return e;
+      if (int e = r.number(mixer, where, "right_scale", &d.scale)) return e;
+      l->branches.push_back(a);
+      l->branches.push_back(d);
+    } else {
+      *known = false;
+    }
+    return PG_OK;
+  });
+}
+
+// Rotated attention with mixed heads, a sink and a window that keeps the first tokens.
+int read_window_attention(const Reader& r, const Json& m, const std::string& where, BranchSpec* b) {
+  b->kind = BranchSpec::ATTENTION;
+  AttentionSpec& a = b->attn;
+  if (int e = read_head_sizes(r, m, where, &a)) return e;
+  const Json *rot = r.object(m, "rot"), *mask = r.object(m, "mask");
+  if (!rot) return r.fail(where + ": missing `rot`");
+  if (!mask) return r.fail(where + ": missing `mask`");
+  if (int e = r.integer(*mask, where + ".mask", "size", 1, 1 << 30, &a.window)) return e;
+  if (int e = r.integer(*mask, where + ".mask", "keep_first", 0, 1 << 30, &a.keep_first)) return e;
+  if (int e = r.integer(*rot, where + ".rot", "dims", 0, a.dim, &a.rot_dims)) return e;
+  if (int e = r.number(*rot, where + ".rot", "base", &a.rot_base)) return e;
+  if (!(a.rot_base > 0)) return r.fail(where + ".rot: base must be > 0");
+  if (a.rot_dims % 2 != 0 || a.vdim % 2 != 0) return r.fail(where + ": rot.dims and vdim must be even");
+  a.bias = a.v_rot = a.head_mix = a.sink = true;
+  return PG_OK;
+}
+
+int read_latent_attention(const Reader& r, const Json& m, const std::string& where, BranchSpec* b) {
+  b->kind = BranchSpec::LATENT;
+  AttentionSpec& a = b->attn;
+  if (int e = r.integer(m, where, "heads", 1, MAX_HEADS, &a.heads)) return e;
+  if (int e = r.integer(m, where, "dim", 1, MAX_HEAD_DIM, &a.dim)) return e;
+  if (int e = r.integer(m, where, "vdim", 1, MAX_HEAD_DIM, &a.vdim)) return e;
+  if (int e = r.integer(m, where, "kv_rank", 1, MAX_LATENT, &a.kv_rank)) return e;
+  if (int e = r.integer(m, where, "q_rank", 1, MAX_WIDTH, &a.q_rank)) return e;
+  if (int e = r.number(m, where, "scale", &a.scale)) return e;
+  a.kv_heads = 1;
+  a.head_gate = true;
+  return PG_OK;
+}
+
+int read_channel_delta(const Reader& r, const Json& m, const std::string& where, BranchSpec* b) {
+  b->kind = BranchSpec::RECURRENCE;
+  RecurrenceSpec& s = b->rec;
+  s.kind = RECUR_CHANNEL;
+  if (int e = r.integer(m, where, "heads", 1, MAX_HEADS, &s.heads)) return e;
+  if (int e = r.integer(m, where, "kv_heads", 1, MAX_HEADS, &s.kv_heads)) return e;
+  if (int e = r.integer(m, where, "dim", 1, MAX_HEAD_DIM, &s.dim)) return e;
+  if (int e = r.integer(m, where, "vdim", 1, MAX_HEAD_DIM, &s.vdim)) return e;
+  if (int e = r.integer(m, where, "conv", 1, MAX_TAPS, &s.conv)) return e;
+  return heads_divide(r, where, s.heads, s.kv_heads);
+}
+
+// Sanesun: layers of type "attention", "channel_delta" and "latent_attention", each beside an optional dense feed-forward
+// that reads the same normed input; RMS norms, no position vectors, a head of its own.
+int parse_sanesun(const Json& root, const std::string& path, LayeredConfig* out) {
+  Reader r{path};
+  out->norm_kind = NORM_RMS;
+  out->activation = ACT_XIELU;
+  out->post_norms = out->sinusoids = out->tied_head = false;
+  out->parallel_ff = true;
+  const Json* embedding = r.object(root, "embedding");
+  if (!embedding) return r.fail("model: missing `embedding`");
+  if (int e = r.number(*embedding, "embedding", "scale", &out->embed_scale)) return e;
+  return read_layers(r, root, out, [&](const std::string& type, const Json& mixer, const std::string& where, LayerSpec* l, bool* known) -> int {
+    BranchSpec b;
+    b.prefix = "mix";
+    int e = PG_OK;
+    if (type == "attention") e = read_window_attention(r, mixer, where, &b);
+    else if (type == "channel_delta") e = read_channel_delta(r, mixer, where, &b);
+    else if (type == "latent_attention") e = read_latent_attention(r, mixer, where, &b);
+    else *known = false;
+    l->branches.push_back(b);
+    return e;
+  });
+}
+
+const Design kDesigns[] = {{"Dirurax", parse_dirurax}, {"Sanesun", parse_sanesun}};
 
 }  // namespace
 
@@ -198,43 +292,69 @@ int check_layered_tensors(const SafeTensorsFile& file, const std::string& path, 
   const int64_t W = cfg->width;
   auto norm = [&](const std::string& name) -> int {
     if (int r = want(name, {W})) return r;
-    return want(name + ".b", {W});
+    return cfg->norm_kind == NORM_LAYER ? want(name + ".b", {W}) : PG_OK;
   };
   if (int r = want("embed", {cfg->vocab, W})) return r;
+  if (!cfg->tied_head)
+    if (int r = want("head", {cfg->vocab, W})) return r;
   if (int r = norm("final.norm")) return r;
   for (size_t i = 0; i < cfg->layers.size(); ++i) {
     LayerSpec& l = cfg->layers[i];
     const std::string p = "l" + std::to_string(i) + ".";
     if (int r = norm(p + "norm1")) return r;
-    if (int r = norm(p + "norm1b")) return r;
+    if (cfg->post_norms)
+      if (int r = norm(p + "norm1b")) return r;
     for (BranchSpec& b : l.branches) {
       const std::string m = p + b.prefix + ".";
-      std::vector<std::pair<std::string, std::vector<int64_t>>> t;
-      int* rank = nullptr;
+      std::vector<std::pair<std::string, std::vector<int64_t>>> t, t2;  // t2: tensors of the second unknown size
+      int *rank = nullptr, *rank2 = nullptr;
       if (b.kind == BranchSpec::ATTENTION) {
         const AttentionSpec& a = b.attn;
         const int64_t H = a.heads, G = a.kv_heads;
         t = {{"q", {H * a.dim, W}}, {"k", {G * a.dim, W}}, {"v", {G * a.vdim, W}}, {"o", {W, H * a.vdim}}};
         if (a.qk_norm) t.insert(t.end(), {{"q.norm", {a.dim}}, {"k.norm", {a.dim}}});
+        if (a.bias) t.insert(t.end(), {{"q.b", {H * a.dim}}, {"k.b", {G * a.dim}}, {"v.b", {G * a.vdim}}});
+        if (a.head_mix) t.push_back({"talk", {H, H}});
+        if (a.sink) t.push_back({"sink", {H}});
+      } else if (b.kind == BranchSpec::LATENT) {
+        const AttentionSpec& a = b.attn;
+        const int64_t H = a.heads;
+        t = {{"dq", {a.q_rank, W}}, {"dq.norm", {a.q_rank}}, {"uq", {H * a.dim, a.q_rank}}, {"dkv", {a.kv_rank, W}},
+             {"dkv.norm", {a.kv_rank}}, {"uk", {H * a.dim, a.kv_rank}}, {"uv", {H * a.vdim, a.kv_rank}}, {"o", {W, H * a.vdim}}};
+        if (a.head_gate) t.push_back({"g", {H, W}});
       } else {
         RecurrenceSpec& s = b.rec;
         rank = &s.rank;
-        const int64_t K = (int64_t)s.heads * s.dim, V = (int64_t)s.heads * s.vdim;
-        if (s.kind == RECUR_GLA)
+        const int64_t K = (int64_t)s.heads * s.dim, V = (int64_t)s.heads * s.vdim, Q = (int64_t)s.kv_heads * s.dim;
+        if (s.kind == RECUR_GLA) {
           t = {{"q", {K, W}}, {"k", {K, W}}, {"v", {V, W}}, {"g", {V, W}}, {"o", {W, V}}, {"norm", {s.vdim}},
                {"a1", {-1, W}}, {"a2", {K, -1}}, {"a2.b", {K}}};
-        else
+        } else if (s.kind == RECUR_DELTA) {
           t = {{"r", {K, W}}, {"k", {K, W}}, {"v", {V, W}}, {"g", {V, W}}, {"o", {W, V}}, {"norm", {V}},
                {"a", {K, W}}, {"a.b", {K}}, {"w1", {-1, W}}, {"w2", {K, -1}}, {"w0", {K}}};
+        } else {
+          t = {{"q", {Q, W}}, {"k", {Q, W}}, {"v", {V, W}}, {"q.conv", {Q, s.conv}}, {"k.conv", {Q, s.conv}}, {"v.conv", {V, s.conv}},
+               {"b", {s.heads, W}}, {"A_log", {s.heads}}, {"norm", {s.vdim}}, {"o", {W, V}}, {"dt_bias", {K}},
+               {"a1", {-1, W}}, {"a2", {K, -1}}};
+          t2 = {{"g1", {-1, W}}, {"g2", {V, -1}}};
+          rank2 = &s.rank2;
+        }
       }
       for (auto& e : t)
         if (int r = want(m + e.first, e.second, rank)) return r;
-      if (rank && (*rank < 1 || *rank > MAX_RANK))
-        return set_error(PG_INVALID_WEIGHTS, m + "* has a decay rank outside 1.." + std::to_string(MAX_RANK));
+      for (auto& e : t2)
+        if (int r = want(m + e.first, e.second, rank2)) return r;
+      for (const int* n : {rank, rank2})
+        if (n && (*n < 1 || *n > MAX_RANK))
+          return set_error(PG_INVALID_WEIGHTS, m + "* has a decay or gate rank outside 1.." + std::to_string(MAX_RANK));
     }
     if (l.ff > 0) {
-      if (int r = norm(p + "norm2")) return r;
-      if (int r = norm(p + "norm2b")) return r;
+      if (!cfg->parallel_ff)
+        if (int r = norm(p + "norm2")) return r;
+      if (cfg->post_norms)
+        if (int r = norm(p + "norm2b")) return r;
+      if (cfg->activation == ACT_XIELU)
+        if (int r = want(p + "mlp.act", {2})) return r;
       if (int r = want(p + "mlp.up", {l.ff, W})) return r;
       if (int r = want(p + "mlp.down", {W, l.ff})) return r;
     }

@@ -38,6 +38,26 @@ __device__ __forceinline__ void gelu_erf_pair(float& x, float& y) {
   y *= py;
 }
 
+__device__ __forceinline__ float exp2_fast(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+// xIELU for results that are rounded to BF16 next: e^z - 1 - z is off by less than 1e-6 here, far below z / 2 wherever that
+// rounds to a BF16 of its own.
+__device__ __forceinline__ float xielu_fast(float z, float a, float b) {
+  const float e = exp2_fast(fminf(z, 0.f) * 1.4426950408889634f) - 1.f - z;
+  return fmaf(0.5f, z, z > 0.f ? a * z * z : b * e);
+}
+__device__ __forceinline__ void activate_pair(const ActArgs& act, float& x, float& y) {
+  if (act.kind == ACT_GELU_ERF) {
+    gelu_erf_pair(x, y);
+  } else if (act.kind == ACT_XIELU) {
+    x = xielu_fast(x, act.a, act.b);
+    y = xielu_fast(y, act.a, act.b);
+  }
+}
+
 __device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, int x, int y, const void* smem_src) {
   asm volatile("cp.async.bulk.tensor.2d.global.shared::cta.bulk_group [%0, {%1, %2}], [%3];" ::"l"(map), "r"(x), "r"(y),
                "r"(smem_u32(smem_src))
@@ -60,7 +80,7 @@ struct BfSmem {
   static constexpr size_t BYTES = (size_t)STAGES * (A_BYTES + B_BYTES) + EPI_BYTES + 1024 /*align*/ + 256 /*barriers*/;
 };
 
-enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_BF16_GELU = 2 };
+enum { OUT_F32 = 0, OUT_BF16 = 1, OUT_BF16_ACT = 2 };
 
 // Persistent over 128 x BN output tiles; two accumulators in tensor memory, so that the epilogue of a tile overlaps the
 // products of the next. Warp 0 loads, warp 1 issues the MMAs and owns the tensor memory, warps 2..5 store. `tma_out`:
@@ -186,9 +206,9 @@ __global__ void __launch_bounds__(192, 1)
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
             if (half) tmem_ld32(tmem_d + (uint32_t)(c0 + 32), v);
-            if (out_kind == OUT_BF16_GELU) {
+            if (out_kind == OUT_BF16_ACT) {
 #pragma unroll
-              for (int j = 0; j < 32; j += 2) gelu_erf_pair(v[j], v[j + 1]);
+              for (int j = 0; j < 32; j += 2) activate_pair(a.act, v[j], v[j + 1]);
             }
             uint32_t p[16];
 #pragma unroll
@@ -357,11 +377,13 @@ __global__ void __launch_bounds__(192, 1)
         float s = 0.f;
 #pragma unroll
         for (int sp = 0; sp < SPLITS; ++sp) s += recv[(size_t)(sp * BN + j) * RP + rl];  // in split order
-        if (out_kind == OUT_BF16_GELU) {
+        const bool split = a.act_from > 0 && feat >= a.act_from;
+        if (out_kind == OUT_BF16_ACT || split) {
           float z = 0.f;
-          gelu_erf_pair(s, z);
+          activate_pair(a.act, s, z);
         }
-        if (out_kind == OUT_F32) a.out[(size_t)j * a.ldo + feat] = s;
+        if (split) static_cast<__nv_bfloat16*>(a.out_act)[(size_t)j * a.ldo_act + feat - a.act_from] = __float2bfloat16_rn(s);
+        else if (out_kind == OUT_F32) a.out[(size_t)j * a.ldo + feat] = s;
         else static_cast<__nv_bfloat16*>(a.out_h)[(size_t)j * a.ldo + feat] = __float2bfloat16_rn(s);
       }
     }
@@ -396,7 +418,7 @@ bool make_out_map(CUtensorMap* map, void* ptr, bool bf16, uint64_t rows, uint64_
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-int out_kind_of(const Bf16GemmArgs& a) { return a.out ? OUT_F32 : a.gelu_erf ? OUT_BF16_GELU : OUT_BF16; }
+int out_kind_of(const Bf16GemmArgs& a) { return a.out ? OUT_F32 : a.act.kind != ACT_NONE ? OUT_BF16_ACT : OUT_BF16; }
 
 template <int BN>
 cudaError_t launch_bn(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
@@ -455,8 +477,11 @@ cudaError_t launch_rows_bn(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
 
 }  // namespace
 
+bool gemm_bf16_rows_kernel(int m, int k) { return m <= 64 && k % KB == 0; }
+
 cudaError_t launch_tc_gemm_bf16(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
   if (a.m <= 0 || a.n <= 0) return cudaSuccess;
+  if (a.act_from > 0 && (!a.w_tiled || !gemm_bf16_rows_kernel(a.m, a.k))) return cudaErrorInvalidValue;
   if (a.k <= 0 || a.k % 8 != 0 || (!a.out && !a.out_h)) return cudaErrorInvalidValue;
   if (a.w_tiled && a.k % KB == 0) {
     if (a.m <= 16) return launch_rows_bn<16>(a, pdl, s);

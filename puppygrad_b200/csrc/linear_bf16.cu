@@ -82,7 +82,7 @@ __global__ void __launch_bounds__(RL_THREADS, 1) rows_linear_kernel(RowsLinearAr
   if (!a.fuse_norm) {
     for (int i = tid; i < MT * (kpad / 4); i += RL_THREADS) {
       const int m = i / (kpad / 4), k = (i % (kpad / 4)) * 4;
-      const float4 v = (m < a.m && k < a.k) ? load4(a.x + (size_t)m * a.ldx + k) : make_float4(0, 0, 0, 0);
+      const float4 v = (m < a.m && k < a.kx) ? mask4(load4(a.x + (size_t)m * a.ldx + k), k, a.kx) : make_float4(0, 0, 0, 0);
       store4(xs + (size_t)m * kpad + act_slot(k), v);
     }
   } else {
@@ -102,23 +102,26 @@ __global__ void __launch_bounds__(RL_THREADS, 1) rows_linear_kernel(RowsLinearAr
         store4(row + act_slot(c), v);
         s += (v.x + v.y) + (v.z + v.w);
       }
-      mean = group_sum(s, red, warp, lane, WPR) * inv_n;
-      float q = 0.f;
-      for (int c = t * 4; c < n.ldx; c += nt * 4) q += norm_step_square(load4(row + act_slot(c)), mean, c, n.width);
-      rstd = 1.f / sqrtf(group_sum(q, red, warp, lane, WPR) * inv_n + n.eps);
+      if (n.post_g) {
+        mean = n.norm == NORM_LAYER ? group_sum(s, red, warp, lane, WPR) * inv_n : 0.f;
+        float q = 0.f;
+        for (int c = t * 4; c < n.ldx; c += nt * 4) q += norm_step_square(load4(row + act_slot(c)), mean, c, n.width);
+        rstd = 1.f / sqrtf(group_sum(q, red, warp, lane, WPR) * inv_n + n.eps);
+      }
     }
     float s = 0.f;
     for (int c = t * 4; c < n.ldx; c += nt * 4) {
       float4 x = on ? norm_step_load_x<__nv_bfloat16>(n, m, c) : make_float4(0, 0, 0, 0);
       if (n.y && on) {
-        const float4 v = norm_step_apply(load4(row + act_slot(c)), mean, rstd, n.post_g, n.post_b, c, n.width);
+        float4 v = load4(row + act_slot(c));
+        if (n.post_g) v = norm_step_apply(v, mean, rstd, n.post_g, n.post_b, c, n.width);
         x.x += v.x; x.y += v.y; x.z += v.z; x.w += v.w;
       }
       if (on && n.x_out && blockIdx.x == 0) store4(n.x_out + (size_t)m * n.ldx + c, x);
       store4(row + act_slot(c), x);
       s += (x.x + x.y) + (x.z + x.w);
     }
-    mean = group_sum(s, red, warp, lane, WPR) * inv_n;
+    mean = n.norm == NORM_LAYER ? group_sum(s, red, warp, lane, WPR) * inv_n : 0.f;
     float q = 0.f;
     for (int c = t * 4; c < n.ldx; c += nt * 4) q += norm_step_square(load4(row + act_slot(c)), mean, c, n.width);
     rstd = 1.f / sqrtf(group_sum(q, red, warp, lane, WPR) * inv_n + n.eps);
@@ -168,8 +171,8 @@ __global__ void __launch_bounds__(RL_THREADS, 1) rows_linear_kernel(RowsLinearAr
       for (int q = 0; q < kparts; ++q) v += part[uu * kparts + q][e];
       const int row = ((round * upc + uu) * (int)gridDim.x + (int)blockIdx.x) * RL_ROWS + r;
       if (row < a.n && m < a.m) {
-        if (a.epilogue == ROWS_GELU_ERF) v = gelu_erf(v);
-        if (a.out) a.out[(size_t)m * a.ldo + row] = v;
+        if (row >= a.act_from) a.out_act[(size_t)m * a.ldo_act + row - a.act_from] = activate(a.act, v);
+        else if (a.out) a.out[(size_t)m * a.ldo + row] = v;
         if (v > bv) {  // a thread's rows only grow: strict > keeps the lowest index
           bv = v;
           bi = row;

@@ -7,6 +7,14 @@
 namespace pg {
 namespace {
 
+// xIELU: expm1 keeps e^z - 1 - z accurate near 0.
+__device__ __forceinline__ float xielu(float z, float a, float b) {
+  return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (expm1f(z) - z));
+}
+__device__ __forceinline__ float activate(const ActArgs& act, float z) {
+  return act.kind == ACT_GELU_ERF ? gelu_erf(z) : act.kind == ACT_XIELU ? xielu(z, act.a, act.b) : z;
+}
+
 // Zeroes the elements of columns >= width.
 __device__ __forceinline__ float4 mask4(float4 v, int c, int width) {
   if (c + 3 >= width) {
@@ -34,19 +42,20 @@ __device__ __forceinline__ float4 norm_step_load_x(const NormStepArgs& a, int ro
   float4 v;
   if (a.ids) {
     v = load4(static_cast<const T*>(a.embed) + (size_t)a.ids[row] * a.ld_embed + c);
-    if (c < a.width) {
+    v.x *= a.embed_scale; v.y *= a.embed_scale; v.z *= a.embed_scale; v.w *= a.embed_scale;
+    if (a.freq && c < a.width) {
       const float2 s = sinusoid(a.pos[row], a.freq[c >> 1]);
       v.x += s.x;
       v.y += s.y;
     }
-    if (c + 2 < a.width) {
+    if (a.freq && c + 2 < a.width) {
       const float2 s = sinusoid(a.pos[row], a.freq[(c >> 1) + 1]);
       v.z += s.x;
       v.w += s.y;
     }
   } else {
     const int src = a.row_index ? a.row_index[row] : row;
-    v = load4(a.x_in + (size_t)src * a.ldx + c);
+    v = c < a.width ? load4(a.x_in + (size_t)src * a.ld_in + c) : make_float4(0, 0, 0, 0);
   }
   return mask4(v, c, a.width);
 }
@@ -61,10 +70,10 @@ __device__ __forceinline__ float norm_step_square(float4 v, float mean, int c, i
   return q;
 }
 
-// (v - mean) * rstd * g + b, zero past width (g and b are padded to the row pitch).
+// (v - mean) * rstd * g [+ b], zero past width (g and b are padded to the row pitch).
 __device__ __forceinline__ float4 norm_step_apply(float4 v, float mean, float rstd, const float* g, const float* b, int c,
                                                   int width) {
-  const float4 gg = load4(g + c), bb = load4(b + c);
+  const float4 gg = load4(g + c), bb = b ? load4(b + c) : make_float4(0, 0, 0, 0);
   float4 o;
   o.x = (v.x - mean) * rstd * gg.x + bb.x;
   o.y = (v.y - mean) * rstd * gg.y + bb.y;

@@ -1,5 +1,5 @@
-// Row kernels of the layered models: embedding with sinusoidal positions, LayerNorm before and after a sublayer fused
-// with the FP32 residual sum, weight packing.
+// Row kernels of the layered models: embedding with sinusoidal positions, LayerNorm or RMS norm before and after a sublayer
+// fused with the FP32 residual sum, activations, weight packing.
 #include "device_util.cuh"
 #include "layered_kernels.cuh"
 #include "norm_step.cuh"
@@ -23,10 +23,13 @@ __global__ void __launch_bounds__(NORM_THREADS) norm_step_kernel(NormStepArgs a)
   }
   const float inv_n = 1.f / (float)a.width;
   auto moments = [&](const float4 (&v)[V4], float* mean, float* rstd) {
-    float s = 0.f;
+    *mean = 0.f;
+    if (a.norm == NORM_LAYER) {
+      float s = 0.f;
 #pragma unroll
-    for (int j = 0; j < V4; ++j) s += (v[j].x + v[j].y) + (v[j].z + v[j].w);  // columns past width are zero
-    *mean = block_sum(s, red) * inv_n;
+      for (int j = 0; j < V4; ++j) s += (v[j].x + v[j].y) + (v[j].z + v[j].w);  // columns past width are zero
+      *mean = block_sum(s, red) * inv_n;
+    }
     float q = 0.f;
 #pragma unroll
     for (int j = 0; j < V4; ++j) q += norm_step_square(v[j], *mean, (tid + j * NORM_THREADS) * 4, a.width);
@@ -39,13 +42,13 @@ __global__ void __launch_bounds__(NORM_THREADS) norm_step_kernel(NormStepArgs a)
       const int c = (tid + j * NORM_THREADS) * 4;
       y[j] = c < a.ldx ? mask4(load4(a.y + (size_t)row * a.ldx + c), c, a.width) : make_float4(0, 0, 0, 0);
     }
-    float mean, rstd;
-    moments(y, &mean, &rstd);
+    float mean = 0.f, rstd = 1.f;
+    if (a.post_g) moments(y, &mean, &rstd);
 #pragma unroll
     for (int j = 0; j < V4; ++j) {
       const int c = (tid + j * NORM_THREADS) * 4;
       if (c < a.width) {
-        const float4 n = norm_step_apply(y[j], mean, rstd, a.post_g, a.post_b, c, a.width);
+        const float4 n = a.post_g ? norm_step_apply(y[j], mean, rstd, a.post_g, a.post_b, c, a.width) : y[j];
         x[j].x += n.x; x[j].y += n.y; x[j].z += n.z; x[j].w += n.w;
       }
     }
@@ -57,14 +60,14 @@ __global__ void __launch_bounds__(NORM_THREADS) norm_step_kernel(NormStepArgs a)
       if (c < a.ldx) store4(a.x_out + (size_t)row * a.ldx + c, x[j]);
     }
   }
-  if (a.pre_g) {
-    float mean, rstd;
-    moments(x, &mean, &rstd);
+  if (a.h || a.h32) {
+    float mean = 0.f, rstd = 1.f;
+    if (a.norm != NORM_COPY) moments(x, &mean, &rstd);
 #pragma unroll
     for (int j = 0; j < V4; ++j) {
       const int c = (tid + j * NORM_THREADS) * 4;
       if (c < a.ldh) {
-        const float4 n = norm_step_apply(x[j], mean, rstd, a.pre_g, a.pre_b, c, a.width);
+        const float4 n = a.norm == NORM_COPY ? x[j] : norm_step_apply(x[j], mean, rstd, a.pre_g, a.pre_b, c, a.width);
         if (a.h32) store4(a.h32 + (size_t)row * a.ldh + c, n);
         else store4(static_cast<T*>(a.h) + (size_t)row * a.ldh + c, n);
       }
@@ -84,11 +87,14 @@ cudaError_t launch_norm_step_t(const NormStepArgs& a, int rows, bool pdl, cudaSt
   return cudaErrorInvalidValue;
 }
 
-__global__ void __launch_bounds__(256) gelu_erf_kernel(float* x, size_t n) {
+__global__ void __launch_bounds__(256) activation_kernel(const float* x, int ldx, float* out, int ldo, int rows, int cols, ActArgs act) {
   grid_dep_launch();
   grid_dep_wait();
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
-    x[i] = gelu_erf(x[i]);
+  const size_t n = (size_t)rows * cols;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / cols, c = i % cols;
+    out[r * ldo + c] = activate(act, x[r * ldx + c]);
+  }
 }
 
 __global__ void __launch_bounds__(256) pack_bf16_kernel(const float* __restrict__ src, __nv_bfloat16* dst, int rows, int cols,
@@ -121,8 +127,9 @@ cudaError_t launch_norm_step(const NormStepArgs& a, int rows, bool bf16, bool pd
   return bf16 ? launch_norm_step_t<__nv_bfloat16>(a, rows, pdl, s) : launch_norm_step_t<float>(a, rows, pdl, s);
 }
 
-cudaError_t launch_gelu_erf(float* x, size_t n, bool pdl, cudaStream_t s) {
-  return launch_kernel(gelu_erf_kernel, dim3(grid_for(n)), dim3(256), 0, s, pdl, x, n);
+cudaError_t launch_activation(const float* x, int ldx, float* out, int ldo, int rows, int cols, ActArgs act, bool pdl, cudaStream_t s) {
+  if (rows <= 0 || cols <= 0) return cudaSuccess;
+  return launch_kernel(activation_kernel, dim3(grid_for((size_t)rows * cols)), dim3(256), 0, s, pdl, x, ldx, out, ldo, rows, cols, act);
 }
 
 size_t tiled_bf16_elems(int rows, int ld) { return (size_t)((rows + 127) / 128) * 128 * ld; }

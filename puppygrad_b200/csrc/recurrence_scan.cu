@@ -135,6 +135,112 @@ __global__ void __launch_bounds__(256) delta_gates_vec_kernel(RecurrenceScanArgs
   }
 }
 
+// Channel delta rule: the convolutions of q, k and v with silu, unit vectors of q and k. A warp takes one head of q or k (2
+// kv_heads units) or of v (heads units) over CONV_ROWS rows; the last inputs stay in registers (TAPS > 0) or are read again.
+constexpr int CONV_ROWS = 16;
+template <int TAPS, int NE>
+__global__ void __launch_bounds__(256) channel_conv_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int lane = threadIdx.x & 31, units = 2 * l.kv_heads + l.heads, ntaps = TAPS > 0 ? TAPS : l.taps;
+  const int groups = (a.rows + CONV_ROWS - 1) / CONV_ROWS;
+  const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  if (w >= (long long)groups * units) return;
+  const int r0 = (int)(w / units) * CONV_ROWS, u = (int)(w % units), r1 = min(r0 + CONV_ROWS, a.rows);
+  const bool is_q = u < l.kv_heads, is_k = !is_q && u < 2 * l.kv_heads;
+  const int h = is_q ? u : is_k ? u - l.kv_heads : u - 2 * l.kv_heads, n = is_q || is_k ? l.dim : l.vdim;
+  const int ch0 = (is_q ? l.off_q : is_k ? l.off_k : l.off_v) - l.off_q + h * n, pitch = (is_q || is_k ? l.kv_heads : l.heads) * n;
+  float* dst = (is_q ? a.rate : is_k ? a.unit : a.vals) + h * n;
+  constexpr int NT = TAPS > 0 ? TAPS : 1;
+  float win[NT][NE], wt[NT][NE];  // inputs (the newest last) and weights
+  if (TAPS > 0) {
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int i = 0; i < NE; ++i) wt[t][i] = lane + i * 32 < n ? l.conv[(size_t)t * l.channels + ch0 + lane + i * 32] : 0.f;
+  }
+  int seq = -1, first = 0;
+  const float* taps = nullptr;
+  for (int r = r0; r < r1; ++r) {
+    const int s = a.row_seq[r];
+    const bool enter = s != seq;
+    if (enter) {
+      seq = s;
+      first = a.seq_start[s];
+      taps = a.taps + (size_t)a.seq_slot[s] * l.taps * l.channels;
+    }
+    const int pos = a.seq_pos[seq] + r - first;
+    float x[NE], sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < NE; ++i) {
+      const int c = lane + i * 32;
+      x[i] = 0.f;
+      if (TAPS > 0) {
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+          if (t + 1 < NT && !enter) win[t][i] = win[t + 1 < NT ? t + 1 : t][i];
+          else win[t][i] = c < n ? conv_input(l, a.p, a.ldp, taps, r, first, pos, NT - 1 - t, ch0 + c) : 0.f;
+        }
+#pragma unroll
+        for (int t = 0; t < NT; ++t) x[i] = fmaf(wt[t][i], win[t][i], x[i]);
+      } else if (c < n) {
+        for (int back = ntaps - 1; back >= 0; --back)
+          x[i] = fmaf(l.conv[(size_t)(ntaps - 1 - back) * l.channels + ch0 + c], conv_input(l, a.p, a.ldp, taps, r, first, pos, back, ch0 + c), x[i]);
+      }
+      x[i] = silu_f(x[i]);
+      sq += x[i] * x[i];
+    }
+    const float inv = is_q || is_k ? 1.f / sqrtf(lane_sum(sq) + UNIT_EPS) : 1.f;
+#pragma unroll
+    for (int i = 0; i < NE; ++i)
+      if (lane + i * 32 < n) dst[(size_t)r * pitch + lane + i * 32] = x[i] * inv;
+  }
+}
+
+// Channel delta rule, after the convolutions: the decays, and what the scan needs to take two tokens at a time: the next
+// token's k times its decay . this one's k, and the write strength. A warp takes a head over GATE_GROUP rows (and looks at
+// the row behind them).
+constexpr int GATE_GROUP = 8;
+template <int NE>
+__global__ void __launch_bounds__(256) channel_gates_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int lane = threadIdx.x & 31, K = l.heads * l.dim, rep = l.heads / l.kv_heads;
+  const int groups = (a.rows + GATE_GROUP - 1) / GATE_GROUP;
+  const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  if (w >= (long long)groups * l.heads) return;
+  const int r0 = (int)(w / l.heads) * GATE_GROUP, head = (int)(w % l.heads), end = min(r0 + GATE_GROUP, a.rows);
+  const int kv_pitch = l.kv_heads * l.dim;
+  float last[NE];
+#pragma unroll
+  for (int i = 0; i < NE; ++i) last[i] = 0.f;
+  for (int r = r0; r <= end && r < a.rows; ++r) {
+    float dot = 0.f;
+#pragma unroll
+    for (int i = 0; i < NE; ++i) {
+      const int c = lane + i * 32;
+      if (c < l.dim) {
+        const float d = channel_decay(l, head, head * l.dim + c, a.z[(size_t)r * a.ldz + head * l.dim + c]);
+        const float k = a.unit[(size_t)r * kv_pitch + head / rep * l.dim + c];
+        if (r < end) a.decay[(size_t)r * K + head * l.dim + c] = d;
+        dot = fmaf(d * k, last[i], dot);
+        last[i] = k;
+      }
+    }
+    dot = lane_sum(dot);
+    if (lane == 0 && r > r0) a.pair[((size_t)(r - 1) * l.heads + head) * 4] = dot;
+    if (lane == 0 && r < end) a.pair[((size_t)r * l.heads + head) * 4 + 1] = sigmoid_f(a.p[(size_t)r * a.ldp + l.off_b + head]);
+  }
+}
+
+// The inputs that the next tokens' convolutions still need. Block = (sequence, one of its last taps - 1 rows).
+__global__ void __launch_bounds__(256) channel_taps_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int seq = blockIdx.x, first = a.seq_start[seq], r = a.seq_start[seq + 1] - 1 - (int)blockIdx.y;
+  if (r < first) return;
+  const int pos = a.seq_pos[seq] + r - first;
+  float* dst = a.taps + ((size_t)a.seq_slot[seq] * l.taps + pos % l.taps) * l.channels;
+  for (int c = threadIdx.x; c < l.channels; c += blockDim.x) dst[c] = a.p[(size_t)r * a.ldp + l.off_q + c];
+}
+
 // ------------------------------------------------------------------ scan
 // Block = one head of one sequence (or of one segment of it), or a part of its columns. The last warp stages the rows of
 // TB tokens at a time in a ring of shared-memory stages (bulk copies where rows are 16-byte aligned); in the others
@@ -154,6 +260,8 @@ struct ScanArgs {
   int mode, tb;
   float *seg_state, *seg_trans;  // [nseq][max_segs][heads][dim][dvp], [nseq][max_segs][heads][dim][dkp] (GLA: [..][dim] decays)
   int dkp;
+  const float *k, *q, *v, *g;  // rows of keys, queries, values and gates (heads side by side) and their pitches
+  int ldk, ldq, ldv, ldg;
   int col_blocks, block_cols;  // column blocks of a head, columns of each (the last may have fewer)
   int vec;      // rows can be copied in 16-byte pieces
   int y_bf16;
@@ -197,14 +305,16 @@ struct GroupSum<N, 0> {
   static __device__ __forceinline__ void run(float*, int) {}
 };
 
-// The delta rule works on two tokens at a time: with e = (u' * w)^T S, where the dash marks the second token,
+// The delta rules work on two tokens at a time: with e = (u' * w)^T S, where the dash marks the second token,
 // u'^T S_t = e - (u' . b) d + (u' . k) v, so that both reads come from one reduction over the state before the pair.
+// Channel delta rule: u = w * k reads, and k x (beta (v - u^T S)) is written.
 template <int KIND, int RPL, int CPL>
 __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kernel(ScanArgs sa) {
   extern __shared__ __align__(16) float sm[];
   __shared__ uint64_t full[SCAN_STAGES], empty[SCAN_STAGES];
   __shared__ int failed_flag;
   constexpr int DKP = 8 * RPL, NA = KIND == KIND_DELTA ? 6 : 3, J = RPL / 4;  // staged key-channel arrays
+  constexpr bool PAIRS = KIND != KIND_GLA;
   const RecurrenceScanArgs& a = sa.a;
   const RecurrenceLayer& l = a.l;
   const int dk = l.dim, K = l.heads * dk, tid = threadIdx.x;
@@ -251,19 +361,25 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
     if (key) {
       off = arr * DKP;
       const float* gates[4] = {a.decay, a.unit, a.rate, a.unit_next};
-      if (arr == 0) src = a.p + l.off_k + head * dk;
-      else if (arr == 2) src = a.p + l.off_q + head * dk;
-      else {
+      const int kv = head / (l.heads / l.kv_heads);
+      if (arr == 0) {
+        src = sa.k + kv * dk;
+        pitch = sa.ldk;
+      } else if (arr == 2) {
+        src = sa.q + kv * dk;
+        pitch = sa.ldq;
+      } else {
         src = gates[arr == 1 ? 0 : arr - 2] + head * dk;
         pitch = K;
       }
     } else if (value || gate) {
       off = NA * DKP + (gate ? COLS : 0);
-      src = a.p + (gate ? l.off_g : l.off_v) + head * l.vdim + cbase;
+      src = (gate ? sa.g : sa.v) + head * l.vdim + cbase;
+      pitch = gate ? sa.ldg : sa.ldv;
     }
     const int count = key ? dk : dv;
     const uint32_t token_bytes = 4u * (uint32_t)((NA - (outputs ? 0 : 1)) * dk + (want_v ? dv : 0) + (want_g ? dv : 0)) +
-                                 (KIND == KIND_DELTA ? 16u : 0u);
+                                 (PAIRS ? 16u : 0u);
     for (int b = 0; b < blocks; ++b) {
       const int s = b % SCAN_STAGES, tb0 = t0 + b * TB, n = min(TB, t1 - tb0);
       if (b >= SCAN_STAGES && !mbar_wait(&empty[s], ((b / SCAN_STAGES) - 1) & 1, failed, a.error_flag, 41)) break;
@@ -275,14 +391,14 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
         if (on)
           for (int t = lane >> 3; t < n; t += 4)
             bulk_row(dst + (size_t)t * stride + off, src + (size_t)(tb0 + t) * pitch, (uint32_t)(4 * count), &full[s]);
-        if (KIND == KIND_DELTA)
+        if (PAIRS)
           for (int t = lane; t < n; t += 32)
             bulk_row(dst + (size_t)t * stride + NA * DKP + 2 * COLS, a.pair + ((size_t)(tb0 + t) * l.heads + head) * 4, 16, &full[s]);
       } else {
         if (on)
           for (int t = lane >> 3; t < n; t += 4)
             for (int i = 0; i < count; ++i) dst[(size_t)t * stride + off + i] = src[(size_t)(tb0 + t) * pitch + i];
-        if (KIND == KIND_DELTA)
+        if (PAIRS)
           for (int t = lane; t < n; t += 32)
             store4(dst + (size_t)t * stride + NA * DKP + 2 * COLS, load4(a.pair + ((size_t)(tb0 + t) * l.heads + head) * 4));
         __syncwarp();
@@ -400,6 +516,62 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
         values(x, v);
         token(t, k, w, q, k, v, nullptr);
       }
+    } else if (KIND == KIND_CHANNEL) {
+      auto times = [](const Row (&x)[J], const Row (&y)[J], Row (&r)[J]) {
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+          r[j].x = mul2(x[j].x, y[j].x);
+          r[j].y = mul2(x[j].y, y[j].y);
+        }
+      };
+      int t = 0;
+      for (; t + 1 < n; t += 2) {
+        const float *xa = x0 + (size_t)t * stride, *xb = xa + stride;
+        float d[2 * CPL], v[CPL];
+        Row k[J], w[J], q[J], r[J];
+        fetch(xa, 0, k);
+        fetch(xa, 1, w);
+        times(k, w, r);
+        dot(r, d);
+        fetch(xb, 0, r);
+        fetch(xb, 1, q);
+        times(r, q, r);
+        times(r, w, r);
+        dot(r, d + CPL);
+        fetch(xa, 2, q);
+        const float2 ca = *reinterpret_cast<const float2*>(xa + NA * DKP + 2 * COLS);
+        const float beta = xb[NA * DKP + 2 * COLS + 1];
+        GroupSum<2 * CPL, 4>::run(d, lr);
+        values(xa, v);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) v[c] = ca.y * (v[c] - d[c]);
+        token(t, k, w, q, k, v, nullptr);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) d[CPL + c] = fmaf(ca.x, v[c], d[CPL + c]);
+        fetch(xb, 0, k);
+        fetch(xb, 1, w);
+        fetch(xb, 2, q);
+        values(xb, v);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) v[c] = beta * (v[c] - d[CPL + c]);
+        token(t + 1, k, w, q, k, v, nullptr);
+      }
+      if (t < n) {
+        const float* xa = x0 + (size_t)t * stride;
+        float d[CPL], v[CPL];
+        Row k[J], w[J], q[J], r[J];
+        fetch(xa, 0, k);
+        fetch(xa, 1, w);
+        times(k, w, r);
+        dot(r, d);
+        fetch(xa, 2, q);
+        values(xa, v);
+        const float beta = xa[NA * DKP + 2 * COLS + 1];
+        GroupSum<CPL, 4>::run(d, lr);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) v[c] = beta * (v[c] - d[c]);
+        token(t, k, w, q, k, v, nullptr);
+      }
     } else {
       int t = 0;
       for (; t + 1 < n; t += 2) {
@@ -472,7 +644,7 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
           for (int i = 0; i < 4; ++i) {
             const int c = lane + i * 32;
             if (c < dv) {
-              const float gate = KIND == KIND_DELTA ? sigmoid_f(g[c]) : silu_f(g[c]);
+              const float gate = KIND == KIND_GLA ? silu_f(g[c]) : sigmoid_f(g[c]);
               const float y = o[i] * rinv * l.norm[KIND == KIND_DELTA ? head * dv + c : c] * gate * l.out_scale;
               if (sa.y_bf16) static_cast<__nv_bfloat16*>(a.y)[base + c] = __float2bfloat16_rn(y);
               else static_cast<float*>(a.y)[base + c] = y;
@@ -504,14 +676,15 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
 
 // Head norm, gate and branch scale of scan outputs that left in several column blocks; a warp per (row, head), at most
 // 256 columns.
-__global__ void __launch_bounds__(256) recurrence_output_kernel(RecurrenceScanArgs a, int y_bf16) {
+__global__ void __launch_bounds__(256) recurrence_output_kernel(ScanArgs sa) {
+  const RecurrenceScanArgs& a = sa.a;
   const RecurrenceLayer& l = a.l;
   const int lane = threadIdx.x & 31, dv = l.vdim;
   const long long total = (long long)a.rows * l.heads;
   for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5; i < total; i += ((long long)gridDim.x * blockDim.x) >> 5) {
     const int row = (int)(i / l.heads), head = (int)(i % l.heads);
     const float* o = a.out_raw + (size_t)row * (l.heads * dv) + head * dv;
-    const float* g = a.p + (size_t)row * a.ldp + l.off_g + head * dv;
+    const float* g = sa.g + (size_t)row * sa.ldg + head * dv;
     float ov[8], gv[8], sq = 0.f;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -525,10 +698,10 @@ __global__ void __launch_bounds__(256) recurrence_output_kernel(RecurrenceScanAr
     for (int j = 0; j < 8; ++j) {
       const int c = lane + j * 32;
       if (c >= dv) break;
-      const float gate = l.kind == KIND_DELTA ? sigmoid_f(gv[j]) : silu_f(gv[j]);
+      const float gate = l.kind == KIND_GLA ? silu_f(gv[j]) : sigmoid_f(gv[j]);
       const float y = ov[j] * rinv * l.norm[l.kind == KIND_DELTA ? head * dv + c : c] * gate * l.out_scale;
       const size_t at = (size_t)row * a.ldy + head * dv + c;
-      if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
+      if (sa.y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
       else static_cast<float*>(a.y)[at] = y;
     }
   }
@@ -702,32 +875,52 @@ cudaError_t launch_scan_any(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
    : dk <= 64  ? launch_scan_cols<KIND_, 8>(sa, grid, bc, cpl, s)                       \
    : dk <= 128 ? launch_scan_cols<KIND_, 16>(sa, grid, bc, cpl, s)                      \
    : dk <= 256 ? launch_scan_cols<KIND_, 32>(sa, grid, bc, cpl, s) : cudaErrorInvalidValue)
-  cudaError_t e = sa.a.l.kind == KIND_DELTA ? PG_SCAN(KIND_DELTA) : PG_SCAN(KIND_GLA);
+  cudaError_t e = sa.a.l.kind == KIND_DELTA ? PG_SCAN(KIND_DELTA) : sa.a.l.kind == KIND_CHANNEL ? PG_SCAN(KIND_CHANNEL) : PG_SCAN(KIND_GLA);
 #undef PG_SCAN
   if (e == cudaSuccess && sa.col_blocks > 1 && (sa.mode == SCAN_FULL || sa.mode == SCAN_OUTPUT)) {
     const long long warps = (long long)sa.a.rows * sa.a.l.heads;
-    e = launch_kernel(recurrence_output_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 32)), dim3(256), 0, s, false, sa.a,
-                      sa.y_bf16);
+    e = launch_kernel(recurrence_output_kernel, dim3((unsigned)std::min<long long>((warps + 7) / 8, 148 * 32)), dim3(256), 0, s, false, sa);
   }
   return e;
+}
+
+cudaError_t launch_channel_gates(const RecurrenceScanArgs& a, cudaStream_t s) {
+  const RecurrenceLayer& l = a.l;
+  const long long cw = (long long)((a.rows + CONV_ROWS - 1) / CONV_ROWS) * (2 * l.kv_heads + l.heads);
+  const long long gw = (long long)((a.rows + GATE_GROUP - 1) / GATE_GROUP) * l.heads;
+  const dim3 cg((unsigned)((cw + 7) / 8)), gg((unsigned)((gw + 7) / 8)), b(256);
+  const int size = std::max(l.dim, l.vdim);
+  cudaError_t e;
+#define PG_CONV(TAPS_)                                                                                  \
+  (size <= 64    ? launch_kernel(channel_conv_kernel<TAPS_, 2>, cg, b, 0, s, false, a)                  \
+   : size <= 128 ? launch_kernel(channel_conv_kernel<TAPS_, 4>, cg, b, 0, s, false, a)                  \
+                 : launch_kernel(channel_conv_kernel<TAPS_, 8>, cg, b, 0, s, false, a))
+  e = l.taps == 2 ? PG_CONV(2) : l.taps == 3 ? PG_CONV(3) : l.taps == 4 ? PG_CONV(4) : PG_CONV(0);
+#undef PG_CONV
+  if (e != cudaSuccess) return e;
+  e = l.dim <= 64    ? launch_kernel(channel_gates_kernel<2>, gg, b, 0, s, false, a)
+      : l.dim <= 128 ? launch_kernel(channel_gates_kernel<4>, gg, b, 0, s, false, a)
+                     : launch_kernel(channel_gates_kernel<8>, gg, b, 0, s, false, a);
+  if (e != cudaSuccess || l.taps == 1) return e;
+  return launch_kernel(channel_taps_kernel, dim3(a.nseq, l.taps - 1), b, 0, s, false, a);
 }
 
 }  // namespace
 
 bool recurrence_use_segments(const RecurrenceLayer& l, int nseq, int max_len, int max_segs) {
   // the transition matrices of the delta rule must fit shared memory twice
-  return max_segs >= 4 && max_len >= 512 && (long long)nseq * l.heads < 48 && (l.kind != KIND_DELTA || l.dim <= 144);
+  return max_segs >= 4 && max_len >= 512 && (long long)nseq * l.heads < 48 && (l.kind == KIND_GLA || l.dim <= 144);
 }
 
 size_t recurrence_segment_floats(const RecurrenceLayer& l, int nseq, int max_segs) {
-  return (size_t)nseq * max_segs * l.heads * l.dim * (l.dvp + (l.kind == KIND_DELTA ? (l.dim + 3) / 4 * 4 : 1));
+  return (size_t)nseq * max_segs * l.heads * l.dim * (l.dvp + (l.kind != KIND_GLA ? (l.dim + 3) / 4 * 4 : 1));
 }
 
 cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cudaStream_t s) {
   if (a.rows <= 0) return cudaSuccess;
   const RecurrenceLayer& l = a.l;
   const int K = l.heads * l.dim;
-  cudaError_t e = launch_kernel(recurrence_decay_kernel, dim3((a.rows + GATE_ROWS - 1) / GATE_ROWS, (K + 255) / 256), dim3(256),
+  cudaError_t e = l.kind == KIND_CHANNEL ? launch_channel_gates(a, s) : launch_kernel(recurrence_decay_kernel, dim3((a.rows + GATE_ROWS - 1) / GATE_ROWS, (K + 255) / 256), dim3(256),
                                 (size_t)GATE_ROWS * l.rank * sizeof(float), s, false, a);
   if (e != cudaSuccess) return e;
   if (l.kind == KIND_DELTA) {
@@ -741,7 +934,15 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   sa.a = a;
   sa.y_bf16 = y_bf16 ? 1 : 0;
   auto m4 = [](int v) { return v % 4 == 0; };
-  sa.vec = m4(l.dim) && m4(l.vdim) && m4(l.off_k) && m4(l.off_q) && m4(l.off_v) && m4(l.off_g) && m4(a.ldp);
+  if (l.kind == KIND_CHANNEL) {
+    sa.k = a.unit; sa.q = a.rate; sa.v = a.vals; sa.g = a.z + K;
+    sa.ldk = sa.ldq = l.kv_heads * l.dim; sa.ldv = l.heads * l.vdim; sa.ldg = a.ldz;
+  } else {
+    sa.k = a.p + l.off_k; sa.q = a.p + l.off_q; sa.v = a.p + l.off_v; sa.g = a.p + l.off_g;
+    sa.ldk = sa.ldq = sa.ldv = sa.ldg = a.ldp;
+  }
+  auto m16 = [](const float* v) { return (reinterpret_cast<uintptr_t>(v) & 15) == 0; };
+  sa.vec = m4(l.dim) && m4(l.vdim) && m16(sa.k) && m16(sa.q) && m16(sa.v) && m16(sa.g) && m4(sa.ldk) && m4(sa.ldv) && m4(sa.ldg);
   if (a.max_segs <= 1 || !a.segments) {
     sa.mode = SCAN_FULL;
     return launch_scan_any(sa, dim3(l.heads, a.nseq, 1), l.vdim, s);
@@ -753,7 +954,7 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   const dim3 grid(l.heads, a.nseq, a.max_segs);
   sa.mode = SCAN_LOCAL;
   if ((e = launch_scan_any(sa, grid, l.vdim, s)) != cudaSuccess) return e;
-  if (l.kind == KIND_DELTA) {
+  if (l.kind != KIND_GLA) {
     sa.mode = SCAN_TRANS;
     e = launch_scan_any(sa, grid, l.dim, s);
   } else {
@@ -761,11 +962,11 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   }
   if (e != cudaSuccess) return e;
   const dim3 cgrid(l.heads, a.nseq, (l.vdim + COMBINE_COLS - 1) / COMBINE_COLS);
-  const size_t csmem = ((size_t)2 * l.dim * COMBINE_COLS + (l.kind == KIND_DELTA ? (size_t)2 * l.dim * (sa.dkp + 4) : 0)) * sizeof(float);
+  const size_t csmem = ((size_t)2 * l.dim * COMBINE_COLS + (l.kind != KIND_GLA ? (size_t)2 * l.dim * (sa.dkp + 4) : 0)) * sizeof(float);
   if (csmem > MAX_SMEM) return cudaErrorInvalidValue;
   e = cudaFuncSetAttribute(recurrence_combine_kernel<KIND_DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
   if (e != cudaSuccess) return e;
-  e = l.kind == KIND_DELTA ? launch_kernel(recurrence_combine_kernel<KIND_DELTA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa)
+  e = l.kind != KIND_GLA ? launch_kernel(recurrence_combine_kernel<KIND_DELTA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa)
                            : launch_kernel(recurrence_combine_kernel<KIND_GLA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa);
   if (e != cudaSuccess) return e;
   sa.mode = SCAN_OUTPUT;

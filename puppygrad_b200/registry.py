@@ -10,8 +10,9 @@ from .decoder import CudaConfig, DecoderModel
 from .dirurax import DiruraxModel
 from .errors import DesignError
 from .gpt2 import Gpt2Model
+from .sanesun import SanesunModel
 
-MODELS: Dict[str, Type[DecoderModel]] = {"gpt2": Gpt2Model, DiruraxModel.architecture: DiruraxModel}
+MODELS: Dict[str, Type[DecoderModel]] = {"gpt2": Gpt2Model, **{m.architecture: m for m in (DiruraxModel, SanesunModel)}}
 
 
 def architecture_of(model_dir: str) -> str:
