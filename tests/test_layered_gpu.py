@@ -4,72 +4,21 @@ against decoding, portions, batches, reuse of pages and slots, edges of blocks a
 A row of logits is compared by the root mean square of its difference (mean removed) over the spread of the expected
 logits: FP32 within 3e-5, BF16 (weights exact, product inputs and cached keys rounded) within 4e-2."""
 import io
-import tempfile
 
 import numpy as np
 import pytest
 
 import puppygrad_b200 as pg
-from puppygrad_b200 import synthetic, trace
+from puppygrad_b200 import trace
+from tests import layered_cases as cases
 from tests import layered_oracle as lo
+from tests.layered_cases import BOUND, MODES, assert_rows, assert_stream, cut, row_errors, run_portions
 
 pytestmark = pytest.mark.gpu
 
-BOUND = {"fp32": 3e-5, "bf16": 4e-2}
-MODES = ("fp32", "bf16")
 
-
-def row_errors(got, want):
-    d = np.asarray(got, np.float64) - want
-    d -= d.mean(axis=-1, keepdims=True)
-    return np.sqrt((d * d).mean(axis=-1)) / want.std()
-
-
-def assert_rows(got, want, mode, factor=1.0):
-    err = row_errors(got, want)
-    assert err.max() <= BOUND[mode] * factor, (mode, float(err.max()), np.nonzero(err > BOUND[mode] * factor)[0][:8])
-
-
-class Case:
-    """A small random model on disk with its expected logits."""
-
-    def __init__(self, cfg, seed, rank=5, edit=None):
-        self.cfg, self.dir = cfg, tempfile.mkdtemp()
-        self.w = lo.random_weights(cfg, seed, rank)
-        if edit:
-            edit(self.w)
-            self.w = {k: synthetic.round_bf16(v) for k, v in self.w.items()}  # what the file holds
-        synthetic.write_design_dir(self.dir, cfg, self.w)
-        self.models, self.known = {}, {}
-
-    def model(self, mode, **kw):
-        key = (mode, tuple(sorted(kw.items())))
-        if key not in self.models:
-            kw.setdefault("max_context", 4096)
-            self.models[key] = pg.load_model(self.dir, pg.CudaConfig(math_mode=mode, **kw))
-        return self.models[key]
-
-    def ids(self, n, seed=0):
-        return np.random.default_rng(1000 + seed).integers(0, self.cfg["vocab"], n)
-
-    def want(self, ids):
-        key = tuple(int(t) for t in ids)
-        if key not in self.known:
-            self.known[key] = lo.forward(self.cfg, self.w, ids)
-        return self.known[key]
-
-
-def cut(ids, sizes):
-    out, at, i = [], 0, 0
-    while at < len(ids):
-        n = sizes[i % len(sizes)]
-        out.append(ids[at:at + n])
-        at, i = at + n, i + 1
-    return out
-
-
-def run_portions(model, cache, slot, portions):
-    return np.concatenate([model.extend([slot], [p], cache, range(len(p))) for p in portions])
+def Case(cfg, seed, **kw):
+    return cases.Case(lo, cfg, seed, **kw)
 
 
 MIXED = lo.config(101, 72, [lo.gla(3, 12, 20, tau=9.0, ff=40), lo.pair(6, 2, 20, 12, 23, 5, 16, left_scale=0.7, right_scale=1.3),
@@ -352,29 +301,10 @@ def test_a_dirty_slot_starts_from_nothing(mixed):
 
 
 # ------------------------------------------------------------------ generation through the usual entry points
-def oracle_greedy(case, prompt, n):
-    ids, gaps = [int(t) for t in prompt], []
-    for _ in range(n):
-        row = lo.forward(case.cfg, case.w, ids)[-1]
-        top = np.sort(row)
-        gaps.append((top[-1] - top[-2]) / row.std())
-        ids.append(int(row.argmax()))
-    return ids, gaps
-
-
 @pytest.fixture(scope="module")
 def greedy(mixed):
     prompts = [mixed.ids(n, 200 + n) for n in (5, 21, 40)]
-    return [(p, *oracle_greedy(mixed, p, 30)) for p in prompts]
-
-
-def assert_stream(tokens, want, gaps, n_prompt, bound):
-    """Equal up to the first choice that is closer than the bound."""
-    for i, (a, b) in enumerate(zip(tokens[n_prompt:], want[n_prompt:])):
-        if a != b:
-            assert gaps[i] < 10 * bound, (i, a, b, gaps[i])
-            return
-    assert len(tokens) == len(want)
+    return [(p, *cases.greedy(mixed, p, 30)) for p in prompts]
 
 
 @pytest.mark.parametrize("mode", MODES)
