@@ -527,17 +527,19 @@ def main():
     ap.add_argument("--skip-extras", action="store_true",
                     help="only the device-timed decode loop (no e2e, per-op profile, CPU baseline)")
     ap.add_argument("--layered", action="store_true",
-                    help="instead: a layered model (Dirurax) beside GPT-2 of equal size, decode and prefill throughput")
+                    help="instead: a layered model beside an older one of equal size (Dirurax beside GPT-2, Sanesun beside Dirurax), "
+                         "decode and prefill throughput")
+    ap.add_argument("--layered-design", default="Dirurax", choices=["Dirurax", "Sanesun"])
     ap.add_argument("--layered-widths", default="1024,2048")
     ap.add_argument("--layered-depth", type=int, default=8)
-    ap.add_argument("--layered-only", action="store_true", help="without the GPT-2 of equal size")
+    ap.add_argument("--layered-only", action="store_true", help="without the older model")
     args = ap.parse_args()
     if args.layered:
         from puppygrad_b200 import layered_bench
         clocks = ClockSampler(0)
         clocks.start()
         result = layered_bench.run(0, [int(w) for w in args.layered_widths.split(",")], args.layered_depth, min(args.steps, 64),
-                                   measured_peaks(), compare=not args.layered_only)
+                                   measured_peaks(), compare=not args.layered_only, design=args.layered_design)
         print(json.dumps({"metric": "layered_model_throughput", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
                           "clocks": clocks.stop(), **result}))
     elif args.impl == "reference":
