@@ -28,6 +28,8 @@ __device__ __forceinline__ float rotated(F x, int c, int dims, const float2* cs)
 }
 
 __global__ void __launch_bounds__(256) angles_kernel(const int* pos, const double* freq, float2* out, int rows, int half) {
+  grid_dep_launch();
+  grid_dep_wait();
   const size_t n = (size_t)rows * half;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
     out[i] = angle(pos[i / half], freq[i % half]);
@@ -82,6 +84,7 @@ __global__ void __launch_bounds__(THREADS) attention_heads_step_kernel(Attention
   T* pool = static_cast<T*>(a.pool);
   const size_t page_elems = (size_t)G * l.page_tokens * (l.dimp + l.vrow), v_at = latent ? 0 : (size_t)G * l.page_tokens * l.dimp;
   const int vpitch = latent ? l.dimp : l.vrow;
+  const int tok = l.wide ? G : 1, hd = l.wide ? 1 : l.page_tokens;  // rows between two tokens, two heads of a page
 
   for (int i = tid; i < (l.rot_dims >> 1); i += THREADS) kcs[i] = angle(pos, l.rot_freq[i]);
   if (l.v_rot)
@@ -153,7 +156,7 @@ __global__ void __launch_bounds__(THREADS) attention_heads_step_kernel(Attention
 #pragma unroll
           for (int k = 0; k < KB; ++k) {
             const int j = jt + k, off = j < n ? koff[j] : -2;
-            if (off >= 0) load8(pool + kbase[j] + (size_t)(kvh * l.page_tokens + off) * l.dimp + c, kv[k]);
+            if (off >= 0) load8(pool + kbase[j] + (size_t)(kvh * hd + off * tok) * l.dimp + c, kv[k]);
             else if (off == -1) load8(kn + kvh * l.dimp + c, kv[k]);
             else
 #pragma unroll
@@ -233,7 +236,7 @@ __global__ void __launch_bounds__(THREADS) attention_heads_step_kernel(Attention
     __syncthreads();
     auto value = [&](int j, int kvh, int vc, float (&v)[8]) {
       if (koff[j] < 0) load8(vn + kvh * l.vdimp + vc * 8, v);
-      else load8(pool + kbase[j] + v_at + (size_t)(kvh * l.page_tokens + koff[j]) * vpitch + vc * 8, v);
+      else load8(pool + kbase[j] + v_at + (size_t)(kvh * hd + koff[j] * tok) * vpitch + vc * 8, v);
     };
     if (one_v) {
 #pragma unroll
@@ -306,11 +309,11 @@ __global__ void __launch_bounds__(THREADS) attention_heads_step_kernel(Attention
   }
   __syncthreads();
   if (a.splits > 1) {
-    const int vd2 = l.vdim + 2;
+    const int vd2 = 4 + ((l.vdim + 3) & ~3);
     for (int i = tid; i < nh * l.vdim; i += THREADS) {
       const int h = i / l.vdim, c = i % l.vdim;
       float* pt = a.part + (((size_t)seq * H + h0 + h) * a.splits + split) * vd2;
-      pt[2 + c] = os[(size_t)h * l.vdimp + c];
+      pt[4 + c] = os[(size_t)h * l.vdimp + c];
       if (c == 0) {
         pt[0] = m_run[h];
         pt[1] = l_run[h];
@@ -342,7 +345,7 @@ __global__ void __launch_bounds__(THREADS) attention_heads_step_kernel(Attention
     __syncthreads();
     for (int i = tid; i < nh * l.vdim; i += THREADS) {
       const int h = i / l.vdim, c = i % l.vdim;
-      const volatile float* pt = a.part + ((size_t)seq * H + h0 + h) * a.splits * vd2 + 2 + c;
+      const volatile float* pt = a.part + ((size_t)seq * H + h0 + h) * a.splits * vd2 + 4 + c;
       float v = 0.f;
       for (int s = 0; s < a.splits; ++s) v = fmaf(raw[h * a.splits + s], pt[s * vd2], v);
       os[(size_t)h * l.vdimp + c] = v;
@@ -370,7 +373,7 @@ __global__ void __launch_bounds__(THREADS) attention_heads_step_kernel(Attention
       y = c < half ? o[c] * vcs[c].x + o[c + half] * vcs[c].y : o[c] * vcs[c - half].x - o[c - half] * vcs[c - half].y;
     }
     y *= corr[h];
-    const size_t at = (size_t)seq * a.ldy + (size_t)(h0 + h) * l.vdim + c;
+    const size_t at = (size_t)seq * a.ldy + (size_t)(h0 + h) * a.ldyh + c;
     if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(y);
     else static_cast<float*>(a.y)[at] = y;
   }
@@ -402,63 +405,99 @@ bool step_shape(const AttentionLayer& l, StepShape* sh) {
 }
 
 // ------------------------------------------------------------------ portions
-// Block = row. Queries with their bias, rotated; with mixed heads head h's query against the row of all key heads:
-// piece c of it = sum over the heads g that read key head c of mix[h][g] q_g.
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+  store4(p, make_float4(v[0], v[1], v[2], v[3]));
+  store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
+  uint32_t u[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    u[i] = *reinterpret_cast<const uint32_t*>(&b);
+  }
+  *reinterpret_cast<uint4*>(p) = make_uint4(u[0], u[1], u[2], u[3]);
+}
+
+// Where a row's key or value of one head goes: the workspace, or (a step) the page of its position.
 template <typename T>
-__global__ void __launch_bounds__(256) attention_rotate_kernel(AttentionPortionArgs a, int mix_in_smem) {
-  extern __shared__ __align__(16) float sm[];  // [heads][dimp] queries, [heads][heads] mixing
+__device__ __forceinline__ T* key_target(const AttentionPortionArgs& a, int row, int head, int which) {
   const AttentionLayer& l = a.l;
-  const int row = blockIdx.x, tid = threadIdx.x, H = l.heads, G = l.kv_heads, rep = H / G;
-  const float* p = a.p + (size_t)row * a.ldp;
+  if (a.step_pos)
+    return page_row(l, static_cast<T*>(a.pool), a.page_table + (size_t)row * l.pages_per_seq, l.life.place(a.step_pos[row]), head, which);
   const int seq = a.row_seq[row];
   const size_t krow = (size_t)a.key_start[seq] + l.life.context(a.seq_pos[seq]) + (row - a.seq_start[seq]);
-  const float2* kcs = a.rot + (size_t)row * (l.rot_dims >> 1);
-  const float2* vcs = a.v_rot + (size_t)row * (l.vdim >> 1);
-  auto entry = [&](int off, const float* bias, int h, int n, int c, int dims, const float2* cs) {
-    const float *x = p + off + h * n, *b = bias ? bias + h * n : nullptr;
-    return c < n ? rotated([=](int e) { return x[e] + (b ? b[e] : 0.f); }, c, dims, cs) : 0.f;
-  };
-  for (int i = tid; i < G * l.dimp; i += 256)
-    static_cast<T*>(a.k)[krow * a.ldk + i] = from_f32<T>(entry(l.off_k, l.k_bias, i / l.dimp, l.dim, i % l.dimp, l.rot_dims, kcs));
-  for (int i = tid; i < G * l.vdimp; i += 256)
-    static_cast<T*>(a.v)[krow * a.ldv + i] = from_f32<T>(entry(l.off_v, l.v_bias, i / l.vdimp, l.vdim, i % l.vdimp, l.v_rot ? l.vdim : 0, vcs));
-  if (!l.mix) {
-    for (int i = tid; i < H * l.dimp; i += 256)
-      static_cast<T*>(a.q)[(size_t)row * H * l.dimp + i] = from_f32<T>(entry(l.off_q, l.q_bias, i / l.dimp, l.dim, i % l.dimp, l.rot_dims, kcs));
-    return;
-  }
+  return which == 0 ? static_cast<T*>(a.k) + krow * a.ldk + head * l.dimp : static_cast<T*>(a.v) + krow * a.ldv + head * l.vdimp;
+}
+
+// Block = ROWS rows and one key head with the query heads that read it: biases, rotation. With mixed heads, piece c of head
+// h's query (the part against key head c) = sum over the heads g that read key head c of mix[h][g] q_g.
+constexpr int ROT_THREADS = 256, ROT_PORTION_ROWS = 8;
+template <typename T, int ROWS>
+__global__ void __launch_bounds__(ROT_THREADS) attention_rotate_kernel(AttentionPortionArgs a) {
+  extern __shared__ __align__(16) float sm[];  // [ROWS][rep][dimp] queries, [heads][rep] mixing
+  const AttentionLayer& l = a.l;
+  const int row0 = blockIdx.x * ROWS, c = blockIdx.y, nrows = min(ROWS, a.rows - row0), tid = threadIdx.x, H = l.heads, G = l.kv_heads, rep = H / G;
+  const int qn = rep * l.dimp, per = qn + l.dimp + l.vdimp;
   float* qs = sm;
-  for (int i = tid; i < H * l.dimp; i += 256) qs[i] = entry(l.off_q, l.q_bias, i / l.dimp, l.dim, i % l.dimp, l.rot_dims, kcs);
-  const float* mix = l.mix;
-  if (mix_in_smem) {
-    float* t = qs + (size_t)H * l.dimp;
-    for (int i = tid; i < H * H; i += 256) t[i] = l.mix[i];
-    mix = t;
+  float* mix = qs + (size_t)ROWS * qn;
+  grid_dep_launch();
+  if (l.mix)
+    for (int i = tid; i < H * rep; i += ROT_THREADS) mix[i] = l.mix[(size_t)(i / rep) * H + c * rep + i % rep];
+  grid_dep_wait();
+  for (int e = tid; e < per; e += ROT_THREADS) {  // a column of the block's rows
+    const bool is_q = e < qn, is_k = !is_q && e < qn + l.dimp;
+    const int x = is_q ? e : is_k ? e - qn : e - qn - l.dimp, np = is_q || is_k ? l.dimp : l.vdimp, n = is_q || is_k ? l.dim : l.vdim;
+    const int head = is_q ? c * rep + x / np : c, col = x % np, dims = is_q || is_k ? l.rot_dims : l.v_rot ? l.vdim : 0;
+    const float* src = a.p + (is_q ? l.off_q : is_k ? l.off_k : l.off_v) + head * n;
+    const float* bias = is_q ? l.q_bias : is_k ? l.k_bias : l.v_bias;
+    const float2* cs = is_q || is_k ? a.rot : a.v_rot;
+    // entry `col` = x cos + sign * partner * sin
+    const int half = dims >> 1, partner = col >= dims || col >= n ? -1 : col < half ? col + half : col - half, turn = col < half ? col : col - half;
+    const float sign = col < half ? -1.f : 1.f;
+    const float b0 = bias && col < n ? bias[head * n + col] : 0.f, b1 = bias && partner >= 0 ? bias[head * n + partner] : 0.f;
+    float v[ROWS];
+#pragma unroll
+    for (int rr = 0; rr < ROWS; ++rr) {
+      v[rr] = 0.f;
+      if (rr < nrows && col < n) {
+        const float* p = src + (size_t)(row0 + rr) * a.ldp;
+        v[rr] = p[col] + b0;
+        if (partner >= 0) {
+          const float2 r = cs[(size_t)(row0 + rr) * half + turn];
+          v[rr] = v[rr] * r.x + sign * ((p[partner] + b1) * r.y);
+        }
+      }
+    }
+#pragma unroll
+    for (int rr = 0; rr < ROWS; ++rr)
+      if (rr < nrows) {
+        if (!is_q) key_target<T>(a, row0 + rr, c, is_k ? 0 : 1)[col] = from_f32<T>(v[rr]);
+        else if (l.mix) qs[rr * qn + x] = v[rr];
+        else static_cast<T*>(a.q)[((size_t)(row0 + rr) * H + head) * l.dimp + col] = from_f32<T>(v[rr]);
+      }
   }
+  if (!l.mix) return;
   __syncthreads();
-  const int width = G * l.dimp;
-  T* out = static_cast<T*>(a.q) + (size_t)row * H * width;
-  for (int i = tid; i < width; i += 256) {
-    const int c = i / l.dimp, e = i % l.dimp;
-    const float* q = qs + (size_t)c * rep * l.dimp + e;
-    const float* t = mix + c * rep;
-    if (rep <= 8) {
-      float x[8];
+  const int no = l.dimp / 8;
+  for (int i = tid; i < H * no; i += ROT_THREADS) {
+    const int o = i % no, h = i / no;
+    const float* t = mix + h * rep;
+    T* out = static_cast<T*>(a.q) + (((size_t)row0 * H + h) * G + c) * l.dimp + o * 8;
 #pragma unroll
-      for (int g = 0; g < 8; ++g) x[g] = g < rep ? q[g * l.dimp] : 0.f;
-      for (int h = 0; h < H; ++h) {
-        float s = 0.f;
+    for (int rr = 0; rr < ROWS; ++rr) {
+      if (rr >= nrows) break;
+      const float* q = qs + rr * qn + o * 8;
+      float acc[8];
 #pragma unroll
-        for (int g = 0; g < 8; ++g)
-          if (g < rep) s = fmaf(t[h * H + g], x[g], s);
-        out[(size_t)h * width + i] = from_f32<T>(s);
+      for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+      for (int g = 0; g < rep; ++g) {
+        float x[8];
+        load8(q + g * l.dimp, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(t[g], x[e], acc[e]);
       }
-    } else {
-      for (int h = 0; h < H; ++h) {
-        float s = 0.f;
-        for (int g = 0; g < rep; ++g) s = fmaf(t[h * H + g], q[g * l.dimp], s);
-        out[(size_t)h * width + i] = from_f32<T>(s);
-      }
+      store8(out + (size_t)rr * H * G * l.dimp, acc);
     }
   }
 }
@@ -467,15 +506,80 @@ template <typename T>
 __global__ void __launch_bounds__(256) attention_latent_kernel(AttentionPortionArgs a) {
   const AttentionLayer& l = a.l;
   const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  grid_dep_launch();
+  grid_dep_wait();
   if (row >= a.rows) return;
-  const int seq = a.row_seq[row];
-  const size_t krow = (size_t)a.key_start[seq] + l.life.context(a.seq_pos[seq]) + (row - a.seq_start[seq]);
-  const float* x = a.p + (size_t)row * a.ldp + l.off_k;
+  T* dst = key_target<T>(a, row, 0, 0);
+  const float* p = a.p + (size_t)row * a.ldp + l.off_k;
+  float4 x[8];  // at most 1024 columns; dimp and the weight are padded, the row is not
   float s = 0.f;
-  for (int c = lane; c < l.dim; c += 32) s += x[c] * x[c];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int c = (i * 32 + lane) * 4;
+    x[i] = make_float4(0, 0, 0, 0);
+    if (c < l.dim) {
+      x[i] = load4(p + c);
+      if (c + 1 >= l.dim) x[i].y = 0.f;
+      if (c + 2 >= l.dim) x[i].z = 0.f;
+      if (c + 3 >= l.dim) x[i].w = 0.f;
+    }
+    s += (x[i].x * x[i].x + x[i].y * x[i].y) + (x[i].z * x[i].z + x[i].w * x[i].w);
+  }
   const float inv = 1.f / sqrtf(lane_sum(s) / (float)l.dim + l.eps);
-  for (int c = lane; c < l.dimp; c += 32)
-    static_cast<T*>(a.k)[krow * a.ldk + c] = from_f32<T>(c < l.dim ? x[c] * inv * l.k_norm[c] : 0.f);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int c = (i * 32 + lane) * 4;
+    if (c < l.dimp) {
+      const float4 g = load4(l.k_norm + c);
+      store4(dst + c, make_float4(x[i].x * inv * g.x, x[i].y * inv * g.y, x[i].z * inv * g.z, x[i].w * inv * g.w));
+    }
+  }
+}
+
+// Block = one head of one sequence. Parts hold maxima and sums in powers of two.
+__global__ void __launch_bounds__(128) attention_merge_kernel(AttentionStepArgs a, const float2* v_rot, int y_bf16) {
+  __shared__ float w[64];
+  const AttentionLayer& l = a.l;
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, pitch = 4 + ((l.vdim + 3) & ~3), half = l.vdim >> 1;
+  constexpr float LOG2E = 1.4426950408889634f;
+  grid_dep_launch();
+  grid_dep_wait();
+  const float* pt = a.part + ((size_t)seq * l.heads + h) * a.splits * pitch;
+  if (tid < 32) {  // at most 32 parts
+    const float sum = tid < a.splits ? pt[tid * pitch + 1] : 0.f, m = sum > 0.f ? pt[tid * pitch] : -1e30f;
+    const float sink = l.sink ? l.sink[h] * LOG2E : -1e30f, top = fmaxf(lane_max(m), sink);
+    const float f = sum > 0.f ? exp2f(m - top) : 0.f;
+    const float den = lane_sum(f * sum) + (l.sink ? exp2f(sink - top) : 0.f);
+    float scale = l.out_scale / den;
+    if (l.off_gate >= 0) scale *= sigmoid_f(a.p[(size_t)seq * a.ldp + l.off_gate + h]);
+    w[tid] = f * scale;
+  }
+  __syncthreads();
+  auto sum = [&](int c) {
+    float v = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < a.splits; ++s) {
+      const float x = pt[s * pitch + 4 + c];  // an empty part holds no numbers
+      v = w[s] != 0.f ? fmaf(w[s], x, v) : v;
+    }
+    return v;
+  };
+  auto put = [&](int c, float v) {
+    const size_t at = (size_t)seq * a.ldy + (size_t)h * a.ldyh + c;
+    if (y_bf16) static_cast<__nv_bfloat16*>(a.y)[at] = __float2bfloat16_rn(v);
+    else static_cast<float*>(a.y)[at] = v;
+  };
+  if (l.v_rot) {
+    for (int c = tid; c < half; c += 128) {
+      const float2 r = v_rot[(size_t)seq * half + c];
+      const float u = sum(c), v = sum(c + half);
+      put(c, u * r.x + v * r.y);
+      put(c + half, v * r.x - u * r.y);
+    }
+  } else {
+    for (int c = tid; c < l.vdim; c += 128) put(c, sum(c));
+    for (int c = l.vdim + tid; c < a.ldyh; c += 128) put(c, 0.f);
+  }
 }
 
 __global__ void __launch_bounds__(256) attention_turn_back_kernel(AttentionPortionArgs a) {
@@ -493,20 +597,35 @@ __global__ void __launch_bounds__(256) attention_turn_back_kernel(AttentionPorti
 
 // ------------------------------------------------------------------ products per head
 // Block = 64 columns of one head for up to MB rows: lane = (eight columns, one of four subsets of k), warps take further
-// subsets; the sums meet by shuffles and through shared memory.
-constexpr int MB = 8;
+// subsets; the sums meet by shuffles and through shared memory. The first weights are requested before the dependency wait.
+constexpr int HP_PRE = 4;
 template <typename T>
+struct Row8 {  // eight weights as they lie
+  uint4 u[sizeof(T) / 2];
+  __device__ __forceinline__ void load(const T* p) {
+#pragma unroll
+    for (int i = 0; i < (int)sizeof(T) / 2; ++i) u[i] = __ldg(reinterpret_cast<const uint4*>(p) + i);
+  }
+  __device__ __forceinline__ void get(float (&v)[8]) const { load8(reinterpret_cast<const T*>(u), v); }
+};
+template <typename T, int MB>
 __global__ void __launch_bounds__(THREADS) head_product_kernel(HeadProductArgs a, int out_bf16) {
-  extern __shared__ __align__(16) float sm[];  // [MB][k] inputs, then [WARPS][MB][64] sums
+  extern __shared__ __align__(16) float sm[];  // [k][MB] inputs, then [WARPS][MB][64] sums
   const int n0 = blockIdx.x * 64, h = blockIdx.y, b0 = blockIdx.z * MB, nb = min(MB, a.batch - b0), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int col = n0 + (lane & 7) * 8, ks = warp * 4 + (lane >> 3);
+  const int col = n0 + (lane & 7) * 8, ks = warp * 4 + (lane >> 3), kstep = 4 * WARPS;
   float* xs = sm;
   float* part = sm + (size_t)MB * a.k;
+  const T* w = static_cast<const T*>(a.w) + (size_t)h * a.k * a.np + col;
+  const bool on = col < a.np;
   grid_dep_launch();
+  Row8<T> pre[HP_PRE];
+#pragma unroll
+  for (int i = 0; i < HP_PRE; ++i)
+    if (on && ks + i * kstep < a.k) pre[i].load(w + (size_t)(ks + i * kstep) * a.np);
   grid_dep_wait();
   for (int i = tid; i < MB * a.k; i += THREADS) {
     const int b = i / a.k, k = i % a.k;
-    xs[i] = b < nb ? a.x[(size_t)(b0 + b) * a.ldx + (size_t)h * a.ldxh + k] : 0.f;
+    xs[k * MB + b] = b < nb ? a.x[(size_t)(b0 + b) * a.ldx + (size_t)h * a.ldxh + k] : 0.f;
   }
   __syncthreads();
   float acc[MB][8];
@@ -514,38 +633,53 @@ __global__ void __launch_bounds__(THREADS) head_product_kernel(HeadProductArgs a
   for (int b = 0; b < MB; ++b)
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc[b][e] = 0.f;
-  if (col < a.np) {
-    const T* w = static_cast<const T*>(a.w) + (size_t)h * a.k * a.np + col;
-#pragma unroll 4
-    for (int k = ks; k < a.k; k += 4 * WARPS) {
-      float v[8];
-      load8(w + (size_t)k * a.np, v);
+  if (on) {
+    for (int k0 = ks; k0 < a.k; k0 += HP_PRE * kstep) {
+      Row8<T> cur[HP_PRE];
 #pragma unroll
-      for (int b = 0; b < MB; ++b) {
-        if (b < nb) {
-          const float x = xs[b * a.k + k];
+      for (int i = 0; i < HP_PRE; ++i) {
+        cur[i] = pre[i];
+        const int next = k0 + (HP_PRE + i) * kstep;
+        if (next < a.k) pre[i].load(w + (size_t)next * a.np);
+      }
 #pragma unroll
-          for (int e = 0; e < 8; ++e) acc[b][e] = fmaf(x, v[e], acc[b][e]);
+      for (int i = 0; i < HP_PRE; ++i) {
+        const int k = k0 + i * kstep;
+        if (k < a.k) {
+          float v[8], x[MB];
+          cur[i].get(v);
+          if (MB % 4 == 0) {
+#pragma unroll
+            for (int b = 0; b < MB; b += 4) {
+              const float4 f = load4(xs + k * MB + b);
+              x[b] = f.x; x[(b + 1) % MB] = f.y; x[(b + 2) % MB] = f.z; x[(b + 3) % MB] = f.w;
+            }
+          } else {
+#pragma unroll
+            for (int b = 0; b < MB; ++b) x[b] = xs[k * MB + b];
+          }
+#pragma unroll
+          for (int b = 0; b < MB; ++b)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc[b][e] = fmaf(x[b], v[e], acc[b][e]);
         }
       }
     }
   }
 #pragma unroll
   for (int b = 0; b < MB; ++b)
-    if (b < nb) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        acc[b][e] += __shfl_xor_sync(ALL_LANES, acc[b][e], 8);
-        acc[b][e] += __shfl_xor_sync(ALL_LANES, acc[b][e], 16);
-        if (lane < 8) part[((size_t)warp * MB + b) * 64 + lane * 8 + e] = acc[b][e];
-      }
+    for (int e = 0; e < 8; ++e) {
+      acc[b][e] += __shfl_xor_sync(ALL_LANES, acc[b][e], 8);
+      acc[b][e] += __shfl_xor_sync(ALL_LANES, acc[b][e], 16);
+      if (lane < 8) part[((size_t)warp * MB + b) * 64 + lane * 8 + e] = acc[b][e];
     }
   __syncthreads();
   for (int i = tid; i < nb * 64; i += THREADS) {
     const int b = i / 64, c = i % 64;
     if (n0 + c >= a.n) continue;
     float v = 0.f;
-    for (int w = 0; w < WARPS; ++w) v += part[((size_t)w * MB + b) * 64 + c];
+    for (int q = 0; q < WARPS; ++q) v += part[((size_t)q * MB + b) * 64 + c];
     const size_t at = (size_t)(b0 + b) * a.ldo + (size_t)h * a.ldh + n0 + c;
     if (out_bf16) static_cast<__nv_bfloat16*>(a.out)[at] = __float2bfloat16_rn(v);
     else static_cast<float*>(a.out)[at] = v;
@@ -571,9 +705,14 @@ cudaError_t heads_step_t(const AttentionStepArgs& a, const StepShape& sh, int yb
 
 }  // namespace
 
+size_t rotate_smem(const AttentionLayer& l) {
+  const int rep = l.heads / l.kv_heads;
+  return l.mix ? ((size_t)ROT_PORTION_ROWS * rep * l.dimp + (size_t)l.heads * rep) * sizeof(float) : 0;
+}
+
 bool attention_heads_supported(const AttentionLayer& l) {
   StepShape sh;
-  return step_shape(l, &sh) && (!l.mix || (size_t)l.heads * l.dimp * sizeof(float) <= MAX_SMEM);
+  return step_shape(l, &sh) && rotate_smem(l) <= MAX_SMEM;
 }
 
 cudaError_t launch_attention_heads_step(const AttentionStepArgs& a, bool bf16, bool y_bf16, bool pdl, cudaStream_t s) {
@@ -582,45 +721,56 @@ cudaError_t launch_attention_heads_step(const AttentionStepArgs& a, bool bf16, b
   return bf16 ? heads_step_t<__nv_bfloat16>(a, sh, y_bf16 ? 1 : 0, pdl, s) : heads_step_t<float>(a, sh, y_bf16 ? 1 : 0, pdl, s);
 }
 
-cudaError_t launch_angles(const int* pos, const double* freq, float2* out, int rows, int half, cudaStream_t s) {
+cudaError_t launch_angles(const int* pos, const double* freq, float2* out, int rows, int half, bool pdl, cudaStream_t s) {
   if (rows <= 0 || half <= 0) return cudaSuccess;
   const size_t blocks = ((size_t)rows * half + 255) / 256;
-  return launch_kernel(angles_kernel, dim3((unsigned)std::min<size_t>(blocks, 148 * 16)), dim3(256), 0, s, false, pos, freq, out, rows, half);
+  return launch_kernel(angles_kernel, dim3((unsigned)std::min<size_t>(blocks, 148 * 16)), dim3(256), 0, s, pdl, pos, freq, out, rows, half);
 }
 
-cudaError_t launch_attention_rotate(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
-  const AttentionLayer& l = a.l;
-  size_t smem = l.mix ? (size_t)l.heads * l.dimp * sizeof(float) : 0;
-  const size_t with = smem + (size_t)l.heads * l.heads * sizeof(float);
-  const int in_smem = l.mix && with <= 96 * 1024 ? 1 : 0;
-  if (in_smem) smem = with;
+cudaError_t launch_attention_rotate(const AttentionPortionArgs& a, bool bf16, cudaStream_t s, bool pdl) {
+  const size_t smem = rotate_smem(a.l);
   if (smem > MAX_SMEM) return cudaErrorInvalidValue;
+  const int rows = a.step_pos ? 1 : ROT_PORTION_ROWS;
+  const dim3 grid((a.rows + rows - 1) / rows, a.l.kv_heads);
   auto run = [&](auto kernel) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
-    return e != cudaSuccess ? e : launch_kernel(kernel, dim3(a.rows), dim3(256), smem, s, false, a, in_smem);
+    return e != cudaSuccess ? e : launch_kernel(kernel, grid, dim3(ROT_THREADS), smem, s, pdl, a);
   };
-  return bf16 ? run(attention_rotate_kernel<__nv_bfloat16>) : run(attention_rotate_kernel<float>);
+  if (a.step_pos) return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, 1>) : run(attention_rotate_kernel<float, 1>);
+  return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, ROT_PORTION_ROWS>) : run(attention_rotate_kernel<float, ROT_PORTION_ROWS>);
 }
 
-cudaError_t launch_attention_latent(const AttentionPortionArgs& a, bool bf16, cudaStream_t s) {
+cudaError_t launch_attention_latent(const AttentionPortionArgs& a, bool bf16, cudaStream_t s, bool pdl) {
   const dim3 grid((a.rows + 7) / 8);
-  return bf16 ? launch_kernel(attention_latent_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, false, a)
-              : launch_kernel(attention_latent_kernel<float>, grid, dim3(256), 0, s, false, a);
+  return bf16 ? launch_kernel(attention_latent_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, pdl, a)
+              : launch_kernel(attention_latent_kernel<float>, grid, dim3(256), 0, s, pdl, a);
+}
+
+cudaError_t launch_attention_merge(const AttentionStepArgs& a, const float2* v_rot, bool y_bf16, bool pdl, cudaStream_t s) {
+  if (a.splits > 32) return cudaErrorInvalidValue;
+  return launch_kernel(attention_merge_kernel, dim3(a.l.heads, a.batch), dim3(128), 0, s, pdl, a, v_rot, y_bf16 ? 1 : 0);
 }
 
 cudaError_t launch_attention_turn_back(const AttentionPortionArgs& a, cudaStream_t s) {
   return launch_kernel(attention_turn_back_kernel, dim3(a.rows), dim3(256), 0, s, false, a);
 }
 
-cudaError_t launch_head_product(const HeadProductArgs& a, bool bf16, bool out_bf16, bool pdl, cudaStream_t s) {
+template <typename T, int MB>
+static cudaError_t head_product_mb(const HeadProductArgs& a, bool out_bf16, bool pdl, cudaStream_t s) {
   const size_t smem = ((size_t)MB * a.k + (size_t)WARPS * MB * 64) * sizeof(float);
   if (smem > MAX_SMEM || a.np % 8 != 0) return cudaErrorInvalidValue;
   const dim3 grid((a.n + 63) / 64, a.heads, (a.batch + MB - 1) / MB);
-  auto run = [&](auto kernel) {
-    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
-    return e != cudaSuccess ? e : launch_kernel(kernel, grid, dim3(THREADS), smem, s, pdl, a, out_bf16 ? 1 : 0);
-  };
-  return bf16 ? run(head_product_kernel<__nv_bfloat16>) : run(head_product_kernel<float>);
+  cudaError_t e = cudaFuncSetAttribute(head_product_kernel<T, MB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
+  return e != cudaSuccess ? e : launch_kernel(head_product_kernel<T, MB>, grid, dim3(THREADS), smem, s, pdl, a, out_bf16 ? 1 : 0);
+}
+
+cudaError_t launch_head_product(const HeadProductArgs& a, bool bf16, bool out_bf16, bool pdl, cudaStream_t s) {
+  if (bf16) {
+    if (a.batch <= 1) return head_product_mb<__nv_bfloat16, 1>(a, out_bf16, pdl, s);
+    if (a.batch <= 4) return head_product_mb<__nv_bfloat16, 4>(a, out_bf16, pdl, s);
+    return head_product_mb<__nv_bfloat16, 8>(a, out_bf16, pdl, s);
+  }
+  return a.batch <= 1 ? head_product_mb<float, 1>(a, out_bf16, pdl, s) : head_product_mb<float, 8>(a, out_bf16, pdl, s);
 }
 
 }  // namespace pg

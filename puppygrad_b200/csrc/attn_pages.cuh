@@ -10,10 +10,10 @@ namespace {
 template <typename T>
 __device__ __forceinline__ T* page_row(const AttentionLayer& l, T* pool, const int* table_row, int c, int head, int which) {
   const size_t page_elems = (size_t)l.kv_heads * l.page_tokens * (l.dimp + l.vrow);
-  T* page = pool + (size_t)table_row[c / l.page_tokens] * page_elems;
-  const int off = c % l.page_tokens;
-  if (which == 0 || l.vrow == 0) return page + ((size_t)head * l.page_tokens + off) * l.dimp;
-  return page + (size_t)l.kv_heads * l.page_tokens * l.dimp + ((size_t)head * l.page_tokens + off) * l.vrow;
+  const bool value = which != 0 && l.vrow != 0;
+  const int off = c % l.page_tokens, width = value ? l.vrow : l.dimp;
+  T* page = pool + (size_t)table_row[c / l.page_tokens] * page_elems + (value ? (size_t)l.kv_heads * l.page_tokens * l.dimp : 0);
+  return page + (l.wide ? (size_t)off * l.kv_heads + head : (size_t)head * l.page_tokens + off) * width;
 }
 
 }  // namespace

@@ -289,7 +289,8 @@ __global__ void __launch_bounds__(192, 1)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n0 = blockIdx.x * TILE_M, split = blockIdx.y;
   const int nkb_all = (a.k + KB - 1) / KB, kb0 = nkb_all * split / SPLITS, nkb = nkb_all * (split + 1) / SPLITS - kb0;
-  const int wrow = ((int)blockIdx.x * nkb_all + kb0) * TILE_M;  // first row of this block's run of weight tiles
+  const int head = blockIdx.z, x0 = head * a.x_head;
+  const int wrow = ((head * (int)gridDim.x + (int)blockIdx.x) * nkb_all + kb0) * TILE_M;  // first row of this block's run of weight tiles
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < S::STAGES; ++s) {
@@ -318,7 +319,7 @@ __global__ void __launch_bounds__(192, 1)
       }
       pdl_wait();
       for (int i = 0; i < ahead; ++i)
-        tma_load_2d(base + (size_t)i * S::STAGE_BYTES + S::A_BYTES, &map_x, (kb0 + i) * KB, 0, &full[i]);
+        tma_load_2d(base + (size_t)i * S::STAGE_BYTES + S::A_BYTES, &map_x, x0 + (kb0 + i) * KB, 0, &full[i]);
       bool ok = true;
       for (int i = ahead; i < nkb; ++i) {
         const int s = i % S::STAGES;
@@ -326,7 +327,7 @@ __global__ void __launch_bounds__(192, 1)
         if (!ok) break;
         mbar_expect_tx(&full[s], S::STAGE_BYTES);
         tma_load_2d(base + (size_t)s * S::STAGE_BYTES, &map_w, 0, wrow + i * TILE_M, &full[s]);
-        tma_load_2d(base + (size_t)s * S::STAGE_BYTES + S::A_BYTES, &map_x, (kb0 + i) * KB, 0, &full[s]);
+        tma_load_2d(base + (size_t)s * S::STAGE_BYTES + S::A_BYTES, &map_x, x0 + (kb0 + i) * KB, 0, &full[s]);
       }
     }
   } else if (warp == 1) {
@@ -382,9 +383,10 @@ __global__ void __launch_bounds__(192, 1)
           float z = 0.f;
           activate_pair(a.act, s, z);
         }
+        const size_t at = (size_t)j * a.ldo + (size_t)head * a.out_head + feat;
         if (split) static_cast<__nv_bfloat16*>(a.out_act)[(size_t)j * a.ldo_act + feat - a.act_from] = __float2bfloat16_rn(s);
-        else if (out_kind == OUT_F32) a.out[(size_t)j * a.ldo + feat] = s;
-        else static_cast<__nv_bfloat16*>(a.out_h)[(size_t)j * a.ldo + feat] = __float2bfloat16_rn(s);
+        else if (out_kind == OUT_F32) a.out[at] = s;
+        else static_cast<__nv_bfloat16*>(a.out_h)[at] = __float2bfloat16_rn(s);
       }
     }
   }
@@ -436,14 +438,14 @@ cudaError_t launch_bn(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
 template <int BN, int SPLITS>
 cudaError_t launch_rows(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
   CUtensorMap mx, mw;
-  const uint64_t tiles = (uint64_t)((a.n + TILE_M - 1) / TILE_M) * (a.k / KB);
-  if (!make_map_bf16(&mx, a.x, a.m, a.k, BN) || !make_map_bf16(&mw, a.w_tiled, tiles * TILE_M, KB, TILE_M)) return cudaErrorInvalidValue;
+  const uint64_t heads = std::max(a.heads, 1), tiles = heads * ((a.n + TILE_M - 1) / TILE_M) * (a.k / KB);
+  if (!make_map_bf16(&mx, a.x, a.m, a.heads ? a.ldx : a.k, BN) || !make_map_bf16(&mw, a.w_tiled, tiles * TILE_M, KB, TILE_M)) return cudaErrorInvalidValue;
   auto kernel = tc_gemm_bf16_rows_kernel<BN, SPLITS>;
   const size_t smem = RowsSmem<BN, SPLITS>::BYTES;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return e;
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3((a.n + TILE_M - 1) / TILE_M, SPLITS);
+  cfg.gridDim = dim3((a.n + TILE_M - 1) / TILE_M, SPLITS, (unsigned)heads);
   cfg.blockDim = dim3(192);
   cfg.dynamicSmemBytes = smem;
   cfg.stream = s;
@@ -463,7 +465,7 @@ template <int BN>
 cudaError_t launch_rows_bn(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
   // As many parts of k as fill the chip once, each at least two k blocks; clusters of eight only where a few of them are
   // needed: sixteen do not run at the same time (measured, 2048 output columns: 19 us in eight parts, 12 us in four).
-  const int tiles = (a.n + TILE_M - 1) / TILE_M, nkb = (a.k + KB - 1) / KB;
+  const int tiles = (a.n + TILE_M - 1) / TILE_M * std::max(a.heads, 1), nkb = (a.k + KB - 1) / KB;
   const int max_splits = tiles <= 8 ? 8 : 4;
   int splits = 1;
   while (splits < max_splits && tiles * splits * 2 <= sm_count() && splits * 4 <= nkb) splits *= 2;
@@ -481,7 +483,8 @@ bool gemm_bf16_rows_kernel(int m, int k) { return m <= 64 && k % KB == 0; }
 
 cudaError_t launch_tc_gemm_bf16(const Bf16GemmArgs& a, bool pdl, cudaStream_t s) {
   if (a.m <= 0 || a.n <= 0) return cudaSuccess;
-  if (a.act_from > 0 && (!a.w_tiled || !gemm_bf16_rows_kernel(a.m, a.k))) return cudaErrorInvalidValue;
+  if (a.heads > 0 && (a.x_head % 8 != 0 || a.ldx % 8 != 0)) return cudaErrorInvalidValue;  // TMA boxes start on 16 bytes
+  if ((a.act_from > 0 || a.heads > 0) && (!a.w_tiled || !gemm_bf16_rows_kernel(a.m, a.k))) return cudaErrorInvalidValue;
   if (a.k <= 0 || a.k % 8 != 0 || (!a.out && !a.out_h)) return cudaErrorInvalidValue;
   if (a.w_tiled && a.k % KB == 0) {
     if (a.m <= 16) return launch_rows_bn<16>(a, pdl, s);

@@ -41,7 +41,8 @@ struct DevBranch {
   int table = -1;      // ... of the page table (by distinct key lifetime)
   int state = -1;      // recurrence: index of the state array (and of the convolution inputs)
   int rot = -1, v_rot = -1;  // indices of the rotations
-  bool heads_step = false;   // decode: all heads of a sequence in one block
+  bool heads_step = false;   // decode: all heads of a sequence in one block ...
+  bool heads_tc = false;     // ... on the tensor cores
   // second step of two-step projections, over columns mid_off.. of the first ones' result (normed where mid_norm is set)
   Matrix mid;
   int mid_off = 0, mid_cols = 0;
@@ -50,6 +51,7 @@ struct DevBranch {
   AttentionLayer full{};
   Matrix up_kv;
   void *to_latent = nullptr, *from_latent = nullptr;  // [heads][dim][attn.dimp], [heads][kv_rank][full.vdimp]
+  Matrix to_latent_rows, from_latent_rows;            // the same for the tensor cores, 128 rows and their multiples per head
 };
 struct DevLayer {
   Norm norm1, norm1b, norm2, norm2b;
@@ -80,14 +82,20 @@ struct LayeredModel {
   std::vector<DevLayer> layers;
   int max_in = 0, max_y = 0, max_ff = 0, max_rec = 0;  // widest projection, mixer output, hidden row, heads * dim ...
   int max_rec_out = 0, max_rec_heads = 0;                  // ... heads * vdim and heads of a recurrence
-  int max_mid_k = 0, max_mid = 0, max_latent = 0;          // widest second-step input and output; heads * latent row
+  int max_mid_k = 0, max_mid = 0, max_latent = 0, max_wide = 0;  // widest second-step input and output; heads * latent row, heads * query
   int n_pools = 0, n_states = 0;
+  bool tc_rotations = false;  // a step needs the angles of its rows
   std::vector<KeyLife> lives;  // one page table each
   std::vector<Rotation> rotations;
   std::vector<void*> allocations;
   uint64_t weight_bytes = 0;
   int device = 0;
   size_t elem() const { return bf16 ? 2 : 4; }
+  size_t rotation_pairs() const {
+    size_t n = 0;
+    for (const Rotation& r : rotations) n += r.dims / 2;
+    return n;
+  }
   ~LayeredModel() {
     if (allocations.empty()) return;
     cudaSetDevice(device);
@@ -104,10 +112,11 @@ struct LayeredRows {  // activations of one pass, all [rows, pitch]
   float *h32 = nullptr, *y32 = nullptr, *ff32 = nullptr, *t32 = nullptr;  // decode with at most 8 BF16 rows: FP32 product inputs
   void* t = nullptr;                                // second-step input, storage type
   float* z = nullptr;                               // ... and output
-  float *q_latent = nullptr, *o_latent = nullptr;   // decode: queries against latent rows, sums of latent rows
+  float *q_latent = nullptr, *o_latent = nullptr;   // decode: queries against wide key rows, sums of latent rows
+  float2* angles = nullptr;                         // decode: (cos, sin) of every rotation, one after the other
   std::vector<void**> buffers() {
     return {(void**)&x[0], (void**)&x[1], (void**)&p,   (void**)&yo, &h, &y, &ff, (void**)&h32, (void**)&y32, (void**)&ff32,
-            (void**)&t32,  &t,            (void**)&z,   (void**)&q_latent, (void**)&o_latent};
+            (void**)&t32,  &t,            (void**)&z,   (void**)&q_latent, (void**)&o_latent, (void**)&angles};
   }
 };
 
@@ -314,11 +323,15 @@ int build_layer(Builder& b, const LayerSpec& spec, const std::string& p, int pag
         a.v_freq = m->rotations[br.v_rot].freq;
       }
       br.heads_step = a.life.window > 0 || a.mix || a.sink || a.q_bias || a.rot_dims || a.v_rot;
+      a.wide = br.heads_step ? 1 : 0;
       a.scale = s.scale; a.eps = eps; a.out_scale = bs.scale;
       a.page_tokens = page_tokens;
       a.pages_per_seq = (a.life.span + page_tokens - 1) / page_tokens;
       br.table = b.table(a.life);
+      m->max_wide = std::max(m->max_wide, s.heads * attention_q_width(a));
       br.pool = m->n_pools++;
+      br.heads_tc = m->bf16 && br.heads_step && attention_heads_tc_supported(a);
+      m->tc_rotations = m->tc_rotations || (br.heads_tc && (br.rot >= 0 || br.v_rot >= 0));
       if (br.heads_step ? !attention_heads_supported(a) : !attention_supported(a))
         return set_error(PG_INVALID_CONFIG, p + bs.prefix + ": " + std::to_string(s.heads / s.kv_heads) + " query heads per key head of size " +
                                                 std::to_string(s.dim) + " exceed what the decode kernel holds");
@@ -341,6 +354,8 @@ int build_layer(Builder& b, const LayerSpec& spec, const std::string& p, int pag
       br.table = b.table(a.life);
       br.pool = m->n_pools++;
       br.heads_step = true;
+      a.wide = 1;
+      br.heads_tc = m->bf16 && attention_heads_tc_supported(a);
       e = a;
       e.kv_heads = H; e.dim = s.dim; e.vdim = s.vdim;
       e.dimp = align_to(s.dim, 8); e.vdimp = e.vrow = align_to(s.vdim, 8);
@@ -358,8 +373,18 @@ int build_layer(Builder& b, const LayerSpec& spec, const std::string& p, int pag
       kv.insert(kv.end(), v.begin(), v.end());
       const uint64_t bytes = m->weight_bytes;  // a step does not read the copy for prompts
       if (int r = b.matrix(kv, H * (e.dimp + e.vdimp), s.kv_rank, N_ALIGN, &br.up_kv)) return r;
+      if (m->bf16) {
+        std::vector<float> ukt((size_t)H * s.kv_rank * s.dim);
+        for (int h = 0; h < H; ++h)
+          for (int c = 0; c < s.dim; ++c)
+            for (int j = 0; j < s.kv_rank; ++j) ukt[((size_t)h * s.kv_rank + j) * s.dim + c] = uk[((size_t)h * s.dim + c) * s.kv_rank + j];
+        const int kn = align_to(a.dimp, 128), vn = align_to(s.vdim, 128);
+        if (int r = b.matrix(pad_heads(ukt, H, s.kv_rank, kn, s.dim), H * kn, s.dim, 128, &br.to_latent_rows)) return r;
+        if (int r = b.matrix(pad_heads(uv, H, s.vdim, vn, s.kv_rank), H * vn, s.kv_rank, 128, &br.from_latent_rows)) return r;
+      }
       m->weight_bytes = bytes;
       m->max_latent = std::max(m->max_latent, H * a.dimp);
+      m->max_wide = std::max(m->max_wide, H * a.dimp);
       if (!attention_heads_supported(a))
         return set_error(PG_INVALID_CONFIG, p + bs.prefix + ": " + std::to_string(H) + " heads with latent rows of " + std::to_string(s.kv_rank) +
                                                 " exceed what the decode kernel holds");
@@ -524,8 +549,11 @@ int alloc_rows(const LayeredModel* m, LayeredRows* r, size_t rows, bool step) {
     if (int q = get(&r->t, rows * m->max_mid_k * e)) return q;
     if (int q = get((void**)&r->z, rows * m->max_mid * 4)) return q;
   }
+  if (step && m->max_wide)
+    if (int q = get((void**)&r->q_latent, rows * m->max_wide * 4)) return q;
+  if (step && m->rotation_pairs())
+    if (int q = get((void**)&r->angles, rows * m->rotation_pairs() * sizeof(float2))) return q;
   if (step && m->max_latent) {
-    if (int q = get((void**)&r->q_latent, rows * m->max_latent * 4)) return q;
     if (int q = get((void**)&r->o_latent, rows * m->max_latent * 4)) return q;
   }
   if (step && m->bf16) {
@@ -638,7 +666,7 @@ int layered_cache_init(pg_cache* c) {
         const size_t bytes = (size_t)c->tables[b.table].num_pages * attention_page_elems(b.attn) * m->elem();
         PG_CUDA_TRY(cudaMalloc(&lc->pools[b.pool], bytes));
         PG_CUDA_TRY(cudaMemsetAsync(lc->pools[b.pool], 0, bytes, c->stream));
-        part = std::max(part, B * b.attn.heads * MAX_SPLITS * (b.attn.vdim + 2));
+        part = std::max(part, B * b.attn.heads * MAX_SPLITS * attention_part_floats(b.attn));
         counters = std::max(counters, B * std::max(b.attn.kv_heads, b.attn.heads));
       } else {
         const size_t bytes = B * recurrence_state_floats(b.rec) * sizeof(float);
@@ -665,22 +693,39 @@ int layered_choose_splits(const pg_cache* c, int batch, int max_len) {
   if (m->backend.attn_splits > 0) return std::min(m->backend.attn_splits, MAX_SPLITS);
   // by the longest key range any layer can have at this length, in powers of two (a step graph per value)
   int span = 0, kv = 1 << 30, piece = 128, most = 8;
+  bool tc = false;
   for (const DevLayer& l : m->layered->layers)
     for (const DevBranch& b : l.branches)
       if (b.kind != BranchSpec::RECURRENCE) {
         span = std::max(span, std::min(b.attn.life.span, max_len));
         kv = std::min(kv, b.heads_step ? 1 : b.attn.kv_heads);
+        tc = tc || b.heads_tc;
         if (b.heads_step) {  // one block would hold all heads: shorter parts, more of them
           piece = 32;
           most = MAX_SPLITS;
         }
       }
   if (!span) return 1;
-  const int by_fill = (2 * m->num_sms + batch * kv - 1) / (batch * kv), by_len = (span + piece - 1) / piece;
   int s = 1;
+  if (tc) {  // tiles of keys; every layer chooses its parts from them (branch_splits)
+    while (s * 128 < span) s *= 2;
+    return s;
+  }
+  const int by_fill = (2 * m->num_sms + batch * kv - 1) / (batch * kv), by_len = (span + piece - 1) / piece;
   while (s * 2 <= std::min(std::min(by_fill, by_len), most)) s *= 2;
   return s;
 }
+
+namespace {
+
+// The parts of a branch's keys in a step, from what layered_choose_splits returned.
+int branch_splits(const pg_model* m, const DevBranch& b, int batch, int chosen) {
+  if (m->backend.attn_splits > 0) return chosen;
+  if (!b.heads_tc) return std::min(chosen, MAX_SPLITS);
+  return attention_heads_tc_splits(b.attn, batch, std::min(chosen, (b.attn.life.span + 127) / 128), m->num_sms);
+}
+
+}  // namespace
 
 namespace {
 
@@ -834,7 +879,77 @@ cudaError_t layered_enqueue_decode(pg_cache* c, int batch, int splits, cudaStrea
     na.h = r.t;
     if ((e = launch_norm_step(na, batch, m->bf16, pdl, s)) != cudaSuccess) return e;
     ++n;
-    return product(m, b.mid, r.t, r.z, nullptr, b.mid.np, b.mid.np, batch, nullptr, c->d_error, pdl, s);
+    const bool half = b.kind == BranchSpec::LATENT && b.heads_tc;  // straight into the next product
+    return product(m, b.mid, r.t, half ? nullptr : r.z, half ? r.z : nullptr, b.mid.np, b.mid.np, batch, nullptr, c->d_error, pdl, s);
+  };
+
+  if (m->tc_rotations) {
+    float2* at = r.angles;
+    for (const Rotation& rot : m->rotations) {
+      PG_L(B_OTHER, launch_angles(c->d_pos, rot.freq, at, batch, rot.dims / 2, pdl, s));
+      at += (size_t)batch * (rot.dims / 2);
+    }
+  }
+  auto angles_of = [&](int rotation) {
+    const float2* at = r.angles;
+    for (int i = 0; i < rotation; ++i) at += (size_t)batch * (m->rotations[i].dims / 2);
+    return at;
+  };
+  // Attention of a step on the tensor cores: queries and the new token's row, the products over the cached rows, the merge.
+  auto heads_tc_step = [&](const DevLayer& l, const DevBranch& b, AttentionStepArgs a, void* yb) -> cudaError_t {
+    AttentionPortionArgs pa{};
+    pa.l = b.attn; pa.p = r.p; pa.ldp = l.ldp; pa.rows = batch; pa.step_pos = c->d_pos; pa.pool = a.pool; pa.page_table = a.page_table;
+    pa.q = r.q_latent;
+    a.q16 = r.q_latent;
+    const float2* v_rot = b.v_rot >= 0 ? angles_of(b.v_rot) : nullptr;
+    if (b.kind == BranchSpec::ATTENTION) {
+      if (b.rot >= 0) pa.rot = angles_of(b.rot);
+      pa.v_rot = v_rot;
+      PG_L(B_ATTN, launch_attention_rotate(pa, true, s, pdl));
+      PG_L(B_ATTN, launch_attention_heads_tc(a, pdl, s));
+      PG_L(B_ATTN, launch_attention_merge(a, v_rot, y_bf16, pdl, s));
+      return cudaSuccess;
+    }
+    const int H = b.attn.heads;
+    PG_L(B_ATTN, launch_attention_latent(pa, true, s, pdl));
+    if (rows_path) {
+      HeadProductArgs hp{};
+      hp.w = b.to_latent; hp.x = r.z; hp.ldx = b.mid.np; hp.ldxh = b.full.dimp;
+      hp.out = r.q_latent; hp.ldo = H * b.attn.dimp; hp.ldh = b.attn.dimp;
+      hp.batch = batch; hp.heads = H; hp.k = b.full.dim; hp.n = hp.np = b.attn.dimp;
+      PG_L(B_ATTN, launch_head_product(hp, true, true, pdl, s));
+      PG_L(B_ATTN, launch_attention_heads_tc(a, pdl, s));
+      a.y = r.o_latent; a.ldy = H * b.attn.dimp; a.ldyh = b.attn.dimp;
+      PG_L(B_ATTN, launch_attention_merge(a, nullptr, false, pdl, s));
+      hp.w = b.from_latent; hp.x = r.o_latent; hp.ldx = a.ldy; hp.ldxh = a.ldyh;
+      hp.out = yb; hp.ldo = l.out.kp; hp.ldh = b.full.vdim;
+      hp.k = b.attn.vdim; hp.n = b.full.vdim; hp.np = b.full.vdimp;
+      PG_L(B_ATTN, launch_head_product(hp, true, false, pdl, s));
+      return cudaSuccess;
+    }
+    // a product per head: the kernel takes 64 rows at a time
+    auto per_head = [&](Bf16GemmArgs g) -> cudaError_t {
+      const char *x = static_cast<const char*>(g.x), *out = static_cast<const char*>(g.out_h);
+      for (int r0 = 0; r0 < batch; r0 += 64) {
+        g.x = x + (size_t)r0 * g.ldx * 2;
+        g.out_h = const_cast<char*>(out) + (size_t)r0 * g.ldo * 2;
+        g.m = std::min(64, batch - r0);
+        PG_L(B_ATTN, launch_tc_gemm_bf16(g, pdl, s));
+      }
+      return cudaSuccess;
+    };
+    Bf16GemmArgs g{};
+    g.w = b.to_latent_rows.w; g.w_tiled = b.to_latent_rows.tiled; g.k = b.to_latent_rows.kp;
+    g.x = r.z; g.ldx = b.mid.np; g.x_head = b.full.dimp; g.heads = H; g.m = batch; g.error_flag = c->d_error;
+    g.out_h = r.q_latent; g.ldo = H * b.attn.dimp; g.out_head = b.attn.dimp; g.n = b.attn.dimp;
+    if ((e = per_head(g)) != cudaSuccess) return e;
+    PG_L(B_ATTN, launch_attention_heads_tc(a, pdl, s));
+    a.y = r.o_latent; a.ldy = H * b.attn.dimp; a.ldyh = b.attn.dimp;
+    PG_L(B_ATTN, launch_attention_merge(a, nullptr, true, pdl, s));
+    g.w = b.from_latent_rows.w; g.w_tiled = b.from_latent_rows.tiled; g.k = b.from_latent_rows.kp;
+    g.x = r.o_latent; g.ldx = a.ldy; g.x_head = a.ldyh;
+    g.out_h = yb; g.ldo = l.out.kp; g.out_head = b.full.vdim; g.n = b.full.vdim;
+    return per_head(g);
   };
 
   for (const DevLayer& l : m->layers) {
@@ -858,9 +973,12 @@ cudaError_t layered_enqueue_decode(pg_cache* c, int batch, int splits, cudaStrea
       if (b.kind != BranchSpec::RECURRENCE) {
         AttentionStepArgs a{};
         a.l = b.attn; a.p = r.p; a.ldp = l.ldp; a.pool = lc->pools[b.pool]; a.page_table = c->tables[b.table].d_table;
-        a.pos = c->d_pos; a.part = lc->attn_part; a.counters = lc->attn_counters;
-        a.y = yb; a.ldy = l.out.kp; a.batch = batch; a.splits = splits;
-        if (b.kind == BranchSpec::ATTENTION) {
+        a.pos = c->d_pos; a.part = lc->attn_part; a.counters = lc->attn_counters; a.num_pages = c->tables[b.table].num_pages;
+        a.y = yb; a.ldy = l.out.kp; a.ldyh = b.attn.vdim; a.batch = batch; a.splits = branch_splits(pm, b, batch, splits);
+        a.error_flag = c->d_error;
+        if (b.heads_tc) {
+          if ((e = heads_tc_step(l, b, a, yb)) != cudaSuccess) return e;
+        } else if (b.kind == BranchSpec::ATTENTION) {
           PG_L(B_ATTN, b.heads_step ? launch_attention_heads_step(a, m->bf16, y_bf16, pdl, s) : launch_attention_step(a, m->bf16, y_bf16, pdl, s));
         } else {  // queries to the latent space, attention over latent rows, values back from it
           HeadProductArgs hp{};
@@ -868,7 +986,7 @@ cudaError_t layered_enqueue_decode(pg_cache* c, int batch, int splits, cudaStrea
           hp.out = r.q_latent; hp.ldo = b.attn.heads * b.attn.dimp; hp.ldh = b.attn.dimp;
           hp.batch = batch; hp.heads = b.attn.heads; hp.k = b.full.dim; hp.n = hp.np = b.attn.dimp;
           PG_L(B_ATTN, launch_head_product(hp, m->bf16, false, pdl, s));
-          a.q = r.q_latent; a.y = r.o_latent; a.ldy = b.attn.heads * b.attn.vdim;
+          a.q = r.q_latent; a.y = r.o_latent; a.ldy = b.attn.heads * b.attn.vdim; a.ldyh = b.attn.vdim;
           PG_L(B_ATTN, launch_attention_heads_step(a, m->bf16, false, pdl, s));
           hp.w = b.from_latent; hp.x = r.o_latent; hp.ldx = a.ldy; hp.ldxh = b.attn.vdim;
           hp.out = yb; hp.ldo = l.out.kp; hp.ldh = b.full.vdim;
@@ -1100,7 +1218,7 @@ int layered_run_portions(pg_cache* c, const PortionPlan& plan, float* logits, St
     if (int r = grow(&lc->angles, &lc->angle_rows, rows, half * sizeof(float2))) return r;
   float2* at = lc->angles;
   for (const Rotation& r : m->rotations) {  // this pass's angles, shared by the layers
-    PG_CUDA_TRY(launch_angles(d.pos, r.freq, at, rows, r.dims / 2, c->stream));
+    PG_CUDA_TRY(launch_angles(d.pos, r.freq, at, rows, r.dims / 2, false, c->stream));
     d.angles.push_back(at);
     at += (size_t)rows * (r.dims / 2);
   }

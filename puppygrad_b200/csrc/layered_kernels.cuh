@@ -91,6 +91,9 @@ struct Bf16GemmArgs {
   int act_from;     // 0: off
   void* out_act;
   int ldo_act;
+  // decode rows only: `heads` products side by side, head h over columns h * x_head.. of x with its own weights (tiled: n rounded up
+  // to 128 rows per head) to columns h * out_head.. of out
+  int heads, x_head, out_head, ldx;  // heads 0: one product; ldx: row pitch of x
 };
 // Whether a product of m rows takes the kernel that knows act_from.
 bool gemm_bf16_rows_kernel(int m, int k);
@@ -190,6 +193,7 @@ struct KeyLife {
 // dimp / vdimp; a latent row (vrow == 0) is key and value in one.
 struct AttentionLayer {
   int heads, kv_heads, dim, vdim, dimp, vdimp, vrow;  // vrow: pitch of the cached value rows
+  int wide;  // page layout: 1: a token's rows of all key heads side by side, 0: a key head's rows of all tokens
   KeyLife life;
   int off_q, off_k, off_v, off_gate;  // off_gate < 0: no gate per head
   const float *q_norm, *k_norm;  // [dim] or nullptr
@@ -201,21 +205,27 @@ struct AttentionLayer {
   float scale, eps, out_scale;
   int page_tokens, pages_per_seq;
 };
-size_t attention_page_elems(const AttentionLayer& l);  // elements of one page: [kv_heads][page_tokens][dimp] keys, then values
+// Elements of one page: keys [kv_heads][page_tokens][dimp] (wide: [page_tokens][kv_heads][dimp]), then the values alike.
+size_t attention_page_elems(const AttentionLayer& l);
 bool attention_supported(const AttentionLayer& l);
 struct AttentionStepArgs {
   AttentionLayer l;
   const float* p;
   int ldp;
-  const float* q;         // latent rows: [batch, heads * dimp] queries against them
+  const float* q;         // latent rows: [batch, heads * dimp] queries against them (FP32 path)
+  const void* q16;        // launch_attention_heads_tc: [batch, heads * attention_q_width()] BF16 queries
+  int num_pages;          // of the pool
   void* pool;
   const int* page_table;  // [slot][pages_per_seq]
   const int* pos;
-  float* part;            // [batch * heads][splits][vdim + 2]
+  float* part;            // [batch * heads][splits][attention_part_floats()]
   unsigned* counters;     // [batch * max(kv_heads, heads)], zero between launches
   void* y;
-  int ldy, batch, splits;
+  int ldy, ldyh, batch, splits;  // ldyh: columns between the outputs of two heads (the merge clears those past vdim)
+  int* error_flag;
 };
+// A part of one head's result: maximum, sum, (padding), sums of values.
+inline int attention_part_floats(const AttentionLayer& l) { return 4 + (l.vdim + 3) / 4 * 4; }
 // One block per key head: no rotation, mixing, sink, window or latent rows.
 cudaError_t launch_attention_step(const AttentionStepArgs& a, bool bf16, bool y_bf16, bool pdl, cudaStream_t s);
 struct AttentionPortionArgs {
@@ -228,6 +238,7 @@ struct AttentionPortionArgs {
   const int* seq_pos;     // [nseq] position of the first row
   const int* row_seq;     // [rows] sequence of each row
   const float2 *rot, *v_rot;  // (cos, sin) of every row: [rows][rot_dims / 2], [rows][vdim / 2]
+  const int* step_pos;    // one new token of slot `row` per row, at this position: keys and values go straight to the pages
   void* pool;
   const int* page_table;
   void *q, *k, *v;        // workspaces in T: [rows][heads * q_width()], [krows][ldk], [krows][ldv]
@@ -237,7 +248,7 @@ struct AttentionPortionArgs {
   int ldy;
 };
 // With mixed heads the mixing is moved to the queries: head h scores all key heads at once, against the whole row of keys.
-inline int attention_q_width(const AttentionLayer& l) { return l.mix ? l.kv_heads * l.dimp : l.dimp; }
+__host__ __device__ inline int attention_q_width(const AttentionLayer& l) { return l.mix ? l.kv_heads * l.dimp : l.dimp; }
 // Makes the rows' queries, keys and values ready in the workspaces, copies the cached keys and values that the first rows
 // still see in front of them, attends, and stores what later tokens can still see into the pages.
 cudaError_t launch_attention_portion(const AttentionPortionArgs& a, bool bf16, cudaStream_t s);
@@ -249,16 +260,28 @@ cudaError_t launch_attention_tc(const AttentionPortionArgs& a, cudaStream_t s); 
 
 // ------------------------------------------------------------------ attn_heads.cu
 // One token per sequence, all heads of it in a block: rotation, mixed heads, sink, window with kept first tokens, latent rows.
+// Makes its queries, keys and values itself and appends the new token.
 cudaError_t launch_attention_heads_step(const AttentionStepArgs& a, bool bf16, bool y_bf16, bool pdl, cudaStream_t s);
 bool attention_heads_supported(const AttentionLayer& l);
 // out[rows][half] = (cos, sin) of pos * freq
-cudaError_t launch_angles(const int* pos, const double* freq, float2* out, int rows, int half, cudaStream_t s);
-// The rows' rotated and mixed queries, rotated keys and values, into the workspaces.
-cudaError_t launch_attention_rotate(const AttentionPortionArgs& a, bool bf16, cudaStream_t s);
-// The rows' normed latents into the key workspace.
-cudaError_t launch_attention_latent(const AttentionPortionArgs& a, bool bf16, cudaStream_t s);
+cudaError_t launch_angles(const int* pos, const double* freq, float2* out, int rows, int half, bool pdl, cudaStream_t s);
+// The rows' rotated and mixed queries, rotated keys and values, into the workspaces (a step's keys and values into the pages).
+cudaError_t launch_attention_rotate(const AttentionPortionArgs& a, bool bf16, cudaStream_t s, bool pdl = false);
+// The rows' normed latents into the key workspace (a step's into the pages).
+cudaError_t launch_attention_latent(const AttentionPortionArgs& a, bool bf16, cudaStream_t s, bool pdl = false);
 // Turns FP32 outputs back by their rows' angles, in place.
 cudaError_t launch_attention_turn_back(const AttentionPortionArgs& a, cudaStream_t s);
+// Adds the parts of a step's heads: sink, turning back, gate, branch scale; y in FP32 or BF16.
+cudaError_t launch_attention_merge(const AttentionStepArgs& a, const float2* v_rot, bool y_bf16, bool pdl, cudaStream_t s);
+
+// ------------------------------------------------------------------ attn_heads_tc.cu
+// One token per sequence on the tensor cores, for heads that share wide key rows (mixed heads, latent rows): BF16 queries a.q16
+// against the cached rows, results as parts for launch_attention_merge. The new token's row must be in its page.
+bool attention_heads_tc_supported(const AttentionLayer& l);
+int attention_heads_tc_splits(const AttentionLayer& l, int batch, int tiles, int sms);  // parts for `tiles` tiles of 128 keys
+cudaError_t launch_attention_heads_tc(const AttentionStepArgs& a, bool pdl, cudaStream_t s);
+
+// ------------------------------------------------------------------ attn_heads.cu
 // out[b, h * ldh + n] = sum_k x[b, h * ldxh + k] w[h][k][n], w in T with rows of np (a multiple of 8)
 struct HeadProductArgs {
   const void* w;

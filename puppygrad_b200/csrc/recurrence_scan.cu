@@ -196,6 +196,66 @@ __global__ void __launch_bounds__(256) channel_conv_kernel(RecurrenceScanArgs a)
   }
 }
 
+// The same when every size and offset is a multiple of four and heads have at most 128 channels: four channels per lane, the
+// rows of a group requested four at a time.
+template <int TAPS>
+__global__ void __launch_bounds__(256) channel_conv_vec_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int lane = threadIdx.x & 31, units = 2 * l.kv_heads + l.heads;
+  const int groups = (a.rows + CONV_ROWS - 1) / CONV_ROWS;
+  const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  if (w >= (long long)groups * units) return;
+  const int r0 = (int)(w / units) * CONV_ROWS, u = (int)(w % units), r1 = min(r0 + CONV_ROWS, a.rows);
+  const bool is_q = u < l.kv_heads, is_k = !is_q && u < 2 * l.kv_heads;
+  const int h = is_q ? u : is_k ? u - l.kv_heads : u - 2 * l.kv_heads, n = is_q || is_k ? l.dim : l.vdim, c = lane * 4;
+  const bool on = c < n;
+  const int ch = (is_q ? l.off_q : is_k ? l.off_k : l.off_v) - l.off_q + h * n + (on ? c : 0), pitch = (is_q || is_k ? l.kv_heads : l.heads) * n;
+  float* dst = (is_q ? a.rate : is_k ? a.unit : a.vals) + h * n + c;
+  const float* src = a.p + l.off_q + ch;
+  float4 win[TAPS], wt[TAPS];  // inputs (the newest last) and weights
+#pragma unroll
+  for (int t = 0; t < TAPS; ++t) wt[t] = load4(l.conv + (size_t)t * l.channels + ch);
+  const bool one = a.row_seq[r0] == a.row_seq[r1 - 1];  // the whole group in one sequence
+  int seq = -1;
+  for (int rb = r0; rb < r1; rb += 4) {
+    float4 x[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) x[j] = load4(src + (size_t)min(rb + j, r1 - 1) * a.ldp);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int r = rb + j;
+      if (r >= r1) break;
+      const int s = one && seq >= 0 ? seq : a.row_seq[r];
+      if (s != seq) {  // entering a sequence: its cached inputs, or what the portion has before this group
+        seq = s;
+        const int first = a.seq_start[s], pos = a.seq_pos[s] + r - first;
+        const float* taps = a.taps + (size_t)a.seq_slot[s] * l.taps * l.channels;
+#pragma unroll
+        for (int t = 0; t + 1 < TAPS; ++t) {
+          const int back = TAPS - 1 - t;
+          win[t + 1] = r - back >= first ? load4(src + (size_t)(r - back) * a.ldp)
+                       : pos - back >= 0 ? load4(taps + (size_t)((pos - back) % TAPS) * l.channels + ch) : make_float4(0, 0, 0, 0);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t + 1 < TAPS; ++t) win[t] = win[t + 1];
+      win[TAPS - 1] = x[j];
+      float4 y = make_float4(0, 0, 0, 0);
+#pragma unroll
+      for (int t = 0; t < TAPS; ++t) {
+        y.x = fmaf(wt[t].x, win[t].x, y.x); y.y = fmaf(wt[t].y, win[t].y, y.y);
+        y.z = fmaf(wt[t].z, win[t].z, y.z); y.w = fmaf(wt[t].w, win[t].w, y.w);
+      }
+      y.x = silu_f(y.x); y.y = silu_f(y.y); y.z = silu_f(y.z); y.w = silu_f(y.w);
+      if (is_q || is_k) {
+        const float sq = on ? (y.x * y.x + y.y * y.y) + (y.z * y.z + y.w * y.w) : 0.f, inv = 1.f / sqrtf(lane_sum(sq) + UNIT_EPS);
+        y.x *= inv; y.y *= inv; y.z *= inv; y.w *= inv;
+      }
+      if (on) store4(dst + (size_t)r * pitch, y);
+    }
+  }
+}
+
 // Channel delta rule, after the convolutions: the decays, and what the scan needs to take two tokens at a time: the next
 // token's k times its decay . this one's k, and the write strength. A warp takes a head over GATE_GROUP rows (and looks at
 // the row behind them).
@@ -231,6 +291,47 @@ __global__ void __launch_bounds__(256) channel_gates_kernel(RecurrenceScanArgs a
   }
 }
 
+// The same for heads of at most 128 channels, a multiple of four: the rows of a group are requested together.
+__global__ void __launch_bounds__(256) channel_gates_vec_kernel(RecurrenceScanArgs a) {
+  const RecurrenceLayer& l = a.l;
+  const int lane = threadIdx.x & 31, K = l.heads * l.dim, rep = l.heads / l.kv_heads;
+  const int groups = (a.rows + GATE_GROUP - 1) / GATE_GROUP;
+  const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+  if (w >= (long long)groups * l.heads) return;
+  const int r0 = (int)(w / l.heads) * GATE_GROUP, head = (int)(w % l.heads), c = lane * 4;
+  const bool on = c < l.dim;
+  const size_t ch = (size_t)head * l.dim + (on ? c : 0);
+  const float* kp = a.unit + head / rep * l.dim + (on ? c : 0);
+  float4 z[GATE_GROUP + 1], k[GATE_GROUP + 1];
+#pragma unroll
+  for (int j = 0; j <= GATE_GROUP; ++j) {
+    const int r = min(r0 + j, a.rows - 1);
+    z[j] = load4(a.z + (size_t)r * a.ldz + ch);
+    k[j] = load4(kp + (size_t)r * l.kv_heads * l.dim);
+  }
+  const float beta = lane < GATE_GROUP && r0 + lane < a.rows ? a.p[(size_t)(r0 + lane) * a.ldp + l.off_b + head] : 0.f;
+  const float4 b = load4(l.b2 + ch);
+  const float na = l.neg_a[head];
+  auto decay = [&](float v, float bias) { return expf(na * softplus_f(v + bias)); };
+  float dots[GATE_GROUP];
+#pragma unroll
+  for (int j = 0; j <= GATE_GROUP; ++j) {
+    const float4 d = make_float4(decay(z[j].x, b.x), decay(z[j].y, b.y), decay(z[j].z, b.z), decay(z[j].w, b.w));
+    if (j < GATE_GROUP && on && r0 + j < a.rows) store4(a.decay + (size_t)(r0 + j) * K + ch, d);
+    if (j > 0) {
+      const float4 o = k[j - 1], q = k[j];
+      dots[j - 1] = on ? (d.x * q.x * o.x + d.y * q.y * o.y) + (d.z * q.z * o.z + d.w * q.w * o.w) : 0.f;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < GATE_GROUP; ++j) dots[j] = lane_sum(dots[j]);
+  float mine = 0.f;
+#pragma unroll
+  for (int j = 0; j < GATE_GROUP; ++j) mine = lane == j ? dots[j] : mine;
+  if (lane < GATE_GROUP && r0 + lane < a.rows)
+    *reinterpret_cast<float2*>(a.pair + ((size_t)(r0 + lane) * l.heads + head) * 4) = make_float2(mine, sigmoid_f(beta));
+}
+
 // The inputs that the next tokens' convolutions still need. Block = (sequence, one of its last taps - 1 rows).
 __global__ void __launch_bounds__(256) channel_taps_kernel(RecurrenceScanArgs a) {
   const RecurrenceLayer& l = a.l;
@@ -238,6 +339,7 @@ __global__ void __launch_bounds__(256) channel_taps_kernel(RecurrenceScanArgs a)
   if (r < first) return;
   const int pos = a.seq_pos[seq] + r - first;
   float* dst = a.taps + ((size_t)a.seq_slot[seq] * l.taps + pos % l.taps) * l.channels;
+#pragma unroll 8
   for (int c = threadIdx.x; c < l.channels; c += blockDim.x) dst[c] = a.p[(size_t)r * a.ldp + l.off_q + c];
 }
 
@@ -890,7 +992,16 @@ cudaError_t launch_channel_gates(const RecurrenceScanArgs& a, cudaStream_t s) {
   const long long gw = (long long)((a.rows + GATE_GROUP - 1) / GATE_GROUP) * l.heads;
   const dim3 cg((unsigned)((cw + 7) / 8)), gg((unsigned)((gw + 7) / 8)), b(256);
   const int size = std::max(l.dim, l.vdim);
+  const bool vec = l.dim % 4 == 0 && l.vdim % 4 == 0 && size <= 128 && l.taps >= 2 && l.taps <= 4 && a.ldp % 4 == 0 && l.off_q % 4 == 0 &&
+                   l.off_k % 4 == 0 && l.off_v % 4 == 0 && l.channels % 4 == 0 && a.ldz % 4 == 0;
   cudaError_t e;
+  if (vec) {
+    e = l.taps == 2   ? launch_kernel(channel_conv_vec_kernel<2>, cg, b, 0, s, false, a)
+        : l.taps == 3 ? launch_kernel(channel_conv_vec_kernel<3>, cg, b, 0, s, false, a)
+                      : launch_kernel(channel_conv_vec_kernel<4>, cg, b, 0, s, false, a);
+    if (e == cudaSuccess) e = launch_kernel(channel_gates_vec_kernel, gg, b, 0, s, false, a);
+    return e != cudaSuccess ? e : launch_kernel(channel_taps_kernel, dim3(a.nseq, l.taps - 1), b, 0, s, false, a);
+  }
 #define PG_CONV(TAPS_)                                                                                  \
   (size <= 64    ? launch_kernel(channel_conv_kernel<TAPS_, 2>, cg, b, 0, s, false, a)                  \
    : size <= 128 ? launch_kernel(channel_conv_kernel<TAPS_, 4>, cg, b, 0, s, false, a)                  \
