@@ -3,8 +3,8 @@
 //
 // Work item = 128 query rows of one head of one sequence; a persistent block takes items in turn, so that the loads and
 // first scores of an item overlap the end of the one before. Warp 0 loads, warp 1 issues the MMAs, warps 2..5 do the
-// softmax (thread = row). S(j + 1) = Q K^T is issued before O += P(j) V, so that the tensor cores work on the next scores
-// while the softmax warps are busy; keys and values have rings of their own. An item walks only the key tiles that some
+// softmax (thread = row). S(j + 1) = Q K^T is issued as soon as the softmax warps hold S(j) in registers, so that the tensor cores
+// work on the next scores while those warps are busy; keys and values have rings of their own. An item walks only the key tiles that some
 // row of it can see: those of the moving range, and before them those of the sequence's kept first keys. Keys come in pieces of
 // 64 columns through a ring; where the queries of an item do not fit beside it, their pieces come with the keys', again for
 // every tile. Every wait is bounded: on expiry the error flag is set, work stops, tensor memory is freed.
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(192, 2)
     attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, AttentionPortionArgs a, TcShape t, int items, int qtiles) {
   extern __shared__ uint8_t smem_raw[];
-  __shared__ uint64_t q_full, q_empty, k_full[MAX_KSTAGES], k_empty[MAX_KSTAGES], v_full[2], v_empty[2], s_full, p_ready, pv_done, o_free;
+  __shared__ uint64_t q_full, q_empty, k_full[MAX_KSTAGES], k_empty[MAX_KSTAGES], v_full[2], v_empty[2], s_full, s_free, p_ready, pv_done, o_free;
   __shared__ uint32_t tmem_slot;
   __shared__ int failed_flag;
   const AttentionLayer& l = a.l;
@@ -102,6 +102,7 @@ __global__ void __launch_bounds__(192, 2)
       mbar_init(&v_empty[i], 1);
     }
     mbar_init(&s_full, 1);
+    mbar_init(&s_free, 4);
     mbar_init(&p_ready, 4);
     mbar_init(&pv_done, 1);
     mbar_init(&o_free, 4);
@@ -170,17 +171,20 @@ __global__ void __launch_bounds__(192, 2)
         umma_commit(&s_full);
         return true;
       };
-      // S(gt) may be overwritten once the softmax warps have read it, which they tell with p_ready(gt): every scores()
-      // but the very first one follows such a wait.
+      // S(gt) may be overwritten once the softmax warps have read it, which they tell with s_free(gt): every scores() but the
+      // very first one follows such a wait.
       for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
         if (!w.set(a, it, qtiles)) continue;
         ok = (!t.q_resident || mbar_wait(&q_full, done & 1, failed, a.error_flag, 24)) && scores(w.tiles == 1);
         for (int j = 0; j < w.tiles && ok; ++j) {
           const uint32_t gt = g + j;
-          ok = mbar_wait(&p_ready, gt & 1, failed, a.error_flag, 25);  // P is written, S has been read
+          ok = mbar_wait(&s_free, gt & 1, failed, a.error_flag, 31);  // S has been read
           if (!ok) break;
           tc_fence_after();
           if (j + 1 < w.tiles) ok = scores(j + 2 == w.tiles);
+          ok = ok && mbar_wait(&p_ready, gt & 1, failed, a.error_flag, 25);  // P is written
+          if (!ok) break;
+          tc_fence_after();
           const uint32_t v = gt % t.vstages;
           ok = ok && mbar_wait(&v_full[v], (gt / t.vstages) & 1, failed, a.error_flag, 26);
           if (ok && j == 0 && done > 0) ok = mbar_wait(&o_free, (done - 1) & 1, failed, a.error_flag, 30);  // O of the item before has been read
@@ -219,6 +223,9 @@ __global__ void __launch_bounds__(192, 2)
 #pragma unroll
           for (int i = 0; i < 32; ++i) s[c * 32 + i] = v[i];
         }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s_free);
         const int k0 = w.start(j), k1 = w.end(j);
         if (j < w.kept_tiles ? k0 + KROWS > k1 : k0 < lo_all || k0 + KROWS - 1 > hi_all) {
           const int lo_i = lo_row - k0, hi_i = min(hi_row, k1 - 1) - k0, keep_i = keep - k0;

@@ -405,20 +405,6 @@ bool step_shape(const AttentionLayer& l, StepShape* sh) {
 }
 
 // ------------------------------------------------------------------ portions
-__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
-  store4(p, make_float4(v[0], v[1], v[2], v[3]));
-  store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
-}
-__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
-  uint32_t u[4];
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-    u[i] = *reinterpret_cast<const uint32_t*>(&b);
-  }
-  *reinterpret_cast<uint4*>(p) = make_uint4(u[0], u[1], u[2], u[3]);
-}
-
 // Where a row's key or value of one head goes: the workspace, or (a step) the page of its position.
 template <typename T>
 __device__ __forceinline__ T* key_target(const AttentionPortionArgs& a, int row, int head, int which) {
@@ -430,76 +416,102 @@ __device__ __forceinline__ T* key_target(const AttentionPortionArgs& a, int row,
   return which == 0 ? static_cast<T*>(a.k) + krow * a.ldk + head * l.dimp : static_cast<T*>(a.v) + krow * a.ldv + head * l.vdimp;
 }
 
-// Block = ROWS rows and one key head with the query heads that read it: biases, rotation. With mixed heads, piece c of head
-// h's query (the part against key head c) = sum over the heads g that read key head c of mix[h][g] q_g.
-constexpr int ROT_THREADS = 256, ROT_PORTION_ROWS = 8;
-template <typename T, int ROWS>
-__global__ void __launch_bounds__(ROT_THREADS) attention_rotate_kernel(AttentionPortionArgs a) {
-  extern __shared__ __align__(16) float sm[];  // [ROWS][rep][dimp] queries, [heads][rep] mixing
+// Block = up to `rows` rows and one key head with the query heads that read it: biases, rotation. With mixed heads, piece c of
+// head h's query (the part against key head c) = sum over the heads g that read key head c of mix[h][g] q_g. UNROLL rows are
+// requested together; what depends on the column only is worked out once per block.
+constexpr int ROT_THREADS = 256, ROT_MAX_ROWS = 32;
+template <typename T, int UNROLL>
+__global__ void __launch_bounds__(ROT_THREADS, 4) attention_rotate_kernel(AttentionPortionArgs a, int rows) {
+  extern __shared__ __align__(16) float sm[];  // [rows][rep][dimp] queries, [heads][rep] mixing
+  __shared__ T* target[2 * ROT_MAX_ROWS];      // where the rows' key and value go
   const AttentionLayer& l = a.l;
-  const int row0 = blockIdx.x * ROWS, c = blockIdx.y, nrows = min(ROWS, a.rows - row0), tid = threadIdx.x, H = l.heads, G = l.kv_heads, rep = H / G;
+  const int row0 = blockIdx.y * rows, c = blockIdx.x, nrows = min(rows, a.rows - row0), tid = threadIdx.x, H = l.heads, G = l.kv_heads, rep = H / G;
   const int qn = rep * l.dimp, per = qn + l.dimp + l.vdimp;
   float* qs = sm;
-  float* mix = qs + (size_t)ROWS * qn;
+  float* mix = qs + (size_t)rows * qn;
   grid_dep_launch();
   if (l.mix)
     for (int i = tid; i < H * rep; i += ROT_THREADS) mix[i] = l.mix[(size_t)(i / rep) * H + c * rep + i % rep];
   grid_dep_wait();
+  if (tid < 2 * nrows) target[tid] = key_target<T>(a, row0 + tid / 2, c, tid & 1);
+  __syncthreads();
   for (int e = tid; e < per; e += ROT_THREADS) {  // a column of the block's rows
     const bool is_q = e < qn, is_k = !is_q && e < qn + l.dimp;
     const int x = is_q ? e : is_k ? e - qn : e - qn - l.dimp, np = is_q || is_k ? l.dimp : l.vdimp, n = is_q || is_k ? l.dim : l.vdim;
     const int head = is_q ? c * rep + x / np : c, col = x % np, dims = is_q || is_k ? l.rot_dims : l.v_rot ? l.vdim : 0;
-    const float* src = a.p + (is_q ? l.off_q : is_k ? l.off_k : l.off_v) + head * n;
     const float* bias = is_q ? l.q_bias : is_k ? l.k_bias : l.v_bias;
-    const float2* cs = is_q || is_k ? a.rot : a.v_rot;
-    // entry `col` = x cos + sign * partner * sin
-    const int half = dims >> 1, partner = col >= dims || col >= n ? -1 : col < half ? col + half : col - half, turn = col < half ? col : col - half;
-    const float sign = col < half ? -1.f : 1.f;
-    const float b0 = bias && col < n ? bias[head * n + col] : 0.f, b1 = bias && partner >= 0 ? bias[head * n + partner] : 0.f;
-    float v[ROWS];
+    // entry `col` = x cos + partner * (-sin or sin); past the rotated entries the factors are 1 and 0
+    const int half = dims >> 1, turn = col < half ? col : col - half;
+    const bool on = col < n, turned = on && col < dims;
+    const int partner = turned ? (col < half ? col + half : col - half) : col;
+    const float sign = !turned ? 0.f : col < half ? -1.f : 1.f;
+    const float* src = a.p + (size_t)row0 * a.ldp + (is_q ? l.off_q : is_k ? l.off_k : l.off_v) + head * n;
+    const float2* cs = turned ? (is_q || is_k ? a.rot : a.v_rot) + (size_t)row0 * half + turn : nullptr;
+    const float b0 = bias && on ? bias[head * n + col] : 0.f, b1 = bias && on ? bias[head * n + partner] : 0.f;
+    T* q16 = static_cast<T*>(a.q) + ((size_t)row0 * H + head) * l.dimp + col;
+    for (int r0 = 0; r0 < nrows; r0 += UNROLL) {
+      float u[UNROLL], v[UNROLL];
+      float2 f[UNROLL];
 #pragma unroll
-    for (int rr = 0; rr < ROWS; ++rr) {
-      v[rr] = 0.f;
-      if (rr < nrows && col < n) {
-        const float* p = src + (size_t)(row0 + rr) * a.ldp;
-        v[rr] = p[col] + b0;
-        if (partner >= 0) {
-          const float2 r = cs[(size_t)(row0 + rr) * half + turn];
-          v[rr] = v[rr] * r.x + sign * ((p[partner] + b1) * r.y);
-        }
+      for (int i = 0; i < UNROLL; ++i) {
+        const int r = min(r0 + i, nrows - 1);
+        const float* p = src + (size_t)r * a.ldp;
+        u[i] = on ? p[col] + b0 : 0.f;
+        v[i] = on ? p[partner] + b1 : 0.f;
+        f[i] = turned ? cs[(size_t)r * half] : make_float2(1.f, 0.f);
+      }
+#pragma unroll
+      for (int i = 0; i < UNROLL; ++i) {
+        const int r = r0 + i;
+        if (r >= nrows) break;
+        const float y = u[i] * f[i].x + sign * (v[i] * f[i].y);
+        if (!is_q) target[2 * r + (is_k ? 0 : 1)][col] = from_f32<T>(y);
+        else if (l.mix) qs[r * qn + x] = y;
+        else q16[(size_t)r * H * l.dimp] = from_f32<T>(y);
       }
     }
-#pragma unroll
-    for (int rr = 0; rr < ROWS; ++rr)
-      if (rr < nrows) {
-        if (!is_q) key_target<T>(a, row0 + rr, c, is_k ? 0 : 1)[col] = from_f32<T>(v[rr]);
-        else if (l.mix) qs[rr * qn + x] = v[rr];
-        else static_cast<T*>(a.q)[((size_t)(row0 + rr) * H + head) * l.dimp + col] = from_f32<T>(v[rr]);
-      }
   }
   if (!l.mix) return;
   __syncthreads();
-  const int no = l.dimp / 8;
-  for (int i = tid; i < H * no; i += ROT_THREADS) {
-    const int o = i % no, h = i / no;
-    const float* t = mix + h * rep;
-    T* out = static_cast<T*>(a.q) + (((size_t)row0 * H + h) * G + c) * l.dimp + o * 8;
+  // thread = four columns of up to HPT heads at a time, whose mixing weights stay in registers over the rows
+  constexpr int HPT = 2, MAX_REP = 8;
+  const int nq = l.dimp / 4, lanes = nq < ROT_THREADS ? nq : ROT_THREADS, nhb = ROT_THREADS / lanes, hb = tid / lanes;
+  if (hb >= nhb) return;
+  for (int o = tid % lanes; o < nq; o += lanes)
+    for (int h0 = hb; h0 < H; h0 += nhb * HPT) {
+      float t[HPT][MAX_REP];
 #pragma unroll
-    for (int rr = 0; rr < ROWS; ++rr) {
-      if (rr >= nrows) break;
-      const float* q = qs + rr * qn + o * 8;
-      float acc[8];
+      for (int i = 0; i < HPT; ++i)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = 0.f;
-      for (int g = 0; g < rep; ++g) {
-        float x[8];
-        load8(q + g * l.dimp, x);
+        for (int g = 0; g < MAX_REP; ++g) t[i][g] = g < rep && h0 + i * nhb < H ? mix[(h0 + i * nhb) * rep + g] : 0.f;
+      T* out = static_cast<T*>(a.q) + (((size_t)row0 * H + h0) * G + c) * l.dimp + o * 4;
+      const size_t out_row = (size_t)H * G * l.dimp, out_head = (size_t)nhb * G * l.dimp;
+      const float* q = qs + o * 4;
+      for (int rr = 0; rr < nrows; ++rr, q += qn, out += out_row) {
+        float4 acc[HPT];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(t[g], x[e], acc[e]);
+        for (int i = 0; i < HPT; ++i) acc[i] = make_float4(0, 0, 0, 0);
+        auto add = [&](float4& v, float f, const float4& x) {
+          v.x = fmaf(f, x.x, v.x); v.y = fmaf(f, x.y, v.y); v.z = fmaf(f, x.z, v.z); v.w = fmaf(f, x.w, v.w);
+        };
+#pragma unroll
+        for (int g = 0; g < MAX_REP; ++g)
+          if (g < rep) {
+            const float4 x = load4(q + g * l.dimp);
+#pragma unroll
+            for (int i = 0; i < HPT; ++i) add(acc[i], t[i][g], x);
+          }
+        for (int g = MAX_REP; g < rep; ++g) {
+          const float4 x = load4(q + g * l.dimp);
+#pragma unroll
+          for (int i = 0; i < HPT; ++i)
+            if (h0 + i * nhb < H) add(acc[i], mix[(h0 + i * nhb) * rep + g], x);
+        }
+#pragma unroll
+        for (int i = 0; i < HPT; ++i)
+          if (h0 + i * nhb < H) store4(out + i * out_head, acc[i]);
       }
-      store8(out + (size_t)rr * H * G * l.dimp, acc);
     }
-  }
 }
 
 template <typename T>
@@ -705,14 +717,14 @@ cudaError_t heads_step_t(const AttentionStepArgs& a, const StepShape& sh, int yb
 
 }  // namespace
 
-size_t rotate_smem(const AttentionLayer& l) {
+size_t rotate_smem(const AttentionLayer& l, int rows) {
   const int rep = l.heads / l.kv_heads;
-  return l.mix ? ((size_t)ROT_PORTION_ROWS * rep * l.dimp + (size_t)l.heads * rep) * sizeof(float) : 0;
+  return l.mix ? ((size_t)rows * rep * l.dimp + (size_t)l.heads * rep) * sizeof(float) : 0;
 }
 
 bool attention_heads_supported(const AttentionLayer& l) {
   StepShape sh;
-  return step_shape(l, &sh) && rotate_smem(l) <= MAX_SMEM;
+  return step_shape(l, &sh) && rotate_smem(l, 1) <= MAX_SMEM;
 }
 
 cudaError_t launch_attention_heads_step(const AttentionStepArgs& a, bool bf16, bool y_bf16, bool pdl, cudaStream_t s) {
@@ -728,16 +740,17 @@ cudaError_t launch_angles(const int* pos, const double* freq, float2* out, int r
 }
 
 cudaError_t launch_attention_rotate(const AttentionPortionArgs& a, bool bf16, cudaStream_t s, bool pdl) {
-  const size_t smem = rotate_smem(a.l);
+  int rows = a.step_pos ? 1 : ROT_MAX_ROWS;
+  while (rows > 1 && rotate_smem(a.l, rows) > 48 * 1024) rows /= 2;
+  const size_t smem = rotate_smem(a.l, rows);
   if (smem > MAX_SMEM) return cudaErrorInvalidValue;
-  const int rows = a.step_pos ? 1 : ROT_PORTION_ROWS;
-  const dim3 grid((a.rows + rows - 1) / rows, a.l.kv_heads);
+  const dim3 grid(a.l.kv_heads, (a.rows + rows - 1) / rows);  // blocks of the same rows together: their queries are neighbours
   auto run = [&](auto kernel) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
-    return e != cudaSuccess ? e : launch_kernel(kernel, grid, dim3(ROT_THREADS), smem, s, pdl, a);
+    return e != cudaSuccess ? e : launch_kernel(kernel, grid, dim3(ROT_THREADS), smem, s, pdl, a, rows);
   };
   if (a.step_pos) return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, 1>) : run(attention_rotate_kernel<float, 1>);
-  return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, ROT_PORTION_ROWS>) : run(attention_rotate_kernel<float, ROT_PORTION_ROWS>);
+  return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, 4>) : run(attention_rotate_kernel<float, 4>);
 }
 
 cudaError_t launch_attention_latent(const AttentionPortionArgs& a, bool bf16, cudaStream_t s, bool pdl) {
