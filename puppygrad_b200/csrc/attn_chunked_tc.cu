@@ -2,8 +2,8 @@
 // S and P and O in tensor memory, FP32 scores and softmax, queries / keys / values by TMA.
 //
 // Work item = 128 query rows of one head of one sequence; a persistent block takes items in turn, so that the loads and
-// first scores of an item overlap the end of the one before. Warp 0 loads, warp 1 issues the MMAs, warps 2..5 do the
-// softmax (thread = row). S(j + 1) = Q K^T is issued as soon as the softmax warps hold S(j) in registers, so that the tensor cores
+// first scores of an item overlap the end of the one before. Warp 0 loads, warp 1 issues the MMAs, warps 2..9 do the
+// softmax: two threads share a row, each with half of a tile's keys; they exchange maxima and sums through shared memory. S(j + 1) = Q K^T is issued as soon as the softmax warps hold S(j) in registers, so that the tensor cores
 // work on the next scores while those warps are busy; keys and values have rings of their own. An item walks only the key tiles that some
 // row of it can see: those of the moving range, and before them those of the sequence's kept first keys. Keys come in pieces of
 // 64 columns through a ring; where the queries of an item do not fit beside it, their pieces come with the keys', again for
@@ -28,7 +28,7 @@ __device__ __forceinline__ float exp2_fast(float x) {
   return r;
 }
 
-constexpr int MAX_KSTAGES = 8;
+constexpr int MAX_KSTAGES = 8, THREADS = 320, SOFTMAX_WARPS = 8;
 
 __device__ __forceinline__ void store8(__nv_bfloat16* p, const float* v) {
   uint32_t u[4];
@@ -74,13 +74,17 @@ struct TcItem {
   __device__ __forceinline__ int end(int j) const { return j < kept_tiles ? kept : 1 << 30; }
 };
 
-__global__ void __launch_bounds__(192, 2)
+__device__ __forceinline__ void pair_barrier(int quarter) { asm volatile("bar.sync %0, 64;" ::"r"(1 + quarter) : "memory"); }
+
+template <int PER_SM>
+__global__ void __launch_bounds__(THREADS, PER_SM)
     attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, AttentionPortionArgs a, TcShape t, int items, int qtiles) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t q_full, q_empty, k_full[MAX_KSTAGES], k_empty[MAX_KSTAGES], v_full[2], v_empty[2], s_full, s_free, p_ready, pv_done, o_free;
   __shared__ uint32_t tmem_slot;
   __shared__ int failed_flag;
+  __shared__ float row_max[2][2][QROWS], row_sum[2][2][QROWS];  // by parity of the tile (item) and side
   const AttentionLayer& l = a.l;
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint8_t* qs = base;
@@ -102,10 +106,10 @@ __global__ void __launch_bounds__(192, 2)
       mbar_init(&v_empty[i], 1);
     }
     mbar_init(&s_full, 1);
-    mbar_init(&s_free, 4);
-    mbar_init(&p_ready, 4);
+    mbar_init(&s_free, SOFTMAX_WARPS);
+    mbar_init(&p_ready, SOFTMAX_WARPS);
     mbar_init(&pv_done, 1);
-    mbar_init(&o_free, 4);
+    mbar_init(&o_free, SOFTMAX_WARPS);
     failed_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -201,44 +205,49 @@ __global__ void __launch_bounds__(192, 2)
       }
     }
   } else {
-    const int q = warp & 3, r = q * 32 + lane;
+    // on expiry these warps go on through their loops without work: the pairs' barriers need both sides
+    const int q = warp & 3, side = (warp - 2) >> 2, r = q * 32 + lane;
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
     const float scale2 = l.scale == 0.f ? 1e-30f : l.scale * LOG2E;  // never 0: the mask is an infinite score
-    for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
+    for (int it = blockIdx.x; it < items; it += gridDim.x) {
       if (!w.set(a, it, qtiles)) continue;
       const int qrow = w.q0 + r, pos = w.p0 + min(qrow, w.n - 1);
       const int lo_row = l.life.low(w.p0, pos), hi_row = l.life.row(w.p0, pos), keep = l.life.keep;
       const int lo_all = l.life.low(w.p0, w.pos_b), hi_all = l.life.row(w.p0, w.pos_a);  // keys every row sees
-      float m_ref = l.sink ? l.sink[w.head] * LOG2E : -1e30f, sum = l.sink ? 1.f : 0.f;
-      for (int j = 0; j < w.tiles && ok; ++j) {
+      float m_ref = l.sink ? l.sink[w.head] * LOG2E : -1e30f, sum = l.sink && side == 0 ? 1.f : 0.f;
+      for (int j = 0; j < w.tiles; ++j) {
         const uint32_t gt = g + j;
-        ok = __all_sync(ALL_LANES, mbar_wait(&s_full, gt & 1, failed, a.error_flag, 27));
-        if (!ok) break;
-        tc_fence_after();
-        float s[128];
+        if (ok) ok = __all_sync(ALL_LANES, mbar_wait(&s_full, gt & 1, failed, a.error_flag, 27));
+        float s[64], m_tile = -INFINITY;
+        if (ok) {
+          tc_fence_after();
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          float v[32];
-          tmem_ld32(tmem + COL_S + lane_addr + (uint32_t)(c * 32), v);
+          for (int c = 0; c < 2; ++c) {
+            float v[32];
+            tmem_ld32(tmem + COL_S + lane_addr + (uint32_t)(side * 64 + c * 32), v);
 #pragma unroll
-          for (int i = 0; i < 32; ++i) s[c * 32 + i] = v[i];
+            for (int i = 0; i < 32; ++i) s[c * 32 + i] = v[i];
+          }
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&s_free);
+          const int k0 = w.start(j) + side * 64, k1 = w.end(j);
+          if (j < w.kept_tiles ? k0 + 64 > k1 : k0 < lo_all || k0 + 63 > hi_all) {
+            const int lo_i = lo_row - k0, hi_i = min(hi_row, k1 - 1) - k0, keep_i = keep - k0;
+#pragma unroll
+            for (int i = 0; i < 64; ++i)
+              if ((i < lo_i && i >= keep_i) || i > hi_i) s[i] = scale2 < 0.f ? INFINITY : -INFINITY;
+          }
+          float mx[4];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) mx[i] = s[i] * scale2;
+#pragma unroll
+          for (int i = 4; i < 64; ++i) mx[i & 3] = fmaxf(mx[i & 3], s[i] * scale2);
+          m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
         }
-        tc_fence_before();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&s_free);
-        const int k0 = w.start(j), k1 = w.end(j);
-        if (j < w.kept_tiles ? k0 + KROWS > k1 : k0 < lo_all || k0 + KROWS - 1 > hi_all) {
-          const int lo_i = lo_row - k0, hi_i = min(hi_row, k1 - 1) - k0, keep_i = keep - k0;
-#pragma unroll
-          for (int i = 0; i < 128; ++i)
-            if ((i < lo_i && i >= keep_i) || i > hi_i) s[i] = scale2 < 0.f ? INFINITY : -INFINITY;
-        }
-        float mx[4];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) mx[i] = s[i] * scale2;
-#pragma unroll
-        for (int i = 4; i < 128; ++i) mx[i & 3] = fmaxf(mx[i & 3], s[i] * scale2);
-        const float m_tile = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+        row_max[gt & 1][side][r] = m_tile;
+        pair_barrier(q);
+        m_tile = fmaxf(m_tile, row_max[gt & 1][side ^ 1][r]);
         // the reference maximum moves only when a row's scores outgrow it by 2^8
         const bool move = __any_sync(ALL_LANES, m_tile > m_ref + 8.f);
         float corr = 1.f;
@@ -248,19 +257,20 @@ __global__ void __launch_bounds__(192, 2)
           m_ref = m_new;
           sum *= corr;
         }
+        if (!ok) continue;
         float part[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int i = 0; i < 128; ++i) {
+        for (int i = 0; i < 64; ++i) {
           s[i] = exp2_fast(fmaf(s[i], scale2, -m_ref));
           part[i & 3] += s[i];
         }
         sum += (part[0] + part[1]) + (part[2] + part[3]);
         if (j > 0) {  // P and O may be touched once O += P(j - 1) V is done (for j = 0 the wait at the end of the item before)
           ok = __all_sync(ALL_LANES, mbar_wait(&pv_done, (gt - 1) & 1, failed, a.error_flag, 28));
-          if (!ok) break;
+          if (!ok) continue;
           tc_fence_after();
           if (move) {
-            for (int c = 0; c < t.vn; c += 16) {
+            for (int c = side * 16; c < t.vn; c += 32) {
               float o[16];
               tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)c, o);
               uint32_t u[16];
@@ -272,21 +282,26 @@ __global__ void __launch_bounds__(192, 2)
         }
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-          uint32_t u[32];
+          uint32_t u[16];
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const __nv_bfloat162 b = __floats2bfloat162_rn(s[h * 64 + 2 * i], s[h * 64 + 2 * i + 1]);
+          for (int i = 0; i < 16; ++i) {
+            const __nv_bfloat162 b = __floats2bfloat162_rn(s[h * 32 + 2 * i], s[h * 32 + 2 * i + 1]);
             u[i] = *reinterpret_cast<const uint32_t*>(&b);
           }
-          tmem_st32(tmem + COL_P + lane_addr + (uint32_t)(h * 32), u);
+          tmem_st16(tmem + COL_P + lane_addr + (uint32_t)(side * 32 + h * 16), u);
         }
         tmem_wait_st();
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&p_ready);
       }
+      row_sum[done & 1][side][r] = sum;
+      pair_barrier(q);
+      sum += row_sum[done & 1][side ^ 1][r];
       if (ok) ok = __all_sync(ALL_LANES, mbar_wait(&pv_done, (g + w.tiles - 1) & 1, failed, a.error_flag, 29));
-      if (!ok) break;
+      g += w.tiles;
+      ++done;
+      if (!ok) continue;
       tc_fence_after();
       float inv = l.out_scale / sum;
       if (l.off_gate >= 0 && qrow < w.n) inv *= sigmoid_f(a.p[(size_t)(w.first + qrow) * a.ldp + l.off_gate + w.head]);
@@ -296,15 +311,10 @@ __global__ void __launch_bounds__(192, 2)
         const int half = l.vdim >> 1;
         const float2* cs = a.v_rot + (size_t)(w.first + min(qrow, w.n - 1)) * half;
         const bool vec2 = vec && half % 8 == 0;
-        for (int c = 0; c < half; c += 16) {
+        for (int c = side * 16; c < half; c += 32) {
           float u[16], v[16];
           tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)c, u);
           tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)(half + c), v);
-          if (c + 16 >= half) {
-            tc_fence_before();
-            __syncwarp();
-            if (lane == 0) mbar_arrive(&o_free);
-          }
           if (qrow < w.n) {
 #pragma unroll
             for (int i = 0; i < 16; ++i)
@@ -332,18 +342,14 @@ __global__ void __launch_bounds__(192, 2)
           }
           __syncwarp();
         }
-        g += w.tiles;
-        ++done;
+        tc_fence_before();  // this side's columns of O are in registers or stored: the next item may overwrite them
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&o_free);
         continue;
       }
-      for (int c = 0; c < t.vn; c += 16) {
+      for (int c = side * 16; c < t.vn; c += 32) {
         float o[16];
         tmem_ld16(tmem + COL_O + lane_addr + (uint32_t)c, o);
-        if (c + 16 >= t.vn) {  // all of O is in registers or stored: the next item may overwrite it
-          tc_fence_before();
-          __syncwarp();
-          if (lane == 0) mbar_arrive(&o_free);
-        }
         if (qrow >= w.n) {  // a row of the next sequence or none: nothing to store
         } else if (vec) {
 #pragma unroll
@@ -360,8 +366,9 @@ __global__ void __launch_bounds__(192, 2)
         }
         __syncwarp();
       }
-      g += w.tiles;
-      ++done;
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&o_free);
     }
   }
   tc_fence_before();
@@ -382,7 +389,7 @@ bool make_head_map(CUtensorMap* map, const void* ptr, uint64_t rows, uint64_t he
             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-constexpr size_t TC_MAX_SMEM = 225 * 1024;
+constexpr size_t TC_MAX_SMEM = 222 * 1024;  // beside the static arrays
 
 }  // namespace
 
@@ -419,15 +426,15 @@ cudaError_t launch_attention_tc(const AttentionPortionArgs& a, cudaStream_t s) {
   if (!make_head_map(&mq, a.q, a.rows, l.heads, width, (uint64_t)l.heads * width) || !make_head_map(&mk, a.k, a.krows, key_heads, width, a.ldk) ||
       !make_head_map(&mv, a.v, a.krows, l.kv_heads, l.vdimp, a.ldv))
     return cudaErrorInvalidValue;
-  cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_MAX_SMEM);
-  if (e != cudaSuccess) return e;
   const int qtiles = (a.max_len + QROWS - 1) / QROWS, items = qtiles * l.heads * a.nseq;
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-  const int per_sm = t.tmem_cols <= 256 && bytes() <= 110 * 1024 ? 2 : 1;
-  return launch_kernel(attention_tc_kernel, dim3(std::min(items, sms * per_sm)), dim3(192), bytes(), s, false, mq, mk, mv, a, t, items,
-                       qtiles);
+  auto run = [&](auto kernel, int per_sm) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC_MAX_SMEM);
+    return e != cudaSuccess ? e : launch_kernel(kernel, dim3(std::min(items, sms * per_sm)), dim3(THREADS), bytes(), s, false, mq, mk, mv, a, t, items, qtiles);
+  };
+  return t.tmem_cols <= 256 && bytes() <= 108 * 1024 ? run(attention_tc_kernel<2>, 2) : run(attention_tc_kernel<1>, 1);
 }
 
 }  // namespace pg
