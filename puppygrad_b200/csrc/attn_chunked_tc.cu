@@ -125,31 +125,31 @@ __global__ void __launch_bounds__(THREADS, PER_SM)
   if (warp == 0) {
     if (lane == 0) {
       const int key_head = l.mix ? 0 : 1;  // mixed heads: all key heads are one wide row
-      uint32_t kp = 0;                     // pieces of keys before the current one
+      RingCursor kr, vr;
       for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
         if (!w.set(a, it, qtiles)) continue;
         if (t.q_resident) {
-          if (done > 0) ok = mbar_wait(&q_empty, (done - 1) & 1, failed, a.error_flag, 20);
+          ok = mbar_wait(&q_empty, (done & 1) ^ 1, failed, a.error_flag, 20);
           if (!ok) break;
           mbar_expect_tx(&q_full, t.dpieces * PIECE);
           for (int d = 0; d < t.dpieces; ++d) tma_load_3d(qs + (size_t)d * PIECE, &map_q, d * 64, w.head, w.first + w.q0, &q_full);
         }
+        const int key0 = a.key_start[w.seq], kh = key_head * w.kvh;
         for (int j = 0; j < w.tiles && ok; ++j) {
-          const int krow = a.key_start[w.seq] + w.start(j);
-          const uint32_t gt = g + j, v = gt % t.vstages;
-          for (int d = 0; d < t.dpieces; ++d, ++kp) {
-            const uint32_t s = kp % t.kstages;
-            if (kp >= (uint32_t)t.kstages) ok = mbar_wait(&k_empty[s], ((kp / t.kstages) - 1) & 1, failed, a.error_flag, 21);
+          const int krow = key0 + w.start(j);
+          for (int d = 0; d < t.dpieces; ++d, kr.next(t.kstages)) {
+            ok = mbar_wait(&k_empty[kr.stage], kr.parity ^ 1, failed, a.error_flag, 21);
             if (!ok) break;
-            mbar_expect_tx(&k_full[s], kstage_bytes);
-            tma_load_3d(ks + (size_t)s * kstage_bytes, &map_k, d * 64, key_head * w.kvh, krow, &k_full[s]);
-            if (!t.q_resident) tma_load_3d(ks + (size_t)s * kstage_bytes + PIECE, &map_q, d * 64, w.head, w.first + w.q0, &k_full[s]);
+            uint8_t* dst = ks + kr.stage * kstage_bytes;
+            mbar_expect_tx(&k_full[kr.stage], kstage_bytes);
+            tma_load_3d(dst, &map_k, d * 64, kh, krow, &k_full[kr.stage]);
+            if (!t.q_resident) tma_load_3d(dst + PIECE, &map_q, d * 64, w.head, w.first + w.q0, &k_full[kr.stage]);
           }
+          if (ok) ok = mbar_wait(&v_empty[vr.stage], vr.parity ^ 1, failed, a.error_flag, 22);
           if (!ok) break;
-          if (gt >= (uint32_t)t.vstages) ok = mbar_wait(&v_empty[v], ((gt / t.vstages) - 1) & 1, failed, a.error_flag, 22);
-          if (!ok) break;
-          mbar_expect_tx(&v_full[v], t.vpieces * PIECE);
-          for (int d = 0; d < t.vpieces; ++d) tma_load_3d(vs + (size_t)(v * t.vpieces + d) * PIECE, &map_v, d * 64, w.kvh, krow, &v_full[v]);
+          mbar_expect_tx(&v_full[vr.stage], t.vpieces * PIECE);
+          for (int d = 0; d < t.vpieces; ++d) tma_load_3d(vs + (vr.stage * t.vpieces + d) * PIECE, &map_v, d * 64, w.kvh, krow, &v_full[vr.stage]);
+          vr.next(t.vstages);
         }
         g += w.tiles;
         ++done;
@@ -158,18 +158,19 @@ __global__ void __launch_bounds__(THREADS, PER_SM)
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc_bf16(QROWS, KROWS), idesc_o = umma_idesc_bf16(QROWS, t.vn, true);
-      uint32_t kp = 0;
+      RingCursor kr, vr;
+      const uint64_t q_desc = umma_desc_sw128(qs), k_desc = umma_desc_sw128(ks), v_desc = umma_desc_mn_sw128(vs, PIECE);
+      const uint32_t kstage16 = kstage_bytes >> 4, vstage16 = (uint32_t)t.vpieces * (PIECE >> 4);
       auto scores = [&](bool last) -> bool {
-        for (int d = 0; d < t.dpieces; ++d, ++kp) {
-          const uint32_t s = kp % t.kstages;
-          if (!mbar_wait(&k_full[s], (kp / t.kstages) & 1, failed, a.error_flag, 23)) return false;
+        for (int d = 0; d < t.dpieces; ++d, kr.next(t.kstages)) {
+          if (!mbar_wait(&k_full[kr.stage], kr.parity, failed, a.error_flag, 23)) return false;
           tc_fence_after();
-          const uint8_t* kt = ks + (size_t)s * kstage_bytes;
-          const uint8_t* qt = t.q_resident ? qs + (size_t)d * PIECE : kt + PIECE;
-          const int steps = min(4, t.ksteps - d * 4);
-          for (int k = 0; k < steps; ++k)
-            umma_bf16_ss(tmem + COL_S, umma_desc_sw128(qt) + (uint64_t)(k * 2), umma_desc_sw128(kt) + (uint64_t)(k * 2), idesc_s, (d | k) != 0);
-          umma_commit(&k_empty[s]);
+          const uint64_t dk = k_desc + kr.stage * kstage16, dq = t.q_resident ? q_desc + (uint32_t)d * (PIECE >> 4) : dk + (PIECE >> 4);
+          const int steps = t.ksteps - d * 4;
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (k < steps) umma_bf16_ss(tmem + COL_S, dq + (uint64_t)(k * 2), dk + (uint64_t)(k * 2), idesc_s, (d | k) != 0);
+          umma_commit(&k_empty[kr.stage]);
         }
         if (last && t.q_resident) umma_commit(&q_empty);
         umma_commit(&s_full);
@@ -189,15 +190,16 @@ __global__ void __launch_bounds__(THREADS, PER_SM)
           ok = ok && mbar_wait(&p_ready, gt & 1, failed, a.error_flag, 25);  // P is written
           if (!ok) break;
           tc_fence_after();
-          const uint32_t v = gt % t.vstages;
-          ok = ok && mbar_wait(&v_full[v], (gt / t.vstages) & 1, failed, a.error_flag, 26);
+          ok = ok && mbar_wait(&v_full[vr.stage], vr.parity, failed, a.error_flag, 26);
           if (ok && j == 0 && done > 0) ok = mbar_wait(&o_free, (done - 1) & 1, failed, a.error_flag, 30);  // O of the item before has been read
           if (!ok) break;
           tc_fence_after();
+          const uint64_t dv = v_desc + vr.stage * vstage16;
+#pragma unroll
           for (int k = 0; k < KROWS / 16; ++k)
-            umma_bf16_ts(tmem + COL_O, tmem + COL_P + (uint32_t)(k * 8),
-                         umma_desc_mn_sw128(vs + (size_t)v * t.vpieces * PIECE + (size_t)k * 2048, PIECE), idesc_o, (j | k) != 0);
-          umma_commit(&v_empty[v]);
+            umma_bf16_ts(tmem + COL_O, tmem + COL_P + (uint32_t)(k * 8), dv + (uint64_t)(k * (2048 >> 4)), idesc_o, (j | k) != 0);
+          umma_commit(&v_empty[vr.stage]);
+          vr.next(t.vstages);
           umma_commit(&pv_done);
         }
         g += w.tiles;

@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(192, 1)
   const int all = (n + ROWS - 1) / ROWS, t0 = all * split / a.splits, t1 = all * (split + 1) / a.splits;
   const int kv0 = l.mix ? h0 / (l.heads / l.kv_heads) : 0;  // first key head whose values are needed
   bool ok = true;
-  uint32_t st = 0;  // stages before the current one: both sides count them alike
+  RingCursor ring_at;
 
   if (warp == 0) {
     if (t0 < t1) {
@@ -113,11 +113,11 @@ __global__ void __launch_bounds__(192, 1)
         for (int part = 0; part < (t.reuse ? 1 : 2) && ok; ++part) {
           const CUtensorMap* map = part == 0 ? &map_k : &map_v;
           const int pieces = part == 0 ? t.kpieces : t.vpieces, x0 = part == 0 ? 0 : kv0 * l.vdimp;
-          for (int d = 0; d < pieces; d += 2, ++st) {
-            const uint32_t s = st % t.stages;
+          for (int d = 0; d < pieces; d += 2, ring_at.next(t.stages)) {
+            const uint32_t s = ring_at.stage;
             const int two = min(2, pieces - d);
             if (lane == 0) {
-              if (st >= (uint32_t)t.stages) ok = mbar_wait(&empty[s], ((st / t.stages) - 1) & 1, failed, a.error_flag, 61);
+              ok = mbar_wait(&empty[s], ring_at.parity ^ 1, failed, a.error_flag, 61);
               if (ok) mbar_expect_tx(&full[s], (uint32_t)two * PIECE);
             }
             ok = __shfl_sync(ALL_LANES, ok ? 1 : 0, 0) != 0;
@@ -133,37 +133,42 @@ __global__ void __launch_bounds__(192, 1)
     if (lane == 0 && t0 < t1) {
       const uint32_t idesc_s = umma_idesc_bf16(ROWS, t.npad), idesc_o = umma_idesc_bf16(ROWS, t.npad) | (1u << 15);  // A of O^T is MN-major
       const int ksteps = (attention_q_width(l) + 15) / 16;
+      const uint64_t k_desc = umma_desc_sw128(ring), v_desc = umma_desc_mn_sw128(ring, PIECE), q_desc = umma_desc_sw128(qs), p_desc = umma_desc_sw128(ps);
+      const uint32_t hpiece16 = hpiece >> 4;
       ok = mbar_wait(&q_full, 0, failed, a.error_flag, 62);
       for (int tile = t0; tile < t1 && ok; ++tile) {
-        const uint32_t turn = (uint32_t)(tile - t0), first = st;
-        for (int d = 0; d < t.kstages; ++d, ++st) {
-          const uint32_t s = st % t.stages;
-          ok = mbar_wait(&full[s], (st / t.stages) & 1, failed, a.error_flag, 63);
+        const uint32_t turn = (uint32_t)(tile - t0);
+        RingCursor first = ring_at;
+        for (int d = 0; d < t.kstages; ++d, ring_at.next(t.stages)) {
+          ok = mbar_wait(&full[ring_at.stage], ring_at.parity, failed, a.error_flag, 63);
           if (!ok) break;
           tc_fence_after();
-          const int steps = min(8, ksteps - d * 8);
-          for (int k = 0; k < steps; ++k)
-            umma_bf16_ss(tmem, umma_desc_sw128(ring + (size_t)s * STAGE + (k >> 2) * PIECE) + (uint64_t)((k & 3) * 2),
-                         umma_desc_sw128(qs + (size_t)(d * 2 + (k >> 2)) * hpiece) + (uint64_t)((k & 3) * 2), idesc_s, (d | k) != 0);
-          if (!t.reuse) umma_commit(&empty[s]);
+          const uint64_t dk = k_desc + ring_at.stage * (STAGE >> 4), dq = q_desc + (uint32_t)(2 * d) * hpiece16;
+          const int steps = ksteps - d * 8;
+#pragma unroll
+          for (int k = 0; k < 8; ++k)
+            if (k < steps)
+              umma_bf16_ss(tmem, dk + (uint64_t)((k >> 2) * (PIECE >> 4) + (k & 3) * 2), dq + (uint64_t)((k >> 2) * hpiece16 + (k & 3) * 2), idesc_s, (d | k) != 0);
+          if (!t.reuse) umma_commit(&empty[ring_at.stage]);
         }
         if (!ok) break;
         umma_commit(&s_full);
         ok = mbar_wait(&p_ready, turn & 1, failed, a.error_flag, 64);  // P is in shared memory, S has been read, O is rescaled
         if (!ok) break;
         tc_fence_after();
-        uint32_t v = t.reuse ? first : st;
-        for (int d = 0; d < t.vstages; ++d, ++v) {
-          const uint32_t s = v % t.stages;
-          if (!t.reuse) ok = mbar_wait(&full[s], (v / t.stages) & 1, failed, a.error_flag, 65);
+        RingCursor v = t.reuse ? first : ring_at;
+        for (int d = 0; d < t.vstages; ++d, v.next(t.stages)) {
+          if (!t.reuse) ok = mbar_wait(&full[v.stage], v.parity, failed, a.error_flag, 65);
           if (!ok) break;
           tc_fence_after();
+          const uint64_t dv = v_desc + v.stage * (STAGE >> 4);
+#pragma unroll
           for (int k = 0; k < ROWS / 16; ++k)
-            umma_bf16_ss(tmem_o + (uint32_t)(d * t.npad), umma_desc_mn_sw128(ring + (size_t)s * STAGE + (size_t)k * 2048, PIECE),
-                         umma_desc_sw128(ps + (size_t)(k >> 2) * hpiece) + (uint64_t)((k & 3) * 2), idesc_o, turn != 0 || k != 0);
-          umma_commit(&empty[s]);
+            umma_bf16_ss(tmem_o + (uint32_t)(d * t.npad), dv + (uint64_t)(k * (2048 >> 4)), p_desc + (uint64_t)((k >> 2) * hpiece16 + (k & 3) * 2), idesc_o,
+                         turn != 0 || k != 0);
+          umma_commit(&empty[v.stage]);
         }
-        st = v;
+        ring_at = v;
         if (ok) umma_commit(&pv_done);
       }
     }

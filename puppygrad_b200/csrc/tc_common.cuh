@@ -49,6 +49,18 @@ __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, volati
   return false;
 }
 
+// Stage and pass parity of a ring of buffers, advanced without divisions. A producer waits for `empty` with parity ^ 1, which a
+// fresh barrier passes; a consumer for `full` with parity.
+struct RingCursor {
+  uint32_t stage = 0, parity = 0;
+  __device__ __forceinline__ void next(uint32_t stages) {
+    if (++stage == stages) {
+      stage = 0;
+      parity ^= 1;
+    }
+  }
+};
+
 __device__ __forceinline__ void tma_load_2d(void* smem_dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
   asm volatile(
       "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
