@@ -85,6 +85,7 @@ struct LayeredModel {
   int max_mid_k = 0, max_mid = 0, max_latent = 0, max_wide = 0;  // widest second-step input and output; heads * latent row, heads * query
   int n_pools = 0, n_states = 0;
   bool tc_rotations = false;  // a step needs the angles of its rows
+  bool channel_rules = false;  // some recurrence is a channel delta rule
   std::vector<KeyLife> lives;  // one page table each
   std::vector<Rotation> rotations;
   std::vector<void*> allocations;
@@ -127,12 +128,13 @@ struct LayeredCache {
   float* attn_part = nullptr;
   unsigned* attn_counters = nullptr;
   // portion workspaces (grow-only)
-  float *decay = nullptr, *unit = nullptr, *rate = nullptr, *unit_next = nullptr, *pair = nullptr, *out_raw = nullptr, *segments = nullptr, *vals = nullptr;
+  float *decay = nullptr, *unit = nullptr, *rate = nullptr, *unit_next = nullptr, *pair = nullptr, *out_raw = nullptr, *segments = nullptr, *vals = nullptr, *writes = nullptr, *quad_decay = nullptr,
+        *quads = nullptr;
   float2* angles = nullptr;
   void *q = nullptr, *k = nullptr, *v = nullptr;
   int* meta = nullptr;
   float* logits = nullptr;
-  size_t q_rows = 0, k_rows = 0, seg_floats = 0, meta_ints = 0, logit_rows = 0, gate_rows = 0, angle_rows = 0;
+  size_t q_rows = 0, k_rows = 0, seg_floats = 0, meta_ints = 0, logit_rows = 0, gate_rows = 0, angle_rows = 0, channel_rows = 0, quad_rows = 0;
   ~LayeredCache() {
     for (void* p : pools) cudaFree(p);
     for (float* p : states) cudaFree(p);
@@ -141,7 +143,7 @@ struct LayeredCache {
     for (LayeredRows* r : {&step, &portion})
       for (void** p : r->buffers())
         if (*p) cudaFree(*p);
-    for (void* p : {(void*)attn_part, (void*)attn_counters, (void*)decay, (void*)unit, (void*)rate, (void*)unit_next, (void*)pair, (void*)out_raw, (void*)segments, (void*)vals, (void*)angles, q, k, v,
+    for (void* p : {(void*)attn_part, (void*)attn_counters, (void*)decay, (void*)unit, (void*)rate, (void*)unit_next, (void*)pair, (void*)out_raw, (void*)segments, (void*)vals, (void*)writes, (void*)quad_decay, (void*)quads, (void*)angles, q, k, v,
                     (void*)meta, (void*)logits})
       if (p) cudaFree(p);
   }
@@ -430,6 +432,7 @@ int build_layer(Builder& b, const LayerSpec& spec, const std::string& p, int pag
         std::copy(g2.begin() + (size_t)i * s.rank2, g2.begin() + (size_t)(i + 1) * s.rank2,
                   mid.begin() + (size_t)(K + i) * br.mid_cols + br.mid_cols - s.rank2);
       if (int r = b.matrix(mid, K + V, br.mid_cols, N_ALIGN, &br.mid)) return r;
+      m->channel_rules = true;
       br.state = m->n_states++;
       m->max_rec = std::max(m->max_rec, K);
       m->max_rec_out = std::max(m->max_rec_out, V);
@@ -1114,6 +1117,7 @@ cudaError_t enqueue_portions(pg_cache* c, const PortionPlan& plan, const Portion
         RecurrenceScanArgs a{};
         a.l = b.rec; a.p = r.p; a.ldp = l.ldp; a.rows = rows; a.nseq = plan.n(); a.row_seq = d.row_seq;
         a.z = r.z; a.ldz = b.mid.np; a.taps = lc->taps[b.state]; a.vals = lc->vals;
+        a.max_len = plan.max_len; a.writes = lc->writes; a.quad_decay = lc->quad_decay; a.quads = lc->quads;
         a.seq_start = d.seq_start; a.seq_slot = d.slot; a.seq_pos = d.start_pos; a.state = lc->states[b.state];
         a.decay = lc->decay; a.unit = lc->unit; a.rate = lc->rate; a.unit_next = lc->unit_next; a.pair = lc->pair;
         a.out_raw = lc->out_raw; a.error_flag = c->d_error;
@@ -1196,14 +1200,26 @@ int layered_run_portions(pg_cache* c, const PortionPlan& plan, float* logits, St
     }
   }
   if (m->max_rec && (size_t)rows > lc->gate_rows) {
-    size_t g = lc->gate_rows, h = g, o = g, x = g, y = g, z = g;
-    if (int r = grow(&lc->vals, &z, rows, m->max_rec_out * sizeof(float))) return r;
+    size_t g = lc->gate_rows, h = g, o = g, x = g, y = g;
     if (int r = grow(&lc->unit_next, &x, rows, m->max_rec * sizeof(float))) return r;
     if (int r = grow(&lc->pair, &y, rows, m->max_rec_heads * 4 * sizeof(float))) return r;
     if (int r = grow(&lc->out_raw, &o, rows, m->max_rec_out * sizeof(float))) return r;
     if (int r = grow(&lc->decay, &g, rows, m->max_rec * sizeof(float))) return r;
     if (int r = grow(&lc->unit, &h, rows, m->max_rec * sizeof(float))) return r;
     if (int r = grow(&lc->rate, &lc->gate_rows, rows, m->max_rec * sizeof(float))) return r;
+  }
+  if (m->channel_rules) {
+    if ((size_t)rows > lc->channel_rows) {
+      size_t v = lc->channel_rows;
+      if (int r = grow(&lc->vals, &v, rows, m->max_rec_out * sizeof(float))) return r;
+      if (int r = grow(&lc->writes, &lc->channel_rows, rows, m->max_rec * sizeof(float))) return r;
+    }
+    const size_t quads = recurrence_quads(rows, ns);
+    if (quads > lc->quad_rows) {
+      size_t d = lc->quad_rows;
+      if (int r = grow(&lc->quad_decay, &d, quads, m->max_rec * sizeof(float))) return r;
+      if (int r = grow(&lc->quads, &lc->quad_rows, quads, (size_t)m->max_rec_heads * 20 * sizeof(float))) return r;
+    }
   }
   if (seg)
     if (int r = grow(&lc->segments, &lc->seg_floats, seg, sizeof(float))) return r;

@@ -144,11 +144,15 @@ struct RecurrenceScanArgs {  // whole portions of `nseq` sequences
   const float* z;        // channel: as in RecurrenceStepArgs
   int ldz;
   float* taps;
-  float* vals;           // channel: [rows, heads * vdim] scratch, values after the convolution (unit and rate hold k and q)
+  int max_len;           // longest portion
+  // channel: scratch. Values after the convolution (unit and rate hold k and q, decay and unit_next what reads the state), writes
+  // into the state, decay of four tokens and their numbers (see recurrence_scan.cu)
+  float *vals, *writes;  // [rows, heads * vdim], [rows, heads * dim]
+  float *quad_decay, *quads;  // [recurrence_quads()][heads * dim], [recurrence_quads()][heads][20]
   float* state;
   float *decay, *unit, *rate;  // [rows, heads * dim] scratch: decay; delta: unit key u, a * u ...
   float *unit_next;            // ... and the next token's u times this token's decay
-  float *pair;                 // [rows, heads, 4] delta: next u . (a * u), next u . k; channel: next k * decay . k, beta
+  float *pair;                 // [rows, heads, 4] delta: next u . (a * u), next u . k
   int* error_flag;
   float* out_raw;              // [rows, heads * vdim] scratch: outputs before the head norm
   float* segments;             // scratch of the segmented scan (may be nullptr)
@@ -158,6 +162,7 @@ struct RecurrenceScanArgs {  // whole portions of `nseq` sequences
 };
 // Whether a portion is cut into segments that run side by side (long sequences that alone would not fill the chip).
 bool recurrence_use_segments(const RecurrenceLayer& l, int nseq, int max_len, int max_segs);
+inline size_t recurrence_quads(int rows, int nseq) { return (size_t)rows / 4 + nseq + 1; }
 size_t recurrence_segment_floats(const RecurrenceLayer& l, int nseq, int max_segs);
 cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cudaStream_t s);
 

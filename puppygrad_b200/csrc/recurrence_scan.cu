@@ -256,80 +256,86 @@ __global__ void __launch_bounds__(256) channel_conv_vec_kernel(RecurrenceScanArg
   }
 }
 
-// Channel delta rule, after the convolutions: the decays, and what the scan needs to take two tokens at a time: the next
-// token's k times its decay . this one's k, and the write strength. A warp takes a head over GATE_GROUP rows (and looks at
-// the row behind them).
-constexpr int GATE_GROUP = 8;
+// Channel delta rule, after the convolutions. The scan takes QUAD tokens at a time from the state S before them. With D_ij the
+// product of the decays of tokens j + 1..i of a quad and P_i that of tokens 0..i, token i reads S through A_i = P_i k_i and
+// answers through Q_i = P_i q_i, and the four writes u_j become
+//   u_i = beta_i (v_i - A_i^T S - sum_{j < i} c_ij u_j),  out_i = Q_i^T S + sum_{j <= i} r_ij u_j,  S = W S + sum_j B_j u_j^T
+// with c_ij = k_i . D_ij k_j, r_ij = q_i . D_ij k_j, B_j = D_3j k_j, W = P_3. Quads are counted from a portion's first row; tokens
+// past its end count as decay 1 and zeros. A warp makes the rows and numbers of one head of one quad.
+constexpr int QUAD = 4, QUAD_NUMBERS = 20;  // c (6), r (10), beta (4)
+__device__ __forceinline__ size_t first_quad(const RecurrenceScanArgs& a, int seq) { return (size_t)(a.seq_start[seq] / QUAD + seq); }
 template <int NE>
-__global__ void __launch_bounds__(256) channel_gates_kernel(RecurrenceScanArgs a) {
+__global__ void __launch_bounds__(256) channel_quads_kernel(RecurrenceScanArgs a) {
   const RecurrenceLayer& l = a.l;
-  const int lane = threadIdx.x & 31, K = l.heads * l.dim, rep = l.heads / l.kv_heads;
-  const int groups = (a.rows + GATE_GROUP - 1) / GATE_GROUP;
+  const int lane = threadIdx.x & 31, K = l.heads * l.dim, rep = l.heads / l.kv_heads, kv_pitch = l.kv_heads * l.dim;
+  const int seq = blockIdx.y, first = a.seq_start[seq], len = a.seq_start[seq + 1] - first;
   const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  if (w >= (long long)groups * l.heads) return;
-  const int r0 = (int)(w / l.heads) * GATE_GROUP, head = (int)(w % l.heads), end = min(r0 + GATE_GROUP, a.rows);
-  const int kv_pitch = l.kv_heads * l.dim;
-  float last[NE];
+  const int quad = (int)(w / l.heads), head = (int)(w % l.heads);
+  if (quad * QUAD >= len) return;
+  const int r0 = first + quad * QUAD, n = min(QUAD, len - quad * QUAD);
+  const float beta = lane < n ? sigmoid_f(a.p[(size_t)(r0 + lane) * a.ldp + l.off_b + head]) : 0.f;
+  float wd[QUAD][NE], k[QUAD][NE], q[QUAD][NE], sums[16];
 #pragma unroll
-  for (int i = 0; i < NE; ++i) last[i] = 0.f;
-  for (int r = r0; r <= end && r < a.rows; ++r) {
-    float dot = 0.f;
+  for (int t = 0; t < QUAD; ++t)
 #pragma unroll
     for (int i = 0; i < NE; ++i) {
       const int c = lane + i * 32;
-      if (c < l.dim) {
-        const float d = channel_decay(l, head, head * l.dim + c, a.z[(size_t)r * a.ldz + head * l.dim + c]);
-        const float k = a.unit[(size_t)r * kv_pitch + head / rep * l.dim + c];
-        if (r < end) a.decay[(size_t)r * K + head * l.dim + c] = d;
-        dot = fmaf(d * k, last[i], dot);
-        last[i] = k;
+      const bool on = t < n && c < l.dim;
+      const size_t r = r0 + t;
+      wd[t][i] = on ? a.z[r * a.ldz + head * l.dim + c] : 0.f;
+      k[t][i] = on ? a.unit[r * kv_pitch + head / rep * l.dim + c] : 0.f;
+      q[t][i] = on ? a.rate[r * kv_pitch + head / rep * l.dim + c] : 0.f;
+    }
+#pragma unroll
+  for (int i = 0; i < 16; ++i) sums[i] = 0.f;
+  const size_t quad_at = first_quad(a, seq) + quad;
+#pragma unroll
+  for (int i = 0; i < NE; ++i) {
+    const int c = lane + i * 32;
+    const bool in = c < l.dim;
+    const float b = in ? l.b2[head * l.dim + c] : 0.f, na = l.neg_a[head];
+#pragma unroll
+    for (int t = 0; t < QUAD; ++t) wd[t][i] = in && t < n ? expf(na * softplus_f(wd[t][i] + b)) : 1.f;
+    float p = 1.f, rest = 1.f;
+#pragma unroll
+    for (int t = 0; t < QUAD; ++t) {
+      p *= wd[t][i];
+      float d = 1.f;
+#pragma unroll
+      for (int j = t; j >= 0; --j) {
+        const float dk = d * k[j][i];
+        sums[6 + t * (t + 1) / 2 + j] = fmaf(q[t][i], dk, sums[6 + t * (t + 1) / 2 + j]);
+        if (j < t) sums[t * (t - 1) / 2 + j] = fmaf(k[t][i], dk, sums[t * (t - 1) / 2 + j]);
+        d *= wd[j][i];
+      }
+      if (in && t < n) {
+        const size_t at = (size_t)(r0 + t) * K + head * l.dim + c;
+        a.decay[at] = p * k[t][i];
+        a.unit_next[at] = p * q[t][i];
       }
     }
-    dot = lane_sum(dot);
-    if (lane == 0 && r > r0) a.pair[((size_t)(r - 1) * l.heads + head) * 4] = dot;
-    if (lane == 0 && r < end) a.pair[((size_t)r * l.heads + head) * 4 + 1] = sigmoid_f(a.p[(size_t)r * a.ldp + l.off_b + head]);
-  }
-}
-
-// The same for heads of at most 128 channels, a multiple of four: the rows of a group are requested together.
-__global__ void __launch_bounds__(256) channel_gates_vec_kernel(RecurrenceScanArgs a) {
-  const RecurrenceLayer& l = a.l;
-  const int lane = threadIdx.x & 31, K = l.heads * l.dim, rep = l.heads / l.kv_heads;
-  const int groups = (a.rows + GATE_GROUP - 1) / GATE_GROUP;
-  const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  if (w >= (long long)groups * l.heads) return;
-  const int r0 = (int)(w / l.heads) * GATE_GROUP, head = (int)(w % l.heads), c = lane * 4;
-  const bool on = c < l.dim;
-  const size_t ch = (size_t)head * l.dim + (on ? c : 0);
-  const float* kp = a.unit + head / rep * l.dim + (on ? c : 0);
-  float4 z[GATE_GROUP + 1], k[GATE_GROUP + 1];
+    if (in) a.quad_decay[quad_at * K + head * l.dim + c] = p;
 #pragma unroll
-  for (int j = 0; j <= GATE_GROUP; ++j) {
-    const int r = min(r0 + j, a.rows - 1);
-    z[j] = load4(a.z + (size_t)r * a.ldz + ch);
-    k[j] = load4(kp + (size_t)r * l.kv_heads * l.dim);
-  }
-  const float beta = lane < GATE_GROUP && r0 + lane < a.rows ? a.p[(size_t)(r0 + lane) * a.ldp + l.off_b + head] : 0.f;
-  const float4 b = load4(l.b2 + ch);
-  const float na = l.neg_a[head];
-  auto decay = [&](float v, float bias) { return expf(na * softplus_f(v + bias)); };
-  float dots[GATE_GROUP];
-#pragma unroll
-  for (int j = 0; j <= GATE_GROUP; ++j) {
-    const float4 d = make_float4(decay(z[j].x, b.x), decay(z[j].y, b.y), decay(z[j].z, b.z), decay(z[j].w, b.w));
-    if (j < GATE_GROUP && on && r0 + j < a.rows) store4(a.decay + (size_t)(r0 + j) * K + ch, d);
-    if (j > 0) {
-      const float4 o = k[j - 1], q = k[j];
-      dots[j - 1] = on ? (d.x * q.x * o.x + d.y * q.y * o.y) + (d.z * q.z * o.z + d.w * q.w * o.w) : 0.f;
+    for (int t = QUAD - 1; t >= 0; --t) {
+      if (in && t < n) a.writes[(size_t)(r0 + t) * K + head * l.dim + c] = rest * k[t][i];
+      rest *= wd[t][i];
     }
   }
+  // sums over the lanes: lane l ends with that of number l >> 1
 #pragma unroll
-  for (int j = 0; j < GATE_GROUP; ++j) dots[j] = lane_sum(dots[j]);
-  float mine = 0.f;
+  for (int o = 16, m = 8; o > 1; o >>= 1, m >>= 1) {
+    const bool up = lane & o;
 #pragma unroll
-  for (int j = 0; j < GATE_GROUP; ++j) mine = lane == j ? dots[j] : mine;
-  if (lane < GATE_GROUP && r0 + lane < a.rows)
-    *reinterpret_cast<float2*>(a.pair + ((size_t)(r0 + lane) * l.heads + head) * 4) = make_float2(mine, sigmoid_f(beta));
+    for (int i = 0; i < 8; ++i)
+      if (i < m) {
+        const float send = up ? sums[i] : sums[i + m], keep = up ? sums[i + m] : sums[i];
+        sums[i] = keep + __shfl_xor_sync(ALL_LANES, send, o);
+      }
+  }
+  const float total = sums[0] + __shfl_xor_sync(ALL_LANES, sums[0], 1);
+  float* out = a.quads + (quad_at * l.heads + head) * QUAD_NUMBERS;
+  if ((lane & 1) == 0) out[lane >> 1] = total;
+  if (lane < QUAD) out[16 + lane] = beta;
 }
 
 // The inputs that the next tokens' convolutions still need. Block = (sequence, one of its last taps - 1 rows).
@@ -407,16 +413,15 @@ struct GroupSum<N, 0> {
   static __device__ __forceinline__ void run(float*, int) {}
 };
 
-// The delta rules work on two tokens at a time: with e = (u' * w)^T S, where the dash marks the second token,
+// The delta rule works on two tokens at a time: with e = (u' * w)^T S, where the dash marks the second token,
 // u'^T S_t = e - (u' . b) d + (u' . k) v, so that both reads come from one reduction over the state before the pair.
-// Channel delta rule: u = w * k reads, and k x (beta (v - u^T S)) is written.
 template <int KIND, int RPL, int CPL>
 __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kernel(ScanArgs sa) {
   extern __shared__ __align__(16) float sm[];
   __shared__ uint64_t full[SCAN_STAGES], empty[SCAN_STAGES];
   __shared__ int failed_flag;
   constexpr int DKP = 8 * RPL, NA = KIND == KIND_DELTA ? 6 : 3, J = RPL / 4;  // staged key-channel arrays
-  constexpr bool PAIRS = KIND != KIND_GLA;
+  constexpr bool PAIRS = KIND == KIND_DELTA;
   const RecurrenceScanArgs& a = sa.a;
   const RecurrenceLayer& l = a.l;
   const int dk = l.dim, K = l.heads * dk, tid = threadIdx.x;
@@ -618,62 +623,6 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
         values(x, v);
         token(t, k, w, q, k, v, nullptr);
       }
-    } else if (KIND == KIND_CHANNEL) {
-      auto times = [](const Row (&x)[J], const Row (&y)[J], Row (&r)[J]) {
-#pragma unroll
-        for (int j = 0; j < J; ++j) {
-          r[j].x = mul2(x[j].x, y[j].x);
-          r[j].y = mul2(x[j].y, y[j].y);
-        }
-      };
-      int t = 0;
-      for (; t + 1 < n; t += 2) {
-        const float *xa = x0 + (size_t)t * stride, *xb = xa + stride;
-        float d[2 * CPL], v[CPL];
-        Row k[J], w[J], q[J], r[J];
-        fetch(xa, 0, k);
-        fetch(xa, 1, w);
-        times(k, w, r);
-        dot(r, d);
-        fetch(xb, 0, r);
-        fetch(xb, 1, q);
-        times(r, q, r);
-        times(r, w, r);
-        dot(r, d + CPL);
-        fetch(xa, 2, q);
-        const float2 ca = *reinterpret_cast<const float2*>(xa + NA * DKP + 2 * COLS);
-        const float beta = xb[NA * DKP + 2 * COLS + 1];
-        GroupSum<2 * CPL, 4>::run(d, lr);
-        values(xa, v);
-#pragma unroll
-        for (int c = 0; c < CPL; ++c) v[c] = ca.y * (v[c] - d[c]);
-        token(t, k, w, q, k, v, nullptr);
-#pragma unroll
-        for (int c = 0; c < CPL; ++c) d[CPL + c] = fmaf(ca.x, v[c], d[CPL + c]);
-        fetch(xb, 0, k);
-        fetch(xb, 1, w);
-        fetch(xb, 2, q);
-        values(xb, v);
-#pragma unroll
-        for (int c = 0; c < CPL; ++c) v[c] = beta * (v[c] - d[CPL + c]);
-        token(t + 1, k, w, q, k, v, nullptr);
-      }
-      if (t < n) {
-        const float* xa = x0 + (size_t)t * stride;
-        float d[CPL], v[CPL];
-        Row k[J], w[J], q[J], r[J];
-        fetch(xa, 0, k);
-        fetch(xa, 1, w);
-        times(k, w, r);
-        dot(r, d);
-        fetch(xa, 2, q);
-        values(xa, v);
-        const float beta = xa[NA * DKP + 2 * COLS + 1];
-        GroupSum<CPL, 4>::run(d, lr);
-#pragma unroll
-        for (int c = 0; c < CPL; ++c) v[c] = beta * (v[c] - d[c]);
-        token(t, k, w, q, k, v, nullptr);
-      }
     } else {
       int t = 0;
       for (; t + 1 < n; t += 2) {
@@ -757,6 +706,267 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) recurrence_scan_kern
     }
     __syncwarp();
     if (lane == 0) mbar_arrive(&empty[sidx]);
+  }
+
+  if (sa.mode == SCAN_OUTPUT) return;
+  float* fin = sa.mode == SCAN_FULL ? a.state + ((size_t)a.seq_slot[seq] * l.heads + head) * dk * l.dvp
+               : trans              ? sa.seg_trans + seg_index * dk * sa.dkp
+                                    : sa.seg_state + seg_index * dk * l.dvp;
+  const int pitch = trans ? sa.dkp : l.dvp;
+#pragma unroll
+  for (int r = 0; r < RPL; r += 2)
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      float v[2];
+      unpack2(s[r / 2][c], v[0], v[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (row_of(r + e) < dk && col0 + c < dv) fin[(size_t)row_of(r + e) * pitch + cbase + col0 + c] = v[e];
+    }
+}
+
+// The channel delta rule, four tokens at a time (see channel_quads_kernel); blocks, lanes, stages and modes as above.
+template <int RPL, int CPL>
+__global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) channel_scan_kernel(ScanArgs sa) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ uint64_t full[SCAN_STAGES], empty[SCAN_STAGES];
+  __shared__ int failed_flag;
+  constexpr int DKP = 8 * RPL, J = RPL / 4;
+  const RecurrenceScanArgs& a = sa.a;
+  const RecurrenceLayer& l = a.l;
+  const int dk = l.dim, K = l.heads * dk, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const bool trans = sa.mode == SCAN_TRANS, outputs = sa.mode == SCAN_FULL || sa.mode == SCAN_OUTPUT;
+  const int head = blockIdx.x / sa.col_blocks, cb = blockIdx.x % sa.col_blocks, seq = blockIdx.y, seg = blockIdx.z;
+  const int all_cols = trans ? dk : l.vdim, cbase = cb * sa.block_cols;
+  const int dv = min(sa.block_cols, all_cols - cbase);  // columns of this block
+  const int W = (blockDim.x >> 5) - 1, COLS = W * 4 * CPL, TB = sa.tb;  // TB: tokens of a stage, a multiple of QUAD
+  // a staged quad: per token A, B, Q, v, gate; then W and the numbers
+  const int stride = 3 * DKP + 2 * COLS, qstride = QUAD * stride + DKP + QUAD_NUMBERS, OP = COLS + 4, quads = TB / QUAD;
+  float* stage = sm;                                            // [SCAN_STAGES][quads][qstride]
+  float* os0 = sm + (size_t)SCAN_STAGES * quads * qstride;      // [2][TB][8 lanes of a group][OP]
+  const bool want_v = !trans, want_g = outputs && sa.col_blocks == 1;
+  volatile int* failed = &failed_flag;
+
+  const int first = a.seq_start[seq];
+  int t0 = first, t1 = a.seq_start[seq + 1];
+  if (sa.mode != SCAN_FULL) {
+    t0 += seg * a.seg_tokens;
+    t1 = min(t1, t0 + a.seg_tokens);
+    if (t0 >= t1) return;
+  }
+  for (int i = tid; i < SCAN_STAGES * quads * qstride; i += blockDim.x) stage[i] = 0.f;  // the padding stays zero
+  if (tid == 0) {
+    for (int i = 0; i < SCAN_STAGES; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], (uint32_t)W);
+    }
+    failed_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // the zeros come before the bulk copies
+  __syncthreads();
+  const int blocks = (t1 - t0 + TB - 1) / TB;
+
+  if (warp == W) {  // ---- stages rows; lane = (token, array) of a quad, then its W and its numbers
+    const int tok = lane / 5, arr = lane % 5;
+    const float* rows[5] = {a.decay + head * dk, a.writes + head * dk, a.unit_next + head * dk, sa.v + head * l.vdim + cbase, sa.g + head * l.vdim + cbase};
+    const bool on = lane >= 20 ? lane < 22 : arr < 2 || (arr == 2 && outputs) || (arr == 3 && want_v) || (arr == 4 && want_g);
+    const float* src = rows[arr];
+    const int pitch = arr < 3 ? K : arr == 3 ? sa.ldv : sa.ldg, count = lane == 21 ? QUAD_NUMBERS : lane == 20 || arr < 3 ? dk : dv;
+    const int off = lane == 21 ? QUAD * stride + DKP : lane == 20 ? QUAD * stride : tok * stride + (arr < 3 ? arr * DKP : 3 * DKP + (arr == 4 ? COLS : 0));
+    const size_t quad0 = first_quad(a, seq) + (t0 - first) / QUAD;
+    const uint32_t token_bytes = 4u * (uint32_t)((outputs ? 3 : 2) * dk + (want_v ? dv : 0) + (want_g ? dv : 0)), quad_bytes = 4u * (uint32_t)(dk + QUAD_NUMBERS);
+    RingCursor r;
+    for (int b = 0; b < blocks; ++b, r.next(SCAN_STAGES)) {
+      const int tb0 = t0 + b * TB, n = min(TB, t1 - tb0), nq = (n + QUAD - 1) / QUAD;
+      if (!mbar_wait(&empty[r.stage], r.parity ^ 1, failed, a.error_flag, 41)) break;
+      __syncwarp();
+      float* dst = stage + (size_t)r.stage * quads * qstride + off;
+      if (sa.vec) {
+        if (lane == 0) mbar_expect_tx(&full[r.stage], (uint32_t)n * token_bytes + (uint32_t)nq * quad_bytes);
+        __syncwarp();
+      }
+      for (int g = 0; g < nq; ++g) {
+        const size_t quad = quad0 + (size_t)b * quads + g;
+        const bool have = on && (lane >= 20 || g * QUAD + tok < n);
+        const float* from = lane == 21 ? a.quads + (quad * l.heads + head) * QUAD_NUMBERS
+                            : lane == 20 ? a.quad_decay + quad * K + head * dk
+                                         : src + (size_t)(tb0 + g * QUAD + tok) * pitch;
+        if (have && sa.vec) bulk_row(dst + (size_t)g * qstride, from, (uint32_t)(4 * count), &full[r.stage]);
+        else if (have)
+          for (int i = 0; i < count; ++i) dst[(size_t)g * qstride + i] = from[i];
+      }
+      if (!sa.vec) {
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&full[r.stage]);
+      }
+    }
+    return;
+  }
+
+  // ---- start state, two neighbouring rows per register pair
+  const int lr = lane & 7, col0 = (warp * 4 + (lane >> 3)) * CPL;
+  unsigned long long s[RPL / 2][CPL];
+  const size_t seg_index = ((size_t)seq * a.max_segs + seg) * l.heads + head;
+  const float* init = nullptr;
+  if (sa.mode == SCAN_FULL && a.seq_pos[seq] > 0) init = a.state + ((size_t)a.seq_slot[seq] * l.heads + head) * dk * l.dvp;
+  if (sa.mode == SCAN_OUTPUT) init = sa.seg_state + seg_index * dk * l.dvp;
+  auto row_of = [&](int r) { return (r >> 2) * 32 + lr * 4 + (r & 3); };
+#pragma unroll
+  for (int r = 0; r < RPL; r += 2)
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) {
+      float v[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int row = row_of(r + e), col = col0 + c;
+        v[e] = 0.f;
+        if (row < dk && col < dv) {
+          if (init) v[e] = init[(size_t)row * l.dvp + cbase + col];
+          else if (trans) v[e] = row == cbase + col ? 1.f : 0.f;
+        }
+      }
+      s[r / 2][c] = pack2(v[0], v[1]);
+    }
+
+  using Row = ulonglong2;  // four entries of a key-channel row
+  auto row = [&](const float* x, int j) { return *reinterpret_cast<const Row*>(x + j * 32 + lr * 4); };
+  RingCursor ring;
+  for (int b = 0; b < blocks; ++b, ring.next(SCAN_STAGES)) {
+    const int tb0 = t0 + b * TB, n = min(TB, t1 - tb0);
+    mbar_wait(&full[ring.stage], ring.parity, failed, a.error_flag, 42);  // on expiry the numbers are void, the barriers below are kept
+    __syncwarp();
+    const float* x0 = stage + (size_t)ring.stage * quads * qstride;
+    float* os = os0 + (size_t)(b & 1) * TB * 8 * OP;
+    for (int g = 0; g * QUAD < n; ++g) {
+      const float* x = x0 + (size_t)g * qstride;
+      const float* num = x + QUAD * stride + DKP;
+      const int have = n - g * QUAD;  // tokens of this quad, if below four
+      float d[QUAD * CPL];
+#pragma unroll
+      for (int i = 0; i < QUAD; ++i) {
+        unsigned long long e[CPL];
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) e[c] = 0;
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+          const Row k = row(x + i * stride, j);
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) e[c] = fma2(k.y, s[2 * j + 1][c], fma2(k.x, s[2 * j][c], e[c]));
+        }
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          float u, v;
+          unpack2(e[c], u, v);
+          d[i * CPL + c] = u + v;
+        }
+      }
+      GroupSum<QUAD * CPL, 4>::run(d, lr);
+      float nr[QUAD_NUMBERS];
+#pragma unroll
+      for (int i = 0; i < QUAD_NUMBERS; i += 4) {
+        const float4 f = load4(num + i);
+        nr[i] = f.x; nr[i + 1] = f.y; nr[i + 2] = f.z; nr[i + 3] = f.w;
+      }
+#pragma unroll
+      for (int i = 0; i < QUAD; ++i)
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          float v = x[i * stride + 3 * DKP + col0 + c] - d[i * CPL + c];
+#pragma unroll
+          for (int j = 0; j < i; ++j) v = fmaf(-nr[i * (i - 1) / 2 + j], d[j * CPL + c], v);
+          d[i * CPL + c] = i < have ? nr[16 + i] * v : 0.f;  // what token i writes
+        }
+      if (outputs) {
+#pragma unroll
+        for (int i = 0; i < QUAD; ++i) {
+          if (i >= have) break;
+          unsigned long long e[CPL];
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) e[c] = 0;
+#pragma unroll
+          for (int j = 0; j < J; ++j) {
+            const Row q = row(x + i * stride + 2 * DKP, j);
+#pragma unroll
+            for (int c = 0; c < CPL; ++c) e[c] = fma2(q.y, s[2 * j + 1][c], fma2(q.x, s[2 * j][c], e[c]));
+          }
+          float r[CPL];
+#pragma unroll
+          for (int c = 0; c < CPL; ++c) {
+            float u, v;
+            unpack2(e[c], u, v);
+            r[c] = u + v;
+            if (lr == 0) {
+#pragma unroll
+              for (int j = 0; j <= i; ++j) r[c] = fmaf(nr[6 + i * (i + 1) / 2 + j], d[j * CPL + c], r[c]);
+            }
+          }
+          float* po = os + (size_t)((g * QUAD + i) * 8 + lr) * OP + col0;
+          if (CPL == 4) store4(po, make_float4(r[0], r[1 % CPL], r[2 % CPL], r[3 % CPL]));
+          else if (CPL == 2) *reinterpret_cast<float2*>(po) = make_float2(r[0], r[1 % CPL]);
+          else po[0] = r[0];
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < J; ++j) {
+        const Row w = row(x + QUAD * stride, j);
+        Row k[QUAD];
+#pragma unroll
+        for (int i = 0; i < QUAD; ++i) k[i] = row(x + i * stride + DKP, j);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          unsigned long long lo = mul2(w.x, s[2 * j][c]), hi = mul2(w.y, s[2 * j + 1][c]);
+#pragma unroll
+          for (int i = 0; i < QUAD; ++i) {
+            const unsigned long long u = pack2(d[i * CPL + c], d[i * CPL + c]);
+            lo = fma2(k[i].x, u, lo);
+            hi = fma2(k[i].y, u, hi);
+          }
+          s[2 * j][c] = lo;
+          s[2 * j + 1][c] = hi;
+        }
+      }
+    }
+    if (outputs) {
+      // every warp's shares are in; this buffer is written again two blocks on, after the next barrier
+      named_barrier(1, W * 32);
+      for (int t = warp; t < n; t += W) {
+        const float* po = os + (size_t)t * 8 * OP;
+        const float* g = x0 + (size_t)(t / QUAD) * qstride + (t % QUAD) * stride + 3 * DKP + COLS;
+        float o[4], sq = 0.f;  // at most 128 columns
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int c = lane + i * 32;
+          float v = 0.f;
+          if (c < dv) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v += po[e * OP + c];
+          }
+          o[i] = v * l.q_scale;
+          sq += o[i] * o[i];
+        }
+        if (sa.col_blocks > 1) {  // recurrence_output_kernel finishes the rows
+          float* out = a.out_raw + (size_t)(tb0 + t) * (l.heads * l.vdim) + head * l.vdim + cbase;
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (lane + i * 32 < dv) out[lane + i * 32] = o[i];
+        } else {
+          const float rinv = 1.f / sqrtf(lane_sum(sq) / (float)dv + l.eps);
+          const size_t base = (size_t)(tb0 + t) * a.ldy + head * dv;
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const int c = lane + i * 32;
+            if (c < dv) {
+              const float y = o[i] * rinv * l.norm[c] * sigmoid_f(g[c]) * l.out_scale;
+              if (sa.y_bf16) static_cast<__nv_bfloat16*>(a.y)[base + c] = __float2bfloat16_rn(y);
+              else static_cast<float*>(a.y)[base + c] = y;
+            }
+          }
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[ring.stage]);
   }
 
   if (sa.mode == SCAN_OUTPUT) return;
@@ -936,21 +1146,33 @@ int sm_count() {
 }
 
 size_t scan_smem(int kind, int rpl, int cpl, int warps, int tb) {
+  if (kind == KIND_CHANNEL) {
+    const size_t c = (size_t)warps * 4 * cpl, quad = QUAD * (3 * 8 * rpl + 2 * c) + 8 * rpl + QUAD_NUMBERS;
+    return ((size_t)SCAN_STAGES * (tb / QUAD) * quad + (size_t)2 * tb * 8 * (c + 4)) * sizeof(float);
+  }
   const size_t na = kind == KIND_DELTA ? 6 : 3, cols = (size_t)warps * 4 * cpl;
   return ((size_t)SCAN_STAGES * tb * (na * 8 * rpl + 2 * cols + 4) + (size_t)2 * tb * 8 * (cols + 4)) * sizeof(float);
+}
+
+template <int KIND, int RPL, int CPL>
+auto scan_kernel() {
+  if constexpr (KIND == KIND_CHANNEL) return channel_scan_kernel<RPL, CPL>;
+  else return recurrence_scan_kernel<KIND, RPL, CPL>;
 }
 
 template <int KIND, int RPL, int CPL>
 cudaError_t launch_scan(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
   const int warps = (cols + 4 * CPL - 1) / (4 * CPL);
   if (warps > SCAN_WARPS) return cudaErrorInvalidValue;
+  const int least = KIND == KIND_CHANNEL ? QUAD : 2;
   sa.tb = 16;
-  while (sa.tb > 2 && scan_smem(KIND, RPL, CPL, warps, sa.tb) > MAX_SMEM) sa.tb /= 2;
+  while (sa.tb > least && scan_smem(KIND, RPL, CPL, warps, sa.tb) > MAX_SMEM) sa.tb /= 2;
   const size_t smem = scan_smem(KIND, RPL, CPL, warps, sa.tb);
   if (smem > MAX_SMEM) return cudaErrorInvalidValue;
-  cudaError_t e = cudaFuncSetAttribute(recurrence_scan_kernel<KIND, RPL, CPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
+  auto kernel = scan_kernel<KIND, RPL, CPL>();
+  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
   if (e != cudaSuccess) return e;
-  return launch_kernel(recurrence_scan_kernel<KIND, RPL, CPL>, grid, dim3((warps + 1) * 32), smem, s, false, sa);
+  return launch_kernel(kernel, grid, dim3((warps + 1) * 32), smem, s, false, sa);
 }
 
 template <int KIND, int RPL>
@@ -989,29 +1211,29 @@ cudaError_t launch_scan_any(ScanArgs sa, dim3 grid, int cols, cudaStream_t s) {
 cudaError_t launch_channel_gates(const RecurrenceScanArgs& a, cudaStream_t s) {
   const RecurrenceLayer& l = a.l;
   const long long cw = (long long)((a.rows + CONV_ROWS - 1) / CONV_ROWS) * (2 * l.kv_heads + l.heads);
-  const long long gw = (long long)((a.rows + GATE_GROUP - 1) / GATE_GROUP) * l.heads;
-  const dim3 cg((unsigned)((cw + 7) / 8)), gg((unsigned)((gw + 7) / 8)), b(256);
+  const long long qw = (long long)((a.max_len + QUAD - 1) / QUAD) * l.heads;
+  const dim3 cg((unsigned)((cw + 7) / 8)), qg((unsigned)((qw + 7) / 8), a.nseq), b(256);
   const int size = std::max(l.dim, l.vdim);
   const bool vec = l.dim % 4 == 0 && l.vdim % 4 == 0 && size <= 128 && l.taps >= 2 && l.taps <= 4 && a.ldp % 4 == 0 && l.off_q % 4 == 0 &&
                    l.off_k % 4 == 0 && l.off_v % 4 == 0 && l.channels % 4 == 0 && a.ldz % 4 == 0;
   cudaError_t e;
-  if (vec) {
-    e = l.taps == 2   ? launch_kernel(channel_conv_vec_kernel<2>, cg, b, 0, s, false, a)
-        : l.taps == 3 ? launch_kernel(channel_conv_vec_kernel<3>, cg, b, 0, s, false, a)
-                      : launch_kernel(channel_conv_vec_kernel<4>, cg, b, 0, s, false, a);
-    if (e == cudaSuccess) e = launch_kernel(channel_gates_vec_kernel, gg, b, 0, s, false, a);
-    return e != cudaSuccess ? e : launch_kernel(channel_taps_kernel, dim3(a.nseq, l.taps - 1), b, 0, s, false, a);
-  }
 #define PG_CONV(TAPS_)                                                                                  \
-  (size <= 64    ? launch_kernel(channel_conv_kernel<TAPS_, 2>, cg, b, 0, s, false, a)                  \
+  (vec           ? launch_kernel(channel_conv_vec_kernel<TAPS_>, cg, b, 0, s, false, a)                 \
+   : size <= 64  ? launch_kernel(channel_conv_kernel<TAPS_, 2>, cg, b, 0, s, false, a)                  \
    : size <= 128 ? launch_kernel(channel_conv_kernel<TAPS_, 4>, cg, b, 0, s, false, a)                  \
                  : launch_kernel(channel_conv_kernel<TAPS_, 8>, cg, b, 0, s, false, a))
-  e = l.taps == 2 ? PG_CONV(2) : l.taps == 3 ? PG_CONV(3) : l.taps == 4 ? PG_CONV(4) : PG_CONV(0);
+  if (l.taps == 2) e = PG_CONV(2);
+  else if (l.taps == 3) e = PG_CONV(3);
+  else if (l.taps == 4) e = PG_CONV(4);
+  else
+    e = size <= 64    ? launch_kernel(channel_conv_kernel<0, 2>, cg, b, 0, s, false, a)
+        : size <= 128 ? launch_kernel(channel_conv_kernel<0, 4>, cg, b, 0, s, false, a)
+                      : launch_kernel(channel_conv_kernel<0, 8>, cg, b, 0, s, false, a);
 #undef PG_CONV
   if (e != cudaSuccess) return e;
-  e = l.dim <= 64    ? launch_kernel(channel_gates_kernel<2>, gg, b, 0, s, false, a)
-      : l.dim <= 128 ? launch_kernel(channel_gates_kernel<4>, gg, b, 0, s, false, a)
-                     : launch_kernel(channel_gates_kernel<8>, gg, b, 0, s, false, a);
+  e = l.dim <= 64    ? launch_kernel(channel_quads_kernel<2>, qg, b, 0, s, false, a)
+      : l.dim <= 128 ? launch_kernel(channel_quads_kernel<4>, qg, b, 0, s, false, a)
+                     : launch_kernel(channel_quads_kernel<8>, qg, b, 0, s, false, a);
   if (e != cudaSuccess || l.taps == 1) return e;
   return launch_kernel(channel_taps_kernel, dim3(a.nseq, l.taps - 1), b, 0, s, false, a);
 }
@@ -1046,8 +1268,8 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   sa.y_bf16 = y_bf16 ? 1 : 0;
   auto m4 = [](int v) { return v % 4 == 0; };
   if (l.kind == KIND_CHANNEL) {
-    sa.k = a.unit; sa.q = a.rate; sa.v = a.vals; sa.g = a.z + K;
-    sa.ldk = sa.ldq = l.kv_heads * l.dim; sa.ldv = l.heads * l.vdim; sa.ldg = a.ldz;
+    sa.v = a.vals; sa.g = a.z + K;
+    sa.ldv = l.heads * l.vdim; sa.ldg = a.ldz;
   } else {
     sa.k = a.p + l.off_k; sa.q = a.p + l.off_q; sa.v = a.p + l.off_v; sa.g = a.p + l.off_g;
     sa.ldk = sa.ldq = sa.ldv = sa.ldg = a.ldp;

@@ -99,7 +99,7 @@ def test_token_by_token_equals_prompt(mixed, mode):
 
 
 @pytest.mark.parametrize("mode", MODES)
-@pytest.mark.parametrize("sizes", [[2], [3, 1], [23], [22, 24, 1], [64], [40, 2, 7, 1, 1, 31], [129]])
+@pytest.mark.parametrize("sizes", [[2], [3, 1], [23], [22, 24, 1], [64], [40, 2, 7, 1, 1, 31], [129], [12, 13, 14, 15, 18, 23, 29, 30, 46]])
 def test_portions(mixed, mode, sizes):
     ids = mixed.ids(200, 1)
     model = mixed.model(mode)
