@@ -413,6 +413,32 @@ struct GroupSum<N, 0> {
   static __device__ __forceinline__ void run(float*, int) {}
 };
 
+// The same sums, each in the lanes that share it only: lane l of the group ends with the values index(l).. (N / 8 of them, or one).
+template <int N, int OFF>
+struct GroupScatter {
+  static __device__ __forceinline__ void run(float* v, int lr) {
+    if (N > 1) {
+      constexpr int H = N > 1 ? N / 2 : 1;
+      const bool up = lr & OFF;
+#pragma unroll
+      for (int i = 0; i < H; ++i) {
+        const float send = up ? v[i] : v[i + H], keep = up ? v[i + H] : v[i];
+        v[i] = keep + __shfl_xor_sync(ALL_LANES, send, OFF);
+      }
+      GroupScatter<H, OFF / 2>::run(v, lr);
+    } else {
+      v[0] += __shfl_xor_sync(ALL_LANES, v[0], OFF);
+      GroupScatter<1, OFF / 2>::run(v, lr);
+    }
+  }
+  static __device__ __forceinline__ int index(int lr) { return (N > 1 && (lr & OFF) ? N / 2 : 0) + GroupScatter<(N > 1 ? N / 2 : 1), OFF / 2>::index(lr); }
+};
+template <int N>
+struct GroupScatter<N, 0> {
+  static __device__ __forceinline__ void run(float*, int) {}
+  static __device__ __forceinline__ int index(int) { return 0; }
+};
+
 // The delta rule works on two tokens at a time: with e = (u' * w)^T S, where the dash marks the second token,
 // u'^T S_t = e - (u' . b) d + (u' . k) v, so that both reads come from one reduction over the state before the pair.
 template <int KIND, int RPL, int CPL>
@@ -743,7 +769,7 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) channel_scan_kernel(
   // a staged quad: per token A, B, Q, v, gate; then W and the numbers
   const int stride = 3 * DKP + 2 * COLS, qstride = QUAD * stride + DKP + QUAD_NUMBERS, OP = COLS + 4, quads = TB / QUAD;
   float* stage = sm;                                            // [SCAN_STAGES][quads][qstride]
-  float* os0 = sm + (size_t)SCAN_STAGES * quads * qstride;      // [2][TB][8 lanes of a group][OP]
+  float* os0 = sm + (size_t)SCAN_STAGES * quads * qstride;      // [2][TB][OP] outputs
   const bool want_v = !trans, want_g = outputs && sa.col_blocks == 1;
   volatile int* failed = &failed_flag;
 
@@ -837,7 +863,7 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) channel_scan_kernel(
     mbar_wait(&full[ring.stage], ring.parity, failed, a.error_flag, 42);  // on expiry the numbers are void, the barriers below are kept
     __syncwarp();
     const float* x0 = stage + (size_t)ring.stage * quads * qstride;
-    float* os = os0 + (size_t)(b & 1) * TB * 8 * OP;
+    float* os = os0 + (size_t)(b & 1) * TB * OP;
     for (int g = 0; g * QUAD < n; ++g) {
       const float* x = x0 + (size_t)g * qstride;
       const float* num = x + QUAD * stride + DKP;
@@ -878,9 +904,9 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) channel_scan_kernel(
           d[i * CPL + c] = i < have ? nr[16 + i] * v : 0.f;  // what token i writes
         }
       if (outputs) {
+        float r[QUAD * CPL];
 #pragma unroll
         for (int i = 0; i < QUAD; ++i) {
-          if (i >= have) break;
           unsigned long long e[CPL];
 #pragma unroll
           for (int c = 0; c < CPL; ++c) e[c] = 0;
@@ -890,22 +916,23 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) channel_scan_kernel(
 #pragma unroll
             for (int c = 0; c < CPL; ++c) e[c] = fma2(q.y, s[2 * j + 1][c], fma2(q.x, s[2 * j][c], e[c]));
           }
-          float r[CPL];
 #pragma unroll
           for (int c = 0; c < CPL; ++c) {
             float u, v;
             unpack2(e[c], u, v);
-            r[c] = u + v;
+            r[i * CPL + c] = u + v;
             if (lr == 0) {
 #pragma unroll
-              for (int j = 0; j <= i; ++j) r[c] = fmaf(nr[6 + i * (i + 1) / 2 + j], d[j * CPL + c], r[c]);
+              for (int j = 0; j <= i; ++j) r[i * CPL + c] = fmaf(nr[6 + i * (i + 1) / 2 + j], d[j * CPL + c], r[i * CPL + c]);
             }
           }
-          float* po = os + (size_t)((g * QUAD + i) * 8 + lr) * OP + col0;
-          if (CPL == 4) store4(po, make_float4(r[0], r[1 % CPL], r[2 % CPL], r[3 % CPL]));
-          else if (CPL == 2) *reinterpret_cast<float2*>(po) = make_float2(r[0], r[1 % CPL]);
-          else po[0] = r[0];
         }
+        using Scatter = GroupScatter<QUAD * CPL, 4>;
+        Scatter::run(r, lr);
+        const int at = Scatter::index(lr), i = at / CPL;
+        float* po = os + (size_t)(g * QUAD + i) * OP + col0 + at % CPL;
+        if (CPL == 4) *reinterpret_cast<float2*>(po) = make_float2(r[0], r[1]);
+        else if (CPL == 2 || (lr & 1) == 0) po[0] = r[0];
       }
 #pragma unroll
       for (int j = 0; j < J; ++j) {
@@ -931,18 +958,13 @@ __global__ void __launch_bounds__((SCAN_WARPS + 1) * 32, 1) channel_scan_kernel(
       // every warp's shares are in; this buffer is written again two blocks on, after the next barrier
       named_barrier(1, W * 32);
       for (int t = warp; t < n; t += W) {
-        const float* po = os + (size_t)t * 8 * OP;
+        const float* po = os + (size_t)t * OP;
         const float* g = x0 + (size_t)(t / QUAD) * qstride + (t % QUAD) * stride + 3 * DKP + COLS;
         float o[4], sq = 0.f;  // at most 128 columns
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int c = lane + i * 32;
-          float v = 0.f;
-          if (c < dv) {
-#pragma unroll
-            for (int e = 0; e < 8; ++e) v += po[e * OP + c];
-          }
-          o[i] = v * l.q_scale;
+          o[i] = c < dv ? po[c] * l.q_scale : 0.f;
           sq += o[i] * o[i];
         }
         if (sa.col_blocks > 1) {  // recurrence_output_kernel finishes the rows
@@ -1096,29 +1118,34 @@ __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(Sca
     asm volatile("cp.async.commit_group;" ::: "memory");
     float* start = sa.seg_state + seg_at(g) * dk * l.dvp;
     const float* m = tr + (size_t)(g & 1) * dk * tp;
+    const int c = tid % COMBINE_COLS, row0 = tid / COMBINE_COLS;  // this thread: one column, rows row0 + q * ROW_STEP
+    constexpr int ROW_STEP = COMBINE_THREADS / COMBINE_COLS;
+    if (KIND == KIND_DELTA) {
+      int j = 0;
+      for (; j + 3 < dk; j += 4) {
+        const float x0 = cur[j * COMBINE_COLS + c], x1 = cur[(j + 1) * COMBINE_COLS + c], x2 = cur[(j + 2) * COMBINE_COLS + c], x3 = cur[(j + 3) * COMBINE_COLS + c];
+#pragma unroll
+        for (int q = 0; q < MAX_PER; ++q)
+          if (q < per) {
+            const float4 t = load4(m + (size_t)min(row0 + q * ROW_STEP, dk - 1) * tp + j);
+            v[q] = fmaf(t.x, x0, v[q]);
+            v[q] = fmaf(t.y, x1, v[q]);
+            v[q] = fmaf(t.z, x2, v[q]);
+            v[q] = fmaf(t.w, x3, v[q]);
+          }
+      }
+      for (; j < dk; ++j)
+#pragma unroll
+        for (int q = 0; q < MAX_PER; ++q)
+          if (q < per) v[q] = fmaf(m[(size_t)min(row0 + q * ROW_STEP, dk - 1) * tp + j], cur[j * COMBINE_COLS + c], v[q]);
+    }
 #pragma unroll
     for (int q = 0; q < MAX_PER; ++q) {
-      const int i = tid + q * COMBINE_THREADS, r = i / COMBINE_COLS, c = i % COMBINE_COLS;
+      const int r = row0 + q * ROW_STEP, i = r * COMBINE_COLS + c;
       if (q < per && r < dk) {
         const float old = cur[i];
-        float x = v[q];
-        if (KIND == KIND_GLA) {
-          x = fmaf(w[q], old, x);
-        } else {
-          float e = 0.f, f = 0.f;
-          int j = 0;
-          for (; j + 3 < dk; j += 4) {
-            const float4 t = load4(m + (size_t)r * tp + j);
-            e = fmaf(t.x, cur[j * COMBINE_COLS + c], e);
-            f = fmaf(t.y, cur[(j + 1) * COMBINE_COLS + c], f);
-            e = fmaf(t.z, cur[(j + 2) * COMBINE_COLS + c], e);
-            f = fmaf(t.w, cur[(j + 3) * COMBINE_COLS + c], f);
-          }
-          for (; j < dk; ++j) e = fmaf(m[(size_t)r * tp + j], cur[j * COMBINE_COLS + c], e);
-          x += e + f;
-        }
         if (c < nc) start[(size_t)r * l.dvp + c0 + c] = old;
-        nxt[i] = x;
+        nxt[i] = KIND == KIND_GLA ? fmaf(w[q], old, v[q]) : v[q];
       }
     }
     __syncthreads();
@@ -1148,7 +1175,7 @@ int sm_count() {
 size_t scan_smem(int kind, int rpl, int cpl, int warps, int tb) {
   if (kind == KIND_CHANNEL) {
     const size_t c = (size_t)warps * 4 * cpl, quad = QUAD * (3 * 8 * rpl + 2 * c) + 8 * rpl + QUAD_NUMBERS;
-    return ((size_t)SCAN_STAGES * (tb / QUAD) * quad + (size_t)2 * tb * 8 * (c + 4)) * sizeof(float);
+    return ((size_t)SCAN_STAGES * (tb / QUAD) * quad + (size_t)2 * tb * (c + 4)) * sizeof(float);
   }
   const size_t na = kind == KIND_DELTA ? 6 : 3, cols = (size_t)warps * 4 * cpl;
   return ((size_t)SCAN_STAGES * tb * (na * 8 * rpl + 2 * cols + 4) + (size_t)2 * tb * 8 * (cols + 4)) * sizeof(float);
