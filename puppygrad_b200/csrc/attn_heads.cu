@@ -421,17 +421,18 @@ __device__ __forceinline__ T* key_target(const AttentionPortionArgs& a, int row,
 // requested together; what depends on the column only is worked out once per block.
 constexpr int ROT_THREADS = 256, ROT_MAX_ROWS = 32;
 template <typename T, int UNROLL>
-__global__ void __launch_bounds__(ROT_THREADS, 4) attention_rotate_kernel(AttentionPortionArgs a, int rows) {
+__global__ void __launch_bounds__(ROT_THREADS, 4) attention_rotate_kernel(AttentionPortionArgs a, int rows, int mix_staged) {
   extern __shared__ __align__(16) float sm[];  // [rows][rep][dimp] queries, [heads][rep] mixing
   __shared__ T* target[2 * ROT_MAX_ROWS];      // where the rows' key and value go
   const AttentionLayer& l = a.l;
   const int row0 = blockIdx.y * rows, c = blockIdx.x, nrows = min(rows, a.rows - row0), tid = threadIdx.x, H = l.heads, G = l.kv_heads, rep = H / G;
   const int qn = rep * l.dimp, per = qn + l.dimp + l.vdimp;
   float* qs = sm;
-  float* mix = qs + (size_t)rows * qn;
+  const float* mix = mix_staged ? qs + (size_t)rows * qn : l.mix + c * rep;
+  const int mix_row = mix_staged ? rep : H;
   grid_dep_launch();
-  if (l.mix)
-    for (int i = tid; i < H * rep; i += ROT_THREADS) mix[i] = l.mix[(size_t)(i / rep) * H + c * rep + i % rep];
+  if (l.mix && mix_staged)
+    for (int i = tid; i < H * rep; i += ROT_THREADS) qs[(size_t)rows * qn + i] = l.mix[(size_t)(i / rep) * H + c * rep + i % rep];
   grid_dep_wait();
   if (tid < 2 * nrows) target[tid] = key_target<T>(a, row0 + tid / 2, c, tid & 1);
   __syncthreads();
@@ -483,7 +484,7 @@ __global__ void __launch_bounds__(ROT_THREADS, 4) attention_rotate_kernel(Attent
 #pragma unroll
       for (int i = 0; i < HPT; ++i)
 #pragma unroll
-        for (int g = 0; g < MAX_REP; ++g) t[i][g] = g < rep && h0 + i * nhb < H ? mix[(h0 + i * nhb) * rep + g] : 0.f;
+        for (int g = 0; g < MAX_REP; ++g) t[i][g] = g < rep && h0 + i * nhb < H ? mix[(size_t)(h0 + i * nhb) * mix_row + g] : 0.f;
       T* out = static_cast<T*>(a.q) + (((size_t)row0 * H + h0) * G + c) * l.dimp + o * 4;
       const size_t out_row = (size_t)H * G * l.dimp, out_head = (size_t)nhb * G * l.dimp;
       const float* q = qs + o * 4;
@@ -505,7 +506,7 @@ __global__ void __launch_bounds__(ROT_THREADS, 4) attention_rotate_kernel(Attent
           const float4 x = load4(q + g * l.dimp);
 #pragma unroll
           for (int i = 0; i < HPT; ++i)
-            if (h0 + i * nhb < H) add(acc[i], mix[(h0 + i * nhb) * rep + g], x);
+            if (h0 + i * nhb < H) add(acc[i], mix[(size_t)(h0 + i * nhb) * mix_row + g], x);
         }
 #pragma unroll
         for (int i = 0; i < HPT; ++i)
@@ -549,7 +550,8 @@ __global__ void __launch_bounds__(256) attention_latent_kernel(AttentionPortionA
 }
 
 // Block = one head of one sequence. Parts hold maxima and sums in powers of two.
-__global__ void __launch_bounds__(128) attention_merge_kernel(AttentionStepArgs a, const float2* v_rot, int y_bf16) {
+constexpr int MERGE_THREADS = 256;
+__global__ void __launch_bounds__(MERGE_THREADS) attention_merge_kernel(AttentionStepArgs a, const float2* v_rot, int y_bf16) {
   __shared__ float w[64];
   const AttentionLayer& l = a.l;
   const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, pitch = 4 + ((l.vdim + 3) & ~3), half = l.vdim >> 1;
@@ -569,7 +571,7 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(AttentionStepArgs 
   __syncthreads();
   auto sum = [&](int c) {
     float v = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int s = 0; s < a.splits; ++s) {
       const float x = pt[s * pitch + 4 + c];  // an empty part holds no numbers
       v = w[s] != 0.f ? fmaf(w[s], x, v) : v;
@@ -582,15 +584,15 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(AttentionStepArgs 
     else static_cast<float*>(a.y)[at] = v;
   };
   if (l.v_rot) {
-    for (int c = tid; c < half; c += 128) {
+    for (int c = tid; c < half; c += MERGE_THREADS) {
       const float2 r = v_rot[(size_t)seq * half + c];
       const float u = sum(c), v = sum(c + half);
       put(c, u * r.x + v * r.y);
       put(c + half, v * r.x - u * r.y);
     }
   } else {
-    for (int c = tid; c < l.vdim; c += 128) put(c, sum(c));
-    for (int c = l.vdim + tid; c < a.ldyh; c += 128) put(c, 0.f);
+    for (int c = tid; c < l.vdim; c += MERGE_THREADS) put(c, sum(c));
+    for (int c = l.vdim + tid; c < a.ldyh; c += MERGE_THREADS) put(c, 0.f);
   }
 }
 
@@ -717,9 +719,10 @@ cudaError_t heads_step_t(const AttentionStepArgs& a, const StepShape& sh, int yb
 
 }  // namespace
 
+bool mix_staged(const AttentionLayer& l) { return l.mix && (size_t)l.heads * (l.heads / l.kv_heads) <= 16384; }
 size_t rotate_smem(const AttentionLayer& l, int rows) {
   const int rep = l.heads / l.kv_heads;
-  return l.mix ? ((size_t)rows * rep * l.dimp + (size_t)l.heads * rep) * sizeof(float) : 0;
+  return l.mix ? ((size_t)rows * rep * l.dimp + (mix_staged(l) ? (size_t)l.heads * rep : 0)) * sizeof(float) : 0;
 }
 
 bool attention_heads_supported(const AttentionLayer& l) {
@@ -747,7 +750,7 @@ cudaError_t launch_attention_rotate(const AttentionPortionArgs& a, bool bf16, cu
   const dim3 grid(a.l.kv_heads, (a.rows + rows - 1) / rows);  // blocks of the same rows together: their queries are neighbours
   auto run = [&](auto kernel) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
-    return e != cudaSuccess ? e : launch_kernel(kernel, grid, dim3(ROT_THREADS), smem, s, pdl, a, rows);
+    return e != cudaSuccess ? e : launch_kernel(kernel, grid, dim3(ROT_THREADS), smem, s, pdl, a, rows, mix_staged(a.l) ? 1 : 0);
   };
   if (a.step_pos) return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, 1>) : run(attention_rotate_kernel<float, 1>);
   return bf16 ? run(attention_rotate_kernel<__nv_bfloat16, 4>) : run(attention_rotate_kernel<float, 4>);
@@ -761,7 +764,7 @@ cudaError_t launch_attention_latent(const AttentionPortionArgs& a, bool bf16, cu
 
 cudaError_t launch_attention_merge(const AttentionStepArgs& a, const float2* v_rot, bool y_bf16, bool pdl, cudaStream_t s) {
   if (a.splits > 32) return cudaErrorInvalidValue;
-  return launch_kernel(attention_merge_kernel, dim3(a.l.heads, a.batch), dim3(128), 0, s, pdl, a, v_rot, y_bf16 ? 1 : 0);
+  return launch_kernel(attention_merge_kernel, dim3(a.l.heads, a.batch), dim3(MERGE_THREADS), 0, s, pdl, a, v_rot, y_bf16 ? 1 : 0);
 }
 
 cudaError_t launch_attention_turn_back(const AttentionPortionArgs& a, cudaStream_t s) {

@@ -36,6 +36,9 @@ ALONE = {
     "attention-own-keys": so.att(5, 5, 24, 8, 17, 6),
     "attention-wide-groups": so.att(18, 2, 8, 8, 25, 3),
     "attention-many-heads": so.att(40, 8, 16, 8, 33, 7),
+    "attention-two-groups-of-heads": so.att(64, 16, 16, 64, 150, 5),
+    "attention-300-heads": so.att(300, 1, 16, 8, 140, 2),
+    "attention-row-of-5120": so.att(40, 40, 128, 8, 21, 3),
     "attention-row-of-320": so.att(5, 5, 64, 64, 40, 3),
     "attention-row-of-544": so.att(4, 4, 136, 72, 50, 2),
     "attention-row-of-1024": so.att(8, 8, 128, 136, 31, 9),
@@ -63,6 +66,7 @@ ALONE = {
     "latent-one": so.latent(1, 16, 8, 8, 12),
     "latent-many-heads": so.latent(40, 8, 8, 64, 16),
     "latent-512": so.latent(16, 64, 72, 512, 200),
+    "latent-two-groups-of-heads": so.latent(130, 8, 8, 500, 16),
     "latent-1000": so.latent(3, 128, 256, 1000, 48),
     "feed-forward": so.delta(1, 1, 4, 4, 2, ff=136),
 }
