@@ -1057,8 +1057,8 @@ __global__ void __launch_bounds__(256) segment_decay_kernel(ScanArgs sa) {
 // Turns the segments' own contributions into their start states, in order: start[0] = cached state (or zero),
 // start[i + 1] = transition[i] start[i] + local[i]; the last one goes to the cache. Block = 16 columns of one head of
 // one sequence; the running state stays in shared memory, the next segment's numbers load one segment ahead.
-constexpr int COMBINE_COLS = 16, COMBINE_THREADS = 256;
-template <int KIND>
+constexpr int COMBINE_COLS = 16, COMBINE_THREADS = 256, ROW_STEP = COMBINE_THREADS / COMBINE_COLS;
+template <int KIND, int PER>  // PER: rows of a thread, PER * ROW_STEP >= dim
 __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(ScanArgs sa) {
   extern __shared__ __align__(16) float sm[];
   const RecurrenceScanArgs& a = sa.a;
@@ -1072,8 +1072,10 @@ __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(Sca
   float* tr = sm + 2 * dk * COMBINE_COLS;  // delta: [2][dk][tp], the next one loading
   float* cached = a.state + ((size_t)a.seq_slot[seq] * l.heads + head) * dk * l.dvp;
   const bool fresh = a.seq_pos[seq] == 0;
-  constexpr int MAX_PER = 256 * COMBINE_COLS / COMBINE_THREADS;  // dk <= 256
-  const int per = (dk * COMBINE_COLS + COMBINE_THREADS - 1) / COMBINE_THREADS;
+  const int c = tid % COMBINE_COLS, row0 = tid / COMBINE_COLS;  // this thread: one column, rows row0 + q * ROW_STEP
+  int at[PER];                                                  // where its rows of a transition matrix start
+#pragma unroll
+  for (int q = 0; q < PER; ++q) at[q] = min(row0 + q * ROW_STEP, dk - 1) * tp;
   auto seg_at = [&](int g) { return ((size_t)seq * a.max_segs + g) * l.heads + head; };
   auto load_trans = [&](int g, float* dst) {
     const float* src = sa.seg_trans + seg_at(g) * dk * sa.dkp;
@@ -1083,13 +1085,13 @@ __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(Sca
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + r * tp + x * 4)), "l"(src + (size_t)i * 4) : "memory");
     }
   };
-  float loc[MAX_PER], dec[MAX_PER];
+  float loc[PER], dec[PER];
   auto load_next = [&](int g) {
     const float* p = sa.seg_state + seg_at(g) * dk * l.dvp;
 #pragma unroll
-    for (int q = 0; q < MAX_PER; ++q) {
-      const int i = tid + q * COMBINE_THREADS, r = i / COMBINE_COLS, c = i % COMBINE_COLS;
-      if (q < per && r < dk) {
+    for (int q = 0; q < PER; ++q) {
+      const int r = row0 + q * ROW_STEP;
+      if (r < dk) {
         loc[q] = c < nc ? p[(size_t)r * l.dvp + c0 + c] : 0.f;
         if (KIND == KIND_GLA) dec[q] = sa.seg_trans[seg_at(g) * dk + r];
       }
@@ -1103,9 +1105,9 @@ __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(Sca
   if (KIND == KIND_DELTA) load_trans(0, tr);
   asm volatile("cp.async.commit_group;" ::: "memory");
   for (int g = 0; g < segs; ++g) {
-    float v[MAX_PER], w[MAX_PER];
+    float v[PER], w[PER];
 #pragma unroll
-    for (int q = 0; q < MAX_PER; ++q) {
+    for (int q = 0; q < PER; ++q) {
       v[q] = loc[q];
       w[q] = KIND == KIND_GLA ? dec[q] : 0.f;
     }
@@ -1118,31 +1120,28 @@ __global__ void __launch_bounds__(COMBINE_THREADS) recurrence_combine_kernel(Sca
     asm volatile("cp.async.commit_group;" ::: "memory");
     float* start = sa.seg_state + seg_at(g) * dk * l.dvp;
     const float* m = tr + (size_t)(g & 1) * dk * tp;
-    const int c = tid % COMBINE_COLS, row0 = tid / COMBINE_COLS;  // this thread: one column, rows row0 + q * ROW_STEP
-    constexpr int ROW_STEP = COMBINE_THREADS / COMBINE_COLS;
     if (KIND == KIND_DELTA) {
       int j = 0;
       for (; j + 3 < dk; j += 4) {
         const float x0 = cur[j * COMBINE_COLS + c], x1 = cur[(j + 1) * COMBINE_COLS + c], x2 = cur[(j + 2) * COMBINE_COLS + c], x3 = cur[(j + 3) * COMBINE_COLS + c];
 #pragma unroll
-        for (int q = 0; q < MAX_PER; ++q)
-          if (q < per) {
-            const float4 t = load4(m + (size_t)min(row0 + q * ROW_STEP, dk - 1) * tp + j);
-            v[q] = fmaf(t.x, x0, v[q]);
-            v[q] = fmaf(t.y, x1, v[q]);
-            v[q] = fmaf(t.z, x2, v[q]);
-            v[q] = fmaf(t.w, x3, v[q]);
-          }
+        for (int q = 0; q < PER; ++q) {
+          const float4 t = load4(m + at[q] + j);
+          v[q] = fmaf(t.x, x0, v[q]);
+          v[q] = fmaf(t.y, x1, v[q]);
+          v[q] = fmaf(t.z, x2, v[q]);
+          v[q] = fmaf(t.w, x3, v[q]);
+        }
       }
       for (; j < dk; ++j)
 #pragma unroll
-        for (int q = 0; q < MAX_PER; ++q)
-          if (q < per) v[q] = fmaf(m[(size_t)min(row0 + q * ROW_STEP, dk - 1) * tp + j], cur[j * COMBINE_COLS + c], v[q]);
+        for (int q = 0; q < PER; ++q)
+          v[q] = fmaf(m[at[q] + j], cur[j * COMBINE_COLS + c], v[q]);
     }
 #pragma unroll
-    for (int q = 0; q < MAX_PER; ++q) {
+    for (int q = 0; q < PER; ++q) {
       const int r = row0 + q * ROW_STEP, i = r * COMBINE_COLS + c;
-      if (q < per && r < dk) {
+      if (r < dk) {
         const float old = cur[i];
         if (c < nc) start[(size_t)r * l.dvp + c0 + c] = old;
         nxt[i] = KIND == KIND_GLA ? fmaf(w[q], old, v[q]) : v[q];
@@ -1324,10 +1323,16 @@ cudaError_t launch_recurrence_scan(const RecurrenceScanArgs& a, bool y_bf16, cud
   const dim3 cgrid(l.heads, a.nseq, (l.vdim + COMBINE_COLS - 1) / COMBINE_COLS);
   const size_t csmem = ((size_t)2 * l.dim * COMBINE_COLS + (l.kind != KIND_GLA ? (size_t)2 * l.dim * (sa.dkp + 4) : 0)) * sizeof(float);
   if (csmem > MAX_SMEM) return cudaErrorInvalidValue;
-  e = cudaFuncSetAttribute(recurrence_combine_kernel<KIND_DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
-  if (e != cudaSuccess) return e;
-  e = l.kind != KIND_GLA ? launch_kernel(recurrence_combine_kernel<KIND_DELTA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa)
-                           : launch_kernel(recurrence_combine_kernel<KIND_GLA>, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa);
+  auto combine = [&](auto kernel) {
+    const cudaError_t r = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MAX_SMEM);
+    return r != cudaSuccess ? r : launch_kernel(kernel, cgrid, dim3(COMBINE_THREADS), csmem, s, false, sa);
+  };
+#define PG_COMBINE(KIND_)                                                              \
+  (l.dim <= 4 * ROW_STEP   ? combine(recurrence_combine_kernel<KIND_, 4>)              \
+   : l.dim <= 8 * ROW_STEP ? combine(recurrence_combine_kernel<KIND_, 8>)              \
+                           : combine(recurrence_combine_kernel<KIND_, 16>))
+  e = l.kind != KIND_GLA ? PG_COMBINE(KIND_DELTA) : PG_COMBINE(KIND_GLA);
+#undef PG_COMBINE
   if (e != cudaSuccess) return e;
   sa.mode = SCAN_OUTPUT;
   return launch_scan_any(sa, grid, l.vdim, s);
