@@ -62,7 +62,7 @@ struct BranchSpec {
   int out_dim() const { return kind == RECURRENCE ? rec.heads * rec.vdim : attn.heads * attn.vdim; }
 };
 
-enum NormKind { NORM_LAYER = 0, NORM_RMS = 1 };  // LayerNorm with weight and bias; x / sqrt(mean(x^2) + eps) * weight
+enum NormKind { NORM_LAYER = 0, NORM_RMS = 1 };  // LayerNorm with weight and bias; weight times x over its root mean square
 enum Activation {
   ACT_NONE = 0,
   ACT_GELU_ERF = 1,

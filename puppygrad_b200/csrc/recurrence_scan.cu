@@ -338,15 +338,15 @@ __global__ void __launch_bounds__(256) channel_quads_kernel(RecurrenceScanArgs a
   if (lane < QUAD) out[16 + lane] = beta;
 }
 
-// The inputs that the next tokens' convolutions still need. Block = (sequence, one of its last taps - 1 rows).
+// The inputs that the next tokens' convolutions still need. Block = (sequence, one of its last taps - 1 rows, 256 channels).
 __global__ void __launch_bounds__(256) channel_taps_kernel(RecurrenceScanArgs a) {
   const RecurrenceLayer& l = a.l;
   const int seq = blockIdx.x, first = a.seq_start[seq], r = a.seq_start[seq + 1] - 1 - (int)blockIdx.y;
   if (r < first) return;
   const int pos = a.seq_pos[seq] + r - first;
   float* dst = a.taps + ((size_t)a.seq_slot[seq] * l.taps + pos % l.taps) * l.channels;
-#pragma unroll 8
-  for (int c = threadIdx.x; c < l.channels; c += blockDim.x) dst[c] = a.p[(size_t)r * a.ldp + l.off_q + c];
+  const int c = blockIdx.z * blockDim.x + threadIdx.x;
+  if (c < l.channels) dst[c] = a.p[(size_t)r * a.ldp + l.off_q + c];
 }
 
 // ------------------------------------------------------------------ scan
@@ -1261,7 +1261,7 @@ cudaError_t launch_channel_gates(const RecurrenceScanArgs& a, cudaStream_t s) {
       : l.dim <= 128 ? launch_kernel(channel_quads_kernel<4>, qg, b, 0, s, false, a)
                      : launch_kernel(channel_quads_kernel<8>, qg, b, 0, s, false, a);
   if (e != cudaSuccess || l.taps == 1) return e;
-  return launch_kernel(channel_taps_kernel, dim3(a.nseq, l.taps - 1), b, 0, s, false, a);
+  return launch_kernel(channel_taps_kernel, dim3(a.nseq, l.taps - 1, (l.channels + 255) / 256), b, 0, s, false, a);
 }
 
 }  // namespace
